@@ -27,6 +27,11 @@
 // > i + q_offset - window), key length (keys >= Tk are masked).  GQA by head grouping.
 // Outputs: O [B, Tq, Hq, D] bf16 (strided) and the log-sum-exp [B, Hq, Tq] fp32 for backward.
 //
+// Distance penalty (template parameter BIAS): a score loses r1_h ln(1 + r2_h (i - j)).  BIAS 1 reads it from a per-head table
+// in shared memory indexed by the distance (windows up to a few thousand keys; distances outside the window hold +inf, so the
+// table is the mask of the second pass too); BIAS 2 evaluates the logarithm per score.  These forms also take head sizes below
+// 128 (a multiple of 8): TMA fills the missing channels with zeros and the Q K^T loop stops at the last real one.
+//
 // The reference calls at::scaled_dot_product_attention, or a query-chunked masked-math fallback
 // for windows (cc/include/tyr_attention.h:58-130).
 #include "common.cuh"
@@ -48,7 +53,13 @@ struct AttnParams {
   long long o_row_stride, o_batch_stride, o_head_stride;
   float* lse;         // [B, Hq, Tq]
   int* err;
+  // distance penalty forms only
+  const float *r1, *r2;   // [Hq]
+  int k_steps;        // 16-channel steps of Q K^T
+  int dv;             // output channels
 };
+
+constexpr int ATT_TBL_PAD = 256;       // table entries below distance 0 and past the window that boundary blocks can touch
 
 struct __align__(1024) AttnSmem {
   uint8_t q[2][ATT_BM * ATT_D * 2];                 // 2 tiles x (2 chunks of [128 x 64])
@@ -134,6 +145,7 @@ __device__ __forceinline__ void kv_range(const AttnParams& p, int r0, int& lo, i
   if (hi < lo) hi = lo;
 }
 
+template <int BIAS>
 __global__ void __launch_bounds__(640, 1)
 flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
                       const __grid_constant__ CUtensorMap tmK,
@@ -177,6 +189,15 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
   }
   for (int i = threadIdx.x; i < 2 * 2 * 2 * ATT_BM; i += blockDim.x) (&s.xch[0][0][0][0])[i] = make_uint2(0u, 0u);
   for (int i = threadIdx.x; i < 2 * 2 * ATT_BM; i += blockDim.x) (&s.xsum[0][0][0])[i] = make_uint2(0u, 0u);
+  float* const table = reinterpret_cast<float*>(&s + 1);     // entry ATT_TBL_PAD + n: penalty at distance n, in log2 units
+  float r1 = 0.f, r2 = 0.f;
+  if constexpr (BIAS != 0) { r1 = p.r1[head]; r2 = p.r2[head]; }
+  if constexpr (BIAS == 1) {
+    for (int i = threadIdx.x; i < p.window + 2 * ATT_TBL_PAD; i += blockDim.x) {
+      const int n = i - ATT_TBL_PAD;
+      table[i] = (n < 0 || n >= p.window) ? INFINITY : r1 * log2f(1.f + r2 * static_cast<float>(n));
+    }
+  }
   if (warp == 16) {
     tmem_alloc(&s.tmem_base, 512);
     tmem_relinquish();
@@ -238,6 +259,7 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
         const uint32_t ka = smem_u32(s.k[st]);
 #pragma unroll
         for (int k = 0; k < ATT_D / 16; ++k) {
+          if (BIAS != 0 && k >= p.k_steps) break;
           const uint32_t off = (k >> 2) * kChunk + (k & 3) * 32;
           umma_f16_ss(tmem_base + t * 128, make_smem_desc_sw128(qa + off, 16, 1024),
                       make_smem_desc_sw128(ka + off, 16, 1024), idesc_s, k > 0 ? 1u : 0u);
@@ -310,6 +332,10 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
     const uint32_t p_addr = tmem_base + t * 128 + h * 64 + lane_addr;     // my 32 packed-probability columns: the start of my own score columns
     const uint32_t o_addr = tmem_base + 256 + t * 128 + h * 64 + lane_addr;
     const bool tile_live = (t == 0) || tile1_live;
+    auto penalty = [&](int n) { return r1 * __log2f(1.f + r2 * static_cast<float>(max(n, 0))); };
+    // Steep penalties: their spread inside one key block could push every probability of a row under the fp32 range when
+    // the reference is only a bound of the row maximum, so those heads take the exact maximum (one more table read per score).
+    const bool exact_max = BIAS != 0 && fabsf(penalty(ATT_BN - 1)) > 48.f;
     float m_used = -INFINITY;   // running maximum the exponentials are taken against
     float l_sum = 0.f;          // this half's part of the row sum
     bool ok = true;
@@ -339,21 +365,30 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
         // scores spilled, and the maximum alone took 500 cycles per block).
         float mx;
         {
-          uint32_t r0[32], r1[32];
-          tmem_ld_32x32_nowait(s_addr, r0);
-          tmem_ld_32x32_nowait(s_addr + 32, r1);
+          uint32_t sa[32], sb[32];
+          tmem_ld_32x32_nowait(s_addr, sa);
+          tmem_ld_32x32_nowait(s_addr + 32, sb);
           tmem_wait_ld();
           if (need_mask) {
-            masked(r0, col0);
-            masked(r1, col0 + 32);
+            masked(sa, col0);
+            masked(sb, col0 + 32);
+          }
+          if (BIAS != 0 && exact_max) {      // scores in units of 1 / scale_log2, like the raw ones
+            const float inv_scale = 1.f / p.scale_log2;
+#pragma unroll
+            for (int c = 0; c < 32; ++c) {
+              const int n0 = qi - (col0 + c), n1 = n0 - 32;
+              sa[c] = __float_as_uint(__uint_as_float(sa[c]) - penalty(n0) * inv_scale);
+              sb[c] = __float_as_uint(__uint_as_float(sb[c]) - penalty(n1) * inv_scale);
+            }
           }
           float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
           for (int c = 0; c < 32; c += 8) {
 #pragma unroll
             for (int u = 0; u < 4; ++u) {
-              mx4[u] = max3(mx4[u], __uint_as_float(r0[c + 2 * u]), __uint_as_float(r0[c + 2 * u + 1]));
-              mx4[u] = max3(mx4[u], __uint_as_float(r1[c + 2 * u]), __uint_as_float(r1[c + 2 * u + 1]));
+              mx4[u] = max3(mx4[u], __uint_as_float(sa[c + 2 * u]), __uint_as_float(sa[c + 2 * u + 1]));
+              mx4[u] = max3(mx4[u], __uint_as_float(sb[c + 2 * u]), __uint_as_float(sb[c + 2 * u + 1]));
             }
           }
           mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
@@ -364,6 +399,12 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
           break;
         }
         mx = fmaxf(mx, other) * p.scale_log2;
+        if (BIAS != 0 && !exact_max) {
+          // bound of the penalised row maximum: raw maximum minus the smallest penalty among this block's visible keys (the
+          // penalty is monotonic in the distance)
+          const int far_col = p.window > 0 ? max(j * ATT_BN, qi - p.window + 1) : j * ATT_BN;
+          mx -= fminf(penalty(qi - min(j * ATT_BN + ATT_BN - 1, qi)), penalty(qi - far_col));
+        }
         // lazy rescale: move the reference maximum only when it grew by more than 8 (log2 units); both halves of a row
         // take the same decision because they see the same maximum
         const bool first = (j == lo[t]);
@@ -384,23 +425,34 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
           tmem_wait_st();
           if (want) l_sum *= f;
         }
-        if (want) m_used = (m_new == -INFINITY) ? 0.f : m_new;
+        if (want) m_used = m_new;           // stays -inf while a row has seen no visible key: its first one sets the reference
         // Pass 2: probabilities exp2(s * scale - m) -> bf16 -> TMEM, 32 scores at a time.  My packed probabilities go to
         // the first 32 columns of MY OWN 64 score columns (chunk c lands on columns 16 c .. 16 c + 15, which chunk c
         // itself or an earlier chunk was read from), so neither half ever writes where the other half still reads.
         float ls4[4] = {0.f, 0.f, 0.f, 0.f};
-        const float neg_m = -m_used;
+        const float neg_m = m_used == -INFINITY ? 0.f : -m_used;
 #pragma unroll
         for (int c = 0; c < 2; ++c) {
           uint32_t r[32];
           tmem_ld_32x32(s_addr + c * 32, r);
           tmem_wait_ld();
-          if (need_mask) masked(r, col0 + c * 32);
+          if (BIAS != 1 && need_mask) masked(r, col0 + c * 32);
+          const float* tb = table + (ATT_TBL_PAD + qi - (col0 + c * 32));
           uint32_t pk[16];
 #pragma unroll
           for (int q = 0; q < 16; ++q) {
-            const float p0 = exp2f(fmaf(__uint_as_float(r[2 * q]), p.scale_log2, neg_m));
-            const float p1 = exp2f(fmaf(__uint_as_float(r[2 * q + 1]), p.scale_log2, neg_m));
+            float e0 = fmaf(__uint_as_float(r[2 * q]), p.scale_log2, neg_m);
+            float e1 = fmaf(__uint_as_float(r[2 * q + 1]), p.scale_log2, neg_m);
+            if constexpr (BIAS == 1) {
+              e0 -= tb[-2 * q];
+              e1 -= tb[-2 * q - 1];
+            } else if constexpr (BIAS == 2) {
+              const int n = qi - (col0 + c * 32 + 2 * q);
+              e0 -= penalty(n);
+              e1 -= penalty(n - 1);
+            }
+            const float p0 = exp2f(e0);
+            const float p1 = exp2f(e1);
             pk[q] = pack_bf16x2(p0, p1);
             ls4[q & 3] += p0 + p1;
           }
@@ -433,6 +485,7 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
           if (row_ok) {
 #pragma unroll
             for (int q = 0; q < 4; ++q) {
+              if (BIAS != 0 && h * 64 + c * 32 + q * 8 >= p.dv) break;
               uint4 u;
               u.x = pack_bf16x2(__uint_as_float(o[q * 8 + 0]) * inv, __uint_as_float(o[q * 8 + 1]) * inv);
               u.y = pack_bf16x2(__uint_as_float(o[q * 8 + 2]) * inv, __uint_as_float(o[q * 8 + 3]) * inv);
@@ -496,6 +549,46 @@ int make_tmap_bthd(CUtensorMap* tm, const void* base, int B, int T, int H, int D
 }  // namespace
 
 // q/k/v/o are [B, T, H, D] views given by (batch, row, head) element strides; D must be 128.
+static int flash_fwd_launch(const void* q, const void* k, const void* v, void* o, float* lse, int B, int Hq, int Hkv, int Tq, int Tk,
+                            int dk, int dv, const long long* st, int causal, int window, int q_offset, float scale, const float* r1,
+                            const float* r2, int* err, void* stream) {
+  if (Hq % Hkv != 0 || B <= 0 || Tq <= 0 || Tk <= 0) return -2;
+  for (int i = 0; i < 12; ++i)
+    if (st[i] & 7) return -3;
+  if (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)o) & 15) return -4;
+  CUtensorMap tq, tk, tv;
+  int r;
+  if ((r = make_tmap_bthd(&tq, q, B, Tq, Hq, dk, st[0], st[1], st[2], ATT_BM))) return 3000 + r;
+  if ((r = make_tmap_bthd(&tk, k, B, Tk, Hkv, dk, st[3], st[4], st[5], ATT_BN))) return 4000 + r;
+  if ((r = make_tmap_bthd(&tv, v, B, Tk, Hkv, dv, st[6], st[7], st[8], ATT_BN))) return 5000 + r;
+  constexpr size_t kBase = sizeof(AttnSmem) + 1024, kMax = 227 * 1024;
+  const size_t table = (static_cast<size_t>(window) + 2 * ATT_TBL_PAD) * sizeof(float);
+  // the table covers a causal window whose distances start at 0 in the query's own block (no key offset)
+  const int bias = r1 == nullptr ? 0 : (causal && window > 0 && q_offset == 0 && kBase + table <= kMax ? 1 : 2);
+  const size_t smem = bias == 1 ? kBase + table : kBase;
+  auto kernel = bias == 0 ? flash_fwd_d128_kernel<0> : (bias == 1 ? flash_fwd_d128_kernel<1> : flash_fwd_d128_kernel<2>);
+  static bool configured_dev[64][3] = {};       // the attribute is per device
+  int cfg_dev = 0;
+  if (cudaGetDevice(&cfg_dev) != cudaSuccess || cfg_dev < 0 || cfg_dev >= 64) cfg_dev = 0;
+  bool& configured = configured_dev[cfg_dev][bias];
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(bias == 1 ? kMax : kBase));
+    if (e != cudaSuccess) return 1000 + (int)e;
+    configured = true;
+  }
+  AttnParams p;
+  p.B = B; p.Hq = Hq; p.Hkv = Hkv; p.Tq = Tq; p.Tk = Tk;
+  p.q_offset = q_offset; p.causal = causal; p.window = window;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.O = (__nv_bfloat16*)o; p.o_batch_stride = st[9]; p.o_row_stride = st[10]; p.o_head_stride = st[11];
+  p.lse = lse; p.err = err;
+  p.r1 = r1; p.r2 = r2; p.k_steps = (dk + 15) / 16; p.dv = dv;
+  dim3 grid((Tq + 2 * ATT_BM - 1) / (2 * ATT_BM), Hq, B);
+  launch_dependent(kernel, dim3(grid), dim3(640), smem, (cudaStream_t)stream, tq, tk, tv, p);
+  cudaError_t e = cudaGetLastError();
+  return e == cudaSuccess ? 0 : 2000 + (int)e;
+}
+
 extern "C" TYR_EXPORT int tyr_flash_fwd(const void* q, const void* k, const void* v, void* o,
                                         float* lse, int B, int Hq, int Hkv, int Tq, int Tk, int D,
                                         long long q_sb, long long q_st, long long q_sh,
@@ -505,33 +598,15 @@ extern "C" TYR_EXPORT int tyr_flash_fwd(const void* q, const void* k, const void
                                         int window, int q_offset, float scale, int* err,
                                         void* stream) {
   if (D != ATT_D) return -1;
-  if (Hq % Hkv != 0 || B <= 0 || Tq <= 0 || Tk <= 0) return -2;
-  if ((q_st | q_sh | q_sb | k_st | k_sh | k_sb | v_st | v_sh | v_sb | o_st | o_sh | o_sb) & 7) return -3;
-  if (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)o) & 15) return -4;
-  CUtensorMap tq, tk, tv;
-  int r;
-  if ((r = make_tmap_bthd(&tq, q, B, Tq, Hq, D, q_sb, q_st, q_sh, ATT_BM))) return 3000 + r;
-  if ((r = make_tmap_bthd(&tk, k, B, Tk, Hkv, D, k_sb, k_st, k_sh, ATT_BN))) return 4000 + r;
-  if ((r = make_tmap_bthd(&tv, v, B, Tk, Hkv, D, v_sb, v_st, v_sh, ATT_BN))) return 5000 + r;
-  constexpr size_t smem = sizeof(AttnSmem) + 1024;
-  static bool configured_dev[64] = {false};     // the attribute is per device
-  int cfg_dev = 0;
-  if (cudaGetDevice(&cfg_dev) != cudaSuccess || cfg_dev < 0 || cfg_dev >= 64) cfg_dev = 0;
-  bool& configured = configured_dev[cfg_dev];
-  if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(flash_fwd_d128_kernel,
-                                         cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e != cudaSuccess) return 1000 + (int)e;
-    configured = true;
-  }
-  AttnParams p;
-  p.B = B; p.Hq = Hq; p.Hkv = Hkv; p.Tq = Tq; p.Tk = Tk;
-  p.q_offset = q_offset; p.causal = causal; p.window = window;
-  p.scale_log2 = scale * 1.4426950408889634f;
-  p.O = (__nv_bfloat16*)o; p.o_row_stride = o_st; p.o_batch_stride = o_sb; p.o_head_stride = o_sh;
-  p.lse = lse; p.err = err;
-  dim3 grid((Tq + 2 * ATT_BM - 1) / (2 * ATT_BM), Hq, B);
-  launch_dependent(flash_fwd_d128_kernel, dim3(grid), dim3(640), smem, (cudaStream_t)stream, tq, tk, tv, p);
-  cudaError_t e = cudaGetLastError();
-  return e == cudaSuccess ? 0 : 2000 + (int)e;
+  const long long st[12] = {q_sb, q_st, q_sh, k_sb, k_st, k_sh, v_sb, v_st, v_sh, o_sb, o_st, o_sh};
+  return flash_fwd_launch(q, k, v, o, lse, B, Hq, Hkv, Tq, Tk, D, D, st, causal, window, q_offset, scale, nullptr, nullptr, err, stream);
+}
+
+// Causal (optionally windowed) attention with the distance penalty r1[h] ln(1 + r2[h] (i - j)) taken off the scores; query and
+// key size dk and value size dv up to 128 (multiples of 8).  strides: (batch, row, head) of q, k, v, o.
+extern "C" TYR_EXPORT int tyr_flash_fwd_biased(const void* q, const void* k, const void* v, void* o, const float* r1,
+                                               const float* r2, int B, int Hq, int Hkv, int T, int dk, int dv,
+                                               const long long* strides, int window, float scale, int* err, void* stream) {
+  if (dk <= 0 || dv <= 0 || dk > ATT_D || dv > ATT_D || (dk & 7) || (dv & 7) || r1 == nullptr || r2 == nullptr || scale <= 0.f) return -1;
+  return flash_fwd_launch(q, k, v, o, nullptr, B, Hq, Hkv, T, T, dk, dv, strides, 1, window, 0, scale, r1, r2, err, stream);
 }

@@ -1,0 +1,191 @@
+// Attention pieces for any head size, fp32 or bf16, with a logarithmic distance penalty on the scores:
+//
+//   score(i, j) = scale q_i . k_j - r1_h ln(1 + r2_h (i - j)),   0 <= i - j < window.
+//
+//   * qk_norm_store: per-head RMSNorm of q and k (no rotation), v copied, rows of the padded batch written to the K/V store at
+//                    their own positions (plain or ring).
+//   * general:       one warp per (query, head), online softmax in fp32; reads keys from the prompt's own rows or from the store.
+//
+// The tensor-core forms are in attention_fwd.cu (prompts) and decode_attention.cu (one token); these kernels take the shapes and
+// the precision those do not.  Compiled without fast math.
+#include "common.cuh"
+
+namespace tyr {
+
+__device__ __forceinline__ float ag_load(const float* p) { return *p; }
+__device__ __forceinline__ float ag_load(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void ag_store(float* p, float v) { *p = v; }
+__device__ __forceinline__ void ag_store(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
+
+struct QkNormArgs {
+  const void* y;               // [B * S, ld]: q (H * dk) | k (G * dk) | v (G * dv); G = 0 when the layer has no keys of its own
+  long long ld;
+  const float *q_w, *k_w;      // [dk] (k_w unused when G == 0)
+  void* q_out;                 // [B * S, H, dkp]
+  void* k_out;                 // [B * S, G, dkp]
+  void* v_out;                 // [B * S, G, dvp] or null
+  void *k_store, *v_store;     // [B, G, cap, dkp / dvp] or null
+  const int* pos;              // position of token 0 of each row (nullable: 0)
+  const int* lens;             // tokens of each row (nullable: S)
+  int B, S, H, G, dk, dv, dkp, dvp, cap, ring;
+  float eps;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(256) qk_norm_store_kernel(QkNormArgs a) {
+  pdl_entry();
+  const int lane = threadIdx.x & 31;
+  const int heads = a.H + 2 * a.G;
+  const long long total = static_cast<long long>(a.B) * a.S * heads;
+  const long long nw = static_cast<long long>(gridDim.x) * 8;
+  for (long long i = blockIdx.x * 8LL + (threadIdx.x >> 5); i < total; i += nw) {
+    const int hd = static_cast<int>(i % heads);
+    const long long row = i / heads;
+    const int b = static_cast<int>(row / a.S), s = static_cast<int>(row % a.S);
+    const T* src = static_cast<const T*>(a.y) + row * a.ld;
+    const bool is_q = hd < a.H, is_v = hd >= a.H + a.G;
+    const int g = is_q ? hd : (is_v ? hd - a.H - a.G : hd - a.H);
+    const int d_in = is_v ? a.dv : a.dk, d_out = is_v ? a.dvp : a.dkp;
+    src += is_v ? static_cast<long long>(a.H + a.G) * a.dk + static_cast<long long>(g) * a.dv : static_cast<long long>(hd) * a.dk;
+    T* dst = is_q ? static_cast<T*>(a.q_out) + (row * a.H + g) * d_out
+                  : (is_v ? (a.v_out ? static_cast<T*>(a.v_out) + (row * a.G + g) * d_out : nullptr)
+                          : static_cast<T*>(a.k_out) + (row * a.G + g) * d_out);
+    T* slot = nullptr;
+    if (!is_q && a.k_store != nullptr) {
+      const int n = a.lens ? a.lens[b] : a.S;
+      const int p0 = a.pos ? a.pos[b] : 0;
+      const int p = p0 + s;
+      const bool keep = s < n && p >= 0 && (a.ring ? p0 + n - p <= a.cap : p < a.cap);     // a ring store keeps the last cap positions
+      if (keep)
+        slot = static_cast<T*>(is_v ? a.v_store : a.k_store) + ((static_cast<long long>(b) * a.G + g) * a.cap + (a.ring ? p % a.cap : p)) * d_out;
+    }
+    float rstd = 1.f;
+    if (!is_v) {
+      float ss = 0.f;
+      for (int d = lane; d < d_in; d += 32) {
+        const float v = ag_load(src + d);
+        ss += v * v;
+      }
+      rstd = 1.f / sqrtf(warp_sum(ss) / d_in + a.eps);
+    }
+    const float* w = is_q ? a.q_w : a.k_w;
+    for (int d = lane; d < d_out; d += 32) {
+      float v = d < d_in ? ag_load(src + d) : 0.f;
+      if (!is_v && d < d_in) v = v * rstd * w[d];
+      if (dst) ag_store(dst + d, v);
+      if (slot) ag_store(slot + d, v);
+    }
+  }
+}
+
+struct GeneralAttnArgs {
+  const void *q, *k, *v;       // q: [B, S, H, .]; k / v: [B, ., G, .] by (batch, position or slot, head) element strides
+  void* out;                   // [B, S, H, dv] contiguous
+  const int* pos;              // position of query 0 of each row (nullable: 0)
+  const float *r1, *r2;        // [H] distance penalty (nullable: none)
+  long long q_sb, q_ss, q_sh, k_sb, k_ss, k_sh, v_sb, v_ss, v_sh;
+  int B, S, H, G, dk, dv, cap, ring, window, keys;
+  float scale;
+  int* err;
+};
+constexpr int GA_WARPS = 4;
+constexpr int GA_DMAX = 256;
+
+template <typename T>
+__global__ void __launch_bounds__(GA_WARPS * 32) general_attention_kernel(GeneralAttnArgs a) {
+  __shared__ float sq[GA_WARPS][GA_DMAX];
+  __shared__ float sp[GA_WARPS][32];
+  pdl_entry();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const long long total = static_cast<long long>(a.B) * a.S * a.H;
+  const long long i = blockIdx.x * static_cast<long long>(GA_WARPS) + warp;
+  if (i >= total) return;
+  const int h = static_cast<int>(i % a.H);
+  const long long row = i / a.H;
+  const int b = static_cast<int>(row / a.S), s = static_cast<int>(row % a.S);
+  const int g = h / (a.H / a.G);
+  const int p = (a.pos ? a.pos[b] : 0) + s;
+  if (p < 0 || (!a.ring && p >= a.keys)) {         // a query without its own key in the store: report, leave the output
+    if (lane == 0) report_error(a.err, ERR_BOUNDS, p);
+    return;
+  }
+  const T* qp = static_cast<const T*>(a.q) + b * a.q_sb + s * a.q_ss + h * a.q_sh;
+  const T* kb = static_cast<const T*>(a.k) + b * a.k_sb + g * a.k_sh;
+  const T* vb = static_cast<const T*>(a.v) + b * a.v_sb + g * a.v_sh;
+  for (int d = lane; d < a.dk; d += 32) sq[warp][d] = ag_load(qp + d);
+  __syncwarp();
+  const float r1 = a.r1 ? a.r1[h] : 0.f, r2 = a.r1 ? a.r2[h] : 0.f;
+  int lo = a.window > 0 ? max(0, p - a.window + 1) : 0;
+  if (a.ring) lo = max(lo, p - a.cap + 1);
+  float m = -INFINITY, l = 0.f, acc[GA_DMAX / 32];
+#pragma unroll
+  for (int j = 0; j < GA_DMAX / 32; ++j) acc[j] = 0.f;
+  for (int base = lo; base <= p; base += 32) {
+    const int j = base + lane;
+    float sc = -INFINITY;
+    if (j <= p) {
+      const T* kr = kb + static_cast<long long>(a.ring ? j % a.cap : j) * a.k_ss;
+      float dot = 0.f;
+      for (int d = 0; d < a.dk; ++d) dot += sq[warp][d] * ag_load(kr + d);
+      sc = dot * a.scale - r1 * log1pf(r2 * static_cast<float>(p - j));
+    }
+    const float mn = fmaxf(m, warp_max(sc));
+    const float f = expf(m - mn), w = expf(sc - mn);
+    l = l * f + warp_sum(w);
+    m = mn;
+    sp[warp][lane] = w;
+    __syncwarp();
+#pragma unroll
+    for (int c = 0; c < GA_DMAX / 32; ++c) acc[c] *= f;
+    const int nk = min(32, p - base + 1);
+    for (int t = 0; t < nk; ++t) {
+      const float wt = sp[warp][t];
+      const T* vr = vb + static_cast<long long>(a.ring ? (base + t) % a.cap : base + t) * a.v_ss;
+#pragma unroll
+      for (int c = 0; c < GA_DMAX / 32; ++c)
+        if (lane + 32 * c < a.dv) acc[c] += wt * ag_load(vr + lane + 32 * c);
+    }
+    __syncwarp();
+  }
+  T* op = static_cast<T*>(a.out) + (row * a.H + h) * a.dv;
+#pragma unroll
+  for (int c = 0; c < GA_DMAX / 32; ++c)
+    if (lane + 32 * c < a.dv) ag_store(op + lane + 32 * c, acc[c] / l);
+}
+
+}  // namespace tyr
+
+using namespace tyr;
+
+extern "C" TYR_EXPORT int tyr_qk_norm_store(const void* y, long long ld, const float* q_w, const float* k_w, void* q_out, void* k_out,
+                                            void* v_out, void* k_store, void* v_store, const int* pos, const int* lens, int B, int S,
+                                            int H, int G, int dk, int dv, int dkp, int dvp, int cap, int ring, float eps, int dtype,
+                                            void* stream) {
+  if (B <= 0 || S <= 0 || H <= 0 || G < 0 || dk <= 0 || dkp < dk || dvp < dv || (G > 0 && dv <= 0)) return -1;
+  if ((k_store != nullptr) != (v_store != nullptr) || (k_store != nullptr && cap <= 0)) return -2;
+  QkNormArgs a{y, ld, q_w, k_w, q_out, k_out, v_out, k_store, v_store, pos, lens, B, S, H, G, dk, dv, dkp, dvp, cap, ring, eps};
+  const long long want = (static_cast<long long>(B) * S * (H + 2 * G) + 7) / 8;
+  const dim3 grid(static_cast<unsigned>(want < 148LL * 32 ? want : 148LL * 32));
+  return (int)(dtype == 1 ? launch_dependent(qk_norm_store_kernel<float>, grid, dim3(256), 0, (cudaStream_t)stream, a)
+                          : launch_dependent(qk_norm_store_kernel<__nv_bfloat16>, grid, dim3(256), 0, (cudaStream_t)stream, a));
+}
+
+// strides: (batch, position or slot, head) element strides of q, k, v.  `keys`: positions the plain form may read (prompt length
+// or capacity).  dk, dv <= 256.
+extern "C" TYR_EXPORT int tyr_general_attention(const void* q, const void* k, const void* v, void* out, const int* pos,
+                                                const float* r1, const float* r2, const long long* strides, int B, int S, int H,
+                                                int G, int dk, int dv, int cap, int ring, int window, int keys, float scale,
+                                                int dtype, int* err, void* stream) {
+  if (B <= 0 || S <= 0 || H <= 0 || G <= 0 || H % G || dk <= 0 || dv <= 0 || dk > GA_DMAX || dv > GA_DMAX) return -1;
+  if ((ring && cap <= 0) || (r1 != nullptr) != (r2 != nullptr)) return -2;
+  GeneralAttnArgs a;
+  a.q = q; a.k = k; a.v = v; a.out = out; a.pos = pos; a.r1 = r1; a.r2 = r2;
+  a.q_sb = strides[0]; a.q_ss = strides[1]; a.q_sh = strides[2];
+  a.k_sb = strides[3]; a.k_ss = strides[4]; a.k_sh = strides[5];
+  a.v_sb = strides[6]; a.v_ss = strides[7]; a.v_sh = strides[8];
+  a.B = B; a.S = S; a.H = H; a.G = G; a.dk = dk; a.dv = dv; a.cap = cap; a.ring = ring; a.window = window; a.keys = keys;
+  a.scale = scale; a.err = err;
+  const dim3 grid(static_cast<unsigned>((static_cast<long long>(B) * S * H + GA_WARPS - 1) / GA_WARPS)), block(GA_WARPS * 32);
+  return (int)(dtype == 1 ? launch_dependent(general_attention_kernel<float>, grid, block, 0, (cudaStream_t)stream, a)
+                          : launch_dependent(general_attention_kernel<__nv_bfloat16>, grid, block, 0, (cudaStream_t)stream, a));
+}

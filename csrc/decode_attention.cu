@@ -9,6 +9,10 @@
 // cannot race with readers.  Split partials {m, l, acc} go to a workspace; the last CTA to arrive for a
 // (batch, K/V head) combines them (atomic ticket, counter reset for the next launch).
 //
+// Each row of the batch has its own position.  Retained keys are walked by distance from the new token (a ring store by position
+// modulo its capacity), so a window may be smaller than the ring and a penalty r1_h ln(1 + r2_h distance) can be taken off the
+// scores (template parameter BIAS).  Key size DK and value size DV may differ.
+//
 // The reference takes the library SDPA over a sliced cache for this step (cc/include/tyr_attention.h:58-130,
 // Tyr/Inference/KVCache.lean:41-215).
 #include <cuda_bf16.h>
@@ -25,11 +29,13 @@ struct DecodeAttnArgs {
   const __nv_bfloat16* q;        // [B, Hq, D], batch stride q_bs, head stride D
   const __nv_bfloat16* k_new;    // [B, Hkv, D], batch stride kn_bs, head stride D
   const __nv_bfloat16* v_new;    // same strides (vn_bs)
-  __nv_bfloat16* k_cache;        // [B, Hkv, cap, D]
+  __nv_bfloat16* k_cache;        // [B, Hkv, cap, DK] and [B, Hkv, cap, DV]
   __nv_bfloat16* v_cache;
-  const int* pos;                // absolute position of the new token
-  __nv_bfloat16* out;            // [B, Hq, D] contiguous
-  float* part_acc;               // [B, Hq, splits, D]
+  const int* pos;                // absolute position of the new token of row b: pos[b * pos_stride]
+  int pos_stride;
+  const float *r1, *r2;          // [Hq] distance penalty (BIAS forms)
+  __nv_bfloat16* out;            // [B, Hq, DV] contiguous
+  float* part_acc;               // [B, Hq, splits, DV]
   float* part_ml;                // [B, Hq, splits, 2]
   int* counters;                 // [B * Hkv], zero on entry, zero on exit
   long long q_bs, kn_bs, vn_bs;
@@ -87,52 +93,62 @@ __device__ __forceinline__ uint32_t prmt(uint32_t a, uint32_t b, uint32_t sel) {
 //   O += P V  : M = heads, N = 8 channels, K = 16 keys.  Lane (g, t) loads 16 bytes (8 channels) of the four key rows
 //   {2t, 2t+1, 2t+8, 2t+9}; byte permutes pair the rows per channel.  The channel order of the accumulators is permuted
 //   (undone when they are written out): accumulator (c, e, u) of lane (g, t) is channel 64c + 16t + 8u + e of head g.
-template <int D, bool WIDE>
+template <int DK, int DV, bool WIDE, bool BIAS>
 __global__ void __launch_bounds__(kDecWarps * 32) decode_attention_kernel(DecodeAttnArgs a) {
   pdl_entry();
-  constexpr int NJ = D / 32;                     // 16-byte chunks per lane of a K (or Q) row
-  constexpr int NC = D / 64;                     // 64-channel blocks of a V row
+  constexpr int NJ = DK / 32;                    // 16-byte chunks per lane of a K (or Q) row
+  constexpr int NC = DV / 64;                    // 64-channel blocks of a V row
   constexpr int R = WIDE ? 2 : 1;                // query heads per lane: g, and g + 8 when more than 8 heads share a K/V head
   constexpr int GM = 8 * R;
   __shared__ float s_m[kDecWarps][GM], s_l[kDecWarps][GM];
-  __shared__ float s_acc[kDecWarps][GM][D];
+  __shared__ float s_acc[kDecWarps][GM][DV];
   __shared__ int s_ticket;
 
   const int split = blockIdx.x, hkv = blockIdx.y, b = blockIdx.z;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int g = lane >> 2, t = lane & 3;
   const int G = a.Hq / a.Hkv;
-  const int pos = *a.pos;
+  const int pos = a.pos[b * a.pos_stride];
   if (pos < 0 || (!a.ring && pos >= a.cap)) {    // position outside the store: report, leave the output untouched
     if (tid == 0) report_error(a.err, ERR_BOUNDS, pos);
     return;
   }
-  int start, n_keys, slot_new;
-  if (a.ring) {
-    start = 0;
-    n_keys = pos + 1 < a.cap ? pos + 1 : a.cap;
-    slot_new = pos % a.cap;
-  } else {
-    start = (a.window > 0 && pos + 1 > a.window) ? pos + 1 - a.window : 0;
-    n_keys = pos + 1 - start;
-    slot_new = pos;
-  }
+  // key index i of 0 .. n_keys - 1 is at distance n_keys - 1 - i from the new token and in slot slot0 + i (modulo cap)
+  int n_keys = pos + 1;
+  if (a.window > 0 && n_keys > a.window) n_keys = a.window;
+  if (a.ring && n_keys > a.cap) n_keys = a.cap;
+  const int start = pos + 1 - n_keys;
+  const int slot0 = a.ring ? start % a.cap : start;
+  const int slot_new = a.ring ? pos % a.cap : pos;
+  auto slot_of = [&](int i) {
+    int sl = slot0 + i;
+    return sl >= a.cap ? sl - a.cap : sl;
+  };
   int chunk = (n_keys + a.splits - 1) / a.splits;
   chunk = (chunk + 63) & ~63;
-  const int lo = start + split * chunk;
+  const int lo = split * chunk;
   int hi = lo + chunk;
-  if (hi > start + n_keys) hi = start + n_keys;
+  if (hi > n_keys) hi = n_keys;
 
-  const long long kv_base = (static_cast<long long>(b) * a.Hkv + hkv) * a.cap * D;
-  const __nv_bfloat16* kc = a.k_cache + kv_base;
-  const __nv_bfloat16* vc = a.v_cache + kv_base;
-  const __nv_bfloat16* kn = a.k_new + b * a.kn_bs + static_cast<long long>(hkv) * D;
-  const __nv_bfloat16* vn = a.v_new + b * a.vn_bs + static_cast<long long>(hkv) * D;
+  const long long kv_row = (static_cast<long long>(b) * a.Hkv + hkv) * a.cap;
+  __nv_bfloat16* kc = a.k_cache + kv_row * DK;
+  __nv_bfloat16* vc = a.v_cache + kv_row * DV;
+  const __nv_bfloat16* kn = a.k_new + b * a.kn_bs + static_cast<long long>(hkv) * DK;
+  const __nv_bfloat16* vn = a.v_new + b * a.vn_bs + static_cast<long long>(hkv) * DV;
 
   if (a.append && split == 0) {                  // fused append; nobody reads this slot from the store in this launch
-    for (int i = tid; i < D / 8; i += kDecWarps * 32) {
-      reinterpret_cast<uint4*>(a.k_cache + kv_base + static_cast<long long>(slot_new) * D)[i] = reinterpret_cast<const uint4*>(kn)[i];
-      reinterpret_cast<uint4*>(a.v_cache + kv_base + static_cast<long long>(slot_new) * D)[i] = reinterpret_cast<const uint4*>(vn)[i];
+    for (int i = tid; i < DK / 8; i += kDecWarps * 32)
+      reinterpret_cast<uint4*>(kc + static_cast<long long>(slot_new) * DK)[i] = reinterpret_cast<const uint4*>(kn)[i];
+    for (int i = tid; i < DV / 8; i += kDecWarps * 32)
+      reinterpret_cast<uint4*>(vc + static_cast<long long>(slot_new) * DV)[i] = reinterpret_cast<const uint4*>(vn)[i];
+  }
+  float r1[R], r2[R];                            // penalty of heads g and g + 8, in log2 units
+  if constexpr (BIAS) {
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      const int head = g + 8 * r < G ? g + 8 * r : 0;
+      r1[r] = a.r1[hkv * G + head];
+      r2[r] = a.r2[hkv * G + head];
     }
   }
 
@@ -140,7 +156,7 @@ __global__ void __launch_bounds__(kDecWarps * 32) decode_attention_kernel(Decode
 #pragma unroll
   for (int r = 0; r < R; ++r) {
     const int head = g + 8 * r;
-    const __nv_bfloat16* qrow = a.q + b * a.q_bs + static_cast<long long>(hkv * G + (head < G ? head : 0)) * D;
+    const __nv_bfloat16* qrow = a.q + b * a.q_bs + static_cast<long long>(hkv * G + (head < G ? head : 0)) * DK;
 #pragma unroll
     for (int j = 0; j < NJ; ++j) qf[r][j] = head < G ? *reinterpret_cast<const uint4*>(qrow + 32 * j + 8 * t) : make_uint4(0u, 0u, 0u, 0u);
   }
@@ -163,7 +179,7 @@ __global__ void __launch_bounds__(kDecWarps * 32) decode_attention_kernel(Decode
     for (int tile = 0; tile < 2; ++tile) {
       int row = base + 8 * tile + g;
       row = row < hi ? row : hi - 1;             // clamped rows are masked below
-      const __nv_bfloat16* krow = (row == slot_new) ? kn : kc + static_cast<long long>(row) * D;
+      const __nv_bfloat16* krow = (row == n_keys - 1) ? kn : kc + static_cast<long long>(slot_of(row)) * DK;
       uint4 kf[NJ];
 #pragma unroll
       for (int j = 0; j < NJ; ++j) kf[j] = *reinterpret_cast<const uint4*>(krow + 32 * j + 8 * t);
@@ -180,6 +196,14 @@ __global__ void __launch_bounds__(kDecWarps * 32) decode_attention_kernel(Decode
         s[1][tile][0] = key0 < hi ? c_hi[0] * a.scale_log2 : -INFINITY;
         s[1][tile][1] = key0 + 1 < hi ? c_hi[1] * a.scale_log2 : -INFINITY;
       }
+      if constexpr (BIAS) {
+        const float n0 = static_cast<float>(max(n_keys - 1 - key0, 0)), n1 = static_cast<float>(max(n_keys - 2 - key0, 0));
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+          s[r][tile][0] -= r1[r] * __log2f(1.f + r2[r] * n0);
+          s[r][tile][1] -= r1[r] * __log2f(1.f + r2[r] * n1);
+        }
+      }
     }
     // ---- V rows of this lane's four keys (issued before the softmax arithmetic so the loads overlap it) ----
     const __nv_bfloat16* vrow[4];
@@ -187,7 +211,7 @@ __global__ void __launch_bounds__(kDecWarps * 32) decode_attention_kernel(Decode
     for (int i = 0; i < 4; ++i) {
       int row = base + 2 * t + (i & 1) + 8 * (i >> 1);
       row = row < hi ? row : hi - 1;
-      vrow[i] = (row == slot_new) ? vn : vc + static_cast<long long>(row) * D;
+      vrow[i] = (row == n_keys - 1) ? vn : vc + static_cast<long long>(slot_of(row)) * DV;
     }
     uint4 vf[NC][4];
 #pragma unroll
@@ -256,8 +280,8 @@ __global__ void __launch_bounds__(kDecWarps * 32) decode_attention_kernel(Decode
   // ---- combine the four warps -------------------------------------------------------------------------------
   __syncthreads();
   const int hq0 = hkv * G;
-  for (int i = tid; i < G * D; i += kDecWarps * 32) {
-    const int g = i / D, d = i - g * D;
+  for (int i = tid; i < G * DV; i += kDecWarps * 32) {
+    const int g = i / DV, d = i - g * DV;
     float M = -INFINITY;
 #pragma unroll
     for (int w = 0; w < kDecWarps; ++w) M = fmaxf(M, s_m[w][g]);
@@ -272,9 +296,9 @@ __global__ void __launch_bounds__(kDecWarps * 32) decode_attention_kernel(Decode
     }
     const long long row = static_cast<long long>(b) * a.Hq + hq0 + g;
     if (a.splits == 1) {
-      a.out[row * D + d] = __float2bfloat16((L > 0.f ? A / L : 0.f) * decode_gate(a, b, hq0 + g, d));
+      a.out[row * DV + d] = __float2bfloat16((L > 0.f ? A / L : 0.f) * decode_gate(a, b, hq0 + g, d));
     } else {
-      a.part_acc[(row * a.splits + split) * D + d] = A;
+      a.part_acc[(row * a.splits + split) * DV + d] = A;
       if (d == 0) {
         a.part_ml[(row * a.splits + split) * 2] = M;
         a.part_ml[(row * a.splits + split) * 2 + 1] = L;
@@ -290,8 +314,8 @@ __global__ void __launch_bounds__(kDecWarps * 32) decode_attention_kernel(Decode
   __syncthreads();
   if (s_ticket != a.splits - 1) return;
   __threadfence();
-  for (int i = tid; i < G * D; i += kDecWarps * 32) {
-    const int g = i / D, d = i - g * D;
+  for (int i = tid; i < G * DV; i += kDecWarps * 32) {
+    const int g = i / DV, d = i - g * DV;
     const long long row = static_cast<long long>(b) * a.Hq + hq0 + g;
     float M = -INFINITY;
     for (int sp = 0; sp < a.splits; ++sp) M = fmaxf(M, __ldcg(&a.part_ml[(row * a.splits + sp) * 2]));
@@ -300,10 +324,10 @@ __global__ void __launch_bounds__(kDecWarps * 32) decode_attention_kernel(Decode
       for (int sp = 0; sp < a.splits; ++sp) {
         const float f = exp2f(__ldcg(&a.part_ml[(row * a.splits + sp) * 2]) - M);
         L += __ldcg(&a.part_ml[(row * a.splits + sp) * 2 + 1]) * f;
-        A += __ldcg(&a.part_acc[(row * a.splits + sp) * D + d]) * f;
+        A += __ldcg(&a.part_acc[(row * a.splits + sp) * DV + d]) * f;
       }
     }
-    a.out[row * D + d] = __float2bfloat16((L > 0.f ? A / L : 0.f) * decode_gate(a, b, hq0 + g, d));
+    a.out[row * DV + d] = __float2bfloat16((L > 0.f ? A / L : 0.f) * decode_gate(a, b, hq0 + g, d));
   }
   if (tid == 0) a.counters[b * a.Hkv + hkv] = 0;
 }
@@ -315,40 +339,23 @@ extern "C" TYR_EXPORT long long tyr_decode_attention_workspace_bytes(int B, int 
   return static_cast<long long>(B) * Hq * splits * (D + 2) * 4 + static_cast<long long>(B) * Hkv * 4;
 }
 
-extern "C" TYR_EXPORT int tyr_decode_attention_gated(const void* q, const void* k_new, const void* v_new, void* k_cache,
-                                                     void* v_cache, const void* pos, void* out, void* workspace, long long q_bs,
-                                                     long long kn_bs, long long vn_bs, int B, int Hq, int Hkv, int D, int cap,
-                                                     int ring, int window, int splits, int append, float scale, const void* gate,
-                                                     long long gate_bs, long long gate_hs, int gate_mode, void* err, void* stream);
-
-// `workspace` must be zero-filled once after allocation (the kernel leaves the counters at zero).
-extern "C" TYR_EXPORT int tyr_decode_attention(const void* q, const void* k_new, const void* v_new, void* k_cache, void* v_cache,
-                                               const void* pos, void* out, void* workspace, long long q_bs, long long kn_bs,
-                                               long long vn_bs, int B, int Hq, int Hkv, int D, int cap, int ring, int window,
-                                               int splits, int append, float scale, void* err, void* stream) {
-  return tyr_decode_attention_gated(q, k_new, v_new, k_cache, v_cache, pos, out, workspace, q_bs, kn_bs, vn_bs, B, Hq, Hkv, D, cap,
-                                    ring, window, splits, append, scale, nullptr, 0, 0, 0, err, stream);
-}
-
-// The same with an output gate folded into the final write (see DecodeAttnArgs::gate).
-extern "C" TYR_EXPORT int tyr_decode_attention_gated(const void* q, const void* k_new, const void* v_new, void* k_cache,
-                                                     void* v_cache, const void* pos, void* out, void* workspace, long long q_bs,
-                                                     long long kn_bs, long long vn_bs, int B, int Hq, int Hkv, int D, int cap,
-                                                     int ring, int window, int splits, int append, float scale, const void* gate,
-                                                     long long gate_bs, long long gate_hs, int gate_mode, void* err, void* stream) {
+static int decode_attention_launch(const void* q, const void* k_new, const void* v_new, void* k_cache, void* v_cache, const void* pos,
+                                   int pos_stride, void* out, void* workspace, long long q_bs, long long kn_bs, long long vn_bs, int B,
+                                   int Hq, int Hkv, int DK, int DV, int cap, int ring, int window, int splits, int append, float scale,
+                                   const void* gate, long long gate_bs, long long gate_hs, int gate_mode, const float* r1,
+                                   const float* r2, void* err, void* stream) {
   using namespace tyr;
   if (gate_mode < 0 || gate_mode > 2 || (gate_mode != 0 && gate == nullptr)) return -5;
   if (B <= 0 || Hq <= 0 || Hkv <= 0 || Hq % Hkv != 0 || Hq / Hkv > 16 || cap <= 0 || splits < 1 || splits > 64) return -1;
-  if (D != 64 && D != 128 && D != 256) return -2;
   const bool wide = Hq / Hkv > 8;
-  if (wide && D == 256) return -4;                                  // 16 heads x 256 channels of accumulators do not fit a warp
   if ((q_bs | kn_bs | vn_bs) & 7) return -3;                       // 16-byte rows
+  if ((r1 != nullptr) != (r2 != nullptr)) return -6;
   DecodeAttnArgs a;
   a.q = (const __nv_bfloat16*)q; a.k_new = (const __nv_bfloat16*)k_new; a.v_new = (const __nv_bfloat16*)v_new;
   a.k_cache = (__nv_bfloat16*)k_cache; a.v_cache = (__nv_bfloat16*)v_cache;
-  a.pos = (const int*)pos; a.out = (__nv_bfloat16*)out;
+  a.pos = (const int*)pos; a.pos_stride = pos_stride; a.r1 = r1; a.r2 = r2; a.out = (__nv_bfloat16*)out;
   a.part_acc = (float*)workspace;
-  a.part_ml = a.part_acc + static_cast<long long>(B) * Hq * splits * D;
+  a.part_ml = a.part_acc + static_cast<long long>(B) * Hq * splits * DV;
   a.counters = (int*)(a.part_ml + static_cast<long long>(B) * Hq * splits * 2);
   a.q_bs = q_bs; a.kn_bs = kn_bs; a.vn_bs = vn_bs;
   a.B = B; a.Hq = Hq; a.Hkv = Hkv; a.cap = cap; a.ring = ring; a.window = window; a.splits = splits; a.append = append;
@@ -358,9 +365,47 @@ extern "C" TYR_EXPORT int tyr_decode_attention_gated(const void* q, const void* 
   const dim3 grid(splits, Hkv, B);
   const cudaStream_t st = (cudaStream_t)stream;
   const dim3 block(kDecWarps * 32);
-  if (D == 64 && !wide) return (int)launch_dependent(decode_attention_kernel<64, false>, grid, block, 0, st, a);
-  if (D == 64) return (int)launch_dependent(decode_attention_kernel<64, true>, grid, block, 0, st, a);
-  if (D == 128 && !wide) return (int)launch_dependent(decode_attention_kernel<128, false>, grid, block, 0, st, a);
-  if (D == 128) return (int)launch_dependent(decode_attention_kernel<128, true>, grid, block, 0, st, a);
-  return (int)launch_dependent(decode_attention_kernel<256, false>, grid, block, 0, st, a);
+  const bool bias = r1 != nullptr;
+#define TYR_DEC(DK_, DV_, WIDE_, BIAS_)                                  \
+  if (DK == DK_ && DV == DV_ && wide == WIDE_ && bias == BIAS_)         \
+    return (int)launch_dependent(decode_attention_kernel<DK_, DV_, WIDE_, BIAS_>, grid, block, 0, st, a);
+  TYR_DEC(64, 64, false, false) TYR_DEC(64, 64, true, false)
+  TYR_DEC(128, 128, false, false) TYR_DEC(128, 128, true, false)
+  TYR_DEC(256, 256, false, false)                                  // 16 heads x 256 channels of accumulators do not fit a warp
+  TYR_DEC(64, 64, false, true) TYR_DEC(64, 64, true, true)
+  TYR_DEC(128, 128, false, true) TYR_DEC(128, 128, true, true)
+  TYR_DEC(64, 128, false, true) TYR_DEC(64, 128, true, true)
+  TYR_DEC(128, 64, false, true) TYR_DEC(128, 64, true, true)
+#undef TYR_DEC
+  return -2;
+}
+
+// `workspace` must be zero-filled once after allocation (the kernel leaves the counters at zero).  An output gate can be folded
+// into the final write (see DecodeAttnArgs::gate).
+extern "C" TYR_EXPORT int tyr_decode_attention_gated(const void* q, const void* k_new, const void* v_new, void* k_cache,
+                                                     void* v_cache, const void* pos, void* out, void* workspace, long long q_bs,
+                                                     long long kn_bs, long long vn_bs, int B, int Hq, int Hkv, int D, int cap,
+                                                     int ring, int window, int splits, int append, float scale, const void* gate,
+                                                     long long gate_bs, long long gate_hs, int gate_mode, void* err, void* stream) {
+  return decode_attention_launch(q, k_new, v_new, k_cache, v_cache, pos, 0, out, workspace, q_bs, kn_bs, vn_bs, B, Hq, Hkv, D, D, cap,
+                                 ring, window, splits, append, scale, gate, gate_bs, gate_hs, gate_mode, nullptr, nullptr, err, stream);
+}
+
+extern "C" TYR_EXPORT int tyr_decode_attention(const void* q, const void* k_new, const void* v_new, void* k_cache, void* v_cache,
+                                               const void* pos, void* out, void* workspace, long long q_bs, long long kn_bs,
+                                               long long vn_bs, int B, int Hq, int Hkv, int D, int cap, int ring, int window,
+                                               int splits, int append, float scale, void* err, void* stream) {
+  return tyr_decode_attention_gated(q, k_new, v_new, k_cache, v_cache, pos, out, workspace, q_bs, kn_bs, vn_bs, B, Hq, Hkv, D, cap,
+                                    ring, window, splits, append, scale, nullptr, 0, 0, 0, err, stream);
+}
+
+// Distance penalty r1[h] ln(1 + r2[h] n) on the scores; own position per row (pos_stride 1) or one for all (0); DK, DV in {64, 128}.
+extern "C" TYR_EXPORT int tyr_decode_attention_biased(const void* q, const void* k_new, const void* v_new, void* k_cache,
+                                                      void* v_cache, const void* pos, int pos_stride, void* out, void* workspace,
+                                                      long long q_bs, long long kn_bs, long long vn_bs, int B, int Hq, int Hkv, int DK,
+                                                      int DV, int cap, int ring, int window, int splits, int append, float scale,
+                                                      const float* r1, const float* r2, void* err, void* stream) {
+  if (r1 == nullptr || r2 == nullptr) return -6;
+  return decode_attention_launch(q, k_new, v_new, k_cache, v_cache, pos, pos_stride, out, workspace, q_bs, kn_bs, vn_bs, B, Hq, Hkv, DK,
+                                 DV, cap, ring, window, splits, append, scale, nullptr, 0, 0, 0, r1, r2, err, stream);
 }

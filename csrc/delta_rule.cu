@@ -175,7 +175,7 @@ gdr_decode_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
                        const float* __restrict__ beta, float* __restrict__ state, __nv_bfloat16* __restrict__ out,
                        int Hk, int Hv, long long q_bstride, long long v_bstride,
                        const __nv_bfloat16* __restrict__ z, long long z_bstride, const __nv_bfloat16* __restrict__ norm_w,
-                       float norm_eps, int* err) {
+                       float norm_eps, int round_o, int* err) {
   constexpr int DV = 128, RG = 8, RPT = DK / RG;
   constexpr uint32_t kBytes = DK * DV * 4, kPiece = kBytes / 4;
   extern __shared__ __align__(128) uint8_t gdr_smem[];
@@ -283,7 +283,8 @@ gdr_decode_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
       float ssq = 0.f;
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
-        o[c] = __bfloat162float(__float2bfloat16(o[c] * qn));
+        o[c] *= qn;
+        if (round_o) o[c] = __bfloat162float(__float2bfloat16(o[c]));    // as separate kernels with a bf16 read-out see it
         ssq += o[c] * o[c];
       }
       ssq = warp_sum(ssq);
@@ -354,10 +355,14 @@ gdn_conv_gates_kernel(const __nv_bfloat16* __restrict__ mixed, const __nv_bfloat
 // come in as fp32.  What is left is a recurrence over the chunks through the [dk, dv] state S,
 //     v_new = u_i - w_i S;   out_i = qg_i S + intra_i v_new;   S <- exp(g_last_i) S + kd_i^T v_new,
 // which the reference runs as a host loop of five small launches per chunk (cc/src/tyr_qwen35.cpp:89-110).  Here one CTA
-// walks all chunks of one (batch, head, 64-column slice of dv): S lives in registers as the accumulator of the last product
-// (each of the 4 warps owns 32 of the 128 state rows) and is mirrored into shared memory as the B operand of the first two;
-// all five products run on tensor cores in TF32 (mma.sync m16n8k8, fp32 accumulate).  The chunk inputs are staged with
-// cp.async in two groups so that the loads of w / qg for the next chunk overlap the last two products of this one.
+// walks all chunks of one (batch, head, 64-column slice of dv) with two groups of four warps: the first computes w_i S and
+// v_new and keeps S in registers as the accumulator of kd_i^T v_new (each warp owns 32 of the 128 state rows; S is mirrored into
+// shared memory as a B operand), the second computes qg_i S and adds intra_i v_new.  The products run on tensor cores with
+// mma.sync m16n8k8 and fp32 accumulation, either in TF32 or (EXACT) with every operand split into two TF32 terms and three
+// products, which keeps about 21 bits of each operand.  The chunk inputs are staged with cp.async in two groups so that the
+// loads of w / qg for the next chunk overlap the last two products of this one.
+//
+// Key sizes below 128 are padded with zero columns by the prepare kernel; value columns past dv hold zeros.
 // ------------------------------------------------------------------------------------------------------------------
 constexpr int GC_C = 64;       // chunk length
 constexpr int GC_DK = 128;     // key dim
@@ -399,30 +404,57 @@ __device__ __forceinline__ void stage_tile(float* dst, const float* src, int row
   }
 }
 
-__global__ void __launch_bounds__(128, 1)
+// One tensor-core operand element, as TF32 (EXACT: leading and trailing TF32 terms).
+template <bool EXACT>
+struct Tf32Op {
+  uint32_t hi, lo;
+  __device__ __forceinline__ explicit Tf32Op(float x) {
+    hi = __float_as_uint(x);
+    lo = 0;
+    if constexpr (EXACT) {
+      hi = (hi + 0x1000u) & 0xffffe000u;            // round to the 10 stored mantissa bits
+      lo = __float_as_uint(x - __uint_as_float(hi));
+    }
+  }
+};
+template <bool EXACT>
+__device__ __forceinline__ void mma_op(float (&c)[4], const Tf32Op<EXACT> (&a)[4], const Tf32Op<EXACT>& b0, const Tf32Op<EXACT>& b1) {
+  if constexpr (EXACT) {
+    mma_tf32(c, a[0].lo, a[1].lo, a[2].lo, a[3].lo, b0.hi, b1.hi);
+    mma_tf32(c, a[0].hi, a[1].hi, a[2].hi, a[3].hi, b0.lo, b1.lo);
+  }
+  mma_tf32(c, a[0].hi, a[1].hi, a[2].hi, a[3].hi, b0.hi, b1.hi);
+}
+__device__ __forceinline__ void store_pair(__nv_bfloat16* p, float x, float y) { *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(x, y); }
+__device__ __forceinline__ void store_pair(float* p, float x, float y) { *reinterpret_cast<float2*>(p) = make_float2(x, y); }
+
+// `dv` columns of the state and the output; `u` has rows of dvp = dv rounded up to 64 columns.
+template <bool EXACT, typename OutT>
+__global__ void __launch_bounds__(256, 1)
 gdr_chunk_scan_kernel(const float* __restrict__ u, const float* __restrict__ w, const float* __restrict__ qg,
                       const float* __restrict__ kd, const float* __restrict__ intra, const float* __restrict__ glast,
-                      const float* __restrict__ state_in, float* __restrict__ state_out, __nv_bfloat16* __restrict__ out, int n,
-                      int dv, int seq, int Hv) {
+                      const float* __restrict__ state_in, float* __restrict__ state_out, OutT* __restrict__ out, int n,
+                      int dk, int dv, int dvp, int seq, int Hv) {
+  using Op = Tf32Op<EXACT>;
   extern __shared__ __align__(16) uint8_t gdr_smem_raw[];
   GdrChunkSmem& sm = *reinterpret_cast<GdrChunkSmem*>(gdr_smem_raw);
   const int bh = blockIdx.y;
   const int col0 = blockIdx.x * GC_DVS;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int grp = threadIdx.x >> 7, warp = (threadIdx.x >> 5) & 3, lane = threadIdx.x & 31;
   const int g = lane >> 2, t = lane & 3;
   const long long chunk_k = static_cast<long long>(GC_C) * GC_DK;      // floats per chunk of w / qg / kd
   const float* w_p = w + static_cast<long long>(bh) * n * chunk_k;
   const float* q_p = qg + static_cast<long long>(bh) * n * chunk_k;
   const float* kd_p = kd + static_cast<long long>(bh) * n * chunk_k;
   const float* in_p = intra + static_cast<long long>(bh) * n * GC_C * GC_C;
-  const float* u_p = u + static_cast<long long>(bh) * n * GC_C * dv + col0;
-  // output rows go straight to the [B, S, Hv, dv] bf16 layout of the layer (rows past the sequence end are dropped)
-  __nv_bfloat16* o_p = out + (static_cast<long long>(bh / Hv) * seq * Hv + (bh % Hv)) * dv + col0;
+  const float* u_p = u + static_cast<long long>(bh) * n * GC_C * dvp + col0;
+  // output rows go straight to the [B, S, Hv, dv] layout of the layer (rows past the sequence end are dropped)
+  OutT* o_p = out + (static_cast<long long>(bh / Hv) * seq * Hv + (bh % Hv)) * dv + col0;
 
-  // state rows [32 warp, 32 warp + 32) x 64 columns as two m-tiles x eight n-tiles of accumulators
+  // group 0: state rows [32 warp, 32 warp + 32) x 64 columns as two m-tiles x eight n-tiles of accumulators
   float S[2][8][4];
-  {
-    const float* si = state_in ? state_in + (static_cast<long long>(bh) * GC_DK) * dv + col0 : nullptr;
+  if (grp == 0) {
+    const float* si = state_in ? state_in + (static_cast<long long>(bh) * dk) * dv + col0 : nullptr;
 #pragma unroll
     for (int mt = 0; mt < 2; ++mt)
 #pragma unroll
@@ -431,7 +463,7 @@ gdr_chunk_scan_kernel(const float* __restrict__ u, const float* __restrict__ w, 
         for (int h2 = 0; h2 < 2; ++h2) {
           const int r = warp * 32 + mt * 16 + g + h2 * 8, c = nt * 8 + 2 * t;
           float2 v = make_float2(0.f, 0.f);
-          if (si) v = *reinterpret_cast<const float2*>(si + static_cast<long long>(r) * dv + c);
+          if (si && r < dk && col0 + c < dv) v = *reinterpret_cast<const float2*>(si + static_cast<long long>(r) * dv + c);
           S[mt][nt][2 * h2] = v.x;
           S[mt][nt][2 * h2 + 1] = v.y;
           *reinterpret_cast<float2*>(&sm.s[r * GC_LDS + c]) = v;
@@ -441,42 +473,37 @@ gdr_chunk_scan_kernel(const float* __restrict__ u, const float* __restrict__ w, 
   stage_tile(sm.q, q_p, GC_C, GC_DK, GC_LDW);
   cp_async_commit();
 
+  const int ar = warp * 16 + g;
   for (int i = 0; i < n; ++i) {
     stage_tile(sm.kd, kd_p + i * chunk_k, GC_C, GC_DK, GC_LDT);
     stage_tile(sm.intra, in_p + static_cast<long long>(i) * GC_C * GC_C, GC_C, GC_C, GC_LDI);
     cp_async_commit();
     cp_async_wait<1>();            // w_i, qg_i landed (this thread's copies); the barrier publishes everyone's and S
     __syncthreads();
-    // ---- X = w_i S, Y = qg_i S : warp rows [16 warp, +16), K = dk
-    float X[8][4], Y[8][4];
+    // ---- group 0: X = w_i S, group 1: X = qg_i S; warp rows [16 warp, +16), K = dk
+    float X[8][4];
 #pragma unroll
     for (int nt = 0; nt < 8; ++nt)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) X[nt][e] = Y[nt][e] = 0.f;
-    const int ar = warp * 16 + g;
-#pragma unroll 4
+      for (int e = 0; e < 4; ++e) X[nt][e] = 0.f;
+    const float* A = grp == 0 ? sm.w : sm.q;
+#pragma unroll 2
     for (int kk = 0; kk < GC_DK / 8; ++kk) {
       const int kc = kk * 8 + t;
-      const uint32_t wa0 = __float_as_uint(sm.w[ar * GC_LDW + kc]), wa1 = __float_as_uint(sm.w[(ar + 8) * GC_LDW + kc]);
-      const uint32_t wa2 = __float_as_uint(sm.w[ar * GC_LDW + kc + 4]), wa3 = __float_as_uint(sm.w[(ar + 8) * GC_LDW + kc + 4]);
-      const uint32_t qa0 = __float_as_uint(sm.q[ar * GC_LDW + kc]), qa1 = __float_as_uint(sm.q[(ar + 8) * GC_LDW + kc]);
-      const uint32_t qa2 = __float_as_uint(sm.q[ar * GC_LDW + kc + 4]), qa3 = __float_as_uint(sm.q[(ar + 8) * GC_LDW + kc + 4]);
+      const Op a[4] = {Op(A[ar * GC_LDW + kc]), Op(A[(ar + 8) * GC_LDW + kc]), Op(A[ar * GC_LDW + kc + 4]), Op(A[(ar + 8) * GC_LDW + kc + 4])};
 #pragma unroll
-      for (int nt = 0; nt < 8; ++nt) {
-        const uint32_t b0 = __float_as_uint(sm.s[kc * GC_LDS + nt * 8 + g]), b1 = __float_as_uint(sm.s[(kc + 4) * GC_LDS + nt * 8 + g]);
-        mma_tf32(X[nt], wa0, wa1, wa2, wa3, b0, b1);
-        mma_tf32(Y[nt], qa0, qa1, qa2, qa3, b0, b1);
-      }
+      for (int nt = 0; nt < 8; ++nt)
+        mma_op<EXACT>(X[nt], a, Op(sm.s[kc * GC_LDS + nt * 8 + g]), Op(sm.s[(kc + 4) * GC_LDS + nt * 8 + g]));
     }
     // ---- v_new = u_i - X  -> shared memory (B operand of the next two products)
-    {
-      const float* ui = u_p + static_cast<long long>(i) * GC_C * dv;
+    if (grp == 0) {
+      const float* ui = u_p + static_cast<long long>(i) * GC_C * dvp;
 #pragma unroll
       for (int nt = 0; nt < 8; ++nt)
 #pragma unroll
         for (int h2 = 0; h2 < 2; ++h2) {
           const int r = ar + h2 * 8, c = nt * 8 + 2 * t;
-          const float2 uu = *reinterpret_cast<const float2*>(ui + static_cast<long long>(r) * dv + c);
+          const float2 uu = *reinterpret_cast<const float2*>(ui + static_cast<long long>(r) * dvp + c);
           *reinterpret_cast<float2*>(&sm.v[r * GC_LDS + c]) = make_float2(uu.x - X[nt][2 * h2], uu.y - X[nt][2 * h2 + 1]);
         }
     }
@@ -487,77 +514,74 @@ gdr_chunk_scan_kernel(const float* __restrict__ u, const float* __restrict__ w, 
       stage_tile(sm.q, q_p + (i + 1) * chunk_k, GC_C, GC_DK, GC_LDW);
     }
     cp_async_commit();
-    // ---- out_i = Y + intra_i v_new : K = chunk
+    if (grp == 1) {
+      // ---- out_i = qg_i S + intra_i v_new : K = chunk
 #pragma unroll 2
-    for (int kk = 0; kk < GC_C / 8; ++kk) {
-      const int kc = kk * 8 + t;
-      const uint32_t a0 = __float_as_uint(sm.intra[ar * GC_LDI + kc]), a1 = __float_as_uint(sm.intra[(ar + 8) * GC_LDI + kc]);
-      const uint32_t a2 = __float_as_uint(sm.intra[ar * GC_LDI + kc + 4]), a3 = __float_as_uint(sm.intra[(ar + 8) * GC_LDI + kc + 4]);
+      for (int kk = 0; kk < GC_C / 8; ++kk) {
+        const int kc = kk * 8 + t;
+        const Op a[4] = {Op(sm.intra[ar * GC_LDI + kc]), Op(sm.intra[(ar + 8) * GC_LDI + kc]), Op(sm.intra[ar * GC_LDI + kc + 4]),
+                         Op(sm.intra[(ar + 8) * GC_LDI + kc + 4])};
 #pragma unroll
-      for (int nt = 0; nt < 8; ++nt) {
-        const uint32_t b0 = __float_as_uint(sm.v[kc * GC_LDS + nt * 8 + g]), b1 = __float_as_uint(sm.v[(kc + 4) * GC_LDS + nt * 8 + g]);
-        mma_tf32(Y[nt], a0, a1, a2, a3, b0, b1);
+        for (int nt = 0; nt < 8; ++nt)
+          mma_op<EXACT>(X[nt], a, Op(sm.v[kc * GC_LDS + nt * 8 + g]), Op(sm.v[(kc + 4) * GC_LDS + nt * 8 + g]));
       }
-    }
-    {
 #pragma unroll
       for (int h2 = 0; h2 < 2; ++h2) {
         const int tok = i * GC_C + ar + h2 * 8;
         if (tok < seq) {
-          __nv_bfloat16* oi = o_p + static_cast<long long>(tok) * Hv * dv;
+          OutT* oi = o_p + static_cast<long long>(tok) * Hv * dv;
 #pragma unroll
           for (int nt = 0; nt < 8; ++nt)
-            *reinterpret_cast<uint32_t*>(oi + nt * 8 + 2 * t) = pack_bf16x2(Y[nt][2 * h2], Y[nt][2 * h2 + 1]);
+            if (col0 + nt * 8 < dv) store_pair(oi + nt * 8 + 2 * t, X[nt][2 * h2], X[nt][2 * h2 + 1]);
         }
       }
-    }
-    // ---- S <- exp(g_last) S + kd_i^T v_new : this warp's 32 state rows, K = chunk
-    const float e = glast[static_cast<long long>(bh) * n + i];
+    } else {
+      // ---- S <- exp(g_last) S + kd_i^T v_new : this warp's 32 state rows, K = chunk
+      const float e = glast[static_cast<long long>(bh) * n + i];
 #pragma unroll
-    for (int mt = 0; mt < 2; ++mt)
+      for (int mt = 0; mt < 2; ++mt)
 #pragma unroll
-      for (int nt = 0; nt < 8; ++nt)
+        for (int nt = 0; nt < 8; ++nt)
 #pragma unroll
-        for (int q4 = 0; q4 < 4; ++q4) S[mt][nt][q4] *= e;
-#pragma unroll 2
-    for (int kk = 0; kk < GC_C / 8; ++kk) {
-      const int kc = kk * 8 + t;
-      uint32_t a[2][4];
+          for (int q4 = 0; q4 < 4; ++q4) S[mt][nt][q4] *= e;
+#pragma unroll 1
+      for (int kk = 0; kk < GC_C / 8; ++kk) {
+        const int kc = kk * 8 + t, m = warp * 32 + g;       // A[m][k] = kd[k][m]
+        const float *k0 = sm.kd + kc * GC_LDT + m, *k4 = sm.kd + (kc + 4) * GC_LDT + m;
+        const Op a0[4] = {Op(k0[0]), Op(k0[8]), Op(k4[0]), Op(k4[8])};
+        const Op a1[4] = {Op(k0[16]), Op(k0[24]), Op(k4[16]), Op(k4[24])};
 #pragma unroll
-      for (int mt = 0; mt < 2; ++mt) {
-        const int m = warp * 32 + mt * 16 + g;          // A[m][k] = kd[k][m]
-        a[mt][0] = __float_as_uint(sm.kd[kc * GC_LDT + m]);
-        a[mt][1] = __float_as_uint(sm.kd[kc * GC_LDT + m + 8]);
-        a[mt][2] = __float_as_uint(sm.kd[(kc + 4) * GC_LDT + m]);
-        a[mt][3] = __float_as_uint(sm.kd[(kc + 4) * GC_LDT + m + 8]);
+        for (int nt = 0; nt < 8; ++nt) {
+          const Op b0(sm.v[kc * GC_LDS + nt * 8 + g]), b1(sm.v[(kc + 4) * GC_LDS + nt * 8 + g]);
+          mma_op<EXACT>(S[0][nt], a0, b0, b1);
+          mma_op<EXACT>(S[1][nt], a1, b0, b1);
+        }
       }
+      // mirror the new state for the next chunk's first products (nobody reads sm.s between the barrier above and the next one)
 #pragma unroll
-      for (int nt = 0; nt < 8; ++nt) {
-        const uint32_t b0 = __float_as_uint(sm.v[kc * GC_LDS + nt * 8 + g]), b1 = __float_as_uint(sm.v[(kc + 4) * GC_LDS + nt * 8 + g]);
-        mma_tf32(S[0][nt], a[0][0], a[0][1], a[0][2], a[0][3], b0, b1);
-        mma_tf32(S[1][nt], a[1][0], a[1][1], a[1][2], a[1][3], b0, b1);
-      }
+      for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+        for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+          for (int h2 = 0; h2 < 2; ++h2)
+            *reinterpret_cast<float2*>(&sm.s[(warp * 32 + mt * 16 + g + h2 * 8) * GC_LDS + nt * 8 + 2 * t]) =
+                make_float2(S[mt][nt][2 * h2], S[mt][nt][2 * h2 + 1]);
     }
-    // mirror the new state for the next chunk's first products (nobody reads sm.s between the barrier above and the next one)
-#pragma unroll
-    for (int mt = 0; mt < 2; ++mt)
-#pragma unroll
-      for (int nt = 0; nt < 8; ++nt)
-#pragma unroll
-        for (int h2 = 0; h2 < 2; ++h2)
-          *reinterpret_cast<float2*>(&sm.s[(warp * 32 + mt * 16 + g + h2 * 8) * GC_LDS + nt * 8 + 2 * t]) =
-              make_float2(S[mt][nt][2 * h2], S[mt][nt][2 * h2 + 1]);
     __syncthreads();               // kd, intra, v free for the next chunk's copies; S mirror complete
   }
-  float* so = state_out + (static_cast<long long>(bh) * GC_DK) * dv + col0;
+  if (grp == 0) {
+    float* so = state_out + (static_cast<long long>(bh) * dk) * dv + col0;
 #pragma unroll
-  for (int mt = 0; mt < 2; ++mt)
+    for (int mt = 0; mt < 2; ++mt)
 #pragma unroll
-    for (int nt = 0; nt < 8; ++nt)
+      for (int nt = 0; nt < 8; ++nt)
 #pragma unroll
-      for (int h2 = 0; h2 < 2; ++h2)
-        *reinterpret_cast<float2*>(so + static_cast<long long>(warp * 32 + mt * 16 + g + h2 * 8) * dv + nt * 8 + 2 * t) =
-            make_float2(S[mt][nt][2 * h2], S[mt][nt][2 * h2 + 1]);
+        for (int h2 = 0; h2 < 2; ++h2) {
+          const int r = warp * 32 + mt * 16 + g + h2 * 8, c = nt * 8 + 2 * t;
+          if (r < dk && col0 + c < dv)
+            *reinterpret_cast<float2*>(so + static_cast<long long>(r) * dv + c) = make_float2(S[mt][nt][2 * h2], S[mt][nt][2 * h2 + 1]);
+        }
+  }
 }
 
 // ------------------------------------------------------------------------------------------------------------------
@@ -572,7 +596,8 @@ gdr_chunk_scan_kernel(const float* __restrict__ u, const float* __restrict__ w, 
 //      its 64 unknowns in registers; the rows of A are broadcast from shared memory.  X = [u | w].
 //   4. qg = q exp(gc), kd = k exp(gc_last - gc), glast = exp(gc_last).
 // The reference builds the same quantities as a graph of library ops over all chunks with a 63-step loop for the solve
-// (cc/src/tyr_qwen35.cpp:21-88).  Rows past the sequence end behave as g = 0, beta = 0, q = k = v = 0.
+// (cc/src/tyr_qwen35.cpp:21-88).  Rows past the sequence end behave as g = 0, beta = 0, q = k = v = 0.  Key sizes below 128 are
+// padded with zero channels, which change neither norms nor products.
 // ------------------------------------------------------------------------------------------------------------------
 constexpr int GP_LDA = GC_C + 4;
 
@@ -590,8 +615,9 @@ struct GdrPrepArgs {
   const __nv_bfloat16 *q, *k, *v;
   const float *g, *beta;               // [B, S, Hv] contiguous
   float *u, *w, *qg, *kd, *intra, *glast;
+  const int* lens;                     // [B] tokens of each row (nullable: S); the rest of a padded row leaves the state alone
   long long q_sb, q_ss, q_sh, k_sb, k_ss, k_sh, v_sb, v_ss, v_sh;
-  int S, n, Hk, Hv, dv;
+  int S, n, Hk, Hv, dk, dv, dvp;       // dvp: dv rounded up to 64, the row length of u
 };
 
 __device__ __forceinline__ uint32_t to_tf32(float x) {
@@ -607,12 +633,13 @@ __global__ void __launch_bounds__(256, 2) gdr_chunk_prepare_kernel(GdrPrepArgs a
   const int b = bh / a.Hv, hv = bh % a.Hv, hk = hv / (a.Hv / a.Hk);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int row0 = c * GC_C;
+  const int len = a.lens ? min(a.lens[b], a.S) : a.S;
   // ---- 1. stage q, k (fp32), g, beta
   for (int i = tid; i < GC_C * (GC_DK / 8); i += 256) {
     const int r = i / (GC_DK / 8), d = (i % (GC_DK / 8)) * 8;
     const int tok = row0 + r;
     uint4 uq = make_uint4(0, 0, 0, 0), uk = make_uint4(0, 0, 0, 0);
-    if (tok < a.S) {
+    if (tok < len && d < a.dk) {
       uq = *reinterpret_cast<const uint4*>(a.q + b * a.q_sb + static_cast<long long>(tok) * a.q_ss + hk * a.q_sh + d);
       uk = *reinterpret_cast<const uint4*>(a.k + b * a.k_sb + static_cast<long long>(tok) * a.k_ss + hk * a.k_sh + d);
     }
@@ -624,18 +651,18 @@ __global__ void __launch_bounds__(256, 2) gdr_chunk_prepare_kernel(GdrPrepArgs a
       sm.k[r * GC_LDW + d + 2 * e] = fk.x; sm.k[r * GC_LDW + d + 2 * e + 1] = fk.y;
     }
   }
-  for (int i = tid; i < GC_C * (a.dv / 8); i += 256) {
-    const int r = i / (a.dv / 8), d = (i % (a.dv / 8)) * 8;
+  for (int i = tid; i < GC_C * (a.dvp / 8); i += 256) {
+    const int r = i / (a.dvp / 8), d = (i % (a.dvp / 8)) * 8;
     const int tok = row0 + r;
     uint4 uv = make_uint4(0, 0, 0, 0);
-    if (tok < a.S) uv = *reinterpret_cast<const uint4*>(a.v + b * a.v_sb + static_cast<long long>(tok) * a.v_ss + hv * a.v_sh + d);
-    *reinterpret_cast<uint4*>(&sm.v[r * a.dv + d]) = uv;
+    if (tok < len && d < a.dv) uv = *reinterpret_cast<const uint4*>(a.v + b * a.v_sb + static_cast<long long>(tok) * a.v_ss + hv * a.v_sh + d);
+    *reinterpret_cast<uint4*>(&sm.v[r * a.dvp + d]) = uv;
   }
   if (tid < GC_C) {
     const int tok = row0 + tid;
     const long long gi = (static_cast<long long>(b) * a.S + tok) * a.Hv + hv;
-    sm.gc[tid] = tok < a.S ? a.g[gi] : 0.f;
-    sm.beta[tid] = tok < a.S ? a.beta[gi] : 0.f;
+    sm.gc[tid] = tok < len ? a.g[gi] : 0.f;
+    sm.beta[tid] = tok < len ? a.beta[gi] : 0.f;
   }
   __syncthreads();
   // inclusive scan of g over the chunk (warp 0: two elements per lane)
@@ -661,7 +688,7 @@ __global__ void __launch_bounds__(256, 2) gdr_chunk_prepare_kernel(GdrPrepArgs a
     }
     sq += __shfl_xor_sync(0xffffffffu, sq, 1); sq += __shfl_xor_sync(0xffffffffu, sq, 2);
     sk += __shfl_xor_sync(0xffffffffu, sk, 1); sk += __shfl_xor_sync(0xffffffffu, sk, 2);
-    const float qn = rsqrtf(sq + 1e-6f) * rsqrtf(static_cast<float>(GC_DK)), kn = rsqrtf(sk + 1e-6f);
+    const float qn = rsqrtf(sq + 1e-6f) * rsqrtf(static_cast<float>(a.dk)), kn = rsqrtf(sk + 1e-6f);
     for (int d = part; d < GC_DK; d += 4) {
       sm.q[r * GC_LDW + d] *= qn;
       sm.k[r * GC_LDW + d] *= kn;
@@ -724,16 +751,16 @@ __global__ void __launch_bounds__(256, 2) gdr_chunk_prepare_kernel(GdrPrepArgs a
   // ---- 3. forward substitution, one right-hand-side column per thread
   {
     const int col = tid;
-    const int ncol = a.dv + GC_DK;
+    const int ncol = a.dvp + GC_DK;
     if (col < ncol) {
       float x[GC_C];
-      const bool is_v = col < a.dv;
+      const bool is_v = col < a.dvp;
       if (is_v) {
 #pragma unroll
-        for (int i = 0; i < GC_C; ++i) x[i] = __bfloat162float(sm.v[i * a.dv + col]) * sm.beta[i];
+        for (int i = 0; i < GC_C; ++i) x[i] = __bfloat162float(sm.v[i * a.dvp + col]) * sm.beta[i];
       } else {
 #pragma unroll
-        for (int i = 0; i < GC_C; ++i) x[i] = sm.k[i * GC_LDW + (col - a.dv)] * sm.beta[i] * sm.eg[i];
+        for (int i = 0; i < GC_C; ++i) x[i] = sm.k[i * GC_LDW + (col - a.dvp)] * sm.beta[i] * sm.eg[i];
       }
 #pragma unroll
       for (int i = 1; i < GC_C; ++i) {
@@ -748,9 +775,9 @@ __global__ void __launch_bounds__(256, 2) gdr_chunk_prepare_kernel(GdrPrepArgs a
         }
         x[i] = acc;
       }
-      float* dst = is_v ? a.u + (static_cast<long long>(bh) * a.n + c) * GC_C * a.dv + col
-                        : a.w + (static_cast<long long>(bh) * a.n + c) * GC_C * GC_DK + (col - a.dv);
-      const int ld = is_v ? a.dv : GC_DK;
+      float* dst = is_v ? a.u + (static_cast<long long>(bh) * a.n + c) * GC_C * a.dvp + col
+                        : a.w + (static_cast<long long>(bh) * a.n + c) * GC_C * GC_DK + (col - a.dvp);
+      const int ld = is_v ? a.dvp : GC_DK;
 #pragma unroll
       for (int i = 0; i < GC_C; ++i) dst[static_cast<long long>(i) * ld] = x[i];
     }
@@ -865,15 +892,15 @@ extern "C" TYR_EXPORT int tyr_causal_conv1d_silu(const void* x, const float* w, 
   return static_cast<int>(cudaGetLastError());
 }
 
-// Chunk-local quantities of the gated delta rule (chunk 64, dk 128, dv 64 or 128).  q, k: bf16 [B, S, Hk, 128] and
-// v: bf16 [B, S, Hv, dv] given by (batch, token, head) element strides; g, beta: fp32 [B, S, Hv] contiguous.  Outputs (fp32,
-// n = ceil(S / 64) chunks): u [B*Hv, n, 64, dv], w / qg / kd [B*Hv, n, 64, 128], intra [B*Hv, n, 64, 64], glast [B*Hv, n].
+// Chunk-local quantities of the gated delta rule (chunk 64, dk and dv multiples of 8 up to 128).  q, k: bf16 [B, S, Hk, dk] and
+// v: bf16 [B, S, Hv, dv] given by (batch, token, head) element strides; g, beta: fp32 [B, S, Hv] contiguous; lens: int32 [B] or
+// null.  Outputs (fp32, n = ceil(S / 64) chunks, dvp = dv rounded up to 64): u [B*Hv, n, 64, dvp], w / qg / kd [B*Hv, n, 64, 128], intra [B*Hv, n, 64, 64], glast [B*Hv, n].
 extern "C" TYR_EXPORT int tyr_gdr_chunk_prepare(const void* q, const void* k, const void* v, const float* g,
                                                 const float* beta, float* u, float* w, float* qg, float* kd,
-                                                float* intra, float* glast, const long long* strides, int B, int S,
+                                                float* intra, float* glast, const int* lens, const long long* strides, int B, int S,
                                                 int Hk, int Hv, int dk, int dv, void* stream) {
   using namespace tyr;
-  if (B <= 0 || S <= 0 || Hk <= 0 || Hv <= 0 || Hv % Hk || dk != GC_DK || (dv != 64 && dv != 128)) return -1;
+  if (B <= 0 || S <= 0 || Hk <= 0 || Hv <= 0 || Hv % Hk || dk <= 0 || dk > GC_DK || (dk & 7) || dv <= 0 || dv > 128 || (dv & 7)) return -1;
   for (int i = 0; i < 9; ++i)
     if (strides[i] & 7) return -3;
   if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v)) & 15) return -4;
@@ -885,7 +912,8 @@ extern "C" TYR_EXPORT int tyr_gdr_chunk_prepare(const void* q, const void* k, co
   a.q_sb = strides[0]; a.q_ss = strides[1]; a.q_sh = strides[2];
   a.k_sb = strides[3]; a.k_ss = strides[4]; a.k_sh = strides[5];
   a.v_sb = strides[6]; a.v_ss = strides[7]; a.v_sh = strides[8];
-  a.S = S; a.n = (S + GC_C - 1) / GC_C; a.Hk = Hk; a.Hv = Hv; a.dv = dv;
+  a.S = S; a.n = (S + GC_C - 1) / GC_C; a.Hk = Hk; a.Hv = Hv; a.dk = dk; a.dv = dv; a.dvp = (dv + 63) & ~63;
+  a.lens = lens;
   constexpr size_t smem = sizeof(GdrPrepSmem);
   static bool configured_dev[64] = {false};     // the attribute is per device
   int cfg_dev = 0;
@@ -900,16 +928,16 @@ extern "C" TYR_EXPORT int tyr_gdr_chunk_prepare(const void* q, const void* k, co
   return static_cast<int>(cudaGetLastError());
 }
 
-// Sequential chunk pass of the gated delta rule (chunk 64, dk 128, dv a multiple of 64), all tensors fp32 and contiguous:
-// u [BH, n, 64, dv], w / qg / kd [BH, n, 64, 128], intra [BH, n, 64, 64], glast [BH, n] (= exp of the chunk's last cumulative
-// log decay), state_in [BH, 128, dv] (nullable = zeros), state_out [BH, 128, dv]; out: bf16 [B, S, Hv, dv] with BH = B * Hv and
-// n = ceil(S / 64).
+// Sequential chunk pass of the gated delta rule (chunk 64, dk <= 128, dv even), all tensors fp32 and contiguous:
+// u [BH, n, 64, dvp], w / qg / kd [BH, n, 64, 128], intra [BH, n, 64, 64], glast [BH, n] (= exp of the chunk's last cumulative
+// log decay), state_in [BH, dk, dv] (nullable = zeros), state_out [BH, dk, dv]; out: [B, S, Hv, dv] with BH = B * Hv and
+// n = ceil(S / 64), bf16, or fp32 with `exact` (split TF32 products).
 extern "C" TYR_EXPORT int tyr_gdr_chunk_scan(const float* u, const float* w, const float* qg, const float* kd,
                                              const float* intra, const float* glast, const float* state_in,
                                              float* state_out, void* out, int BH, int n, int dk, int dv, int chunk, int S,
-                                             int Hv, void* stream) {
+                                             int Hv, int exact, void* stream) {
   using namespace tyr;
-  if (BH <= 0 || n <= 0 || dk != GC_DK || chunk != GC_C || dv <= 0 || dv % GC_DVS || Hv <= 0 || BH % Hv || S <= 0 || S > n * GC_C) return -1;
+  if (BH <= 0 || n <= 0 || dk <= 0 || dk > GC_DK || chunk != GC_C || dv <= 0 || (dv & 7) || Hv <= 0 || BH % Hv || S <= 0 || S > n * GC_C) return -1;
   if ((reinterpret_cast<uintptr_t>(u) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(qg) |
        reinterpret_cast<uintptr_t>(kd) | reinterpret_cast<uintptr_t>(intra) | reinterpret_cast<uintptr_t>(out) |
        reinterpret_cast<uintptr_t>(state_out) | reinterpret_cast<uintptr_t>(state_in)) & 15)
@@ -920,12 +948,20 @@ extern "C" TYR_EXPORT int tyr_gdr_chunk_scan(const float* u, const float* w, con
   if (cudaGetDevice(&cfg_dev) != cudaSuccess || cfg_dev < 0 || cfg_dev >= 64) cfg_dev = 0;
   bool& configured = configured_dev[cfg_dev];
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(gdr_chunk_scan_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(gdr_chunk_scan_kernel<false, __nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(gdr_chunk_scan_kernel<true, float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return 1000 + (int)e;
     configured = true;
   }
-  gdr_chunk_scan_kernel<<<dim3(dv / GC_DVS, BH), 128, smem, reinterpret_cast<cudaStream_t>(stream)>>>(
-      u, w, qg, kd, intra, glast, state_in, state_out, reinterpret_cast<__nv_bfloat16*>(out), n, dv, S, Hv);
+  const int slices = (dv + GC_DVS - 1) / GC_DVS, dvp = slices * GC_DVS;
+  const dim3 grid(slices, BH);
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  if (exact)
+    gdr_chunk_scan_kernel<true, float><<<grid, 256, smem, st>>>(u, w, qg, kd, intra, glast, state_in, state_out, reinterpret_cast<float*>(out),
+                                                                n, dk, dv, dvp, S, Hv);
+  else
+    gdr_chunk_scan_kernel<false, __nv_bfloat16><<<grid, 256, smem, st>>>(u, w, qg, kd, intra, glast, state_in, state_out,
+                                                                         reinterpret_cast<__nv_bfloat16*>(out), n, dk, dv, dvp, S, Hv);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -958,11 +994,12 @@ extern "C" TYR_EXPORT int tyr_gdr_decode(const void* q, const void* k, const voi
 }
 
 // dv == 128, dk 64 or 128, v / z rows 8-byte aligned (strides multiples of 4 elements): the shared-memory tile form of the
-// step (gdr_decode_tile_kernel); `z` / `norm_w` may be null (no gated RMSNorm).  `err`: the device error record.
+// step (gdr_decode_tile_kernel); `z` / `norm_w` may be null (no gated RMSNorm); `round_o`: the norm sees the
+// read-out rounded to bf16 (else fp32).  `err`: the device error record.
 extern "C" TYR_EXPORT int tyr_gdr_decode_tile(const void* q, const void* k, const void* v, const float* g, const float* beta,
                                               float* state, void* out, int B, int Hk, int Hv, int dk,
                                               long long q_bstride, long long v_bstride, const void* z, long long z_bstride,
-                                              const void* norm_w, float norm_eps, int* err, void* stream) {
+                                              const void* norm_w, float norm_eps, int round_o, int* err, void* stream) {
   using namespace tyr;
   if (B <= 0 || Hk <= 0 || Hv <= 0 || Hv % Hk != 0 || (dk != 64 && dk != 128)) return -1;
   if (z != nullptr && norm_w == nullptr) return -3;
@@ -990,10 +1027,10 @@ extern "C" TYR_EXPORT int tyr_gdr_decode_tile(const void* q, const void* k, cons
   cudaError_t e;
   if (dk == 128)
     e = launch_dependent(gdr_decode_tile_kernel<128>, dim3(B * Hv), dim3(256), smem, st, qq, kk, vv, g, beta, state, oo, Hk, Hv,
-                         q_bstride, v_bstride, zz, z_bstride, nw, norm_eps, err);
+                         q_bstride, v_bstride, zz, z_bstride, nw, norm_eps, round_o, err);
   else
     e = launch_dependent(gdr_decode_tile_kernel<64>, dim3(B * Hv), dim3(256), smem, st, qq, kk, vv, g, beta, state, oo, Hk, Hv,
-                         q_bstride, v_bstride, zz, z_bstride, nw, norm_eps, err);
+                         q_bstride, v_bstride, zz, z_bstride, nw, norm_eps, round_o, err);
   return static_cast<int>(e);
 }
 

@@ -114,6 +114,7 @@ struct RouteArgs {
   int softmax;           // 0 = sigmoid scores, 1 = softmax scores
   int renorm;
   float softcap, scale;
+  int groups, keep;      // groups > 1: E / groups neighbouring experts form a group; only the `keep` groups with the best expert compete
 };
 
 // One warp routes one token from its row of logits.  The row may have been written by other CTAs of the same launch, so it is
@@ -148,6 +149,33 @@ __device__ __forceinline__ void route_token_n(const RouteArgs& a, const float* r
   for (int j = 0; j < kMaxPer; ++j) {
     const int e = lane + 32 * j;
     sel[j] = (j < per && e < a.E) ? score[j] + (a.bias ? a.bias[e] : 0.f) : -INFINITY;
+  }
+  if (a.groups > 1) {
+    // lane g holds the best choice score of group g (groups <= 32), then the groups are ranked by it (ties: lower group); experts
+    // of the other groups leave the competition whatever the sign of their scores
+    const int size = a.E / a.groups;
+    float mine = -INFINITY;
+    for (int g = 0; g < a.groups; ++g) {
+      float best = -INFINITY;
+#pragma unroll
+      for (int j = 0; j < kMaxPer; ++j) {
+        const int e = lane + 32 * j;
+        if (e < a.E && e / size == g) best = fmaxf(best, sel[j]);
+      }
+      best = warp_max(best);
+      if (lane == g) mine = best;
+    }
+    int rank = 0;
+    for (int g = 0; g < a.groups; ++g) {
+      const float other = __shfl_sync(0xffffffffu, mine, g);
+      rank += (other > mine || (other == mine && g < lane)) ? 1 : 0;
+    }
+    const unsigned kept = __ballot_sync(0xffffffffu, lane < a.groups && rank < a.keep);
+#pragma unroll
+    for (int j = 0; j < kMaxPer; ++j) {
+      const int e = lane + 32 * j;
+      if (e < a.E && !((kept >> (e / size)) & 1u)) sel[j] = -INFINITY;
+    }
   }
   float wsum = 0.f;
   float my_w = 0.f;
@@ -638,9 +666,10 @@ extern "C" TYR_EXPORT int tyr_nvfp4_dequant(const void* packed, const void* scal
 
 extern "C" TYR_EXPORT int tyr_moe_route(const float* logits, const float* bias, int* ids, float* weights, int* counts,
                                         int T, int E, int k, int softmax, int renorm, float softcap, float scale,
-                                        void* stream) {
+                                        int groups, int keep, void* stream) {
   if (T <= 0 || E <= 0 || E > 512 || k <= 0 || k > 32 || k > E) return -1;
-  RouteArgs a{logits, bias, ids, weights, counts, T, E, k, softmax, renorm, softcap, scale};
+  if (groups > 1 && (groups > 32 || E % groups || keep <= 0 || keep > groups || k > keep * (E / groups))) return -4;
+  RouteArgs a{logits, bias, ids, weights, counts, T, E, k, softmax, renorm, softcap, scale, groups, keep};
   moe_route_kernel<<<(T + 7) / 8, 256, 0, (cudaStream_t)stream>>>(a);
   return (int)cudaGetLastError();
 }
@@ -649,8 +678,10 @@ extern "C" TYR_EXPORT int tyr_moe_route(const float* logits, const float* bias, 
 // T * E floats, `tickets` ceil(T / 4) zeroed ints.
 extern "C" TYR_EXPORT int tyr_moe_route_fused(const void* x, const float* router_w, const float* bias, float* logits,
                                               int* tickets, int* ids, float* weights, int* counts, int T, int E, int k,
-                                              int h, int softmax, int renorm, float softcap, float scale, void* stream) {
+                                              int h, int softmax, int renorm, float softcap, float scale, int groups, int keep,
+                                              void* stream) {
   if (T <= 0 || E <= 0 || E > 512 || k <= 0 || k > 32 || k > E || h <= 0 || (h & 7)) return -1;
+  if (groups > 1 && (groups > 32 || E % groups || keep <= 0 || keep > groups || k > keep * (E / groups))) return -4;
   if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(router_w)) & 15) return -2;
   const size_t smem = sizeof(__nv_bfloat16) * static_cast<size_t>(h) * kRouteTok;
   if (smem > 160 * 1024) return -3;
@@ -659,7 +690,7 @@ extern "C" TYR_EXPORT int tyr_moe_route_fused(const void* x, const float* router
     cudaFuncSetAttribute(moe_route_fused_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     configured = smem;
   }
-  RouteArgs a{nullptr, bias, ids, weights, counts, T, E, k, softmax, renorm, softcap, scale};
+  RouteArgs a{nullptr, bias, ids, weights, counts, T, E, k, softmax, renorm, softcap, scale, groups, keep};
   dim3 grid((T + kRouteTok - 1) / kRouteTok, (E + kRouteExp - 1) / kRouteExp);
   return (int)launch_dependent(moe_route_fused_kernel, grid, dim3(256), smem, (cudaStream_t)stream, a, (const __nv_bfloat16*)x,
                                router_w, logits, tickets, h);

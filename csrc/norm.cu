@@ -334,6 +334,115 @@ __global__ void __launch_bounds__(256) rmsnorm_weighted_row_kernel(RmsWArgs a) {
   }
 }
 
+// Norm on a sublayer's output, added to an fp32 residual stream:
+//   r = (resid ? resid : 0) + x / sqrt(mean(x^2) + eps) * gain,   resid_out = r,   y = r in the compute dtype.
+// `gain` holds one number for all channels (n_gain == 1) or one per channel.  One CTA per row; a thread keeps up to kPnVecs
+// vectors of 8 channels in registers between the reduction and the write.
+struct PostNormArgs {
+  const void* x;           // [rows, D] (TX)
+  const float* gain;
+  float* resid;            // [rows, D] in place (nullable: plain norm)
+  void* y;                 // [rows, D] (TY), nullable
+  long long x_stride;      // elements between rows of x
+  int D, n_gain;
+  float eps;
+};
+constexpr int kPnVecs = 4;
+
+__device__ __forceinline__ void pn_load8(const __nv_bfloat16* p, float (&f)[8]) {
+  const uint4 u = *reinterpret_cast<const uint4*>(p);
+  const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    const float2 t = unpack_bf16x2(w[e]);
+    f[2 * e] = t.x; f[2 * e + 1] = t.y;
+  }
+}
+__device__ __forceinline__ void pn_load8(const float* p, float (&f)[8]) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+__device__ __forceinline__ void pn_store8(__nv_bfloat16* p, const float (&f)[8]) {
+  uint4 u;
+  u.x = pack_bf16x2(f[0], f[1]); u.y = pack_bf16x2(f[2], f[3]); u.z = pack_bf16x2(f[4], f[5]); u.w = pack_bf16x2(f[6], f[7]);
+  *reinterpret_cast<uint4*>(p) = u;
+}
+__device__ __forceinline__ void pn_store8(float* p, const float (&f)[8]) {
+  reinterpret_cast<float4*>(p)[0] = make_float4(f[0], f[1], f[2], f[3]);
+  reinterpret_cast<float4*>(p)[1] = make_float4(f[4], f[5], f[6], f[7]);
+}
+__device__ __forceinline__ float pn_get(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ float pn_get(const float* p) { return *p; }
+__device__ __forceinline__ void pn_put(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
+__device__ __forceinline__ void pn_put(float* p, float v) { *p = v; }
+
+template <typename TX, typename TY, bool VEC>
+__global__ void __launch_bounds__(256) post_norm_residual_kernel(PostNormArgs a) {
+  __shared__ float red[8];
+  const long long row = blockIdx.x;
+  const int tid = threadIdx.x, nw = blockDim.x >> 5;
+  const TX* x = static_cast<const TX*>(a.x) + row * a.x_stride;
+  float* resid = a.resid ? a.resid + row * a.D : nullptr;
+  TY* y = a.y ? static_cast<TY*>(a.y) + row * a.D : nullptr;
+  pdl_entry();
+  float f[kPnVecs][8], ss = 0.f;
+  if constexpr (VEC) {
+#pragma unroll
+    for (int j = 0; j < kPnVecs; ++j) {
+      const int v = (tid + j * blockDim.x) * 8;
+      if (v < a.D) {
+        pn_load8(x + v, f[j]);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss += f[j][e] * f[j][e];
+      }
+    }
+  } else {
+    for (int d = tid; d < a.D; d += blockDim.x) {
+      const float t = pn_get(x + d);
+      ss += t * t;
+    }
+  }
+  ss = warp_sum(ss);
+  if ((tid & 31) == 0) red[tid >> 5] = ss;
+  __syncthreads();
+  float tot = 0.f;
+  for (int i = 0; i < nw; ++i) tot += red[i];
+  const float rstd = rsqrtf(tot / a.D + a.eps);
+  if constexpr (VEC) {
+#pragma unroll
+    for (int j = 0; j < kPnVecs; ++j) {
+      const int v = (tid + j * blockDim.x) * 8;
+      if (v >= a.D) continue;
+      float w[8];
+      if (a.n_gain == 1) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) w[e] = a.gain[0];
+      } else {
+        pn_load8(a.gain + v, w);
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[j][e] *= rstd * w[e];
+      if (resid) {
+        float r[8];
+        pn_load8(resid + v, r);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[j][e] += r[e];
+        pn_store8(resid + v, f[j]);
+      }
+      if (y) pn_store8(y + v, f[j]);
+    }
+  } else {
+    for (int d = tid; d < a.D; d += blockDim.x) {
+      float t = pn_get(x + d) * rstd * a.gain[a.n_gain == 1 ? 0 : d];
+      if (resid) {
+        t += resid[d];
+        resid[d] = t;
+      }
+      if (y) pn_put(y + d, t);
+    }
+  }
+}
+
 static int grid_for_rows(long long rows, int warps_per_block) {
   long long blocks = (rows + warps_per_block - 1) / warps_per_block;
   const long long cap = 148LL * 16;
@@ -406,4 +515,23 @@ extern "C" TYR_EXPORT int tyr_rmsnorm_weighted(const void* x, const void* w, con
   if (rows <= 2048 && D >= 1024 && D <= 256 * kRowVecs * 8)
     return (int)launch_dependent(rmsnorm_weighted_row_kernel, dim3(rows), dim3(256), 0, (cudaStream_t)stream, a);
   return (int)launch_dependent(rmsnorm_weighted_kernel, dim3(grid_for_rows(rows, 8)), dim3(256), 0, (cudaStream_t)stream, a);
+}
+
+// x_dtype / y_dtype: 0 = bf16, 1 = fp32; `gain` fp32 of one or D numbers; `resid` fp32 in place or null; `y` may be null.
+extern "C" TYR_EXPORT int tyr_post_norm_residual(const void* x, long long x_stride, const float* gain, int n_gain, float* resid, void* y,
+                                                 long long rows, int D, float eps, int x_dtype, int y_dtype, void* stream) {
+  if (rows <= 0 || D <= 0 || (n_gain != 1 && n_gain != D) || (resid == nullptr && y == nullptr)) return -1;
+  PostNormArgs a{x, gain, resid, y, x_stride, D, n_gain, eps};
+  const uintptr_t al = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(resid) | reinterpret_cast<uintptr_t>(y) |
+                       (n_gain == 1 ? 0 : reinterpret_cast<uintptr_t>(gain));
+  const bool vec = (D & 7) == 0 && (x_stride & 7) == 0 && (al & 15) == 0 && D <= 256 * 8 * kPnVecs;
+  int threads = 256;
+  while (threads > 32 && threads * 4 >= D) threads >>= 1;       // narrow rows: no idle warps
+  const dim3 grid(static_cast<unsigned>(rows)), block(threads);
+  cudaStream_t st = (cudaStream_t)stream;
+#define TYR_PN(TX, TY) (vec ? launch_dependent(post_norm_residual_kernel<TX, TY, true>, grid, block, 0, st, a) \
+                            : launch_dependent(post_norm_residual_kernel<TX, TY, false>, grid, block, 0, st, a))
+  if (x_dtype == 0) return (int)(y_dtype == 0 ? TYR_PN(__nv_bfloat16, __nv_bfloat16) : TYR_PN(__nv_bfloat16, float));
+  return (int)(y_dtype == 0 ? TYR_PN(float, __nv_bfloat16) : TYR_PN(float, float));
+#undef TYR_PN
 }

@@ -22,7 +22,28 @@ class NativeLibraryMissing(RuntimeError):
     pass
 
 
+_units = None
+
+
+def use_units(units) -> None:
+    """Kernel units (names of csrc/*.cu without suffix) this process needs.  Where the whole library has not been built, the first
+    kernel call then compiles these units alone instead of every source."""
+    global _units
+    _units = tuple(sorted(units))
+
+
 def _load(name: str):
+    if name == "libtyr_kernels.so" and _units is not None and not (_HERE / name).exists():
+        from . import build as _b
+        part = _b.partial_name(_units)
+        if not (_HERE / part).exists():
+            if os.environ.get("TYR_B200_AUTOBUILD", "1") == "0":
+                raise NativeLibraryMissing(f"{_HERE / part} not found and automatic builds are off")
+            try:
+                _b.build_kernels(units=_units)
+            except Exception as e:  # pragma: no cover - build environment specific
+                raise NativeLibraryMissing(f"building the kernel units {', '.join(_units)} failed: {e}") from e
+        name = part
     path = _HERE / name
     if not path.exists():
         if os.environ.get("TYR_B200_AUTOBUILD", "1") != "0":

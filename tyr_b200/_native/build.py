@@ -30,10 +30,13 @@ OBJ_DIR = ROOT / "build" / "obj"
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
-    "-lineinfo", "-O3", "-std=c++17", "--use_fast_math",
+    "-lineinfo", "-O3", "-std=c++17",
     "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=hidden",
     "--expt-relaxed-constexpr",
 ]
+# Units whose results are carried through thousands of steps or stand for the fp32 mode: correctly rounded division, square root
+# and library exponentials.  Every other unit is compiled with fast math.
+PRECISE_UNITS = ("delta_general", "attention_general")
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-pthread"]
 
 
@@ -69,17 +72,27 @@ def _link(cmd, out: Path):
 CHECKED_UNITS = ("moe_nvfp4", "rope")       # translation units with index checks; the checked library holds only these
 
 
-def build_kernels(verbose: bool = False, force: bool = False, checked: bool = False) -> Path:
+def partial_name(units) -> str:
+    """Library of a subset of the kernel units; its name follows the subset and the sources, so an old one is never picked up."""
+    hdrs = sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
+    dig = _digest([CSRC / f"{u}.cu" for u in units] + hdrs, " ".join(NVCC_FLAGS))
+    return f"libtyr_kernels_part_{dig[:12]}.so"
+
+
+def build_kernels(verbose: bool = False, force: bool = False, checked: bool = False, units=None) -> Path:
     """``checked=True`` builds ``libtyr_kernels_checked.so``: the units listed in ``CHECKED_UNITS`` compiled with
-    ``-DTYR_BOUNDS_CHECK`` (data-dependent indices are tested and violations recorded, see csrc/common.cuh)."""
+    ``-DTYR_BOUNDS_CHECK`` (data-dependent indices are tested and violations recorded, see csrc/common.cuh).  ``units`` names a
+    subset of the sources (without suffix): only those are compiled, into a library of their own (:func:`partial_name`)."""
     srcs = sorted(CSRC.glob("*.cu"))
     if checked:
         srcs = [s for s in srcs if s.stem in CHECKED_UNITS]
     hdrs = sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
-    out = OUT_DIR / ("libtyr_kernels_checked.so" if checked else "libtyr_kernels.so")
+    if units is not None:
+        srcs = [s for s in srcs if s.stem in units]
+    out = OUT_DIR / ("libtyr_kernels_checked.so" if checked else partial_name(units) if units is not None else "libtyr_kernels.so")
     OBJ_DIR.mkdir(parents=True, exist_ok=True)
     base_flags = NVCC_FLAGS + (["-DTYR_BOUNDS_CHECK"] if checked else [])
-    hdr_digest = _digest(hdrs, " ".join(base_flags))
+    hdr_digest = _digest(hdrs, " ".join(base_flags) + " precise: " + " ".join(PRECISE_UNITS))
     nvcc = _nvcc()
     jobs = []
     objs = []
@@ -93,7 +106,7 @@ def build_kernels(verbose: bool = False, force: bool = False, checked: bool = Fa
 
     def compile_one(job):
         s, obj, stamp, dig = job
-        flags = list(base_flags)
+        flags = list(base_flags) + ([] if s.stem in PRECISE_UNITS else ["--use_fast_math"])
         if verbose:
             flags += ["-Xptxas", "-v"]
         log = _run([nvcc, *flags, "-I", str(CSRC), "-c", str(s), "-o", str(obj)])

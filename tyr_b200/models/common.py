@@ -5,6 +5,7 @@
 * rotary tables (plain / YaRN / partial), HF rotate-half application.
 * ``KVCache``: static and ring (sliding-window) stores with in-place writes; the session owns the
   tensors (Tyr/Model/Laguna/Model.lean:351-406, Tyr/Model/Qwen/Model.lean KVCache).
+* ``LinearState``: convolution window and recurrent state of a linear-attention layer.
 """
 from __future__ import annotations
 
@@ -135,11 +136,11 @@ class KVCache:
     length: int = 0           # absolute positions written so far
 
     @staticmethod
-    def allocate(batch: int, kv_heads: int, cap: int, head_dim: int, device, dtype, ring: bool = False) -> "KVCache":
+    def allocate(batch: int, kv_heads: int, cap: int, head_dim: int, device, dtype, ring: bool = False, v_dim: Optional[int] = None) -> "KVCache":
         if cap <= 0:
             raise ValueError("cache capacity must be positive")
-        shape = (batch, kv_heads, cap, head_dim)
-        return KVCache(torch.zeros(shape, device=device, dtype=dtype), torch.zeros(shape, device=device, dtype=dtype), ring)
+        zeros = lambda d: torch.zeros((batch, kv_heads, cap, d), device=device, dtype=dtype)
+        return KVCache(zeros(head_dim), zeros(head_dim if v_dim is None else v_dim), ring)
 
     @property
     def cap(self) -> int:
@@ -172,8 +173,27 @@ class KVCache:
     def clone(self) -> "KVCache":
         return KVCache(self.k.clone(), self.v.clone(), self.ring, self.length)
 
+    def retain(self, rows: torch.Tensor) -> None:
+        """Keep only these rows of the batch, in this order; the others' memory is given back."""
+        self.k, self.v = self.k.index_select(0, rows), self.v.index_select(0, rows)
+
     def nbytes(self) -> int:
-        return self.k.numel() * self.k.element_size() * 2
+        return self.k.numel() * self.k.element_size() + self.v.numel() * self.v.element_size()
+
+
+@dataclass
+class LinearState:
+    conv: Optional[torch.Tensor] = None        # [B, conv_dim, K] last K pre-conv inputs
+    rec: Optional[torch.Tensor] = None         # fp32 [B, Hv, dk, dv]
+
+    def retain(self, rows: torch.Tensor) -> None:
+        if self.conv is not None:
+            self.conv = self.conv.index_select(0, rows)
+        if self.rec is not None:
+            self.rec = self.rec.index_select(0, rows)
+
+    def nbytes(self) -> int:
+        return sum(t.numel() * t.element_size() for t in (self.conv, self.rec) if t is not None)
 
 
 def cached_attention(q: torch.Tensor, k_new: torch.Tensor, v_new: torch.Tensor, cache: Optional[KVCache],

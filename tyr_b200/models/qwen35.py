@@ -21,9 +21,10 @@ from ..ops import moe as moe_ops
 from ..ops.attention import attention
 from ..ops.decode_attention import decode_attention, geometry_supported
 from ..ops.rope import rope_norm
-from .common import KVCache, apply_rotary_partial, cached_attention, cos_sin_tables, head_norm, lin, norm_w, plain_inv_freq, swiglu_mlp
+from .common import KVCache, LinearState, apply_rotary_partial, cached_attention, cos_sin_tables, head_norm, lin, norm_w, plain_inv_freq, swiglu_mlp
 from .generation import SamplingStrategy, generate_cached
 from .laguna import name_candidates
+from .session import HybridSession
 
 LINEAR, FULL = "linear_attention", "full_attention"
 
@@ -286,12 +287,6 @@ def attention_forward(cfg: Qwen35Config, a: Attention, x, cos, sin, cache: Optio
     return lin(o, a.o_proj)
 
 
-@dataclass
-class LinearState:
-    conv: Optional[torch.Tensor] = None        # [B, conv_dim, K] last K pre-conv inputs
-    rec: Optional[torch.Tensor] = None         # fp32 [B, Hv, dk, dv]
-
-
 def rms_norm_gated(x, gate, w, eps):
     xf = x.float()
     y = xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * w.float()
@@ -390,36 +385,45 @@ def forward(m: Qwen35ForCausalLM, input_ids=None, attn_mask=None, inputs_embeds=
     return lin(forward_hidden(m, input_ids, attn_mask, inputs_embeds), m.lm_head)
 
 
-class HybridCache:
+class HybridCache(HybridSession):
     """KV caches for full layers, conv + recurrent states for linear layers (Model.lean:784-860)."""
+    name = "Qwen3.5"
 
     def __init__(self, m: Qwen35ForCausalLM, batch: int, max_len: int):
         cfg = m.cfg
-        self.m, self.pos, self.max_len, self.batch = m, 0, max_len, batch
+        super().__init__(batch, max_len, m.device)
+        self.m = m
         self.cos, self.sin = rope_tables(cfg, max_len, m.device)
         self.kv = [KVCache.allocate(batch, cfg.num_key_value_heads, max_len, cfg.head_dim, m.device, m.dtype) if cfg.is_full(i) else None
                    for i in range(cfg.num_hidden_layers)]
         self.lin = [None if cfg.is_full(i) else LinearState() for i in range(cfg.num_hidden_layers)]
 
-    def state_bytes(self) -> int:
-        n = sum(c.nbytes() for c in self.kv if c is not None)
-        for s in self.lin:
-            if s is not None:
-                n += sum(t.numel() * t.element_size() for t in (s.conv, s.rec) if t is not None)
-        return n
-
     @torch.no_grad()
-    def run(self, x: torch.Tensor) -> torch.Tensor:
+    def run_hidden(self, x: torch.Tensor) -> torch.Tensor:
         cfg, S = self.m.cfg, x.shape[1]
-        if self.pos + S > self.max_len:
-            raise ValueError("Qwen3.5 cache overflow")
+        self._check_room(S)
         cos, sin = self.cos[self.pos:self.pos + S], self.sin[self.pos:self.pos + S]
         for i, l in enumerate(self.m.layers):
             x = layer_forward(cfg, i, l, x, cos, sin, self.kv[i], self.lin[i])
-        self.pos += S
-        return lin(rms(x[:, -1], self.m.norm, cfg.rms_norm_eps), self.m.lm_head)
+        self._advance([S] * self.batch)
+        return x
 
-    def prefill(self, ids): return self.run(F.embedding(ids, self.m.embed_tokens))
+    def run(self, x: torch.Tensor) -> torch.Tensor:
+        return self.head(self._norm(self.run_hidden(x)[:, -1]))
+
+    def _norm(self, x): return rms(x, self.m.norm, self.m.cfg.rms_norm_eps)
+
+    def hidden(self, ids, lengths=None):
+        if lengths is not None and any(n != ids.shape[1] for n in lengths):
+            raise ValueError("Qwen3.5 prefills prompts of one length")
+        return self._norm(self.run_hidden(F.embedding(ids, self.m.embed_tokens)))
+
+    def head(self, h): return lin(h, self.m.lm_head)
+
+    def prefill(self, ids, lengths=None):
+        if lengths is not None:
+            return super().prefill(ids, lengths)
+        return self.run(F.embedding(ids, self.m.embed_tokens))
 
     # -- decode with the position on the device (CUDA-graph body) ---------------------------------------------------
     def device_step_supported(self) -> bool:
@@ -449,26 +453,6 @@ class HybridCache:
             h1, x = norm_w(f, next_w, eps, one_plus_w=True, residual=h2, return_residual=True)
         self.pos_t += 1
         return lin(h1[:, -1], m.lm_head)
-
-    def _advance_host(self):
-        self.pos += 1
-        for c in self.kv:
-            if c is not None:
-                c.length += 1
-
-    def step(self, tok):
-        if self.pos == 0 or not self.device_step_supported():
-            return self.run(F.embedding(tok.reshape(-1, 1), self.m.embed_tokens))
-        if self.pos + 1 > self.max_len:
-            raise ValueError("Qwen3.5 cache overflow")
-        if getattr(self, "_graph", None) is None:
-            from ..utils.graph import GraphedStep
-            self.pos_t = torch.full((1,), self.pos, dtype=torch.int32, device=self.m.device)
-            state = [self.pos_t] + [t for s in self.lin if s is not None for t in (s.conv, s.rec)]
-            self._graph = GraphedStep(self._device_step, (tok.reshape(-1).clone(),), advancing_state=state)
-        out = self._graph(tok.reshape(-1))
-        self._advance_host()
-        return out
 
 
 def generate(m: Qwen35ForCausalLM, input_ids, max_new_tokens=64, strategy=SamplingStrategy(), eos_token_ids=None, on_step=None):

@@ -27,6 +27,10 @@ def _sigs(lib_):
         if g is not None:
             g.argtypes = [P, P, P, P, P, P, P, P, L, L, L, I, I, I, I, I, I, I, I, I, F, P, L, L, I, P, P]
             g.restype = I
+        g = getattr(lib_, "tyr_decode_attention_biased", None)
+        if g is not None:
+            g.argtypes = [P, P, P, P, P, P, I, P, P, L, L, L, I, I, I, I, I, I, I, I, I, I, F, P, P, P, P]
+            g.restype = I
         lib_.tyr_decode_attention_workspace_bytes.argtypes = [I, I, I, I, I]
         lib_.tyr_decode_attention_workspace_bytes.restype = L
 

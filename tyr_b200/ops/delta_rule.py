@@ -28,7 +28,7 @@ def _sigs(lib_):
         fn.restype = ctypes.c_int
     fn = getattr(lib_, "tyr_gdr_decode_tile", None)
     if fn is not None:
-        fn.argtypes = [P, P, P, P, P, P, P, I, I, I, I, L, L, P, L, P, ctypes.c_float, P, P]
+        fn.argtypes = [P, P, P, P, P, P, P, I, I, I, I, L, L, P, L, P, ctypes.c_float, I, P, P]
         fn.restype = ctypes.c_int
     fn = getattr(lib_, "tyr_gdn_conv_gates", None)
     if fn is not None:
@@ -36,16 +36,35 @@ def _sigs(lib_):
         fn.restype = ctypes.c_int
     fn = getattr(lib_, "tyr_gdr_chunk_scan", None)
     if fn is not None:
-        fn.argtypes = [P] * 9 + [I, I, I, I, I, I, I, P]
+        fn.argtypes = [P] * 9 + [I, I, I, I, I, I, I, I, P]
         fn.restype = ctypes.c_int
     fn = getattr(lib_, "tyr_gdr_chunk_prepare", None)
     if fn is not None:
-        fn.argtypes = [P] * 11 + [ctypes.POINTER(L), I, I, I, I, I, I, P]
+        fn.argtypes = [P] * 12 + [ctypes.POINTER(L), I, I, I, I, I, I, P]
         fn.restype = ctypes.c_int
     fn = getattr(lib_, "tyr_causal_conv1d_silu", None)
     if fn is not None:
         fn.argtypes = [P, P, P, P, I, I, I, I, L, L, P]
         fn.restype = ctypes.c_int
+    F = ctypes.c_float
+    for name, args in (("tyr_conv_silu", [P, P, P, I, I, I, I, L, L, I, P]),
+                       ("tyr_delta_conv_gates", [P, P, P, L, L, L] + [P] * 7 + [I, I, I, I, I, P]),
+                       ("tyr_delta_gates", [P, P, L, L, P, P, P, P, L, I, I, P]),
+                       ("tyr_gdr_recurrent", [P] * 8 + [ctypes.POINTER(L), I, I, I, I, I, I, I, P]),
+                       ("tyr_gated_norm", [P, P, L, P, P, L, I, I, F, I, P])):
+        fn = getattr(lib_, name, None)
+        if fn is not None:
+            fn.argtypes = args
+            fn.restype = ctypes.c_int
+
+
+def _dt(t: torch.Tensor) -> int:
+    """Activation type code of csrc/delta_general.cu."""
+    if t.dtype == torch.bfloat16:
+        return 0
+    if t.dtype == torch.float32:
+        return 1
+    raise TypeError(f"delta rule kernels take bf16 or fp32 activations, got {t.dtype}")
 
 
 _CHUNK_KERNEL = os.environ.get("TYR_GDR_CHUNK_KERNEL", "1") != "0"
@@ -75,32 +94,36 @@ def recurrent_gated_delta_rule(q, k, v, g, beta, state: Optional[torch.Tensor] =
 
 
 def chunk_kernels_supported(q, k, v, chunk_size: int = 64) -> bool:
-    """Both chunk kernels (csrc/delta_rule.cu) apply: bf16 on CUDA, dk 128, dv 64 or 128, chunk 64, 16-byte aligned q / k rows;
-    q and k may carry fewer heads than v (grouped keys)."""
+    """Both chunk kernels (csrc/delta_rule.cu) apply: bf16 on CUDA, dk and dv multiples of 8 up to 128, chunk 64, 16-byte aligned
+    q / k / v rows; q and k may carry fewer heads than v (grouped keys)."""
+    dk, dv = q.shape[-1], v.shape[-1]
     ok_view = lambda t: t.stride(3) == 1 and all(x % 8 == 0 for x in t.stride()[:3]) and t.data_ptr() % 16 == 0
-    return (_CHUNK_KERNEL and q.is_cuda and q.dtype == k.dtype == v.dtype == torch.bfloat16 and q.shape[-1] == 128 and v.shape[-1] in (64, 128)
+    return (_CHUNK_KERNEL and q.is_cuda and q.dtype == k.dtype == v.dtype == torch.bfloat16 and 0 < dk <= 128 and dk % 8 == 0 and 0 < dv <= 128 and dv % 8 == 0
             and chunk_size == 64 and v.shape[2] % q.shape[2] == 0 and q.shape[2] == k.shape[2] and ok_view(q) and ok_view(k) and ok_view(v)
             and hasattr(lib(), "tyr_gdr_chunk_prepare") and hasattr(lib(), "tyr_gdr_chunk_scan"))
 
 
-def chunk_gated_delta_rule_fused(q, k, v, g, beta, state: Optional[torch.Tensor] = None):
+def chunk_gated_delta_rule_fused(q, k, v, g, beta, state: Optional[torch.Tensor] = None, lens: Optional[torch.Tensor] = None,
+                                 exact: bool = False, state_out: Optional[torch.Tensor] = None):
     """Two launches: the chunk-local quantities (normalisation, decay, the two 64 x 64 products, the triangular solve) and the
-    recurrence over the chunks.  q, k: [B, S, Hk, 128] with Hk dividing Hv (keys are not repeated); see :func:`chunk_kernels_supported`."""
+    recurrence over the chunks.  q, k: [B, S, Hk, dk] with Hk dividing Hv (keys are not repeated); see :func:`chunk_kernels_supported`.
+    ``lens`` (int32 [B]): tokens of each row; the padding after them leaves the state alone.  ``exact``: split-TF32 products
+    against the state and an fp32 read-out."""
     import ctypes
     B, S, Hk, dk = q.shape
     Hv, dv = v.shape[2], v.shape[3]
     n, BH, dev = (S + 63) // 64, B * Hv, q.device
     f32 = lambda *shape: torch.empty(shape, dtype=torch.float32, device=dev)
-    u, w, qg, kd, intra, glast = f32(BH, n, 64, dv), f32(BH, n, 64, dk), f32(BH, n, 64, dk), f32(BH, n, 64, dk), f32(BH, n, 64, 64), f32(BH, n)
+    u, w, qg, kd, intra, glast = f32(BH, n, 64, -(-dv // 64) * 64), f32(BH, n, 64, 128), f32(BH, n, 64, 128), f32(BH, n, 64, 128), f32(BH, n, 64, 64), f32(BH, n)
     strides = (ctypes.c_longlong * 9)(*[t.stride(i) for t in (q, k, v) for i in range(3)])
     gc, bc = g.float().contiguous(), beta.float().contiguous()
     st = cur_stream(dev)
-    check(lib().tyr_gdr_chunk_prepare(ptr(q), ptr(k), ptr(v), ptr(gc), ptr(bc), ptr(u), ptr(w), ptr(qg), ptr(kd), ptr(intra), ptr(glast), strides,
+    check(lib().tyr_gdr_chunk_prepare(ptr(q), ptr(k), ptr(v), ptr(gc), ptr(bc), ptr(u), ptr(w), ptr(qg), ptr(kd), ptr(intra), ptr(glast), ptr(lens), strides,
                                       B, S, Hk, Hv, dk, dv, st), "gdr_chunk_prepare")
     st_in = None if state is None else state.float().contiguous()
-    st_out = f32(B, Hv, dk, dv)
-    out = torch.empty((B, S, Hv, dv), dtype=torch.bfloat16, device=dev)          # written in the layer's layout by the scan kernel
-    check(lib().tyr_gdr_chunk_scan(ptr(u), ptr(w), ptr(qg), ptr(kd), ptr(intra), ptr(glast), ptr(st_in), ptr(st_out), ptr(out), BH, n, dk, dv, 64, S, Hv, st),
+    st_out = f32(B, Hv, dk, dv) if state_out is None else state_out
+    out = torch.empty((B, S, Hv, dv), dtype=torch.float32 if exact else torch.bfloat16, device=dev)   # the layer's layout, from the scan kernel
+    check(lib().tyr_gdr_chunk_scan(ptr(u), ptr(w), ptr(qg), ptr(kd), ptr(intra), ptr(glast), ptr(st_in), ptr(st_out), ptr(out), BH, n, dk, dv, 64, S, Hv, 1 if exact else 0, st),
           "gdr_chunk_scan")
     return out, st_out
 
@@ -109,6 +132,11 @@ def causal_conv1d_silu(x: torch.Tensor, weight: torch.Tensor, bias: Optional[tor
     """x: [B, S, C] (channels last), weight: [C, K] -> silu(causal depthwise conv + bias) as [B, S, C], zero history."""
     B, S, C = x.shape
     K = weight.shape[-1]
+    if x.is_cuda and bias is None and x.stride(2) == 1 and (x.dtype == torch.float32 or K > 4 or C % 8):
+        y = torch.empty((B, S, C), dtype=x.dtype, device=x.device)
+        wf = weight.reshape(C, K).float().contiguous()
+        check(lib().tyr_conv_silu(ptr(x), ptr(wf), ptr(y), B, S, C, K, x.stride(0), x.stride(1), _dt(x), cur_stream(x.device)), "conv_silu")
+        return y
     if (x.is_cuda and x.dtype == torch.bfloat16 and C % 8 == 0 and K <= 4 and x.stride(2) == 1 and x.stride(0) % 8 == 0 and x.stride(1) % 8 == 0
             and x.data_ptr() % 16 == 0 and hasattr(lib(), "tyr_causal_conv1d_silu")):
         y = torch.empty((B, S, C), dtype=x.dtype, device=x.device)
@@ -174,7 +202,7 @@ def gdr_decode_step(q, k, v, g, beta, state: torch.Tensor) -> torch.Tensor:
         gc, bc = g.float().contiguous(), beta.float().contiguous()
         if _tile_ok(dv, v, None, B * Hv):
             check(lib().tyr_gdr_decode_tile(ptr(q), ptr(k), ptr(v), ptr(gc), ptr(bc), ptr(state), ptr(out), B, Hk, Hv, dk,
-                                            q.stride(0), v.stride(0), None, 0, None, 0.0, ptr(err_word(q.device)),
+                                            q.stride(0), v.stride(0), None, 0, None, 0.0, 1, ptr(err_word(q.device)),
                                             cur_stream(q.device)), "gdr_decode_tile")
             return out
         check(lib().tyr_gdr_decode(ptr(q), ptr(k), ptr(v), ptr(gc), ptr(bc), ptr(state), ptr(out), B, Hk, Hv, dk, dv,
@@ -213,14 +241,14 @@ def gdn_decode_fused_supported(mixed, conv_state, rec_state, dk: int, dv: int) -
 
 
 def gdn_decode_fused(mixed, z, b, a, conv_state, conv_w, conv_b, dt_bias, a_log, norm_w, eps: float, rec_state,
-                     Hk: int, Hv: int, dk: int, dv: int) -> torch.Tensor:
+                     Hk: int, Hv: int, dk: int, dv: int, exact: bool = False) -> torch.Tensor:
     """One GatedDeltaNet decode token between the input and output projections in two launches.
 
     ``mixed`` [B, 1, cd] (q | k | v channels), ``z`` [B, 1, Hv*dv], ``b`` / ``a`` [B, 1, Hv]: column windows of one projection
     output or separate tensors (rows may be strided).  Kernel 1: causal conv + bias + SiLU with ``conv_state`` ([B, cd, K] bf16) shifted in place,
     beta = sigmoid(b), g = -softplus(a + dt_bias) * exp(a_log).  Kernel 2: the recurrent step on ``rec_state`` (fp32
     [B, Hv, dk, dv], in place; L2-normalised q / k inside) with the gated RMSNorm ``norm(o) * norm_w * silu(z)`` in its
-    epilogue.  Returns [B, 1, Hv*dv].  Model.lean:642-779 of the reference, which issues library ops."""
+    epilogue (``exact``: of the fp32 read-out, else of the read-out rounded to bf16; tile form only).  Returns [B, 1, Hv*dv].  Model.lean:642-779 of the reference, which issues library ops."""
     B, _, cd = mixed.shape
     K = conv_state.shape[-1]
     assert b.stride(-1) == 1 and a.stride(-1) == 1 and z.stride(-1) == 1 and b.dtype == a.dtype == z.dtype == torch.bfloat16
@@ -241,8 +269,104 @@ def gdn_decode_fused(mixed, z, b, a, conv_state, conv_w, conv_b, dt_bias, a_log,
     nw = norm_w if (norm_w.dtype == torch.bfloat16 and norm_w.is_contiguous()) else norm_w.to(torch.bfloat16).contiguous()
     if _tile_ok(dv, v, z, B * Hv):
         check(lib().tyr_gdr_decode_tile(ptr(q), ptr(k), ptr(v), ptr(g), ptr(beta), ptr(rec_state), ptr(out), B, Hk, Hv, dk, cd, cd,
-                                        ptr(z), z.stride(0), ptr(nw), eps, ptr(err_word(dev)), cur_stream(dev)), "gdr_decode_tile")
+                                        ptr(z), z.stride(0), ptr(nw), eps, 0 if exact else 1, ptr(err_word(dev)), cur_stream(dev)), "gdr_decode_tile")
         return out
     check(lib().tyr_gdr_decode_norm(ptr(q), ptr(k), ptr(v), ptr(g), ptr(beta), ptr(rec_state), ptr(out), B, Hk, Hv, dk, dv, cd, cd,
                                     ptr(z), z.stride(0), ptr(nw), eps, cur_stream(dev)), "gdr_decode_norm")
     return out
+
+
+# ---- any head size, bf16 or fp32, rows of unequal length (csrc/delta_general.cu; plain PyTorch off the GPU) ---------------------
+def delta_gates(b: torch.Tensor, a: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor):
+    """b, a: [B, S, Hv] projections (rows may be strided) -> fp32 (g, beta): log decay ``-exp(a_log) softplus(a + dt_bias)`` and
+    write strength ``sigmoid(b)``."""
+    if not b.is_cuda:
+        return -torch.exp(a_log.float()) * torch.nn.functional.softplus(a.float() + dt_bias.float()), torch.sigmoid(b.float())
+    B, S, Hv = b.shape
+    g = torch.empty((B, S, Hv), dtype=torch.float32, device=b.device)
+    beta = torch.empty_like(g)
+    assert b.stride(2) == a.stride(2) == 1 and b.stride(0) == S * b.stride(1) and a.stride(0) == S * a.stride(1) and b.dtype == a.dtype
+    check(lib().tyr_delta_gates(ptr(b), ptr(a), b.stride(1), a.stride(1), ptr(dt_bias), ptr(a_log), ptr(g), ptr(beta), B * S, Hv, _dt(b),
+                                cur_stream(b.device)), "delta_gates")
+    return g, beta
+
+
+def recurrent_delta(q, k, v, g, beta, state: torch.Tensor, lens: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The recurrence token by token with fp32 state, arithmetic and read-out.  q, k: [B, S, Hk, dk]; v: [B, S, Hv, dv] (views with
+    contiguous channels); ``state`` fp32 [B, Hv, dk, dv] is advanced IN PLACE over the first ``lens[b]`` tokens of row b; the
+    read-out [B, S, Hv, dv] is zero past them."""
+    B, S, Hk, dk = q.shape
+    Hv, dv = v.shape[2], v.shape[3]
+    if not q.is_cuda:
+        rep = Hv // Hk
+        n = lens.tolist() if lens is not None else [S] * B
+        out = torch.zeros(B, S, Hv, dv, dtype=torch.float32)
+        for r in range(B):
+            sl = lambda t: t[r:r + 1, :n[r]].float()
+            o, st = recurrent_gated_delta_rule(sl(q).repeat_interleave(rep, 2), sl(k).repeat_interleave(rep, 2), sl(v), sl(g), sl(beta), state[r:r + 1])
+            out[r, :n[r]] = o[0]
+            state[r] = st[0]
+        return out
+    import ctypes
+    assert state.dtype == torch.float32 and state.is_contiguous() and q.stride(3) == k.stride(3) == v.stride(3) == 1 and q.dtype == k.dtype == v.dtype
+    out = torch.empty((B, S, Hv, dv), dtype=torch.float32, device=q.device)
+    strides = (ctypes.c_longlong * 9)(*[t.stride(i) for t in (q, k, v) for i in range(3)])
+    check(lib().tyr_gdr_recurrent(ptr(q), ptr(k), ptr(v), ptr(g.contiguous()), ptr(beta.contiguous()), ptr(state), ptr(out), ptr(lens), strides,
+                                  B, S, Hk, Hv, dk, dv, _dt(q), cur_stream(q.device)), "gdr_recurrent")
+    return out
+
+
+def delta_prefill(q, k, v, g, beta, state: torch.Tensor, lens: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Fresh prompts (the state starts at zero): fp32 read-out [B, S, Hv, dv]; ``state`` receives the state after each row's last
+    token.  The tensor-core chunk form where it applies, else the recurrence."""
+    if q.is_cuda and q.shape[1] > 1 and chunk_kernels_supported(q, k, v):
+        return chunk_gated_delta_rule_fused(q, k, v, g, beta, None, lens, exact=True, state_out=state)[0]
+    state.zero_()
+    return recurrent_delta(q, k, v, g, beta, state, lens)
+
+
+def gated_norm(o: torch.Tensor, z: torch.Tensor, w: torch.Tensor, eps: float) -> torch.Tensor:
+    """``o / sqrt(mean(o^2) + eps) * w * silu(z)`` per head: o fp32 [B, S, Hv, dv], z [B, S, Hv*dv] (rows may be strided),
+    w fp32 [dv] -> [B, S, Hv*dv] in z's dtype."""
+    B, S, Hv, dv = o.shape
+    if not o.is_cuda:
+        y = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+        return (y * torch.nn.functional.silu(z.float()).reshape(B, S, Hv, dv)).reshape(B, S, Hv * dv).to(z.dtype)
+    assert z.stride(2) == 1 and z.stride(0) == S * z.stride(1) and o.is_contiguous()
+    y = torch.empty((B, S, Hv * dv), dtype=z.dtype, device=z.device)
+    check(lib().tyr_gated_norm(ptr(o), ptr(z), z.stride(1), ptr(w), ptr(y), B * S, Hv, dv, eps, _dt(z), cur_stream(z.device)), "gated_norm")
+    return y
+
+
+def conv_window(x: torch.Tensor, K: int, lens: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The last K inputs of every channel at the end of each row ([B, S, C] -> [B, C, K], zeros before the start): the state a
+    decode step continues from."""
+    B, S, C = x.shape
+    end = torch.full((B,), S, device=x.device, dtype=torch.long) if lens is None else lens.long()
+    t = end[:, None] - K + torch.arange(K, device=x.device)
+    win = torch.gather(x, 1, t.clamp_min(0)[:, :, None].expand(B, K, C))
+    return (win * (t >= 0).to(x.dtype)[:, :, None]).transpose(1, 2).contiguous()
+
+
+def delta_decode(mixed, z, b, a, conv_state, conv_w, dt_bias, a_log, norm_w, eps: float, rec_state, Hk: int, Hv: int, dk: int, dv: int):
+    """One token of a gated delta layer between its input and output projections: convolution window and state advanced in
+    place, fp32 gates, recurrence, read-out and norm.  Shapes as in :func:`gdn_decode_fused` (no convolution bias)."""
+    if gdn_decode_fused_supported(mixed, conv_state, rec_state, dk, dv) and conv_state.shape[-1] <= 8 and _tile_ok(dv, mixed, z, mixed.shape[0] * Hv):
+        return gdn_decode_fused(mixed, z, b, a, conv_state, conv_w, None, dt_bias, a_log, norm_w, eps, rec_state, Hk, Hv, dk, dv, exact=True)
+    B, _, C = mixed.shape
+    K = conv_state.shape[-1]
+    if mixed.is_cuda:
+        dev = mixed.device
+        y = torch.empty((B, 1, C), dtype=mixed.dtype, device=dev)
+        g = torch.empty((B, 1, Hv), dtype=torch.float32, device=dev)
+        beta = torch.empty_like(g)
+        assert conv_state.is_contiguous() and conv_state.dtype == mixed.dtype and mixed.stride(2) == b.stride(2) == a.stride(2) == 1
+        check(lib().tyr_delta_conv_gates(ptr(mixed), ptr(b), ptr(a), mixed.stride(0), b.stride(0), a.stride(0), ptr(conv_state), ptr(conv_w.float()),
+                                         ptr(dt_bias), ptr(a_log), ptr(y), ptr(g), ptr(beta), B, C, K, Hv, _dt(mixed), cur_stream(dev)), "delta_conv_gates")
+    else:
+        conv_state.copy_(torch.cat([conv_state[:, :, 1:], mixed.transpose(1, 2)], dim=2))
+        y = torch.nn.functional.silu((conv_state.float() * conv_w.float()).sum(-1)).to(mixed.dtype).unsqueeze(1)
+        g, beta = delta_gates(b, a, dt_bias, a_log)
+    kd = Hk * dk
+    q, k, v = y[..., :kd].reshape(B, 1, Hk, dk), y[..., kd:2 * kd].reshape(B, 1, Hk, dk), y[..., 2 * kd:].reshape(B, 1, Hv, dv)
+    return gated_norm(recurrent_delta(q, k, v, g, beta, rec_state), z, norm_w.float(), eps)

@@ -31,6 +31,10 @@ def _sigs(lib_):
         if fn is not None:
             fn.argtypes = args
             fn.restype = ctypes.c_int
+    fn = getattr(lib_, "tyr_flash_fwd_biased", None)
+    if fn is not None:
+        fn.argtypes = [P, P, P, P, P, P, I, I, I, I, I, I, ctypes.POINTER(L), I, F, P, P]
+        fn.restype = ctypes.c_int
     fn = getattr(lib_, "tyr_flash_bwd_workspace_bytes", None)
     if fn is not None:
         fn.argtypes = [I, I, I]
@@ -72,6 +76,25 @@ def flash_fwd_bthd(q, k, v, *, causal: bool, window: Optional[int], scale: Optio
                               *_bthd_strides(out), 1 if causal else 0, int(window or 0), q_offset, sc,
                               ptr(err_word(q.device)), cur_stream(q.device)), "flash_fwd")
     return out, lse
+
+
+def biased_supported(q, k, v) -> bool:
+    """[B, T, H, D] bf16 views; query / key and value sizes up to 128, multiples of 8."""
+    return (has_fwd() and q.is_cuda and q.dtype == k.dtype == v.dtype == torch.bfloat16 and q.shape[2] % k.shape[2] == 0
+            and all(t.shape[3] <= 128 and t.shape[3] % 8 == 0 and _ok_view(t) for t in (q, k, v)))
+
+
+def flash_fwd_biased(q, k, v, r1, r2, *, window: Optional[int], scale: float) -> torch.Tensor:
+    """Causal attention of whole prompts with ``r1[h] ln(1 + r2[h] (i - j))`` taken off the scores.  q: [B, T, Hq, dk],
+    k: [B, T, Hkv, dk], v: [B, T, Hkv, dv] (views), r1 / r2 fp32 [Hq] -> [B, T, Hq, dv]."""
+    import ctypes
+    B, T, Hq, dk = q.shape
+    Hkv, dv = k.shape[2], v.shape[3]
+    out = torch.empty((B, T, Hq, dv), dtype=q.dtype, device=q.device)
+    strides = (ctypes.c_longlong * 12)(*[x for t in (q, k, v, out) for x in _bthd_strides(t)])
+    check(lib().tyr_flash_fwd_biased(ptr(q), ptr(k), ptr(v), ptr(out), ptr(r1), ptr(r2), B, Hq, Hkv, T, dk, dv, strides, int(window or 0), scale,
+                                     ptr(err_word(q.device)), cur_stream(q.device)), "flash_fwd_biased")
+    return out
 
 
 def flash_bwd_bthd(do, q, k, v, o, lse, *, causal, window, scale, q_offset=None):

@@ -12,6 +12,7 @@ from __future__ import annotations
 
 import collections
 import os
+import weakref
 from dataclasses import dataclass
 from typing import Dict, Optional, Tuple
 
@@ -30,8 +31,8 @@ def _sigs(lib_):
     P, I, L, F = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong, ctypes.c_float
     table = {
         "tyr_nvfp4_quantize": [P, P, P, P, L, L, P], "tyr_nvfp4_dequant": [P, P, P, P, L, L, P],
-        "tyr_moe_route": [P, P, P, P, P, I, I, I, I, I, F, F, P],
-        "tyr_moe_route_fused": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, F, P],
+        "tyr_moe_route": [P, P, P, P, P, I, I, I, I, I, F, F, I, I, P],
+        "tyr_moe_route_fused": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, F, I, I, P],
         "tyr_moe_layout": [P, P, P, P, P, P, P, P, I, I, P], "tyr_moe_count": [P, P, I, I, P],
         "tyr_moe_gather_rows": [P, P, P, I, I, I, P], "tyr_moe_combine": [P, P, P, P, P, I, I, I, P],
         "tyr_moe_fp4_gemv": [P] * 17 + [I, I, I, I, I, P], "tyr_moe_finalize": [P, P, P, L, P],
@@ -111,10 +112,12 @@ def nvfp4_dequant(packed: torch.Tensor, scales: torch.Tensor, global_scale: torc
 
 # ---- routing -------------------------------------------------------------------------------------------
 def route(logits: torch.Tensor, k: int, *, softmax: bool = False, bias: Optional[torch.Tensor] = None,
-          renorm: bool = True, softcap: float = 0.0, scale: float = 1.0, want_counts: bool = True):
+          renorm: bool = True, softcap: float = 0.0, scale: float = 1.0, want_counts: bool = True, groups: int = 1, keep: int = 1):
     """logits fp32 [T, E] -> (ids int32 [T, k], weights fp32 [T, k], counts int32 [E]).
     Sigmoid (Laguna, Tyr/Model/Laguna/MoE.lean:71-90) or softmax (Qwen3.5) scores; the selection
-    bias only influences WHICH experts are picked; ties go to the lower expert index."""
+    bias only influences WHICH experts are picked; ties go to the lower expert index.  With ``groups`` > 1 the experts form
+    that many equal groups of neighbours, a group counts by its best selection score (bias included), and only experts of the
+    ``keep`` best groups compete."""
     T, E = logits.shape
     if logits.is_cuda:
         lg = logits.float().contiguous()
@@ -123,13 +126,17 @@ def route(logits: torch.Tensor, k: int, *, softmax: bool = False, bias: Optional
         counts = torch.zeros(E, dtype=torch.int32, device=logits.device)
         b = bias.float().contiguous() if bias is not None else None
         check(lib().tyr_moe_route(ptr(lg), ptr(b), ptr(ids), ptr(w), ptr(counts), T, E, k, 1 if softmax else 0,
-                                  1 if renorm else 0, softcap, scale, cur_stream(logits.device)), "moe_route")
+                                  1 if renorm else 0, softcap, scale, groups, keep, cur_stream(logits.device)), "moe_route")
         return ids, w, counts
     l = logits.float()
     if softcap > 0:
         l = softcap * torch.tanh(l / softcap)
     scores = torch.softmax(l, -1) if softmax else torch.sigmoid(l)
     sel = scores + bias.float() if bias is not None else scores
+    if groups > 1:
+        best = sel.reshape(T, groups, E // groups).amax(-1)
+        kept = torch.zeros(T, groups, dtype=torch.bool).scatter_(1, torch.argsort(best, dim=-1, descending=True, stable=True)[:, :keep], True)
+        sel = sel.masked_fill(~kept.repeat_interleave(E // groups, dim=1), float("-inf"))
     order = torch.argsort(sel, dim=-1, descending=True, stable=True)[:, :k]
     w = torch.gather(scores, 1, order)
     if renorm:
@@ -163,7 +170,7 @@ def route_fused_supported(x: torch.Tensor, router_w: torch.Tensor) -> bool:
 
 
 def route_fused(x: torch.Tensor, router_w: torch.Tensor, k: int, *, softmax: bool = False, bias: Optional[torch.Tensor] = None,
-                renorm: bool = True, softcap: float = 0.0, scale: float = 1.0):
+                renorm: bool = True, softcap: float = 0.0, scale: float = 1.0, groups: int = 1, keep: int = 1):
     """x bf16 [T, h], router_w fp32 [E, h] -> (ids, weights, counts) as :func:`route` of ``x.float() @ router_w.T`` (fp32
     accumulation inside the kernel; the logits are never written out)."""
     T, E = x.shape[0], router_w.shape[0]
@@ -174,7 +181,7 @@ def route_fused(x: torch.Tensor, router_w: torch.Tensor, k: int, *, softmax: boo
     logits = torch.empty((T, E), dtype=torch.float32, device=x.device)
     b = bias.float().contiguous() if bias is not None else None
     check(lib().tyr_moe_route_fused(ptr(x), ptr(router_w), ptr(b), ptr(logits), ptr(tickets), ptr(ids), ptr(w), ptr(counts), T, E, k, x.shape[1], 1 if softmax else 0,
-                                    1 if renorm else 0, softcap, scale, cur_stream(x.device)), "moe_route_fused")
+                                    1 if renorm else 0, softcap, scale, groups, keep, cur_stream(x.device)), "moe_route_fused")
     return ids, w, counts
 
 
@@ -358,7 +365,7 @@ def moe_fp4_forward(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, e
     return fp4.moe_fp4_tc_forward(x, ids, wf, ex, offsets, order, tiles, add=add)
 
 
-_gu_cache: Dict[int, torch.Tensor] = {}
+_gu_cache: Dict[int, Tuple["weakref.ref", torch.Tensor]] = {}
 
 
 def interleave_gate_up(gate_up: torch.Tensor) -> torch.Tensor:
@@ -366,8 +373,16 @@ def interleave_gate_up(gate_up: torch.Tensor) -> torch.Tensor:
     SwiGLU epilogue; mi is padded to a multiple of 128 with zero rows.  Cached per source tensor."""
     key = gate_up.data_ptr()
     hit = _gu_cache.get(key)
-    if hit is not None and hit.shape[0] == gate_up.shape[0]:
-        return hit
+    if hit is not None and hit[0]() is gate_up:             # an address alone may belong to a new tensor by now
+        return hit[1]
+    out = _interleave(gate_up)
+    if len(_gu_cache) > 256:
+        _gu_cache.clear()
+    _gu_cache[key] = (weakref.ref(gate_up), out)
+    return out
+
+
+def _interleave(gate_up: torch.Tensor) -> torch.Tensor:
     E, two_mi, h = gate_up.shape
     mi = two_mi // 2
     g, u = gate_up[:, :mi], gate_up[:, mi:]
@@ -375,11 +390,53 @@ def interleave_gate_up(gate_up: torch.Tensor) -> torch.Tensor:
     if pad:
         g, u = torch.nn.functional.pad(g, (0, 0, 0, pad)), torch.nn.functional.pad(u, (0, 0, 0, pad))
     mp = mi + pad
-    out = torch.stack([g.reshape(E, mp // 128, 128, h), u.reshape(E, mp // 128, 128, h)], dim=2).reshape(E, 2 * mp, h).contiguous()
-    if len(_gu_cache) > 256:
-        _gu_cache.clear()
-    _gu_cache[key] = out
-    return out
+    return torch.stack([g.reshape(E, mp // 128, 128, h), u.reshape(E, mp // 128, 128, h)], dim=2).reshape(E, 2 * mp, h).contiguous()
+
+
+def _deinterleave(tiled: torch.Tensor, mi: int) -> torch.Tensor:
+    E, rows, h = tiled.shape
+    gu = tiled.reshape(E, rows // 256, 2, 128, h).transpose(1, 2).reshape(E, 2, rows // 2, h)
+    return torch.cat([gu[:, 0, :mi], gu[:, 1, :mi]], dim=1)
+
+
+class ExpertBank:
+    """Expert banks ``gate_up`` [E, 2*mi, h] and ``down`` [E, h, mi].  The first grouped product turns them into the layout that
+    GEMM reads (gate / up interleaved per 128 rows, mi padded to a multiple of 128), which then replaces the plain one."""
+
+    def __init__(self, gate_up: torch.Tensor, down: torch.Tensor):
+        self.num_experts, self.moe_int = gate_up.shape[0], gate_up.shape[1] // 2
+        self._plain: Optional[Tuple[torch.Tensor, torch.Tensor]] = (gate_up, down)
+        self._tiled: Optional[Tuple[torch.Tensor, torch.Tensor]] = None
+
+    @property
+    def gate_up(self) -> torch.Tensor:
+        return self._plain[0] if self._plain is not None else _deinterleave(self._tiled[0], self.moe_int)
+
+    @property
+    def down(self) -> torch.Tensor:
+        return self._plain[1] if self._plain is not None else self._tiled[1][..., :self.moe_int].contiguous()
+
+    def tiled(self) -> Tuple[torch.Tensor, torch.Tensor]:
+        if self._tiled is None:
+            gate_up, down = self._plain
+            self._tiled = (_interleave(gate_up), torch.nn.functional.pad(down, (0, (-self.moe_int) % 128)).contiguous())
+            self._plain = None
+        return self._tiled
+
+
+def grouped_supported(x: torch.Tensor, mi: int) -> bool:
+    """The grouped tensor-core path of :func:`moe_bank_forward` applies (no host synchronisation, so a step can be captured)."""
+    return x.is_cuda and x.dtype == torch.bfloat16 and x.shape[-1] % 8 == 0 and mi % 8 == 0
+
+
+def moe_bank_forward(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, bank: ExpertBank, counts: Optional[torch.Tensor] = None,
+                     add: Optional[torch.Tensor] = None, act: str = "swiglu") -> torch.Tensor:
+    """``sum_s weights[t, s] expert_{ids[t, s]}(x[t])`` (+ ``add``) over an :class:`ExpertBank`; x: [T, h]."""
+    if not grouped_supported(x, bank.moe_int):
+        gu, mi = bank.gate_up, bank.moe_int
+        y = moe_eager(x, ids, weights, gu[:, :mi], gu[:, mi:], bank.down, act=act)
+        return y if add is None else (y.float() + add.float()).to(x.dtype)
+    return _moe_grouped(x, ids, weights, *bank.tiled(), counts, add, act)
 
 
 def moe_dense_forward(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor,
@@ -387,23 +444,25 @@ def moe_dense_forward(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
     """bf16 expert banks: ``gate_up`` [E, 2*mi, h], ``down`` [E, h, mi].  Grouped tensor-core path on the
     GPU for bf16; per-expert loop otherwise (Tyr/Model/Qwen35/Model.lean:200-248 computes the same sum
     by gathering one expert matrix per (token, slot))."""
-    T, h = x.shape
-    E, two_mi, _ = gate_up.shape
-    mi = two_mi // 2
-    k = ids.shape[1]
-    if not (x.is_cuda and x.dtype == torch.bfloat16 and gate_up.dtype == torch.bfloat16 and h % 8 == 0 and mi % 8 == 0):
+    mi = gate_up.shape[1] // 2
+    if not (grouped_supported(x, mi) and gate_up.dtype == torch.bfloat16):
         y = moe_eager(x, ids, weights, gate_up[:, :mi], gate_up[:, mi:], down, act=act)
         return y if add is None else (y.float() + add.float()).to(x.dtype)
+    dn = down if mi % 128 == 0 else torch.nn.functional.pad(down, (0, (-mi) % 128))
+    return _moe_grouped(x, ids, weights, interleave_gate_up(gate_up), dn.contiguous(), counts, add, act)
+
+
+def _moe_grouped(x, ids, weights, gu, dn, counts, add, act):
+    T, h = x.shape
+    k = ids.shape[1]
     if counts is None:
-        counts = count_experts(ids, E)
+        counts = count_experts(ids, gu.shape[0])
     offsets, order, pos, tiles = layout(ids.to(torch.int32), counts, want_tiles=True)
     st = cur_stream(x.device)
-    gu = interleave_gate_up(gate_up)
-    dn = down if mi % 128 == 0 else torch.nn.functional.pad(down, (0, (-mi) % 128)).contiguous()
     xs = torch.empty((T * k, h), dtype=x.dtype, device=x.device)
     check(lib().tyr_moe_gather_rows(ptr(x.contiguous()), ptr(order), ptr(xs), T * k, k, h, st), "moe_gather_rows")
     hid = grouped_gemm(xs, gu, offsets, tiles, act=act)
-    y = grouped_gemm(hid, dn.contiguous(), offsets, tiles)
+    y = grouped_gemm(hid, dn, offsets, tiles)
     out = torch.empty_like(x)
     check(lib().tyr_moe_combine(ptr(y), ptr(pos), ptr(weights.float().contiguous()), ptr(add.contiguous() if add is not None else None),
                                 ptr(out), T, k, h, st), "moe_combine")

@@ -13,7 +13,17 @@ from typing import Optional, Sequence
 
 import torch
 
+from .._native import register_signatures
 from ._common import check, cur_stream, lib, ptr
+
+
+@register_signatures
+def _sigs(lib_):
+    P, I, L, F = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong, ctypes.c_float
+    fn = getattr(lib_, "tyr_post_norm_residual", None)
+    if fn is not None:
+        fn.argtypes = [P, L, P, I, P, P, L, I, F, I, I, P]
+        fn.restype = I
 
 EPS = 1e-6
 
@@ -132,3 +142,28 @@ def rms_norm_weighted(x: torch.Tensor, weight: Optional[torch.Tensor], eps: floa
         y = y * torch.nn.functional.silu(gate.float())
     y = y.to(x.dtype)
     return (y, r_out) if (return_residual and residual is not None) else y
+
+
+def post_norm_residual(x: torch.Tensor, gain: torch.Tensor, eps: float, resid: Optional[torch.Tensor] = None,
+                       out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """``r = resid + norm(x) * gain`` with an fp32 residual stream updated IN PLACE (``norm(x) * gain`` alone without one), returned
+    as a copy in ``out_dtype`` (default: x's).  ``gain``: fp32, one number for all channels or one per channel.  An fp32 result of
+    an fp32 stream is the stream itself."""
+    D = x.shape[-1]
+    out_dtype = x.dtype if out_dtype is None else out_dtype
+    if not x.is_cuda:
+        y = rms_norm_ref(x, eps) * gain
+        if resid is not None:
+            resid += y
+            y = resid
+        return y.to(out_dtype)
+    kinds = {torch.bfloat16: 0, torch.float32: 1}
+    xr = x if x.dim() == 2 and x.stride(1) == 1 else x.reshape(-1, D)
+    if xr.stride(-1) != 1:
+        xr = xr.contiguous()
+    assert gain.dtype == torch.float32 and (resid is None or (resid.dtype == torch.float32 and resid.is_contiguous() and resid.numel() == xr.numel()))
+    same = resid is not None and out_dtype == torch.float32
+    y = None if same else torch.empty(x.shape, dtype=out_dtype, device=x.device)
+    check(lib().tyr_post_norm_residual(ptr(xr), xr.stride(0), ptr(gain), gain.numel(), ptr(resid), ptr(y), xr.shape[0], D, eps, kinds[x.dtype],
+                                       kinds[out_dtype], cur_stream(x.device)), "post_norm_residual")
+    return resid.view(x.shape) if same else y

@@ -2,7 +2,8 @@
 
 The step function must be free of host reads and host-dependent shapes: positions live in device tensors, stores are
 updated in place.  State that a step advances non-idempotently (position counters, recurrent states) is listed by the
-caller; it is saved before the warm-up runs and the capture, and restored afterwards, so capturing costs no step."""
+caller; it is saved before the warm-up runs and the capture, and restored after each of them, so capturing costs no step and
+every warm-up run writes the store slots of the step itself (a second position would overwrite the oldest key of a full ring)."""
 from __future__ import annotations
 
 from typing import Callable, Optional, Sequence
@@ -21,6 +22,8 @@ class GraphedStep:
         with torch.cuda.stream(side), torch.no_grad():
             for _ in range(warmup):                       # allocates workspaces, builds fused weights, loads modules
                 fn(*self.static_in)
+                for t, s in zip(advancing_state, saved):
+                    t.copy_(s)
         torch.cuda.current_stream().wait_stream(side)
         torch.cuda.synchronize()
         from ..ops import _common as opc
