@@ -25,6 +25,10 @@ __device__ __forceinline__ float dg_log_decay(float a, float dt_bias, float a_lo
   return -expf(a_log) * sp;
 }
 
+// exp(g) for a log decay g <= 0.  Close to 1 the result is 1 + expm1(g), rounded once: a one-ulp bias of exp itself, applied at
+// every token, would add up over the memory of a slowly decaying head.
+__device__ __forceinline__ float dg_decay(float g) { return g > -0.5f ? 1.f + expm1f(g) : expf(g); }
+
 // y[b, s, c] = silu(sum_j w[c, j] x[b, s - (K - 1) + j, c]); x rows strided, y contiguous
 template <typename T>
 __global__ void __launch_bounds__(256) conv_silu_kernel(const T* __restrict__ x, const float* __restrict__ w, T* __restrict__ y,
@@ -153,7 +157,7 @@ __global__ void __launch_bounds__(REC_WARPS * 32) gdr_recurrent_kernel(Recurrent
       const int d = lane + 32 * e;
       if (d < DKM) { sq[warp][d] = nq[e] * qn; sk[warp][d] = nk[e] * kn; }
     }
-    const float v = nv, decay = expf(ng), beta = nb;
+    const float v = nv, decay = dg_decay(ng), beta = nb;
     __syncwarp();
     if (t + 1 < n) fetch(t + 1);
     float kv = 0.f;

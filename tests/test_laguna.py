@@ -161,6 +161,9 @@ def test_gpu_laguna_bf16_fused_decode_matches_eager():
                    num_experts_per_tok=4, moe_intermediate_size=128, shared_expert_intermediate_size=128,
                    intermediate_size=512, sliding_window=128)
     m = L.init(cfg, device="cuda", dtype=torch.bfloat16)
+    for l in m.layers:
+        if not isinstance(l.ffn, L.DenseMLP):         # a fixed order of the experts: no near-tie in a router can flip a choice
+            l.ffn.router.e_score_correction_bias = torch.randperm(cfg.num_experts, device="cuda").float()
     ids = torch.randint(3, 97, (2, 200), device="cuda")
     with torch.no_grad():
         ref = L.forward(m, ids, use_fused=False).float()
@@ -172,9 +175,7 @@ def test_gpu_laguna_bf16_fused_decode_matches_eager():
             for t in range(190, 200):
                 errs.append((sess.step(ids[:, t], use_fused=fused).float() - ref[:, t]).abs().amax(dim=1))
             ok = (torch.stack(errs) < 0.05 * scale).float().mean().item()
-            # a near-tie in a router can pick a different expert once the arithmetic differs in the last bf16
-            # bit, which changes that row discretely; everything else must agree
-            assert ok >= 0.85, (fused, ok)
+            assert ok == 1.0, (fused, ok)
 
 
 def test_tiny_fixture_generator_is_deterministic_and_self_consistent(tmp_path):

@@ -521,6 +521,22 @@ class CacheSession:
         self.pos += S
         return norm_w(x, self.m.norm, cfg.rms_norm_eps)
 
+    def hidden(self, ids: torch.Tensor, lengths: Optional[Sequence[int]] = None) -> torch.Tensor:
+        """Final normed hidden states [B, S, h] of whole prompts of one length."""
+        if lengths is not None and any(n != ids.shape[1] for n in lengths):
+            raise ValueError("Laguna prefills prompts of one length")
+        return self._run(F.embedding(ids, self.m.embed_tokens), True)
+
+    def head(self, h: torch.Tensor) -> torch.Tensor:
+        return lin(h, self.m.lm_head)
+
+    def retain(self, rows: Sequence[int]) -> None:
+        """Keep these rows of the batch and give back what the others hold."""
+        idx = torch.tensor(list(rows), device=self.m.device)
+        for c in self.caches:
+            c.retain(idx)
+        self.batch, self._graph = len(rows), None
+
     def prefill(self, input_ids: torch.Tensor, use_fused: bool = True) -> torch.Tensor:
         """Returns last-position logits [B, V]."""
         h = self._run(F.embedding(input_ids, self.m.embed_tokens), use_fused)

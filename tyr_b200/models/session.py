@@ -15,7 +15,6 @@ from .common import KVCache, LinearState
 
 class HybridSession:
     name = "hybrid"
-    ragged = False                 # rows of one prefill may have different lengths
 
     def __init__(self, batch: int, max_len: int, device):
         if max_len <= 0:

@@ -445,7 +445,6 @@ class CacheSession(HybridSession):
     """K/V stores of the layers with keys of their own (ring stores of the widest window that reads them) and convolution /
     recurrent states of the delta layers; ``retain`` gives finished rows back."""
     name = "Zatorax"
-    ragged = True
 
     def __init__(self, m: ZatoraxForCausalLM, batch: int, max_len: int):
         super().__init__(batch, max_len, m.device)
