@@ -1,11 +1,12 @@
 """Shared runner for the pretrained text families (counterpart of Examples/ModelRunner.lean and the per-family RunHF
-executables: Qwen3, Qwen2.5-Omni thinker, Qwen3.5 / 3.6, Gemma 4) plus the speech demos (Whisper, Qwen3-ASR).
+executables: Qwen3, Qwen2.5-Omni thinker, Qwen3.5 / 3.6, Gemma 4, Zatorax) plus the speech demos (Whisper, Qwen3-ASR).
 
     python -m tyr_b200.cli.model_runner --family gemma4 --source google/gemma-4-e2b --prompt "Hi" --max-new-tokens 64 --stream
     python -m tyr_b200.cli.model_runner --family qwen3 --source Qwen/Qwen3-4B --prompt-file prompts.txt --batch-size 4
+    python -m tyr_b200.cli.model_runner --source <zatorax dir> --prompt "5 17 3" --max-new-tokens 16        # family from config.json
     python -m tyr_b200.cli.model_runner --family whisper --source openai/whisper-small --audio speech.wav
 
-Common flags: ``--source`` (directory or hub repo id), ``--prompt`` / ``--prompt-file``, ``--batch-size``, ``--max-new-tokens``,
+Common flags: ``--family`` (default ``auto``: by config.json, ``models/registry.py``), ``--source`` (directory or hub repo id), ``--prompt`` / ``--prompt-file``, ``--batch-size``, ``--max-new-tokens``,
 ``--stream``, ``--device`` (auto | cpu | cuda | cuda:N, falling back to CPU with a warning), ``--bench``.
 """
 from __future__ import annotations
@@ -18,10 +19,11 @@ from typing import Callable, List, Optional, Tuple
 import torch
 
 from ..io import hub
+from ..models import registry
 from ..models.generation import SamplingStrategy
 from ..tokenizer import hf as tok_hf
 
-TEXT_FAMILIES = ("qwen3", "qwen25omni", "qwen35", "gemma4")
+TEXT_FAMILIES = ("qwen3", "qwen25omni", "qwen35", "gemma4", "zatorax")
 SPEECH_FAMILIES = ("whisper", "qwen3asr")
 
 
@@ -62,8 +64,14 @@ def left_pad(rows: List[List[int]], pad: int) -> torch.Tensor:
     return torch.tensor([[pad] * (w - len(r)) + r for r in rows])
 
 
+def right_pad(rows: List[List[int]], pad: int) -> Tuple[torch.Tensor, List[int]]:
+    """(ids padded at the end, row lengths)."""
+    w = max(len(r) for r in rows)
+    return torch.tensor([r + [pad] * (w - len(r)) for r in rows]), [len(r) for r in rows]
+
+
 def load_text_family(family: str, model_dir: str, device, dtype):
-    """Returns (generate(ids, max_new, strategy, on_step) -> ids, tokenizer, render(prompt) -> str, eos ids, pad id)."""
+    """Returns (generate(ids, max_new, strategy, on_step[, lengths]) -> ids, tokenizer, render(prompt) -> str, eos ids, pad id)."""
     if family in ("qwen3", "qwen25omni"):
         from ..models import qwen as Q
         lm = Q.load_qwen25_omni_thinker(model_dir, device, dtype) if family == "qwen25omni" else Q.load_from_pretrained(model_dir, device, dtype)
@@ -87,21 +95,40 @@ def load_text_family(family: str, model_dir: str, device, dtype):
         tok = tok_hf.load_gemma4(model_dir)
         gen = lambda ids, n, st_, cb: G.generate(m, ids, n, st_, cfg.eos_token_id, cb)
         return gen, tok, lambda p: tok_hf.gemma_prompt([{"role": "user", "content": p}]), list(cfg.eos_token_id), cfg.pad_token_id or 0
+    if family == "zatorax":
+        import os
+        from ..models import zatorax as Z
+        from ..tokenizer.ids import IdTokenizer
+        m = Z.load_pretrained(model_dir, device, dtype)
+        has_tok = os.path.exists(os.path.join(model_dir, "tokenizer.json"))
+        tok = tok_hf.HFTokenizer.from_file(model_dir) if has_tok else IdTokenizer(m.cfg.vocab)
+        gen = lambda ids, n, st, cb, lengths=None: Z.generate(m, ids, n, st, (), cb, lengths=lengths)
+        return gen, tok, lambda p: p, [], 0
     raise ValueError(f"unknown text family {family}")
 
 
 def run_text(a, device, dtype, out=print) -> int:
     model_dir = hub.resolve_pretrained_dir(a.source, a.revision)
+    if a.family == "auto":
+        a.family = registry.detect_dir(model_dir).name
+        if a.family not in TEXT_FAMILIES:
+            raise ValueError(f"{a.family} has its own command line")
     gen, tok, render, eos, pad = load_text_family(a.family, model_dir, device, dtype)
     strategy = SamplingStrategy.greedy() if a.temperature <= 0 else SamplingStrategy.multinomial(a.temperature, a.top_k, a.top_p)
     prompts = load_prompts(a.prompt_file, a.prompt)
     for chunk in batches(prompts, a.batch_size):
-        ids = left_pad([tok.encode(render(p)) for p in chunk], pad).to(device)
+        rows, extra = [tok.encode(render(p)) for p in chunk], ()
+        if registry.by_name(a.family).ragged:        # prompts padded at the end, their lengths passed on
+            ids, lengths = right_pad(rows, pad)
+            extra = (lengths,)
+        else:
+            ids = left_pad(rows, pad)
+        ids = ids.to(device)
         on_step = None
         if a.stream and len(chunk) == 1:
             on_step = lambda step, t: print(tok.decode([int(t[0])], skip_special=True), end="", flush=True)
         t0 = time.perf_counter()
-        res = gen(ids, a.max_new_tokens, strategy, on_step)
+        res = gen(ids, a.max_new_tokens, strategy, on_step, *extra)
         if device.type == "cuda":
             torch.cuda.synchronize(device)
         dt = time.perf_counter() - t0
@@ -144,7 +171,7 @@ def run_speech(a, device, dtype, out=print) -> int:
 
 def parse(argv):
     p = argparse.ArgumentParser(prog="model_runner")
-    p.add_argument("--family", required=True, choices=TEXT_FAMILIES + SPEECH_FAMILIES)
+    p.add_argument("--family", default="auto", choices=("auto",) + TEXT_FAMILIES + SPEECH_FAMILIES)
     p.add_argument("--source", required=True)
     p.add_argument("--revision", default=None)
     p.add_argument("--prompt", default="Hello!")
