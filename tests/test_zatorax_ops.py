@@ -232,7 +232,7 @@ def test_step_attention_rows_at_their_own_positions(place, H, G, dk, dv, window,
     """Twelve tokens per row from unequal positions, over plain stores and over rings whose windows are as wide or narrower;
     a layer that reads the same keys with half the window and without appending."""
     dev, dt = place
-    B, steps, eps, scale = 3, 12, 1e-5, 0.4
+    B, steps, eps, scale = 3, 12, 1e-5, 1.6 * dk ** -0.5
     T = max(start) + steps
     y, qw, kw = rnd(B, T, (H + G) * dk + G * dv), rnd(dk).abs() + 0.5, rnd(dk).abs() + 0.5
     r1, r2 = rnd(H).abs(), rnd(H).abs() * 0.3

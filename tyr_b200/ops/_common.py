@@ -64,6 +64,14 @@ def raise_on_device_error(device=None):
             "(1=mbarrier timeout, 2=peer flag timeout, 3=bounds, 4=tmem)")
 
 
+def row_stride(t: torch.Tensor) -> int:
+    """Elements between consecutive rows of a [B, S, C] view with contiguous channels whose B * S rows are evenly spaced."""
+    B, S = t.shape[:2]
+    if t.stride(2) != 1 or (B > 1 and S > 1 and t.stride(0) != S * t.stride(1)):
+        raise ValueError(f"rows of a [B, S, C] operand must be evenly spaced, got strides {t.stride()} for {tuple(t.shape)}")
+    return t.stride(1) if S > 1 else t.stride(0)
+
+
 def is_cuda(*ts) -> bool:
     return any(t is not None and t.is_cuda for t in ts)
 

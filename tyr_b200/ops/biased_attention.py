@@ -16,7 +16,7 @@ import torch
 from .._native import register_signatures
 from . import decode_attention as da
 from . import flash
-from ._common import check, cur_stream, err_word, lib, ptr
+from ._common import check, cur_stream, err_word, lib, ptr, row_stride
 
 MAX_HEAD = 256
 
@@ -75,11 +75,10 @@ def qk_norm_store(y: torch.Tensor, q_w: torch.Tensor, k_w: Optional[torch.Tensor
                 store.k[b, :, slots] = k[b, s0:n].transpose(0, 1)
                 store.v[b, :, slots] = v[b, s0:n].transpose(0, 1)
         return q, k, v
-    assert y.stride(2) == 1 and y.stride(0) == S * y.stride(1)
     q = torch.empty((B, S, H, dkp), dtype=y.dtype, device=y.device)
     k = torch.empty((B, S, G, dkp), dtype=y.dtype, device=y.device) if G else None
     v = torch.empty((B, S, G, dvp), dtype=y.dtype, device=y.device) if G and want_v else None
-    check(lib().tyr_qk_norm_store(ptr(y), y.stride(1), ptr(q_w), ptr(k_w), ptr(q), ptr(k), ptr(v), ptr(store.k) if store is not None else None,
+    check(lib().tyr_qk_norm_store(ptr(y), row_stride(y), ptr(q_w), ptr(k_w), ptr(q), ptr(k), ptr(v), ptr(store.k) if store is not None else None,
                                   ptr(store.v) if store is not None else None, ptr(pos), ptr(lens), B, S, H, G, dk, dv, dkp, dvp,
                                   store.cap if store is not None else 0, 1 if store is not None and store.ring else 0, eps, _dt(y),
                                   cur_stream(y.device)), "qk_norm_store")

@@ -11,7 +11,7 @@ from typing import Optional, Tuple
 import torch
 
 from .._native import register_signatures
-from ._common import check, cur_stream, err_word, lib, ptr
+from ._common import check, cur_stream, err_word, lib, ptr, row_stride
 
 
 @register_signatures
@@ -285,8 +285,8 @@ def delta_gates(b: torch.Tensor, a: torch.Tensor, dt_bias: torch.Tensor, a_log: 
     B, S, Hv = b.shape
     g = torch.empty((B, S, Hv), dtype=torch.float32, device=b.device)
     beta = torch.empty_like(g)
-    assert b.stride(2) == a.stride(2) == 1 and b.stride(0) == S * b.stride(1) and a.stride(0) == S * a.stride(1) and b.dtype == a.dtype
-    check(lib().tyr_delta_gates(ptr(b), ptr(a), b.stride(1), a.stride(1), ptr(dt_bias), ptr(a_log), ptr(g), ptr(beta), B * S, Hv, _dt(b),
+    assert b.dtype == a.dtype
+    check(lib().tyr_delta_gates(ptr(b), ptr(a), row_stride(b), row_stride(a), ptr(dt_bias), ptr(a_log), ptr(g), ptr(beta), B * S, Hv, _dt(b),
                                 cur_stream(b.device)), "delta_gates")
     return g, beta
 
@@ -332,9 +332,9 @@ def gated_norm(o: torch.Tensor, z: torch.Tensor, w: torch.Tensor, eps: float) ->
     if not o.is_cuda:
         y = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * w.float()
         return (y * torch.nn.functional.silu(z.float()).reshape(B, S, Hv, dv)).reshape(B, S, Hv * dv).to(z.dtype)
-    assert z.stride(2) == 1 and z.stride(0) == S * z.stride(1) and o.is_contiguous()
+    assert o.is_contiguous()
     y = torch.empty((B, S, Hv * dv), dtype=z.dtype, device=z.device)
-    check(lib().tyr_gated_norm(ptr(o), ptr(z), z.stride(1), ptr(w), ptr(y), B * S, Hv, dv, eps, _dt(z), cur_stream(z.device)), "gated_norm")
+    check(lib().tyr_gated_norm(ptr(o), ptr(z), row_stride(z), ptr(w), ptr(y), B * S, Hv, dv, eps, _dt(z), cur_stream(z.device)), "gated_norm")
     return y
 
 
