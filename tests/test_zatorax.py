@@ -49,19 +49,20 @@ CONFIGS = {
         delta(2, 1, 128, 128, 4, moe(16, 4, 128, (4, 2), 64)), attn(4, 2, 128, 128, 0.09, 150, moe(8, 2, 72, (2, 1), 64)),
         attn(4, 2, 128, 128, 0.08, 60, None, kv_from=1), delta(4, 2, 64, 128, 2, moe(8, 2, 64, None, 32))]},
 }
-TOL = {torch.float32: 2e-4, torch.bfloat16: 0.06}
+TOL = {torch.float32: 2e-4, torch.bfloat16: 0.12}
 
 
-def weights(cfg, seed=0):
+def weights(cfg, dtype=torch.float32, seed=0):
     """Exact in bf16.  Sharp queries and keys (scores of several units), decays from forgetful to nearly lossless, negative
-    corrections."""
+    corrections.  For 16-bit arithmetic the corrections outweigh the scores, so that no near-tie of two experts can flip, and the
+    attention is less sharp."""
     gen = torch.Generator().manual_seed(seed)
     out = {}
     for n, shape in Z.tensor_shapes(Z.ZatoraxConfig.from_json(cfg)).items():
         t = torch.randn(shape, generator=gen)
         last = n.rsplit(".", 1)[-1]
         if n.endswith("q.norm") or n.endswith("k.norm"):
-            t = 1.5 + 0.5 * t
+            t = 1.5 + 0.5 * t if dtype == torch.float32 else 1.0 + 0.2 * t
         elif n.endswith("mix.norm"):
             t = 1.0 + 0.3 * t
         elif last in ("norm1", "norm2", "norm"):
@@ -75,7 +76,7 @@ def weights(cfg, seed=0):
         elif last == "r2":
             t = 0.05 + 0.2 * t.abs()
         elif last == "correction":
-            t = -1.5 + 0.4 * t
+            t = -1.5 + 0.4 * t if dtype == torch.float32 else -0.5 - 1.5 * torch.randperm(shape[0], generator=gen)
         elif n != "embed":
             t = t * shape[-1] ** -0.5
         out[n] = t.bfloat16()
@@ -89,25 +90,23 @@ def tokens(cfg, n, seed=1):
 _known = {}
 
 
-def expected(name, toks):
-    key = (name, tuple(toks))
+def expected(name, toks, dtype=torch.float32):
+    key = (name, tuple(toks), dtype)
     if key not in _known:
-        _known[key] = O.logits(CONFIGS[name], {k: v.double() for k, v in weights(CONFIGS[name]).items()}, toks)
+        _known[key] = O.logits(CONFIGS[name], {k: v.double() for k, v in weights(CONFIGS[name], dtype).items()}, toks)
     return _known[key]
 
 
 def model(name, place):
-    w = weights(CONFIGS[name])
+    w = weights(CONFIGS[name], place[1])
     return Z.build(Z.ZatoraxConfig.from_json(CONFIGS[name]), w.__getitem__, *place)
 
 
 def close(got, want, dtype):
-    """Root mean square of the logits' difference per position; at most one position in twenty may differ by a flipped choice of
-    experts in 16-bit arithmetic."""
+    """Root mean square of the logits' difference at every position."""
     d = got.detach().double().cpu() - want
     err = (d - d.mean(-1, keepdim=True)).pow(2).mean(-1).sqrt() / want.std()
-    bad = int((err > TOL[dtype]).sum())
-    assert bad <= (len(err) // 20 if dtype == torch.bfloat16 else 0), err
+    assert bool((err < TOL[dtype]).all()) and float(err.median()) < TOL[dtype] / 4, err
 
 
 # ---- configuration, weights, registry -----------------------------------------------------------------------------
@@ -145,9 +144,9 @@ def test_registry_picks_the_family():
         registry.detect({"model_type": "other"})
 
 
-def save(tmp_path, name):
+def save(tmp_path, name, dtype=torch.float32):
     (tmp_path / "config.json").write_text(json.dumps(CONFIGS[name]))
-    st.save_file(weights(CONFIGS[name]), str(tmp_path / "model.safetensors"))
+    st.save_file(weights(CONFIGS[name], dtype), str(tmp_path / "model.safetensors"))
     return str(tmp_path)
 
 
@@ -179,7 +178,7 @@ def test_missing_or_misshapen_weights_are_named(tmp_path):
 def test_whole_prompt(place, name, n):
     toks = tokens(CONFIGS[name], n)
     got = Z.forward(model(name, place), torch.tensor([toks], device=place[0]))
-    close(got[0], expected(name, toks), place[1])
+    close(got[0], expected(name, toks, place[1]), place[1])
 
 
 def run_split(m, toks, first):
@@ -197,7 +196,7 @@ def run_split(m, toks, first):
 def test_decoding_continues_a_prompt(place, name, n, first):
     """Cuts before, at and past the windows, the convolutions' reach and a chunk; rings wrap while decoding."""
     toks = tokens(CONFIGS[name], n)
-    close(run_split(model(name, place), toks, first), expected(name, toks)[first - 1:], place[1])
+    close(run_split(model(name, place), toks, first), expected(name, toks, place[1])[first - 1:], place[1])
 
 
 @pytest.mark.parametrize("place", PLACES)
@@ -222,14 +221,14 @@ def test_unequal_requests_in_one_batch(place, name, lens):
         for i, r in enumerate(rows):
             out[r].append(lg[i])
     got = torch.cat([torch.stack(o) for o in out])
-    want = torch.cat([expected(name, s[:n + len(o) - 1])[n - 1:] for s, n, o in zip(seqs, lens, out)])
+    want = torch.cat([expected(name, s[:n + len(o) - 1], place[1])[n - 1:] for s, n, o in zip(seqs, lens, out)])
     close(got, want, place[1])
 
 
 @pytest.mark.parametrize("place", PLACES)
 def test_long_decoding(place):
     toks = tokens(CONFIGS["mixed"], 260, seed=3)
-    close(run_split(model("mixed", place), toks, 4)[-120:], expected("mixed", toks)[-120:], place[1])
+    close(run_split(model("mixed", place), toks, 4)[-120:], expected("mixed", toks, place[1])[-120:], place[1])
 
 
 @pytest.mark.parametrize("place", PLACES)
@@ -301,7 +300,7 @@ def test_command_line_generates_from_token_ids(tmp_path, capsys):
 # ---- trace replay -------------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("place", PLACES)
 def test_trace_replay(tmp_path, capsys, place):
-    d = save(tmp_path, "mixed")
+    d = save(tmp_path, "mixed", place[1])
     a, b, c = (tokens(CONFIGS["mixed"], n, seed=n) for n in (30, 14, 22))
     steps = [{"step": 0, "entries": [{"id": "a", "tokens": a[:20], "want": [0, 19]}, {"id": "b", "tokens": b[:12], "want": [11]}], "end": []},
              {"step": 1, "entries": [{"id": "b", "tokens": [b[12]], "want": [0]}, {"id": "a", "tokens": [a[20]], "want": []}], "end": []},
@@ -316,7 +315,7 @@ def test_trace_replay(tmp_path, capsys, place):
     assert capsys.readouterr().out.split() == [x for s in steps for x in ("done", str(s["step"]))]
     assert sorted(p.name for p in out.iterdir()) == ["0.f32", "1.f32", "2.f32", "4.f32", "5.f32"]
     got = torch.cat([torch.frombuffer(bytearray((out / f"{i}.f32").read_bytes()), dtype=torch.float32).reshape(-1, 88) for i in (0, 1, 2, 4, 5)])
-    ea, eb, ec = (expected("mixed", t) for t in (a, b, c))
+    ea, eb, ec = (expected("mixed", t, place[1]) for t in (a, b, c))
     close(got, torch.stack([ea[0], ea[19], eb[11], eb[12], eb[13], ea[22], ec[21]]), place[1])
 
 
