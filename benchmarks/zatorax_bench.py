@@ -2,7 +2,7 @@
 of the new design beside the like kernels of the older models.
 
     python bench.py --workload zatorax --steps 10 --warmup 3          # one JSON line
-    python -m benchmarks.zatorax_bench kernels                        # the kernels alone
+    python -m benchmarks.zatorax_bench kernels ["prompt attention"]   # the kernels alone (cases whose name starts so)
 
 Both stacks have the same width, head counts, head size 128, expert count, top-k, expert and shared FFN, vocabulary and order
 of layers (three delta-rule layers, then one attention layer).  Qwen3.5 attends the whole prompt, Zatorax a window.  CUDA events
@@ -107,7 +107,7 @@ def run(warmup: int = 3, steps: int = 10, sizes=tuple(SIZES)) -> dict:
 
 
 @torch.no_grad()
-def kernels(warmup: int = 3, steps: int = 20, device="cuda") -> dict:
+def kernels(only: str = "", warmup: int = 3, steps: int = 20, device="cuda") -> dict:
     """{case: {"new": ms, "like": ms, "floor": ms}}: a kernel of the new design, the like kernel of the older models on the same
     shapes, and the time of the algorithmic bytes or operations at the measured peaks."""
     from tyr_b200.models.common import KVCache
@@ -126,6 +126,8 @@ def kernels(warmup: int = 3, steps: int = 20, device="cuda") -> dict:
     mk = lambda *s, dt=bf: torch.randn(*s, device=device).to(dt)
 
     def case(name, new, like, floor):
+        if not name.startswith(only):
+            return
         out[name] = {"new": t(new), "like": t(like), "floor": floor}
         print(f"{name}: new {out[name]['new'] * 1e3:.1f} us, like {out[name]['like'] * 1e3:.1f} us, floor {floor * 1e3:.1f} us", flush=True)
 
@@ -183,7 +185,7 @@ def kernels(warmup: int = 3, steps: int = 20, device="cuda") -> dict:
 
 
 if __name__ == "__main__":
-    if sys.argv[1:] == ["kernels"]:
-        print(json.dumps(kernels()))
+    if sys.argv[1:2] == ["kernels"]:
+        kernels(*sys.argv[2:3])
     else:
         print(json.dumps(run()))

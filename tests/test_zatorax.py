@@ -44,6 +44,10 @@ CONFIGS = {
     # every count that can be one is one
     "ones": {"architecture": "Zatorax", "vocab": 40, "width": 16, "norm": {"eps": 1e-6}, "layers": [
         delta(1, 1, 8, 8, 1, moe(1, 1, 8, (1, 1), 8)), attn(1, 1, 8, 8, 1.0, 1, moe(2, 1, 8, (2, 1), 8))]},
+    # sizes no tensor-core kernel tiles
+    "odd": {"architecture": "Zatorax", "vocab": 77, "width": 50, "norm": {"eps": 1e-5}, "layers": [
+        delta(3, 1, 10, 14, 2, moe(5, 2, 20, None, 13)), attn(18, 1, 20, 12, 0.3, 11, moe(9, 3, 17, (3, 2), 20)), delta(2, 2, 12, 130, 9, None),
+        attn(2, 1, 130, 30, 0.1, 6, None)]},
     # head sizes of the fused decode kernels
     "wide": {"architecture": "Zatorax", "vocab": 120, "width": 128, "norm": {"eps": 1e-5}, "layers": [
         delta(2, 1, 128, 128, 4, moe(16, 4, 128, (4, 2), 64)), attn(4, 2, 128, 128, 0.09, 150, moe(8, 2, 72, (2, 1), 64)),
@@ -174,7 +178,7 @@ def test_missing_or_misshapen_weights_are_named(tmp_path):
 
 # ---- whole prompts and decoding -----------------------------------------------------------------------------------
 @pytest.mark.parametrize("place", PLACES)
-@pytest.mark.parametrize("name,n", [("mixed", 75), ("ones", 20), ("wide", 200), ("mixed", 1), ("mixed", 2), ("wide", 3)])
+@pytest.mark.parametrize("name,n", [("mixed", 75), ("ones", 20), ("odd", 40), ("wide", 200), ("mixed", 1), ("mixed", 2), ("wide", 3)])
 def test_whole_prompt(place, name, n):
     toks = tokens(CONFIGS[name], n)
     got = Z.forward(model(name, place), torch.tensor([toks], device=place[0]))
@@ -191,7 +195,7 @@ def run_split(m, toks, first):
 
 
 @pytest.mark.parametrize("place", PLACES)
-@pytest.mark.parametrize("name,n,first", [("mixed", 75, 1), ("mixed", 75, 2), ("mixed", 75, 9), ("mixed", 75, 40), ("ones", 20, 1), ("wide", 200, 1), ("wide", 200, 149),
+@pytest.mark.parametrize("name,n,first", [("mixed", 75, 1), ("mixed", 75, 2), ("mixed", 75, 9), ("mixed", 75, 40), ("ones", 20, 1), ("odd", 40, 8), ("wide", 200, 1), ("wide", 200, 149),
                                           ("wide", 200, 64)])
 def test_decoding_continues_a_prompt(place, name, n, first):
     """Cuts before, at and past the windows, the convolutions' reach and a chunk; rings wrap while decoding."""
