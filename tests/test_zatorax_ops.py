@@ -325,7 +325,7 @@ def test_group_choice_follows_the_corrected_best_expert(place):
     assert ids.tolist() == [[5, 0, 4]]                    # 0.02 of the kept group, not 0.25 of the group that lost
 
 
-@GPU
+@pytest.mark.gpu
 @pytest.mark.parametrize("T", [1, 3, 130])
 def test_fused_routing_matches(T):
     h, E = 64, 16

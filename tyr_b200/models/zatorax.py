@@ -1,7 +1,7 @@
 """Zatorax: hybrid decoder of gated delta-rule layers and sliding-window attention with a logarithmic distance penalty, group-limited
 mixture of experts with a shared expert, norms with a single gain on the sublayers' outputs, fp32 residual stream.
 
-    x <- x + norm1(mixer(x));   x <- x + norm2(experts(x))
+    x += norm1(mix(x));   x += norm2(moe(x))
 
 An attention layer may read the keys and values of an earlier one (``kv_from``): it has queries, window and penalty of its own and
 no store.  Prompts run through the chunked delta-rule kernels and the flash kernel with the penalty table; a decode step through

@@ -5,7 +5,7 @@
 ``prompt_attention`` runs over whole prompts (tcgen05 flash kernel), ``step_attention`` over one new token per row with the K/V
 append fused in (split-KV kernel, a position per row, plain or ring store).  Shapes and dtypes those do not take go to the
 one-warp-per-query kernel of csrc/attention_general.cu, which also norms q / k and fills the store (``qk_norm_store``).  Plain
-PyTorch states the same contract off the GPU."""
+PyTorch computes the same off the GPU."""
 from __future__ import annotations
 
 import ctypes
