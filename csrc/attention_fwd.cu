@@ -32,6 +32,9 @@
 // table is the mask of the second pass too); BIAS 2 evaluates the logarithm per score.  These forms also take head sizes below
 // 128 (a multiple of 8): TMA fills the missing channels with zeros and the Q K^T loop stops at the last real one.
 //
+// Sink and gate (BIAS 3): the same head sizes without a penalty; the softmax denominator also holds exp(sink_h), and the output is
+// multiplied by out_scale * sigmoid(gate), both in the epilogue.
+//
 // The reference calls at::scaled_dot_product_attention, or a query-chunked masked-math fallback
 // for windows (cc/include/tyr_attention.h:58-130).
 #include "common.cuh"
@@ -57,6 +60,11 @@ struct AttnParams {
   const float *r1, *r2;   // [Hq]
   int k_steps;        // 16-channel steps of Q K^T
   int dv;             // output channels
+  // sink and gate form only (both nullable)
+  const float* sink;  // [Hq]
+  const __nv_bfloat16* gate;
+  long long g_row_stride, g_batch_stride, g_head_stride;
+  float out_scale;
 };
 
 constexpr int ATT_TBL_PAD = 256;       // table entries below distance 0 and past the window that boundary blocks can touch
@@ -150,6 +158,7 @@ __global__ void __launch_bounds__(640, 1)
 flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
                       const __grid_constant__ CUtensorMap tmK,
                       const __grid_constant__ CUtensorMap tmV, AttnParams p) {
+  constexpr bool kPenalty = BIAS == 1 || BIAS == 2;
   pdl_trigger();
   extern __shared__ uint8_t smem_raw[];
   AttnSmem& s = *reinterpret_cast<AttnSmem*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
@@ -191,7 +200,7 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
   for (int i = threadIdx.x; i < 2 * 2 * ATT_BM; i += blockDim.x) (&s.xsum[0][0][0])[i] = make_uint2(0u, 0u);
   float* const table = reinterpret_cast<float*>(&s + 1);     // entry ATT_TBL_PAD + n: penalty at distance n, in log2 units
   float r1 = 0.f, r2 = 0.f;
-  if constexpr (BIAS != 0) { r1 = p.r1[head]; r2 = p.r2[head]; }
+  if constexpr (kPenalty) { r1 = p.r1[head]; r2 = p.r2[head]; }
   if constexpr (BIAS == 1) {
     for (int i = threadIdx.x; i < p.window + 2 * ATT_TBL_PAD; i += blockDim.x) {
       const int n = i - ATT_TBL_PAD;
@@ -335,7 +344,7 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
     auto penalty = [&](int n) { return r1 * __log2f(1.f + r2 * static_cast<float>(max(n, 0))); };
     // Steep penalties: their spread inside one key block could push every probability of a row under the fp32 range when
     // the reference is only a bound of the row maximum, so those heads take the exact maximum (one more table read per score).
-    const bool exact_max = BIAS != 0 && fabsf(penalty(ATT_BN - 1)) > 48.f;
+    const bool exact_max = kPenalty && fabsf(penalty(ATT_BN - 1)) > 48.f;
     float m_used = -INFINITY;   // running maximum the exponentials are taken against
     float l_sum = 0.f;          // this half's part of the row sum
     bool ok = true;
@@ -373,7 +382,7 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
             masked(sa, col0);
             masked(sb, col0 + 32);
           }
-          if (BIAS != 0 && exact_max) {      // scores in units of 1 / scale_log2, like the raw ones
+          if (kPenalty && exact_max) {      // scores in units of 1 / scale_log2, like the raw ones
             const float inv_scale = 1.f / p.scale_log2;
 #pragma unroll
             for (int c = 0; c < 32; ++c) {
@@ -399,7 +408,7 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
           break;
         }
         mx = fmaxf(mx, other) * p.scale_log2;
-        if (BIAS != 0 && !exact_max) {
+        if (kPenalty && !exact_max) {
           // bound of the penalised row maximum: raw maximum minus the smallest penalty among this block's visible keys (the
           // penalty is monotonic in the distance)
           const int far_col = p.window > 0 ? max(j * ATT_BN, qi - p.window + 1) : j * ATT_BN;
@@ -473,8 +482,17 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
         l_sum += other;
       }
       if (ok && hi[t] > lo[t]) {
-        const float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
+        float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
         const bool row_ok = row < p.Tq;
+        const __nv_bfloat16* gate = nullptr;
+        if constexpr (BIAS == 3) {
+          if (p.sink) {                          // both terms relative to the larger of the row's reference and the sink
+            const float sk = p.sink[head] * 1.4426950408889634f, m = fmaxf(m_used, sk), f = exp2f(m_used - m);
+            inv = f / (l_sum * f + exp2f(sk - m));
+          }
+          inv *= p.out_scale;
+          if (p.gate) gate = p.gate + batch * p.g_batch_stride + static_cast<long long>(row) * p.g_row_stride + head * p.g_head_stride + h * 64;
+        }
         __nv_bfloat16* out = p.O + batch * p.o_batch_stride + static_cast<long long>(row) * p.o_row_stride +
                              head * p.o_head_stride + h * 64;
 #pragma unroll
@@ -486,6 +504,16 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
 #pragma unroll
             for (int q = 0; q < 4; ++q) {
               if (BIAS != 0 && h * 64 + c * 32 + q * 8 >= p.dv) break;
+              if (BIAS == 3 && gate) {
+                const uint4 gu = *reinterpret_cast<const uint4*>(gate + c * 32 + q * 8);
+                const uint32_t gw[4] = {gu.x, gu.y, gu.z, gu.w};
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                  const float2 g2 = unpack_bf16x2(gw[e]);
+                  o[q * 8 + 2 * e] = __float_as_uint(__fdividef(__uint_as_float(o[q * 8 + 2 * e]), 1.f + __expf(-g2.x)));
+                  o[q * 8 + 2 * e + 1] = __float_as_uint(__fdividef(__uint_as_float(o[q * 8 + 2 * e + 1]), 1.f + __expf(-g2.y)));
+                }
+              }
               uint4 u;
               u.x = pack_bf16x2(__uint_as_float(o[q * 8 + 0]) * inv, __uint_as_float(o[q * 8 + 1]) * inv);
               u.y = pack_bf16x2(__uint_as_float(o[q * 8 + 2]) * inv, __uint_as_float(o[q * 8 + 3]) * inv);
@@ -549,9 +577,16 @@ int make_tmap_bthd(CUtensorMap* tm, const void* base, int B, int T, int H, int D
 }  // namespace
 
 // q/k/v/o are [B, T, H, D] views given by (batch, row, head) element strides; D must be 128.
+struct FlashExtra {           // sink and gate form
+  const float* sink;
+  const void* gate;
+  const long long* gate_strides;
+  float out_scale;
+};
+
 static int flash_fwd_launch(const void* q, const void* k, const void* v, void* o, float* lse, int B, int Hq, int Hkv, int Tq, int Tk,
                             int dk, int dv, const long long* st, int causal, int window, int q_offset, float scale, const float* r1,
-                            const float* r2, int* err, void* stream) {
+                            const float* r2, int* err, void* stream, const FlashExtra* extra = nullptr) {
   if (Hq % Hkv != 0 || B <= 0 || Tq <= 0 || Tk <= 0) return -2;
   for (int i = 0; i < 12; ++i)
     if (st[i] & 7) return -3;
@@ -564,10 +599,11 @@ static int flash_fwd_launch(const void* q, const void* k, const void* v, void* o
   constexpr size_t kBase = sizeof(AttnSmem) + 1024, kMax = 227 * 1024;
   const size_t table = (static_cast<size_t>(window) + 2 * ATT_TBL_PAD) * sizeof(float);
   // the table covers a causal window whose distances start at 0 in the query's own block (no key offset)
-  const int bias = r1 == nullptr ? 0 : (causal && window > 0 && q_offset == 0 && kBase + table <= kMax ? 1 : 2);
+  const int bias = extra != nullptr ? 3 : r1 == nullptr ? 0 : (causal && window > 0 && q_offset == 0 && kBase + table <= kMax ? 1 : 2);
   const size_t smem = bias == 1 ? kBase + table : kBase;
-  auto kernel = bias == 0 ? flash_fwd_d128_kernel<0> : (bias == 1 ? flash_fwd_d128_kernel<1> : flash_fwd_d128_kernel<2>);
-  static bool configured_dev[64][3] = {};       // the attribute is per device
+  auto kernel = bias == 0 ? flash_fwd_d128_kernel<0>
+                          : (bias == 1 ? flash_fwd_d128_kernel<1> : (bias == 2 ? flash_fwd_d128_kernel<2> : flash_fwd_d128_kernel<3>));
+  static bool configured_dev[64][4] = {};       // the attribute is per device
   int cfg_dev = 0;
   if (cudaGetDevice(&cfg_dev) != cudaSuccess || cfg_dev < 0 || cfg_dev >= 64) cfg_dev = 0;
   bool& configured = configured_dev[cfg_dev][bias];
@@ -576,7 +612,13 @@ static int flash_fwd_launch(const void* q, const void* k, const void* v, void* o
     if (e != cudaSuccess) return 1000 + (int)e;
     configured = true;
   }
-  AttnParams p;
+  AttnParams p{};
+  if (extra != nullptr) {
+    p.sink = extra->sink;
+    p.gate = static_cast<const __nv_bfloat16*>(extra->gate);
+    p.g_batch_stride = extra->gate_strides[0]; p.g_row_stride = extra->gate_strides[1]; p.g_head_stride = extra->gate_strides[2];
+    p.out_scale = extra->out_scale;
+  }
   p.B = B; p.Hq = Hq; p.Hkv = Hkv; p.Tq = Tq; p.Tk = Tk;
   p.q_offset = q_offset; p.causal = causal; p.window = window;
   p.scale_log2 = scale * 1.4426950408889634f;
@@ -609,4 +651,15 @@ extern "C" TYR_EXPORT int tyr_flash_fwd_biased(const void* q, const void* k, con
                                                const long long* strides, int window, float scale, int* err, void* stream) {
   if (dk <= 0 || dv <= 0 || dk > ATT_D || dv > ATT_D || (dk & 7) || (dv & 7) || r1 == nullptr || r2 == nullptr || scale <= 0.f) return -1;
   return flash_fwd_launch(q, k, v, o, nullptr, B, Hq, Hkv, T, T, dk, dv, strides, 1, window, 0, scale, r1, r2, err, stream);
+}
+
+// Causal attention with a sink per head (nullable) in the softmax denominator and the output multiplied by out_scale * sigmoid(gate)
+// (gate nullable); sizes as above.  strides: (batch, row, head) of q, k, v, o, gate.  v may be k.
+extern "C" TYR_EXPORT int tyr_flash_fwd_sink(const void* q, const void* k, const void* v, void* o, const float* sink, const void* gate, int B,
+                                             int Hq, int Hkv, int T, int dk, int dv, const long long* strides, float scale, float out_scale,
+                                             int* err, void* stream) {
+  if (dk <= 0 || dv <= 0 || dk > ATT_D || dv > ATT_D || (dk & 7) || (dv & 7) || scale <= 0.f) return -1;
+  if (gate != nullptr && (((strides[12] | strides[13] | strides[14]) & 7) || (reinterpret_cast<uintptr_t>(gate) & 15))) return -3;
+  const FlashExtra ex{sink, gate, strides + 12, out_scale};
+  return flash_fwd_launch(q, k, v, o, nullptr, B, Hq, Hkv, T, T, dk, dv, strides, 1, 0, 0, scale, nullptr, nullptr, err, stream, &ex);
 }

@@ -1,6 +1,8 @@
 // Attention pieces for any head size, fp32 or bf16, with a logarithmic distance penalty on the scores:
 //
-//   score(i, j) = scale q_i . k_j - r1_h ln(1 + r2_h (i - j)),   0 <= i - j < window.
+//   score(i, j) = scale q_i . k_j - r1_h ln(1 + r2_h (i - j)),   0 <= i - j < window,
+//
+// a sink (the softmax denominator also holds exp(sink_h)) and an output gate (element by element, out_scale sigmoid(gate)).
 //
 //   * qk_norm_store: per-head RMSNorm of q and k (no rotation), v copied, rows of the padded batch written to the K/V store at
 //                    their own positions (plain or ring).
@@ -80,12 +82,14 @@ __global__ void __launch_bounds__(256) qk_norm_store_kernel(QkNormArgs a) {
 
 struct GeneralAttnArgs {
   const void *q, *k, *v;       // q: [B, S, H, .]; k / v: [B, ., G, .] by (batch, position or slot, head) element strides
-  void* out;                   // [B, S, H, dv] contiguous
+  void* out;                   // [B * S, .] rows of out_ld elements, channel h * dv + d
   const int* pos;              // position of query 0 of each row (nullable: 0)
   const float *r1, *r2;        // [H] distance penalty (nullable: none)
-  long long q_sb, q_ss, q_sh, k_sb, k_ss, k_sh, v_sb, v_ss, v_sh;
+  const float* sink;           // [H] (nullable: none)
+  const void* gate;            // [B * S, .] rows of gate_ld elements, channel h * dv + d (nullable: none)
+  long long q_sb, q_ss, q_sh, k_sb, k_ss, k_sh, v_sb, v_ss, v_sh, gate_ld, out_ld;
   int B, S, H, G, dk, dv, cap, ring, window, keys;
-  float scale;
+  float scale, out_scale;
   int* err;
 };
 constexpr int GA_WARPS = 4;
@@ -117,7 +121,7 @@ __global__ void __launch_bounds__(GA_WARPS * 32) general_attention_kernel(Genera
   const float r1 = a.r1 ? a.r1[h] : 0.f, r2 = a.r1 ? a.r2[h] : 0.f;
   int lo = a.window > 0 ? max(0, p - a.window + 1) : 0;
   if (a.ring) lo = max(lo, p - a.cap + 1);
-  float m = -INFINITY, l = 0.f, acc[GA_DMAX / 32];
+  float m = a.sink ? a.sink[h] : -INFINITY, l = a.sink ? 1.f : 0.f, acc[GA_DMAX / 32];
 #pragma unroll
   for (int j = 0; j < GA_DMAX / 32; ++j) acc[j] = 0.f;
   for (int base = lo; base <= p; base += 32) {
@@ -147,10 +151,14 @@ __global__ void __launch_bounds__(GA_WARPS * 32) general_attention_kernel(Genera
     }
     __syncwarp();
   }
-  T* op = static_cast<T*>(a.out) + (row * a.H + h) * a.dv;
+  T* op = static_cast<T*>(a.out) + row * a.out_ld + static_cast<long long>(h) * a.dv;
+  const T* gp = a.gate ? static_cast<const T*>(a.gate) + row * a.gate_ld + static_cast<long long>(h) * a.dv : nullptr;
 #pragma unroll
   for (int c = 0; c < GA_DMAX / 32; ++c)
-    if (lane + 32 * c < a.dv) ag_store(op + lane + 32 * c, acc[c] / l);
+    if (lane + 32 * c < a.dv) {
+      const float g = gp ? a.out_scale / (1.f + expf(-ag_load(gp + lane + 32 * c))) : a.out_scale;
+      ag_store(op + lane + 32 * c, acc[c] / l * g);
+    }
 }
 
 }  // namespace tyr
@@ -170,22 +178,40 @@ extern "C" TYR_EXPORT int tyr_qk_norm_store(const void* y, long long ld, const f
                           : launch_dependent(qk_norm_store_kernel<__nv_bfloat16>, grid, dim3(256), 0, (cudaStream_t)stream, a));
 }
 
+static int general_attention_launch(GeneralAttnArgs& a, const long long* strides, int dtype, void* stream) {
+  if (a.B <= 0 || a.S <= 0 || a.H <= 0 || a.G <= 0 || a.H % a.G || a.dk <= 0 || a.dv <= 0 || a.dk > GA_DMAX || a.dv > GA_DMAX) return -1;
+  if ((a.ring && a.cap <= 0) || (a.r1 != nullptr) != (a.r2 != nullptr)) return -2;
+  a.q_sb = strides[0]; a.q_ss = strides[1]; a.q_sh = strides[2];
+  a.k_sb = strides[3]; a.k_ss = strides[4]; a.k_sh = strides[5];
+  a.v_sb = strides[6]; a.v_ss = strides[7]; a.v_sh = strides[8];
+  const dim3 grid(static_cast<unsigned>((static_cast<long long>(a.B) * a.S * a.H + GA_WARPS - 1) / GA_WARPS)), block(GA_WARPS * 32);
+  return (int)(dtype == 1 ? launch_dependent(general_attention_kernel<float>, grid, block, 0, (cudaStream_t)stream, a)
+                          : launch_dependent(general_attention_kernel<__nv_bfloat16>, grid, block, 0, (cudaStream_t)stream, a));
+}
+
 // strides: (batch, position or slot, head) element strides of q, k, v.  `keys`: positions the plain form may read (prompt length
-// or capacity).  dk, dv <= 256.
+// or capacity).  dk, dv <= 256.  out contiguous.
 extern "C" TYR_EXPORT int tyr_general_attention(const void* q, const void* k, const void* v, void* out, const int* pos,
                                                 const float* r1, const float* r2, const long long* strides, int B, int S, int H,
                                                 int G, int dk, int dv, int cap, int ring, int window, int keys, float scale,
                                                 int dtype, int* err, void* stream) {
-  if (B <= 0 || S <= 0 || H <= 0 || G <= 0 || H % G || dk <= 0 || dv <= 0 || dk > GA_DMAX || dv > GA_DMAX) return -1;
-  if ((ring && cap <= 0) || (r1 != nullptr) != (r2 != nullptr)) return -2;
-  GeneralAttnArgs a;
+  GeneralAttnArgs a{};
   a.q = q; a.k = k; a.v = v; a.out = out; a.pos = pos; a.r1 = r1; a.r2 = r2;
-  a.q_sb = strides[0]; a.q_ss = strides[1]; a.q_sh = strides[2];
-  a.k_sb = strides[3]; a.k_ss = strides[4]; a.k_sh = strides[5];
-  a.v_sb = strides[6]; a.v_ss = strides[7]; a.v_sh = strides[8];
   a.B = B; a.S = S; a.H = H; a.G = G; a.dk = dk; a.dv = dv; a.cap = cap; a.ring = ring; a.window = window; a.keys = keys;
-  a.scale = scale; a.err = err;
-  const dim3 grid(static_cast<unsigned>((static_cast<long long>(B) * S * H + GA_WARPS - 1) / GA_WARPS)), block(GA_WARPS * 32);
-  return (int)(dtype == 1 ? launch_dependent(general_attention_kernel<float>, grid, block, 0, (cudaStream_t)stream, a)
-                          : launch_dependent(general_attention_kernel<__nv_bfloat16>, grid, block, 0, (cudaStream_t)stream, a));
+  a.out_ld = static_cast<long long>(H) * dv;
+  a.scale = scale; a.out_scale = 1.f; a.err = err;
+  return general_attention_launch(a, strides, dtype, stream);
+}
+
+// The same over all earlier positions with a sink per head, an output gate and a factor (sink and gate nullable).  strides: as above,
+// then the row strides of gate and out.
+extern "C" TYR_EXPORT int tyr_general_attention_sink(const void* q, const void* k, const void* v, void* out, const int* pos, const float* sink,
+                                                     const void* gate, const long long* strides, int B, int S, int H, int G, int dk, int dv,
+                                                     int keys, float scale, float out_scale, int dtype, int* err, void* stream) {
+  GeneralAttnArgs a{};
+  a.q = q; a.k = k; a.v = v; a.out = out; a.pos = pos; a.sink = sink; a.gate = gate;
+  a.B = B; a.S = S; a.H = H; a.G = G; a.dk = dk; a.dv = dv; a.cap = keys; a.keys = keys;
+  a.gate_ld = strides[9]; a.out_ld = strides[10];
+  a.scale = scale; a.out_scale = out_scale; a.err = err;
+  return general_attention_launch(a, strides, dtype, stream);
 }

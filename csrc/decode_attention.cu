@@ -11,7 +11,8 @@
 //
 // Each row of the batch has its own position.  Retained keys are walked by distance from the new token (a ring store by position
 // modulo its capacity), so a window may be smaller than the ring and a penalty r1_h ln(1 + r2_h distance) can be taken off the
-// scores (template parameter BIAS).  Key size DK and value size DV may differ.
+// scores (template parameter BIAS).  Key size DK and value size DV may differ.  The softmax denominator may also hold exp(sink_h),
+// added once when a row's result is written, and the values may be the keys (one store: its rows are read from memory once).
 //
 // The reference takes the library SDPA over a sliced cache for this step (cc/include/tyr_attention.h:58-130,
 // Tyr/Inference/KVCache.lean:41-215).
@@ -34,7 +35,7 @@ struct DecodeAttnArgs {
   const int* pos;                // absolute position of the new token of row b: pos[b * pos_stride]
   int pos_stride;
   const float *r1, *r2;          // [Hq] distance penalty (BIAS forms)
-  __nv_bfloat16* out;            // [B, Hq, DV] contiguous
+  __nv_bfloat16* out;            // [B, Hq, dv], batch stride out_bs
   float* part_acc;               // [B, Hq, splits, DV]
   float* part_ml;                // [B, Hq, splits, 2]
   int* counters;                 // [B * Hkv], zero on entry, zero on exit
@@ -48,6 +49,10 @@ struct DecodeAttnArgs {
   const __nv_bfloat16* gate;
   long long gate_bs, gate_hs;
   int gate_mode;
+  const float* sink;             // [Hq] (nullable)
+  long long out_bs;              // batch stride of out
+  int dv;                        // channels of a head that are written (heads of out are packed)
+  float out_scale;
 };
 
 __device__ __forceinline__ float decode_gate(const DecodeAttnArgs& a, int b, int h, int d) {
@@ -60,6 +65,17 @@ __device__ __forceinline__ float decode_gate(const DecodeAttnArgs& a, int b, int
     return 1.f / (1.f + __expf(-g));
   }
   return 1.f;
+}
+
+// Channel d of a head: A / L over all keys relative to 2^M, with the sink, the gate and the factor.
+__device__ __forceinline__ void decode_write(const DecodeAttnArgs& a, int b, int h, int d, float M, float L, float A) {
+  if (d >= a.dv) return;
+  if (a.sink != nullptr) {
+    const float sk = a.sink[h] * 1.4426950408889634f, m = fmaxf(M, sk), f = exp2f(M - m);
+    A *= f;
+    L = L * f + exp2f(sk - m);
+  }
+  a.out[b * a.out_bs + static_cast<long long>(h) * a.dv + d] = __float2bfloat16((L > 0.f ? A / L : 0.f) * decode_gate(a, b, h, d) * a.out_scale);
 }
 
 // One m16n8k16 step.  `lo` accumulates the tile's rows 0..7 (query head g of the lane), `hi` rows 8..15 (head g + 8).
@@ -296,7 +312,7 @@ __global__ void __launch_bounds__(kDecWarps * 32) decode_attention_kernel(Decode
     }
     const long long row = static_cast<long long>(b) * a.Hq + hq0 + g;
     if (a.splits == 1) {
-      a.out[row * DV + d] = __float2bfloat16((L > 0.f ? A / L : 0.f) * decode_gate(a, b, hq0 + g, d));
+      decode_write(a, b, hq0 + g, d, M, L, A);
     } else {
       a.part_acc[(row * a.splits + split) * DV + d] = A;
       if (d == 0) {
@@ -327,7 +343,7 @@ __global__ void __launch_bounds__(kDecWarps * 32) decode_attention_kernel(Decode
         A += __ldcg(&a.part_acc[(row * a.splits + sp) * DV + d]) * f;
       }
     }
-    a.out[row * DV + d] = __float2bfloat16((L > 0.f ? A / L : 0.f) * decode_gate(a, b, hq0 + g, d));
+    decode_write(a, b, hq0 + g, d, M, L, A);
   }
   if (tid == 0) a.counters[b * a.Hkv + hkv] = 0;
 }
@@ -343,7 +359,8 @@ static int decode_attention_launch(const void* q, const void* k_new, const void*
                                    int pos_stride, void* out, void* workspace, long long q_bs, long long kn_bs, long long vn_bs, int B,
                                    int Hq, int Hkv, int DK, int DV, int cap, int ring, int window, int splits, int append, float scale,
                                    const void* gate, long long gate_bs, long long gate_hs, int gate_mode, const float* r1,
-                                   const float* r2, void* err, void* stream) {
+                                   const float* r2, void* err, void* stream, const float* sink = nullptr, int dv_out = 0,
+                                   long long out_bs = 0, float out_scale = 1.f) {
   using namespace tyr;
   if (gate_mode < 0 || gate_mode > 2 || (gate_mode != 0 && gate == nullptr)) return -5;
   if (B <= 0 || Hq <= 0 || Hkv <= 0 || Hq % Hkv != 0 || Hq / Hkv > 16 || cap <= 0 || splits < 1 || splits > 64) return -1;
@@ -362,6 +379,10 @@ static int decode_attention_launch(const void* q, const void* k_new, const void*
   a.scale_log2 = scale * 1.4426950408889634f;
   a.err = (int*)err;
   a.gate = (const __nv_bfloat16*)gate; a.gate_bs = gate_bs; a.gate_hs = gate_hs; a.gate_mode = gate == nullptr ? 0 : gate_mode;
+  a.sink = sink;
+  a.dv = dv_out > 0 ? dv_out : DV;
+  a.out_bs = out_bs > 0 ? out_bs : static_cast<long long>(Hq) * DV;
+  a.out_scale = out_scale;
   const dim3 grid(splits, Hkv, B);
   const cudaStream_t st = (cudaStream_t)stream;
   const dim3 block(kDecWarps * 32);
@@ -408,4 +429,18 @@ extern "C" TYR_EXPORT int tyr_decode_attention_biased(const void* q, const void*
   if (r1 == nullptr || r2 == nullptr) return -6;
   return decode_attention_launch(q, k_new, v_new, k_cache, v_cache, pos, pos_stride, out, workspace, q_bs, kn_bs, vn_bs, B, Hq, Hkv, DK,
                                  DV, cap, ring, window, splits, append, scale, nullptr, 0, 0, 0, r1, r2, err, stream);
+}
+
+// Sink per head (nullable), output gate out_scale * sigmoid(gate) (gate nullable: [B, Hq, dv] packed heads, batch stride gate_bs), own position
+// per row (pos_stride 1) or one for all (0); stores of D in {64, 128} channels, of which dv are written to out [B, Hq, dv] (batch
+// stride out_bs).  v_new / v_cache may be k_new / k_cache.
+extern "C" TYR_EXPORT int tyr_decode_attention_sink(const void* q, const void* k_new, const void* v_new, void* k_cache, void* v_cache,
+                                                    const void* pos, void* out, void* workspace, long long q_bs, long long kn_bs,
+                                                    long long vn_bs, int B, int Hq, int Hkv, int D, int dv, int cap, int splits, int append,
+                                                    int pos_stride, float scale, const float* sink, const void* gate, long long gate_bs,
+                                                    long long out_bs, float out_scale, void* err, void* stream) {
+  if (dv <= 0 || dv > D || (D != 64 && D != 128)) return -2;
+  return decode_attention_launch(q, k_new, v_new, k_cache, v_cache, pos, pos_stride, out, workspace, q_bs, kn_bs, vn_bs, B, Hq, Hkv, D, D, cap, 0, 0,
+                                 splits, append, scale, gate, gate_bs, dv, gate == nullptr ? 0 : 2, nullptr, nullptr, err, stream, sink, dv,
+                                 out_bs, out_scale);
 }

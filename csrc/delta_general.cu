@@ -5,8 +5,9 @@
 //   * conv_gates:    one decode token: convolution window shifted in place, SiLU, and the per-head gates.
 //   * gates:         log decay -exp(A_log) softplus(a + dt_bias) and write strength sigmoid(b) for whole prompts.
 //   * recurrent:     the recurrence itself, token by token, the state in registers (one token for decode, any number for
-//                    prompts; rows of a batch may be shorter than the padded length).
-//   * gated_norm:    o / rms(o) * w * silu(z) per head on the fp32 read-out.
+//                    prompts; rows of a batch may be shorter than the padded length).  The decay is one number per token and
+//                    value head, or (CHANNEL) one per key channel, computed here from its projection together with the write strength.
+//   * gated_norm:    o / rms(o) * w * silu(z) or sigmoid(z) per head on the fp32 read-out.
 //
 // This unit is compiled without fast math: a decay close to 1 is applied thousands of times, and the few-ulp bias of the
 // approximate exponential would grow with the sequence.
@@ -100,6 +101,9 @@ __global__ void __launch_bounds__(256) delta_gates_kernel(const T* __restrict__ 
 struct RecurrentArgs {
   const void *q, *k, *v;                 // [B, S, H, d] by (batch, token, head) element strides
   const float *g, *beta;                 // [B, S, Hv]
+  const void *a_raw, *b_raw;             // CHANNEL: projections of decay [B * S, .] (channel hv * dk + d) and write strength (channel hv)
+  const float *dt_bias, *a_log;          // CHANNEL: [Hv * dk], [Hv]
+  long long a_ld, b_ld;                  // CHANNEL: row strides
   float* state;                          // [B, Hv, dk, dv], in place
   float* out;                            // [B, S, Hv, dv]
   const int* lens;                       // [B] tokens of each row (nullable: S)
@@ -108,11 +112,11 @@ struct RecurrentArgs {
 };
 constexpr int REC_WARPS = 4;
 
-template <typename T, int RPL>
+template <typename T, int RPL, bool CHANNEL>
 __global__ void __launch_bounds__(REC_WARPS * 32) gdr_recurrent_kernel(RecurrentArgs a) {
   constexpr int DKM = 4 * RPL;           // largest dk of this instance
   constexpr int EPL = (DKM + 31) / 32;   // q / k elements a lane loads per token
-  __shared__ float sk[REC_WARPS][DKM], sq[REC_WARPS][DKM];
+  __shared__ float sk[REC_WARPS][DKM], sq[REC_WARPS][DKM], sd[REC_WARPS][CHANNEL ? DKM : 1];
   const int bh = blockIdx.x, b = bh / a.Hv, hv = bh % a.Hv, hk = hv / (a.Hv / a.Hk);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int col = (blockIdx.y * REC_WARPS + warp) * 8 + (lane & 7), rg = lane >> 3;
@@ -133,17 +137,30 @@ __global__ void __launch_bounds__(REC_WARPS * 32) gdr_recurrent_kernel(Recurrent
     s[i] = (col_ok && r < a.dk) ? sp[static_cast<long long>(r) * a.dv] : 0.f;
   }
   const float q_scale = 1.f / sqrtf(static_cast<float>(a.dk));
-  float nq[EPL], nk[EPL], nv = 0.f, ng = 0.f, nb = 0.f;
+  const T* ap = static_cast<const T*>(a.a_raw) + static_cast<long long>(b) * a.S * a.a_ld + static_cast<long long>(hv) * a.dk;
+  const T* brp = static_cast<const T*>(a.b_raw) + static_cast<long long>(b) * a.S * a.b_ld + hv;
+  float bias[CHANNEL ? EPL : 1], a_log = 0.f;
+  if constexpr (CHANNEL) {
+    a_log = a.a_log[hv];
+#pragma unroll
+    for (int e = 0; e < EPL; ++e) bias[e] = lane + 32 * e < a.dk ? a.dt_bias[static_cast<long long>(hv) * a.dk + lane + 32 * e] : 0.f;
+  }
+  float nq[EPL], nk[EPL], na[CHANNEL ? EPL : 1], nv = 0.f, ng = 0.f, nb = 0.f;
   auto fetch = [&](int t) {
 #pragma unroll
     for (int e = 0; e < EPL; ++e) {
       const int d = lane + 32 * e;
       nq[e] = d < a.dk ? dg_load(qp + t * a.q_ss + d) : 0.f;
       nk[e] = d < a.dk ? dg_load(kp + t * a.k_ss + d) : 0.f;
+      if constexpr (CHANNEL) na[e] = d < a.dk ? dg_load(ap + t * a.a_ld + d) : 0.f;
     }
     nv = col_ok ? dg_load(vp + t * a.v_ss) : 0.f;
-    ng = gp[static_cast<long long>(t) * a.Hv];
-    nb = bp[static_cast<long long>(t) * a.Hv];
+    if constexpr (CHANNEL) {
+      nb = dg_sigmoid(dg_load(brp + t * a.b_ld));
+    } else {
+      ng = gp[static_cast<long long>(t) * a.Hv];
+      nb = bp[static_cast<long long>(t) * a.Hv];
+    }
   };
   if (n > 0) fetch(0);
   for (int t = 0; t < n; ++t) {
@@ -156,14 +173,16 @@ __global__ void __launch_bounds__(REC_WARPS * 32) gdr_recurrent_kernel(Recurrent
     for (int e = 0; e < EPL; ++e) {
       const int d = lane + 32 * e;
       if (d < DKM) { sq[warp][d] = nq[e] * qn; sk[warp][d] = nk[e] * kn; }
+      if constexpr (CHANNEL)
+        if (d < DKM) sd[warp][d] = dg_decay(dg_log_decay(na[e], bias[e], a_log));
     }
-    const float v = nv, decay = dg_decay(ng), beta = nb;
+    const float v = nv, decay = CHANNEL ? 1.f : dg_decay(ng), beta = nb;
     __syncwarp();
     if (t + 1 < n) fetch(t + 1);
     float kv = 0.f;
 #pragma unroll
     for (int i = 0; i < RPL; ++i) {
-      s[i] *= decay;
+      s[i] *= CHANNEL ? sd[warp][4 * i + rg] : decay;
       kv += s[i] * sk[warp][4 * i + rg];
     }
     kv += __shfl_xor_sync(0xffffffffu, kv, 8);
@@ -189,19 +208,22 @@ __global__ void __launch_bounds__(REC_WARPS * 32) gdr_recurrent_kernel(Recurrent
   }
 }
 
-// o: fp32 [rows, Hv, dv]; z: rows of stride ld_z; w: fp32 [dv]; y: [rows, Hv * dv].  One warp per (row, head).
+// the gate of gated_norm: SiLU, or the sigmoid alone (act 1)
+__device__ __forceinline__ float dg_gate(float z, int act) { return act == 1 ? dg_sigmoid(z) : z * dg_sigmoid(z); }
+
+// o: fp32 [rows, Hv, dv]; z and y: rows of stride ld_z / ld_y, channel h * dv + d; w: fp32 [dv].  One warp per (row, head).
 template <typename T>
 __global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict__ o, const T* __restrict__ z, long long ld_z,
-                                                         const float* __restrict__ w, T* __restrict__ y, long long rows, int Hv,
-                                                         int dv, float eps) {
+                                                         const float* __restrict__ w, T* __restrict__ y, long long ld_y, long long rows,
+                                                         int Hv, int dv, float eps, int act) {
   pdl_entry();
   const int lane = threadIdx.x & 31;
   const long long nw = static_cast<long long>(gridDim.x) * 8;
   for (long long i = blockIdx.x * 8LL + (threadIdx.x >> 5); i < rows * Hv; i += nw) {
     const float* op = o + i * dv;
     const T* zp = z + (i / Hv) * ld_z + (i % Hv) * dv;
-    T* yp = y + i * dv;
-    if ((dv & 3) == 0 && dv <= 256 && sizeof(T) == 2 && (ld_z & 3) == 0 && (reinterpret_cast<uintptr_t>(z) & 7) == 0) {
+    T* yp = y + (i / Hv) * ld_y + (i % Hv) * dv;
+    if ((dv & 3) == 0 && dv <= 256 && sizeof(T) == 2 && ((ld_z | ld_y) & 3) == 0 && ((reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(y)) & 7) == 0) {
       float4 v[2];
       float ss = 0.f;
 #pragma unroll
@@ -219,8 +241,8 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict
           const float2 z0 = unpack_bf16x2(zu.x), z1 = unpack_bf16x2(zu.y);
           const float4 wv = *reinterpret_cast<const float4*>(w + d);
           uint2 r;
-          r.x = pack_bf16x2(v[j].x * rstd * wv.x * (z0.x * dg_sigmoid(z0.x)), v[j].y * rstd * wv.y * (z0.y * dg_sigmoid(z0.y)));
-          r.y = pack_bf16x2(v[j].z * rstd * wv.z * (z1.x * dg_sigmoid(z1.x)), v[j].w * rstd * wv.w * (z1.y * dg_sigmoid(z1.y)));
+          r.x = pack_bf16x2(v[j].x * rstd * wv.x * dg_gate(z0.x, act), v[j].y * rstd * wv.y * dg_gate(z0.y, act));
+          r.y = pack_bf16x2(v[j].z * rstd * wv.z * dg_gate(z1.x, act), v[j].w * rstd * wv.w * dg_gate(z1.y, act));
           *reinterpret_cast<uint2*>(reinterpret_cast<char*>(yp + d)) = r;
         }
       }
@@ -230,7 +252,7 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict
       const float rstd = 1.f / sqrtf(warp_sum(ss) / dv + eps);
       for (int d = lane; d < dv; d += 32) {
         const float zz = dg_load(zp + d);
-        dg_store(yp + d, op[d] * rstd * w[d] * (zz * dg_sigmoid(zz)));
+        dg_store(yp + d, op[d] * rstd * w[d] * dg_gate(zz, act));
       }
     }
   }
@@ -283,36 +305,57 @@ extern "C" TYR_EXPORT int tyr_delta_gates(const void* b_in, const void* a_in, lo
 }
 
 // strides: (batch, token, head) element strides of q, k, v.  dk <= 256.
-extern "C" TYR_EXPORT int tyr_gdr_recurrent(const void* q, const void* k, const void* v, const float* g, const float* beta,
-                                            float* state, float* out, const int* lens, const long long* strides, int B, int S,
-                                            int Hk, int Hv, int dk, int dv, int dtype, void* stream) {
-  if (B <= 0 || S <= 0 || Hk <= 0 || Hv <= 0 || Hv % Hk || dk <= 0 || dk > 256 || dv <= 0) return -1;
-  RecurrentArgs a;
-  a.q = q; a.k = k; a.v = v; a.g = g; a.beta = beta; a.state = state; a.out = out; a.lens = lens;
+static int recurrent_launch(RecurrentArgs& a, const long long* strides, int B, int dtype, bool channel, void* stream) {
+  if (B <= 0 || a.S <= 0 || a.Hk <= 0 || a.Hv <= 0 || a.Hv % a.Hk || a.dk <= 0 || a.dk > 256 || a.dv <= 0) return -1;
   a.q_sb = strides[0]; a.q_ss = strides[1]; a.q_sh = strides[2];
   a.k_sb = strides[3]; a.k_ss = strides[4]; a.k_sh = strides[5];
   a.v_sb = strides[6]; a.v_ss = strides[7]; a.v_sh = strides[8];
-  a.S = S; a.Hk = Hk; a.Hv = Hv; a.dk = dk; a.dv = dv;
-  const dim3 grid(B * Hv, (dv + 8 * REC_WARPS - 1) / (8 * REC_WARPS)), block(REC_WARPS * 32);
+  const int dk = a.dk;
+  const dim3 grid(B * a.Hv, (a.dv + 8 * REC_WARPS - 1) / (8 * REC_WARPS)), block(REC_WARPS * 32);
   cudaStream_t st = (cudaStream_t)stream;
-#define TYR_REC(T)                                                                                      \
-  (dk <= 32 ? launch_dependent(gdr_recurrent_kernel<T, 8>, grid, block, 0, st, a)                       \
-            : dk <= 64 ? launch_dependent(gdr_recurrent_kernel<T, 16>, grid, block, 0, st, a)           \
-                       : dk <= 128 ? launch_dependent(gdr_recurrent_kernel<T, 32>, grid, block, 0, st, a) \
-                                   : launch_dependent(gdr_recurrent_kernel<T, 64>, grid, block, 0, st, a))
-  return (int)(dtype == 1 ? TYR_REC(float) : TYR_REC(__nv_bfloat16));
+#define TYR_REC(T, CH)                                                                                      \
+  (dk <= 32 ? launch_dependent(gdr_recurrent_kernel<T, 8, CH>, grid, block, 0, st, a)                       \
+            : dk <= 64 ? launch_dependent(gdr_recurrent_kernel<T, 16, CH>, grid, block, 0, st, a)           \
+                       : dk <= 128 ? launch_dependent(gdr_recurrent_kernel<T, 32, CH>, grid, block, 0, st, a) \
+                                   : launch_dependent(gdr_recurrent_kernel<T, 64, CH>, grid, block, 0, st, a))
+  if (channel) return (int)(dtype == 1 ? TYR_REC(float, true) : TYR_REC(__nv_bfloat16, true));
+  return (int)(dtype == 1 ? TYR_REC(float, false) : TYR_REC(__nv_bfloat16, false));
 #undef TYR_REC
 }
 
-extern "C" TYR_EXPORT int tyr_gated_norm(const float* o, const void* z, long long ld_z, const float* w, void* y, long long rows,
-                                         int Hv, int dv, float eps, int dtype, void* stream) {
-  if (rows <= 0 || Hv <= 0 || dv <= 0) return -1;
-  if ((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(y)) & 15) return -2;
+extern "C" TYR_EXPORT int tyr_gdr_recurrent(const void* q, const void* k, const void* v, const float* g, const float* beta,
+                                            float* state, float* out, const int* lens, const long long* strides, int B, int S,
+                                            int Hk, int Hv, int dk, int dv, int dtype, void* stream) {
+  RecurrentArgs a{};
+  a.q = q; a.k = k; a.v = v; a.g = g; a.beta = beta; a.state = state; a.out = out; a.lens = lens;
+  a.S = S; a.Hk = Hk; a.Hv = Hv; a.dk = dk; a.dv = dv;
+  return recurrent_launch(a, strides, B, dtype, false, stream);
+}
+
+// A decay per key channel: a_raw [B * S, .] (channel hv * dk + d) and b_raw (channel hv) in the activations' type, strides[9] and
+// strides[10] their row strides; log decay -exp(a_log[hv]) softplus(a_raw + dt_bias), write strength sigmoid(b_raw).
+extern "C" TYR_EXPORT int tyr_gdr_recurrent_channel(const void* q, const void* k, const void* v, const void* a_raw, const void* b_raw,
+                                                    const float* dt_bias, const float* a_log, float* state, float* out, const int* lens,
+                                                    const long long* strides, int B, int S, int Hk, int Hv, int dk, int dv, int dtype,
+                                                    void* stream) {
+  RecurrentArgs a{};
+  a.q = q; a.k = k; a.v = v; a.a_raw = a_raw; a.b_raw = b_raw; a.dt_bias = dt_bias; a.a_log = a_log;
+  a.a_ld = strides[9]; a.b_ld = strides[10];
+  a.state = state; a.out = out; a.lens = lens;
+  a.S = S; a.Hk = Hk; a.Hv = Hv; a.dk = dk; a.dv = dv;
+  return recurrent_launch(a, strides, B, dtype, true, stream);
+}
+
+// act: 0 = SiLU gate, 1 = sigmoid gate
+extern "C" TYR_EXPORT int tyr_gated_norm(const float* o, const void* z, long long ld_z, const float* w, void* y, long long ld_y, long long rows,
+                                         int Hv, int dv, float eps, int act, int dtype, void* stream) {
+  if (rows <= 0 || Hv <= 0 || dv <= 0 || act < 0 || act > 1) return -1;
+  if ((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(w)) & 15) return -2;
   const long long want = (rows * Hv + 7) / 8;
   const dim3 grid(static_cast<unsigned>(want < 148LL * 32 ? want : 148LL * 32));
   cudaStream_t st = (cudaStream_t)stream;
   if (dtype == 1)
-    return (int)launch_dependent(gated_norm_kernel<float>, grid, dim3(256), 0, st, o, (const float*)z, ld_z, w, (float*)y, rows, Hv, dv, eps);
-  return (int)launch_dependent(gated_norm_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, o, (const __nv_bfloat16*)z, ld_z, w, (__nv_bfloat16*)y,
-                               rows, Hv, dv, eps);
+    return (int)launch_dependent(gated_norm_kernel<float>, grid, dim3(256), 0, st, o, (const float*)z, ld_z, w, (float*)y, ld_y, rows, Hv, dv, eps, act);
+  return (int)launch_dependent(gated_norm_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, o, (const __nv_bfloat16*)z, ld_z, w, (__nv_bfloat16*)y, ld_y,
+                               rows, Hv, dv, eps, act);
 }

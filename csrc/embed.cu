@@ -68,6 +68,35 @@ embed_grad_sorted_kernel(const __nv_bfloat16* __restrict__ dy, const long long* 
   }
 }
 
+// Input rows of a decoder with sinusoidal positions: x[r, d] = table[ids[r], d] * scale + sin / cos(p * freq[d / 2]), fp32, channel 2i the
+// sine and 2i + 1 the cosine.  `turns` holds the frequencies over 2 pi in double, so that the angle is reduced to a fraction of a turn
+// before it is rounded and far positions keep their accuracy.  p = pos[r] (a decode step), else r % S.
+template <typename T>
+__global__ void __launch_bounds__(256) embed_positions_kernel(const long long* __restrict__ ids, const T* __restrict__ table, const double* __restrict__ turns,
+                                                              const int* __restrict__ pos, float* __restrict__ x, long long rows, int S, int D,
+                                                              int vocab, float scale, int* err) {
+  pdl_entry();
+  const int half = (D + 1) / 2;
+  const long long total = rows * half;
+  for (long long i = blockIdx.x * 256LL + threadIdx.x; i < total; i += gridDim.x * 256LL) {
+    const long long r = i / half;
+    const int k = static_cast<int>(i % half);
+    const long long id = ids[r];
+    if (id < 0 || id >= vocab) {
+      if (k == 0) report_error(err, ERR_BOUNDS, static_cast<int>(id));
+      continue;
+    }
+    const int p = pos ? pos[r] : static_cast<int>(r % S);
+    const double t = p * turns[k];
+    float sn, cs;
+    sincospif(2.f * static_cast<float>(t - rint(t)), &sn, &cs);
+    const T* e = table + id * D + 2 * k;
+    float* o = x + r * D + 2 * k;
+    o[0] = static_cast<float>(e[0]) * scale + sn;
+    if (2 * k + 1 < D) o[1] = static_cast<float>(e[1]) * scale + cs;
+  }
+}
+
 }  // namespace tyr
 
 // Returns 0 on success, -1 on a bad shape / alignment.
@@ -80,4 +109,21 @@ extern "C" TYR_EXPORT int tyr_embed_grad_sorted(const void* dy, const long long*
   tyr::launch_dependent(tyr::embed_grad_sorted_kernel, dim3(blocks), dim3(threads), 0, reinterpret_cast<cudaStream_t>(stream),
       reinterpret_cast<const __nv_bfloat16*>(dy), order, sorted_ids, grad, N, d, ld, V);
   return static_cast<int>(cudaGetLastError());
+}
+
+// ids int64 [rows]; table [vocab, D] (dtype 0 = bf16, 1 = fp32); turns double [(D + 1) / 2]; pos int32 [rows] or null; x fp32 [rows, D].
+// An id outside the table is recorded in `err` and its row left alone.
+extern "C" TYR_EXPORT int tyr_embed_positions(const void* ids, const void* table, const double* turns, const int* pos, float* x, long long rows,
+                                              int S, int D, int vocab, float scale, int dtype, int* err, void* stream) {
+  using namespace tyr;
+  if (rows <= 0 || S <= 0 || D <= 0 || vocab <= 0) return -1;
+  const long long want = (rows * ((D + 1) / 2) + 255) / 256;
+  const dim3 grid(static_cast<unsigned>(want < 148LL * 32 ? want : 148LL * 32));
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  auto* id = static_cast<const long long*>(ids);
+  if (dtype == 1)
+    return (int)launch_dependent(embed_positions_kernel<float>, grid, dim3(256), 0, st, id, static_cast<const float*>(table), turns, pos, x, rows, S, D,
+                                 vocab, scale, err);
+  return (int)launch_dependent(embed_positions_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, id, static_cast<const __nv_bfloat16*>(table), turns, pos,
+                               x, rows, S, D, vocab, scale, err);
 }

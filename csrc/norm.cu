@@ -443,6 +443,77 @@ __global__ void __launch_bounds__(256) post_norm_residual_kernel(PostNormArgs a)
   }
 }
 
+// A sublayer's output added to an fp32 residual stream, and the norm the next layer reads:
+//   r = resid + x (x null: r = resid),   resid_out = r,   y = r / sqrt(mean(r^2) + eps) * gain.
+struct AddNormArgs {
+  const void* x;           // [rows, D] (TX), nullable
+  const float* gain;       // [D]
+  float* resid;            // [rows, D], in place
+  void* y;                 // [rows, D] (TY)
+  long long x_stride, r_stride;      // elements between rows
+  int D;
+  float eps;
+};
+
+template <typename TX, typename TY, bool VEC>
+__global__ void __launch_bounds__(256) add_norm_kernel(AddNormArgs a) {
+  __shared__ float red[8];
+  const long long row = blockIdx.x;
+  const int tid = threadIdx.x, nw = blockDim.x >> 5;
+  const TX* x = a.x ? static_cast<const TX*>(a.x) + row * a.x_stride : nullptr;
+  float* resid = a.resid + row * a.r_stride;
+  TY* y = static_cast<TY*>(a.y) + row * a.D;
+  pdl_entry();
+  float f[kPnVecs][8], ss = 0.f;
+  if constexpr (VEC) {
+#pragma unroll
+    for (int j = 0; j < kPnVecs; ++j) {
+      const int v = (tid + j * blockDim.x) * 8;
+      if (v < a.D) {
+        pn_load8(resid + v, f[j]);
+        if (x) {
+          float t[8];
+          pn_load8(x + v, t);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) f[j][e] += t[e];
+          pn_store8(resid + v, f[j]);
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) ss += f[j][e] * f[j][e];
+      }
+    }
+  } else {
+    for (int d = tid; d < a.D; d += blockDim.x) {
+      float t = resid[d];
+      if (x) {
+        t += pn_get(x + d);
+        resid[d] = t;
+      }
+      ss += t * t;
+    }
+  }
+  ss = warp_sum(ss);
+  if ((tid & 31) == 0) red[tid >> 5] = ss;
+  __syncthreads();
+  float tot = 0.f;
+  for (int i = 0; i < nw; ++i) tot += red[i];
+  const float rstd = rsqrtf(tot / a.D + a.eps);
+  if constexpr (VEC) {
+#pragma unroll
+    for (int j = 0; j < kPnVecs; ++j) {
+      const int v = (tid + j * blockDim.x) * 8;
+      if (v >= a.D) continue;
+      float w[8];
+      pn_load8(a.gain + v, w);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[j][e] *= rstd * w[e];
+      pn_store8(y + v, f[j]);
+    }
+  } else {
+    for (int d = tid; d < a.D; d += blockDim.x) pn_put(y + d, resid[d] * rstd * a.gain[d]);
+  }
+}
+
 static int grid_for_rows(long long rows, int warps_per_block) {
   long long blocks = (rows + warps_per_block - 1) / warps_per_block;
   const long long cap = 148LL * 16;
@@ -534,4 +605,21 @@ extern "C" TYR_EXPORT int tyr_post_norm_residual(const void* x, long long x_stri
   if (x_dtype == 0) return (int)(y_dtype == 0 ? TYR_PN(__nv_bfloat16, __nv_bfloat16) : TYR_PN(__nv_bfloat16, float));
   return (int)(y_dtype == 0 ? TYR_PN(float, __nv_bfloat16) : TYR_PN(float, float));
 #undef TYR_PN
+}
+
+extern "C" TYR_EXPORT int tyr_add_norm(const void* x, long long x_stride, const float* gain, float* resid, long long r_stride, void* y, long long rows,
+                                       int D, float eps, int x_dtype, int y_dtype, void* stream) {
+  if (rows <= 0 || D <= 0 || gain == nullptr || resid == nullptr || y == nullptr) return -1;
+  AddNormArgs a{x, gain, resid, y, x_stride, r_stride, D, eps};
+  const uintptr_t al = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(resid) | reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(gain);
+  const bool vec = (D & 7) == 0 && (x_stride & 7) == 0 && (r_stride & 3) == 0 && (al & 15) == 0 && D <= 256 * 8 * kPnVecs;
+  int threads = 256;
+  while (threads > 32 && threads * 4 >= D) threads >>= 1;       // narrow rows: no idle warps
+  const dim3 grid(static_cast<unsigned>(rows)), block(threads);
+  cudaStream_t st = (cudaStream_t)stream;
+#define TYR_AN(TX, TY) (vec ? launch_dependent(add_norm_kernel<TX, TY, true>, grid, block, 0, st, a) \
+                            : launch_dependent(add_norm_kernel<TX, TY, false>, grid, block, 0, st, a))
+  if (x_dtype == 0) return (int)(y_dtype == 0 ? TYR_AN(__nv_bfloat16, __nv_bfloat16) : TYR_AN(__nv_bfloat16, float));
+  return (int)(y_dtype == 0 ? TYR_AN(float, __nv_bfloat16) : TYR_AN(float, float));
+#undef TYR_AN
 }

@@ -1,9 +1,9 @@
 """Shared runner for the pretrained text families (counterpart of Examples/ModelRunner.lean and the per-family RunHF
-executables: Qwen3, Qwen2.5-Omni thinker, Qwen3.5 / 3.6, Gemma 4, Zatorax) plus the speech demos (Whisper, Qwen3-ASR).
+executables: Qwen3, Qwen2.5-Omni thinker, Qwen3.5 / 3.6, Gemma 4, Zatorax, Kinetar) plus the speech demos (Whisper, Qwen3-ASR).
 
     python -m tyr_b200.cli.model_runner --family gemma4 --source google/gemma-4-e2b --prompt "Hi" --max-new-tokens 64 --stream
     python -m tyr_b200.cli.model_runner --family qwen3 --source Qwen/Qwen3-4B --prompt-file prompts.txt --batch-size 4
-    python -m tyr_b200.cli.model_runner --source <zatorax dir> --prompt "5 17 3" --max-new-tokens 16        # family from config.json
+    python -m tyr_b200.cli.model_runner --source <zatorax or kinetar dir> --prompt "5 17 3" --max-new-tokens 16        # family from config.json
     python -m tyr_b200.cli.model_runner --family whisper --source openai/whisper-small --audio speech.wav
 
 Common flags: ``--family`` (default ``auto``: by config.json, ``models/registry.py``), ``--source`` (directory or hub repo id), ``--prompt`` / ``--prompt-file``, ``--batch-size``, ``--max-new-tokens``,
@@ -23,7 +23,7 @@ from ..models import registry
 from ..models.generation import SamplingStrategy
 from ..tokenizer import hf as tok_hf
 
-TEXT_FAMILIES = ("qwen3", "qwen25omni", "qwen35", "gemma4", "zatorax")
+TEXT_FAMILIES = ("qwen3", "qwen25omni", "qwen35", "gemma4", "zatorax", "kinetar")
 SPEECH_FAMILIES = ("whisper", "qwen3asr")
 
 
@@ -95,10 +95,11 @@ def load_text_family(family: str, model_dir: str, device, dtype):
         tok = tok_hf.load_gemma4(model_dir)
         gen = lambda ids, n, st_, cb: G.generate(m, ids, n, st_, cfg.eos_token_id, cb)
         return gen, tok, lambda p: tok_hf.gemma_prompt([{"role": "user", "content": p}]), list(cfg.eos_token_id), cfg.pad_token_id or 0
-    if family == "zatorax":
+    if registry.by_name(family).ragged:
+        import importlib
         import os
-        from ..models import zatorax as Z
         from ..tokenizer.ids import IdTokenizer
+        Z = importlib.import_module(f"tyr_b200.models.{registry.by_name(family).module}")
         m = Z.load_pretrained(model_dir, device, dtype)
         has_tok = os.path.exists(os.path.join(model_dir, "tokenizer.json"))
         tok = tok_hf.HFTokenizer.from_file(model_dir) if has_tok else IdTokenizer(m.cfg.vocab)

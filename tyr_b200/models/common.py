@@ -54,6 +54,23 @@ def lin(x: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor] = None, act:
     return y
 
 
+def project(x: torch.Tensor, w: torch.Tensor, act: Optional[str] = None, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``act(x @ w^T)`` for rows of views: x [B, S, K] and ``out`` [B, S, N] may be column windows of wider buffers, which the tensor-core
+    product reads and writes in place."""
+    rows = x.shape[0] * x.shape[1]
+    ok = lambda t: t.stride(2) == 1 and (t.shape[0] == 1 or t.shape[1] == 1 or t.stride(0) == t.shape[1] * t.stride(1)) and t.data_ptr() % 16 == 0
+    ld = lambda t: t.stride(1) if t.shape[1] > 1 else t.stride(0)
+    if (x.is_cuda and x.dtype == w.dtype == torch.bfloat16 and rows >= TCGEN05_MIN_ROWS and not torch.is_grad_enabled() and w.shape[0] % 8 == 0
+            and w.shape[1] % 8 == 0 and w.stride(1) == 1 and w.stride(0) % 8 == 0 and w.data_ptr() % 16 == 0 and ok(x) and ld(x) % 8 == 0
+            and (out is None or (ok(out) and ld(out) % 8 == 0))):
+        y = torch.empty((*x.shape[:2], w.shape[0]), dtype=x.dtype, device=x.device) if out is None else out
+        flat = lambda t: t.as_strided((rows, t.shape[2]), (ld(t), 1))
+        _gemm(flat(x), w, act=act, out=flat(y))
+        return y
+    y = lin(x, w, act=act)
+    return y if out is None else out.copy_(y)
+
+
 def swiglu_mlp(x, gate_w, up_w, down_w):
     rows = x.numel() // x.shape[-1]
     if rows <= _decode_gemm.MAX_ROWS and x.is_cuda and not torch.is_grad_enabled():
@@ -136,11 +153,14 @@ class KVCache:
     length: int = 0           # absolute positions written so far
 
     @staticmethod
-    def allocate(batch: int, kv_heads: int, cap: int, head_dim: int, device, dtype, ring: bool = False, v_dim: Optional[int] = None) -> "KVCache":
+    def allocate(batch: int, kv_heads: int, cap: int, head_dim: int, device, dtype, ring: bool = False, v_dim: Optional[int] = None,
+                 shared: bool = False) -> "KVCache":
+        """``shared``: the values are the keys, and one store serves both."""
         if cap <= 0:
             raise ValueError("cache capacity must be positive")
         zeros = lambda d: torch.zeros((batch, kv_heads, cap, d), device=device, dtype=dtype)
-        return KVCache(zeros(head_dim), zeros(head_dim if v_dim is None else v_dim), ring)
+        k = zeros(head_dim)
+        return KVCache(k, k if shared else zeros(head_dim if v_dim is None else v_dim), ring)
 
     @property
     def cap(self) -> int:
@@ -175,16 +195,18 @@ class KVCache:
 
     def retain(self, rows: torch.Tensor) -> None:
         """Keep only these rows of the batch, in this order; the others' memory is given back."""
-        self.k, self.v = self.k.index_select(0, rows), self.v.index_select(0, rows)
+        shared = self.v is self.k
+        self.k = self.k.index_select(0, rows)
+        self.v = self.k if shared else self.v.index_select(0, rows)
 
     def nbytes(self) -> int:
-        return self.k.numel() * self.k.element_size() + self.v.numel() * self.v.element_size()
+        return sum(t.numel() * t.element_size() for t in ((self.k,) if self.v is self.k else (self.k, self.v)))
 
 
 @dataclass
 class LinearState:
     conv: Optional[torch.Tensor] = None        # [B, conv_dim, K] last K pre-conv inputs
-    rec: Optional[torch.Tensor] = None         # fp32 [B, Hv, dk, dv]
+    rec: Optional[torch.Tensor] = None         # fp32 [B, Hv, dk, dv] (delta rule) or [B, channels, states] (selective scan)
 
     def retain(self, rows: torch.Tensor) -> None:
         if self.conv is not None:
@@ -192,8 +214,11 @@ class LinearState:
         if self.rec is not None:
             self.rec = self.rec.index_select(0, rows)
 
+    def tensors(self) -> List[torch.Tensor]:
+        return [t for t in (self.conv, self.rec) if t is not None]
+
     def nbytes(self) -> int:
-        return sum(t.numel() * t.element_size() for t in (self.conv, self.rec) if t is not None)
+        return sum(t.numel() * t.element_size() for t in self.tensors())
 
 
 def cached_attention(q: torch.Tensor, k_new: torch.Tensor, v_new: torch.Tensor, cache: Optional[KVCache],

@@ -35,6 +35,9 @@ class Family:
 
 
 FAMILIES: List[Family] = [
+    Family("kinetar", ("kinetar",), "kinetar", "CacheSession",
+           ("attention_fwd", "attention_general", "decode_attention", "decode_gemm", "delta_general", "delta_rule", "embed", "gemm_tcgen05", "mix_conv",
+            "norm", "selective_scan", "skinny_gemm"), ragged=True),
     Family("zatorax", ("zatorax",), "zatorax", "CacheSession",
            ("attention_fwd", "attention_general", "decode_attention", "decode_gemm", "delta_general", "delta_rule", "gemm_tcgen05", "moe_nvfp4",
             "norm", "skinny_gemm"), ragged=True),

@@ -90,7 +90,7 @@ class HybridSession:
         else:
             if self._graph is None:
                 from ..utils.graph import GraphedStep
-                state = [self.pos_t] + [t for s in self.lin if s is not None for t in (s.conv, s.rec)]
+                state = [self.pos_t] + [t for s in self.lin if s is not None for t in s.tensors()]
                 self._graph = GraphedStep(self._device_step, (tok.clone(),), advancing_state=state)
             out = self._graph(tok)
         self._advance_host()

@@ -51,7 +51,8 @@ def _sigs(lib_):
                        ("tyr_delta_conv_gates", [P, P, P, L, L, L] + [P] * 7 + [I, I, I, I, I, P]),
                        ("tyr_delta_gates", [P, P, L, L, P, P, P, P, L, I, I, P]),
                        ("tyr_gdr_recurrent", [P] * 8 + [ctypes.POINTER(L), I, I, I, I, I, I, I, P]),
-                       ("tyr_gated_norm", [P, P, L, P, P, L, I, I, F, I, P])):
+                       ("tyr_gdr_recurrent_channel", [P] * 10 + [ctypes.POINTER(L), I, I, I, I, I, I, I, P]),
+                       ("tyr_gated_norm", [P, P, L, P, P, L, L, I, I, F, I, I, P])):
         fn = getattr(lib_, name, None)
         if fn is not None:
             fn.argtypes = args
@@ -325,16 +326,20 @@ def delta_prefill(q, k, v, g, beta, state: torch.Tensor, lens: Optional[torch.Te
     return recurrent_delta(q, k, v, g, beta, state, lens)
 
 
-def gated_norm(o: torch.Tensor, z: torch.Tensor, w: torch.Tensor, eps: float) -> torch.Tensor:
-    """``o / sqrt(mean(o^2) + eps) * w * silu(z)`` per head: o fp32 [B, S, Hv, dv], z [B, S, Hv*dv] (rows may be strided),
-    w fp32 [dv] -> [B, S, Hv*dv] in z's dtype."""
+def gated_norm(o: torch.Tensor, z: torch.Tensor, w: torch.Tensor, eps: float, act: str = "silu", out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``o / sqrt(mean(o^2) + eps) * w * act(z)`` per head, ``act`` SiLU or sigmoid: o fp32 [B, S, Hv, dv], z [B, S, Hv*dv] (rows may be
+    strided), w fp32 [dv] -> [B, S, Hv*dv] in z's dtype (``out``: a view with evenly spaced rows)."""
     B, S, Hv, dv = o.shape
     if not o.is_cuda:
         y = o * torch.rsqrt(o.pow(2).mean(-1, keepdim=True) + eps) * w.float()
-        return (y * torch.nn.functional.silu(z.float()).reshape(B, S, Hv, dv)).reshape(B, S, Hv * dv).to(z.dtype)
+        f = torch.sigmoid if act == "sigmoid" else torch.nn.functional.silu
+        y = (y * f(z.float()).reshape(B, S, Hv, dv)).reshape(B, S, Hv * dv).to(z.dtype)
+        return y if out is None else out.copy_(y)
     assert o.is_contiguous()
-    y = torch.empty((B, S, Hv * dv), dtype=z.dtype, device=z.device)
-    check(lib().tyr_gated_norm(ptr(o), ptr(z), row_stride(z), ptr(w), ptr(y), B * S, Hv, dv, eps, _dt(z), cur_stream(z.device)), "gated_norm")
+    y = torch.empty((B, S, Hv * dv), dtype=z.dtype, device=z.device) if out is None else out
+    assert y.dtype == z.dtype and y.shape == (B, S, Hv * dv)
+    check(lib().tyr_gated_norm(ptr(o), ptr(z), row_stride(z), ptr(w), ptr(y), row_stride(y), B * S, Hv, dv, eps, {"silu": 0, "sigmoid": 1}[act], _dt(z),
+                               cur_stream(z.device)), "gated_norm")
     return y
 
 
@@ -370,3 +375,50 @@ def delta_decode(mixed, z, b, a, conv_state, conv_w, dt_bias, a_log, norm_w, eps
     kd = Hk * dk
     q, k, v = y[..., :kd].reshape(B, 1, Hk, dk), y[..., kd:2 * kd].reshape(B, 1, Hk, dk), y[..., 2 * kd:].reshape(B, 1, Hv, dv)
     return gated_norm(recurrent_delta(q, k, v, g, beta, rec_state), z, norm_w.float(), eps)
+
+
+# ---- a decay per key channel ------------------------------------------------------------------------------------------------------
+def channel_log_decay(a: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor) -> torch.Tensor:
+    """a: [B, S, Hv * dk] -> fp32 [B, S, Hv, dk]: ``-exp(a_log) softplus(a + dt_bias)``."""
+    z = torch.nn.functional.softplus(a.float() + dt_bias).reshape(*a.shape[:2], a_log.numel(), -1)
+    return -torch.exp(a_log.float())[:, None] * z
+
+
+def recurrent_channel_delta(q, k, v, a, b, dt_bias, a_log, state: torch.Tensor, lens: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """:func:`recurrent_delta` with a decay per key channel: ``a`` [B, S, Hv * dk] and ``b`` [B, S, Hv] are the projections of decay and
+    write strength (rows may be strided), dt_bias fp32 [Hv * dk], a_log fp32 [Hv]."""
+    import ctypes
+    B, S, Hk, dk = q.shape
+    Hv, dv = v.shape[2], v.shape[3]
+    if not q.is_cuda:
+        rep = Hv // Hk
+        decay, beta = torch.exp(channel_log_decay(a, dt_bias, a_log)), torch.sigmoid(b.float())
+        qf, kf = (l2norm(t.float()).repeat_interleave(rep, 2) for t in (q, k))
+        qf = qf * dk ** -0.5
+        out = torch.zeros(B, S, Hv, dv, dtype=torch.float32)
+        for r in range(B):
+            st = state[r]
+            for t in range(S if lens is None else int(lens[r])):
+                st = st * decay[r, t][..., None]
+                u = beta[r, t][:, None] * (v[r, t].float() - torch.einsum("hd,hdv->hv", kf[r, t], st))
+                st = st + kf[r, t][..., None] * u[:, None]
+                out[r, t] = torch.einsum("hd,hdv->hv", qf[r, t], st)
+            state[r] = st
+        return out
+    assert state.dtype == torch.float32 and state.is_contiguous() and q.stride(3) == k.stride(3) == v.stride(3) == 1 and q.dtype == k.dtype == v.dtype == a.dtype == b.dtype
+    out = torch.empty((B, S, Hv, dv), dtype=torch.float32, device=q.device)
+    strides = (ctypes.c_longlong * 11)(*[t.stride(i) for t in (q, k, v) for i in range(3)], row_stride(a), row_stride(b))
+    check(lib().tyr_gdr_recurrent_channel(ptr(q), ptr(k), ptr(v), ptr(a), ptr(b), ptr(dt_bias), ptr(a_log), ptr(state), ptr(out), ptr(lens), strides,
+                                          B, S, Hk, Hv, dk, dv, _dt(q), cur_stream(q.device)), "gdr_recurrent_channel")
+    return out
+
+
+def channel_delta_prefill(q, k, v, a, b, dt_bias, a_log, state: torch.Tensor, lens: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """:func:`delta_prefill` with a decay per key channel (operands of :func:`recurrent_channel_delta`)."""
+    state.zero_()
+    return recurrent_channel_delta(q, k, v, a, b, dt_bias, a_log, state, lens)
+
+
+def channel_delta_decode(q, k, v, a, b, z, dt_bias, a_log, norm_w: torch.Tensor, eps: float, state: torch.Tensor, out: torch.Tensor) -> None:
+    """One token per row: recurrence on ``state`` (in place), norm of the read-out and sigmoid gate ``z`` [B, 1, Hv * dv] -> ``out``."""
+    gated_norm(recurrent_channel_delta(q, k, v, a, b, dt_bias, a_log, state), z, norm_w, eps, "sigmoid", out)

@@ -1,13 +1,14 @@
-"""Embedding-table gradient from rows sorted by token id (csrc/embed.cu)."""
+"""Embedding kernels (csrc/embed.cu): table gradient from rows sorted by token id; scaled rows with sinusoidal positions."""
 from __future__ import annotations
 
 import ctypes
-from typing import Tuple
+import math
+from typing import Optional, Tuple
 
 import torch
 
 from .._native import register_signatures
-from ._common import check, cur_stream, lib, ptr
+from ._common import check, cur_stream, err_word, lib, ptr
 
 
 @register_signatures
@@ -16,6 +17,10 @@ def _sigs(lib_):
     fn = getattr(lib_, "tyr_embed_grad_sorted", None)
     if fn is not None:
         fn.argtypes = [P, P, P, P, I, I, L, I, P]
+        fn.restype = I
+    fn = getattr(lib_, "tyr_embed_positions", None)
+    if fn is not None:
+        fn.argtypes = [P, P, P, P, P, L, I, I, I, ctypes.c_float, I, P, P]
         fn.restype = I
 
 
@@ -39,3 +44,28 @@ def embedding_grad_(grad_table: torch.Tensor, dy: torch.Tensor, idx: torch.Tenso
                                           grad_table.shape[0], cur_stream(flat.device)), "embed_grad_sorted")
         return
     grad_table.index_add_(0, idx.reshape(-1), flat.to(grad_table.dtype))
+
+
+def position_turns(width: int, base: float = 10000.0, device="cpu") -> torch.Tensor:
+    """Frequencies of the sinusoidal position vector over 2 pi, in double: channel pair i turns ``base^(-2i / width) / 2 pi`` per position."""
+    i = torch.arange((width + 1) // 2, dtype=torch.float64)
+    return (base ** (-2.0 * i / width) / (2.0 * math.pi)).to(device)
+
+
+def embed_positions(ids: torch.Tensor, table: torch.Tensor, turns: torch.Tensor, scale: float, pos: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """fp32 [B, S, D]: ``table[ids] * scale`` plus the sinusoidal vector of each position (channel 2i the sine, 2i + 1 the cosine).
+    ``pos``: int32 [B] positions of single tokens (S == 1); without it positions count from 0 in every row."""
+    B, S = ids.shape
+    V, D = table.shape
+    if not ids.is_cuda:
+        p = (torch.arange(S)[None] if pos is None else pos[:, None]).double()
+        angle = 2.0 * math.pi * torch.frac(p[..., None] * turns)
+        vec = torch.stack([torch.sin(angle), torch.cos(angle)], -1).flatten(-2)[..., :D].float()
+        return torch.nn.functional.embedding(ids, table).float() * scale + vec
+    assert ids.dtype == torch.int64 and table.is_contiguous() and turns.dtype == torch.float64 and turns.numel() == (D + 1) // 2
+    assert pos is None or (S == 1 and pos.dtype == torch.int32 and pos.numel() == B)
+    x = torch.empty((B, S, D), dtype=torch.float32, device=ids.device)
+    kind = {torch.bfloat16: 0, torch.float32: 1}[table.dtype]
+    check(lib().tyr_embed_positions(ptr(ids.contiguous()), ptr(table), ptr(turns), ptr(pos), ptr(x), B * S, S, D, V, scale, kind, ptr(err_word(ids.device)),
+                                    cur_stream(ids.device)), "embed_positions")
+    return x

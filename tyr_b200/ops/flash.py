@@ -35,6 +35,10 @@ def _sigs(lib_):
     if fn is not None:
         fn.argtypes = [P, P, P, P, P, P, I, I, I, I, I, I, ctypes.POINTER(L), I, F, P, P]
         fn.restype = ctypes.c_int
+    fn = getattr(lib_, "tyr_flash_fwd_sink", None)
+    if fn is not None:
+        fn.argtypes = [P, P, P, P, P, P, I, I, I, I, I, I, ctypes.POINTER(L), F, F, P, P]
+        fn.restype = ctypes.c_int
     fn = getattr(lib_, "tyr_flash_bwd_workspace_bytes", None)
     if fn is not None:
         fn.argtypes = [I, I, I]
@@ -170,3 +174,26 @@ class _FlashPackedFn(torch.autograd.Function):
 
 def flash_attention_packed(qkv, B, T, H, D, *, causal=True, window=None, scale=None):
     return _FlashPackedFn.apply(qkv, B, T, H, D, causal, window, scale)
+
+
+def sink_supported(q, k, v, gate, out) -> bool:
+    """[B, T, H, D] bf16 views with query / key and value sizes up to 128, multiples of 8; 16-byte aligned rows of gate and output."""
+    rows = lambda t: t is None or (t.dtype == torch.bfloat16 and t.stride(2) == 1 and t.stride(0) % 8 == 0 and t.stride(1) % 8 == 0 and t.data_ptr() % 16 == 0)
+    return biased_supported(q, k, v) and hasattr(lib(), "tyr_flash_fwd_sink") and rows(gate) and rows(out)
+
+
+def flash_fwd_sink(q, k, v, *, scale: float, sink=None, gate=None, out_scale: float = 1.0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Causal attention of whole prompts with ``exp(sink[h])`` in the softmax denominator and the output multiplied by
+    ``out_scale * sigmoid(gate)``.  q: [B, T, Hq, dk], k: [B, T, Hkv, dk], v: [B, T, Hkv, dv] (views), sink fp32 [Hq], gate
+    [B, T, Hq * dv] -> [B, T, Hq * dv]."""
+    import ctypes
+    B, T, Hq, dk = q.shape
+    Hkv, dv = k.shape[2], v.shape[3]
+    if out is None:
+        out = torch.empty((B, T, Hq * dv), dtype=q.dtype, device=q.device)
+    o4 = out.unflatten(2, (Hq, dv))
+    strides = (ctypes.c_longlong * 15)(*[x for t in (q, k, v, o4) for x in _bthd_strides(t)],
+                                       *((0, 0, 0) if gate is None else _bthd_strides(gate.unflatten(2, (Hq, dv)))))
+    check(lib().tyr_flash_fwd_sink(ptr(q), ptr(k), ptr(v), ptr(out), ptr(sink), ptr(gate), B, Hq, Hkv, T, dk, dv, strides, scale, out_scale,
+                                   ptr(err_word(q.device)), cur_stream(q.device)), "flash_fwd_sink")
+    return out

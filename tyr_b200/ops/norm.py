@@ -24,6 +24,10 @@ def _sigs(lib_):
     if fn is not None:
         fn.argtypes = [P, L, P, I, P, P, L, I, F, I, I, P]
         fn.restype = I
+    fn = getattr(lib_, "tyr_add_norm", None)
+    if fn is not None:
+        fn.argtypes = [P, L, P, P, L, P, L, I, F, I, I, P]
+        fn.restype = I
 
 EPS = 1e-6
 
@@ -167,3 +171,23 @@ def post_norm_residual(x: torch.Tensor, gain: torch.Tensor, eps: float, resid: O
     check(lib().tyr_post_norm_residual(ptr(xr), xr.stride(0), ptr(gain), gain.numel(), ptr(resid), ptr(y), xr.shape[0], D, eps, kinds[x.dtype],
                                        kinds[out_dtype], cur_stream(x.device)), "post_norm_residual")
     return resid.view(x.shape) if same else y
+
+
+def add_norm(x: Optional[torch.Tensor], gain: torch.Tensor, eps: float, resid: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
+    """``resid += x`` IN PLACE on an fp32 residual stream [..., D] (left alone without ``x``), and ``norm(resid) * gain`` of the sum in
+    ``out_dtype``: a sublayer's residual add and the next sublayer's norm in one launch.  ``gain``: fp32, one per channel.  ``resid`` may
+    be rows of a view (evenly spaced)."""
+    D = resid.shape[-1]
+    if not resid.is_cuda:
+        if x is not None:
+            resid += x
+        return (rms_norm_ref(resid, eps) * gain).to(out_dtype)
+    kinds = {torch.bfloat16: 0, torch.float32: 1}
+    r = resid.view(-1, D)
+    x2 = None if x is None else x.reshape(-1, D)
+    assert gain.dtype == resid.dtype == torch.float32 and gain.shape == (D,) and gain.is_contiguous() and r.stride(1) == 1
+    assert x2 is None or (x2.stride(1) == 1 and x2.shape == r.shape)
+    y = torch.empty(resid.shape, dtype=out_dtype, device=resid.device)
+    check(lib().tyr_add_norm(ptr(x2), 0 if x2 is None else x2.stride(0), ptr(gain), ptr(r), r.stride(0), ptr(y), r.shape[0], D, eps,
+                             kinds[out_dtype if x2 is None else x2.dtype], kinds[out_dtype], cur_stream(resid.device)), "add_norm")
+    return y
