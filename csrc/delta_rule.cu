@@ -168,19 +168,28 @@ __device__ __forceinline__ void gdr_bulk_store(void* dst, const void* src, uint3
                : "memory");
 }
 
-template <int DK>
+//
+// CHANNEL: a decay per key channel, computed here together with the write strength from their projections, and a gate that is the
+// sigmoid alone.
+struct GdrChannelStep {
+  const __nv_bfloat16 *a_raw, *b_raw;      // [B, Hv * DK] and [B, Hv], batch strides below
+  long long a_bs, b_bs;
+  const float *dt_bias, *a_log;            // [Hv * DK], [Hv]
+};
+
+template <int DK, bool CHANNEL>
 __global__ void __launch_bounds__(256)
 gdr_decode_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k,
                        const __nv_bfloat16* __restrict__ v, const float* __restrict__ g,
                        const float* __restrict__ beta, float* __restrict__ state, __nv_bfloat16* __restrict__ out,
                        int Hk, int Hv, long long q_bstride, long long v_bstride,
                        const __nv_bfloat16* __restrict__ z, long long z_bstride, const __nv_bfloat16* __restrict__ norm_w,
-                       float norm_eps, int round_o, int* err) {
+                       float norm_eps, int round_o, long long out_bstride, GdrChannelStep cs, int* err) {
   constexpr int DV = 128, RG = 8, RPT = DK / RG;
   constexpr uint32_t kBytes = DK * DV * 4, kPiece = kBytes / 4;
   extern __shared__ __align__(128) uint8_t gdr_smem[];
   float* tile = reinterpret_cast<float*>(gdr_smem);                      // [DK][128]
-  __shared__ float sq[DK], sk[DK];
+  __shared__ float sq[DK], sk[DK], sd[CHANNEL ? DK : 1];
   __shared__ float red[2][RG];
   __shared__ __align__(16) float part[RG][DV];
   __shared__ __align__(8) uint64_t bar;
@@ -209,6 +218,10 @@ gdr_decode_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
     const float a = __bfloat162float(qp[tid]), c = __bfloat162float(kp[tid]);
     sq[tid] = a; sk[tid] = c;
     qs = a * a; ks = c * c;
+    if constexpr (CHANNEL) {
+      const float z = __bfloat162float(cs.a_raw[b * cs.a_bs + hv * DK + tid]) + cs.dt_bias[hv * DK + tid];
+      sd[tid] = __expf(-__expf(cs.a_log[hv]) * (fmaxf(z, 0.f) + log1pf(__expf(-fabsf(z)))));
+    }
   }
   qs = warp_sum(qs); ks = warp_sum(ks);
   if (quad == 0) { red[0][rg] = qs; red[1][rg] = ks; }
@@ -218,8 +231,8 @@ gdr_decode_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
   for (int i = 0; i < RG; ++i) { qs += red[0][i]; ks += red[1][i]; }
   const float qn = rsqrtf(qs + 1e-6f) * rsqrtf(static_cast<float>(DK));
   const float kn = rsqrtf(ks + 1e-6f);
-  const float decay = __expf(g[bh]);
-  const float bt = beta[bh];
+  const float decay = CHANNEL ? 1.f : __expf(g[bh]);
+  const float bt = CHANNEL ? 1.f / (1.f + __expf(-__bfloat162float(cs.b_raw[b * cs.b_bs + hv]))) : beta[bh];
   const int col = 4 * quad;
   const __nv_bfloat16* vp = v + b * v_bstride + static_cast<long long>(hv) * DV;
   float vt[4];
@@ -237,7 +250,7 @@ gdr_decode_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
 #pragma unroll
   for (int r = 0; r < RPT; ++r) {
     const float4 t = trow[r * (DV / 4)];
-    const float kk = sk[rg * RPT + r];
+    const float kk = CHANNEL ? sk[rg * RPT + r] * sd[rg * RPT + r] : sk[rg * RPT + r];
     kv[0] += t.x * kk; kv[1] += t.y * kk; kv[2] += t.z * kk; kv[3] += t.w * kk;
   }
   *reinterpret_cast<float4*>(&part[rg][col]) = make_float4(kv[0], kv[1], kv[2], kv[3]);
@@ -256,9 +269,9 @@ gdr_decode_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
 #pragma unroll
   for (int r = 0; r < RPT; ++r) {
     float4 t = trow[r * (DV / 4)];
-    const float kk = sk[rg * RPT + r], qq = sq[rg * RPT + r];
-    t.x = t.x * decay + kk * delta[0]; t.y = t.y * decay + kk * delta[1];
-    t.z = t.z * decay + kk * delta[2]; t.w = t.w * decay + kk * delta[3];
+    const float kk = sk[rg * RPT + r], qq = sq[rg * RPT + r], de = CHANNEL ? sd[rg * RPT + r] : decay;
+    t.x = t.x * de + kk * delta[0]; t.y = t.y * de + kk * delta[1];
+    t.z = t.z * de + kk * delta[2]; t.w = t.w * de + kk * delta[3];
     o[0] += t.x * qq; o[1] += t.y * qq; o[2] += t.z * qq; o[3] += t.w * qq;
     trow[r * (DV / 4)] = t;
   }
@@ -278,7 +291,7 @@ gdr_decode_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
       const float4 t = *reinterpret_cast<const float4*>(&part[i][col]);
       o[0] += t.x; o[1] += t.y; o[2] += t.z; o[3] += t.w;
     }
-    __nv_bfloat16* op = out + static_cast<long long>(bh) * DV + col;
+    __nv_bfloat16* op = out + b * out_bstride + static_cast<long long>(hv) * DV + col;
     if (z != nullptr) {
       float ssq = 0.f;
 #pragma unroll
@@ -293,7 +306,7 @@ gdr_decode_tile_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16*
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         const float zz = __bfloat162float(zp[c]);
-        o[c] = o[c] * rstd * __bfloat162float(norm_w[col + c]) * (zz / (1.f + __expf(-zz)));
+        o[c] = o[c] * rstd * __bfloat162float(norm_w[col + c]) * ((CHANNEL ? 1.f : zz) / (1.f + __expf(-zz)));
       }
     } else {
 #pragma unroll
@@ -428,11 +441,12 @@ __device__ __forceinline__ void mma_op(float (&c)[4], const Tf32Op<EXACT> (&a)[4
 __device__ __forceinline__ void store_pair(__nv_bfloat16* p, float x, float y) { *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(x, y); }
 __device__ __forceinline__ void store_pair(float* p, float x, float y) { *reinterpret_cast<float2*>(p) = make_float2(x, y); }
 
-// `dv` columns of the state and the output; `u` has rows of dvp = dv rounded up to 64 columns.
+// `dv` columns of the state and the output; `u` has rows of dvp = dv rounded up to 64 columns.  `glast` holds the chunk's decay of the
+// state: one number (gl_ld 1) or one per key channel (gl_ld GC_DK).
 template <bool EXACT, typename OutT>
 __global__ void __launch_bounds__(256, 1)
 gdr_chunk_scan_kernel(const float* __restrict__ u, const float* __restrict__ w, const float* __restrict__ qg,
-                      const float* __restrict__ kd, const float* __restrict__ intra, const float* __restrict__ glast,
+                      const float* __restrict__ kd, const float* __restrict__ intra, const float* __restrict__ glast, int gl_ld,
                       const float* __restrict__ state_in, float* __restrict__ state_out, OutT* __restrict__ out, int n,
                       int dk, int dv, int dvp, int seq, int Hv) {
   using Op = Tf32Op<EXACT>;
@@ -537,13 +551,18 @@ gdr_chunk_scan_kernel(const float* __restrict__ u, const float* __restrict__ w, 
       }
     } else {
       // ---- S <- exp(g_last) S + kd_i^T v_new : this warp's 32 state rows, K = chunk
-      const float e = glast[static_cast<long long>(bh) * n + i];
+      const float* gl = glast + (static_cast<long long>(bh) * n + i) * gl_ld;
 #pragma unroll
       for (int mt = 0; mt < 2; ++mt)
 #pragma unroll
-        for (int nt = 0; nt < 8; ++nt)
+        for (int h2 = 0; h2 < 2; ++h2) {
+          const float e = gl[gl_ld == 1 ? 0 : warp * 32 + mt * 16 + g + h2 * 8];
 #pragma unroll
-          for (int q4 = 0; q4 < 4; ++q4) S[mt][nt][q4] *= e;
+          for (int nt = 0; nt < 8; ++nt) {
+            S[mt][nt][2 * h2] *= e;
+            S[mt][nt][2 * h2 + 1] *= e;
+          }
+        }
 #pragma unroll 1
       for (int kk = 0; kk < GC_C / 8; ++kk) {
         const int kc = kk * 8 + t, m = warp * 32 + g;       // A[m][k] = kd[k][m]
@@ -799,6 +818,285 @@ __global__ void __launch_bounds__(256, 2) gdr_chunk_prepare_kernel(GdrPrepArgs a
   }
 }
 
+// ------------------------------------------------------------------------------------------------------------------
+// The same chunk-local quantities with a decay per key channel: with G the cumulative log decay of a channel,
+//     (k_i . k_j) exp(gc_i - gc_j)   becomes   sum_d k_id k_jd exp(G_id - G_jd).
+// To stay on tensor cores the exponential is split into factors that belong to one operand each and cannot overflow: the chunk is
+// cut into four blocks of 16 tokens, and with P_b the cumulative log decay up to the start of block b and gl the one inside a block,
+//     kh_i = k_i exp(gl_i) <= k_i,   kt_j = k_j exp(gl_end - gl_j) <= k_j,   exp(G_i - G_j) = [kh_i exp(P_I - P_(J+1))] kt_j
+// for row i in block I and column j in block J <= I; the scale is at most 1 for J < I and exp(|decay of one block|) for J = I.  A chunk
+// with a block whose decay passes exp(-60) in some channel (GP_STEEP) evaluates its diagonal blocks pair by pair instead.
+// Decay and write strength are computed here from their projections.
+// ------------------------------------------------------------------------------------------------------------------
+constexpr float GP_STEEP = -60.f;
+
+struct GdrPrepChannelSmem {
+  float k[GC_C * GC_LDW];            // raw, then kh
+  float q[GC_C * GC_LDW];            // raw, then q exp(gl); then the matrix of the triangular solve [64][GP_LDA]
+  float kt[GC_C * GC_LDW];
+  float pre[5][GC_DK];               // P_b
+  float beta[GC_C];
+};
+
+struct GdrPrepChannelArgs {
+  const __nv_bfloat16 *q, *k, *v, *a_raw, *b_raw;
+  const float *dt_bias, *a_log;        // [Hv * dk], [Hv]
+  float *u, *w, *qg, *kd, *intra, *glast;
+  const int* lens;
+  long long q_sb, q_ss, q_sh, k_sb, k_ss, k_sh, v_sb, v_ss, v_sh, a_ld, b_ld;
+  int S, n, Hk, Hv, dk, dv, dvp;
+};
+
+__global__ void __launch_bounds__(256, 2) gdr_chunk_prepare_channel_kernel(GdrPrepChannelArgs a) {
+  extern __shared__ __align__(16) uint8_t gdr_smem_raw[];
+  GdrPrepChannelSmem& sm = *reinterpret_cast<GdrPrepChannelSmem*>(gdr_smem_raw);
+  const int c = blockIdx.x, bh = blockIdx.y;
+  const int b = bh / a.Hv, hv = bh % a.Hv, hk = hv / (a.Hv / a.Hk);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int row0 = c * GC_C;
+  const int len = a.lens ? min(a.lens[b], a.S) : a.S;
+  // ---- 1. stage q, k (fp32) and beta
+  for (int i = tid; i < GC_C * (GC_DK / 8); i += 256) {
+    const int r = i / (GC_DK / 8), d = (i % (GC_DK / 8)) * 8;
+    const int tok = row0 + r;
+    uint4 uq = make_uint4(0, 0, 0, 0), uk = make_uint4(0, 0, 0, 0);
+    if (tok < len && d < a.dk) {
+      uq = *reinterpret_cast<const uint4*>(a.q + b * a.q_sb + static_cast<long long>(tok) * a.q_ss + hk * a.q_sh + d);
+      uk = *reinterpret_cast<const uint4*>(a.k + b * a.k_sb + static_cast<long long>(tok) * a.k_ss + hk * a.k_sh + d);
+    }
+    const uint32_t qq[4] = {uq.x, uq.y, uq.z, uq.w}, kk[4] = {uk.x, uk.y, uk.z, uk.w};
+    float4 fq[2], fk[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const float2 q0 = unpack_bf16x2(qq[2 * e]), q1 = unpack_bf16x2(qq[2 * e + 1]), k0 = unpack_bf16x2(kk[2 * e]), k1 = unpack_bf16x2(kk[2 * e + 1]);
+      fq[e] = make_float4(q0.x, q0.y, q1.x, q1.y);
+      fk[e] = make_float4(k0.x, k0.y, k1.x, k1.y);
+      *reinterpret_cast<float4*>(&sm.q[r * GC_LDW + d + 4 * e]) = fq[e];
+      *reinterpret_cast<float4*>(&sm.k[r * GC_LDW + d + 4 * e]) = fk[e];
+    }
+  }
+  if (tid < GC_C) {
+    const int tok = row0 + tid;
+    sm.beta[tid] = tok < len ? 1.f / (1.f + __expf(-__bfloat162float(a.b_raw[(static_cast<long long>(b) * a.S + tok) * a.b_ld + hv]))) : 0.f;
+  }
+  // ---- 2. log decays: a thread owns one channel of two blocks; gl = cumulative inside a block
+  const int d = tid & (GC_DK - 1), half = tid >> 7;
+  float gl[2][16];
+  {
+    const bool live = d < a.dk;
+    const float bias = live ? a.dt_bias[hv * a.dk + d] : 0.f, rate = -__expf(a.a_log[hv]);
+    const __nv_bfloat16* ap = a.a_raw + static_cast<long long>(b) * a.S * a.a_ld + static_cast<long long>(hv) * a.dk + d;
+#pragma unroll
+    for (int h = 0; h < 2; ++h)
+#pragma unroll
+      for (int t = 0; t < 16; ++t) {
+        const int tok = row0 + (half * 2 + h) * 16 + t;
+        gl[h][t] = live && tok < len ? __bfloat162float(ap[tok * a.a_ld]) + bias : -INFINITY;
+      }
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      float run = 0.f;
+#pragma unroll
+      for (int t = 0; t < 16; ++t) {
+        const float z = gl[h][t];
+        run += rate * (z == -INFINITY ? 0.f : fmaxf(z, 0.f) + log1pf(__expf(-fabsf(z))));
+        gl[h][t] = run;
+      }
+    }
+  }
+  const bool steep = __syncthreads_or(gl[0][15] < GP_STEEP || gl[1][15] < GP_STEEP);
+  // L2 normalisation: 4 threads per row
+  {
+    const int r = tid >> 2, part = tid & 3;
+    float sq = 0.f, sk = 0.f;
+    for (int e = part; e < GC_DK; e += 4) {
+      const float x = sm.q[r * GC_LDW + e], y = sm.k[r * GC_LDW + e];
+      sq += x * x; sk += y * y;
+    }
+    sq += __shfl_xor_sync(0xffffffffu, sq, 1); sq += __shfl_xor_sync(0xffffffffu, sq, 2);
+    sk += __shfl_xor_sync(0xffffffffu, sk, 1); sk += __shfl_xor_sync(0xffffffffu, sk, 2);
+    const float qn = rsqrtf(sq + 1e-6f) * rsqrtf(static_cast<float>(a.dk)), kn = rsqrtf(sk + 1e-6f);
+    for (int e = part; e < GC_DK; e += 4) {
+      sm.q[r * GC_LDW + e] *= qn;
+      sm.k[r * GC_LDW + e] *= kn;
+    }
+  }
+  float dia_k[4], dia_q[4];                          // steep chunks: this thread's pair of each diagonal block
+  if (steep) {
+#pragma unroll
+    for (int h = 0; h < 2; ++h)
+#pragma unroll
+      for (int t = 0; t < 16; ++t) sm.kt[((half * 2 + h) * 16 + t) * GC_LDW + d] = gl[h][t];
+    __syncthreads();
+    const int pi = tid >> 4, pj = tid & 15;
+#pragma unroll 1
+    for (int blk = 0; blk < 4; ++blk) {
+      const float *ki = sm.k + (blk * 16 + pi) * GC_LDW, *qi = sm.q + (blk * 16 + pi) * GC_LDW, *gi = sm.kt + (blk * 16 + pi) * GC_LDW;
+      const float *kj = sm.k + (blk * 16 + pj) * GC_LDW, *gj = sm.kt + (blk * 16 + pj) * GC_LDW;
+      float sk = 0.f, sq = 0.f;
+      if (pj <= pi)
+        for (int e = 0; e < GC_DK; ++e) {
+          const float w = __expf(gi[e] - gj[e]) * kj[e];
+          sk += ki[e] * w;
+          sq += qi[e] * w;
+        }
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (e == blk) { dia_k[e] = sk; dia_q[e] = sq; }
+    }
+  }
+  __syncthreads();
+  // ---- 3. kh, q exp(gl), kt
+#pragma unroll
+  for (int h = 0; h < 2; ++h)
+#pragma unroll
+    for (int t = 0; t < 16; ++t) {
+      const int i = ((half * 2 + h) * 16 + t) * GC_LDW + d;
+      const float e = __expf(gl[h][t]), kk = sm.k[i];
+      sm.k[i] = kk * e;
+      sm.q[i] *= e;
+      sm.kt[i] = kk * __expf(gl[h][15] - gl[h][t]);
+    }
+  sm.pre[half * 2 + 1][d] = gl[0][15];               // the blocks' own decays first, then their running sum
+  sm.pre[half * 2 + 2][d] = gl[1][15];
+  __syncthreads();
+  if (tid < GC_DK) {
+    float run = 0.f;
+    sm.pre[0][tid] = 0.f;
+#pragma unroll
+    for (int i = 1; i <= 4; ++i) {
+      run += sm.pre[i][tid];
+      sm.pre[i][tid] = run;
+    }
+  }
+  __syncthreads();
+  // ---- 4. warps 0-3: k k^T strips, warps 4-7: q k^T strips (one block of 16 rows each), 3-term TF32
+  const int g8 = lane >> 2, t4 = lane & 3;
+  const bool is_q = warp >= 4;
+  const int I = warp & 3, ar = I * 16 + g8;
+  float acc[8][4];
+#pragma unroll
+  for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[nt][e] = 0.f;
+  {
+    const float* A = is_q ? sm.q : sm.k;
+    const int last = steep ? I - 1 : I;
+#pragma unroll 1
+    for (int kk = 0; kk < GC_DK / 8; ++kk) {
+      const int kc = kk * 8 + t4;
+      const float af[4] = {A[ar * GC_LDW + kc], A[(ar + 8) * GC_LDW + kc], A[ar * GC_LDW + kc + 4], A[(ar + 8) * GC_LDW + kc + 4]};
+      const float p0 = sm.pre[I][kc], p1 = sm.pre[I][kc + 4];
+#pragma unroll
+      for (int J = 0; J < 4; ++J) {
+        if (J > last) break;
+        const float s0 = __expf(p0 - sm.pre[J + 1][kc]), s1 = __expf(p1 - sm.pre[J + 1][kc + 4]);
+        uint32_t ah[4], al[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const float x = af[e] * (e < 2 ? s0 : s1);
+          ah[e] = to_tf32(x);
+          al[e] = to_tf32(x - __uint_as_float(ah[e]));
+        }
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const int nt = 2 * J + h;
+          const float b0f = sm.kt[(nt * 8 + g8) * GC_LDW + kc], b1f = sm.kt[(nt * 8 + g8) * GC_LDW + kc + 4];
+          const uint32_t b0h = to_tf32(b0f), b1h = to_tf32(b1f);
+          const uint32_t b0l = to_tf32(b0f - __uint_as_float(b0h)), b1l = to_tf32(b1f - __uint_as_float(b1h));
+          mma_tf32(acc[nt], al[0], al[1], al[2], al[3], b0h, b1h);
+          mma_tf32(acc[nt], ah[0], ah[1], ah[2], ah[3], b0l, b1l);
+          mma_tf32(acc[nt], ah[0], ah[1], ah[2], ah[3], b0h, b1h);
+        }
+      }
+    }
+  }
+  // ---- 5. qg = q exp(G), kd = k exp(G_last - G), glast = exp(G_last)
+  {
+    float* qg_o = a.qg + (static_cast<long long>(bh) * a.n + c) * GC_C * GC_DK;
+    float* kd_o = a.kd + (static_cast<long long>(bh) * a.n + c) * GC_C * GC_DK;
+    for (int i = tid; i < GC_C * (GC_DK / 4); i += 256) {
+      const int r = i / (GC_DK / 4), e = (i % (GC_DK / 4)) * 4, blk = r >> 4;
+      const float4 p = *reinterpret_cast<const float4*>(&sm.pre[blk][e]), pn = *reinterpret_cast<const float4*>(&sm.pre[blk + 1][e]);
+      const float4 pl = *reinterpret_cast<const float4*>(&sm.pre[4][e]);
+      const float4 fq = *reinterpret_cast<const float4*>(&sm.q[r * GC_LDW + e]), fk = *reinterpret_cast<const float4*>(&sm.kt[r * GC_LDW + e]);
+      *reinterpret_cast<float4*>(qg_o + r * GC_DK + e) = make_float4(fq.x * __expf(p.x), fq.y * __expf(p.y), fq.z * __expf(p.z), fq.w * __expf(p.w));
+      *reinterpret_cast<float4*>(kd_o + r * GC_DK + e) =
+          make_float4(fk.x * __expf(pl.x - pn.x), fk.y * __expf(pl.y - pn.y), fk.z * __expf(pl.z - pn.z), fk.w * __expf(pl.w - pn.w));
+    }
+    if (tid < GC_DK) a.glast[(static_cast<long long>(bh) * a.n + c) * GC_DK + tid] = __expf(sm.pre[4][tid]);
+  }
+  __syncthreads();                                   // sm.q is free: it becomes the matrix of the solve
+  float* const mat = sm.q;
+  float* const intra_o = a.intra + (static_cast<long long>(bh) * a.n + c) * GC_C * GC_C;
+#pragma unroll
+  for (int nt = 0; nt < 8; ++nt)
+#pragma unroll
+    for (int h2 = 0; h2 < 2; ++h2) {
+      const int i = ar + h2 * 8, j = nt * 8 + 2 * t4;
+      const float v0 = acc[nt][2 * h2], v1 = acc[nt][2 * h2 + 1];
+      if (is_q) {
+        *reinterpret_cast<float2*>(intra_o + i * GC_C + j) = make_float2(j <= i ? v0 : 0.f, j + 1 <= i ? v1 : 0.f);
+      } else {
+        const float bi = sm.beta[i];
+        mat[i * GP_LDA + j] = j < i ? v0 * bi : 0.f;
+        mat[i * GP_LDA + j + 1] = j + 1 < i ? v1 * bi : 0.f;
+      }
+    }
+  __syncthreads();
+  if (steep) {
+    const int pi = tid >> 4, pj = tid & 15;
+    if (pj <= pi)
+#pragma unroll
+      for (int blk = 0; blk < 4; ++blk) {
+        const int i = blk * 16 + pi, j = blk * 16 + pj;
+        intra_o[i * GC_C + j] = dia_q[blk];
+        if (pj < pi) mat[i * GP_LDA + j] = dia_k[blk] * sm.beta[i];
+      }
+    __syncthreads();
+  }
+  // ---- 6. forward substitution, one right-hand-side column per thread
+  const int col = tid;
+  if (col < a.dvp + GC_DK) {
+    float x[GC_C];
+    const bool is_v = col < a.dvp;
+    if (is_v) {
+      const __nv_bfloat16* vp = a.v + b * a.v_sb + hv * a.v_sh + col;
+#pragma unroll
+      for (int i = 0; i < GC_C; ++i) {
+        const int tok = row0 + i;
+        x[i] = tok < len && col < a.dv ? __bfloat162float(vp[static_cast<long long>(tok) * a.v_ss]) * sm.beta[i] : 0.f;
+      }
+    } else {
+      const int e = col - a.dvp;
+#pragma unroll
+      for (int blk = 0; blk < 4; ++blk) {
+        const float p = __expf(sm.pre[blk][e]);
+#pragma unroll
+        for (int t = 0; t < 16; ++t) x[blk * 16 + t] = sm.k[(blk * 16 + t) * GC_LDW + e] * p * sm.beta[blk * 16 + t];
+      }
+    }
+#pragma unroll
+    for (int i = 1; i < GC_C; ++i) {
+      float s = x[i];
+#pragma unroll
+      for (int j4 = 0; j4 < (i + 3) / 4; ++j4) {
+        const float4 r4 = *reinterpret_cast<const float4*>(&mat[i * GP_LDA + 4 * j4]);     // entries at j >= i are zero
+        s -= r4.x * x[4 * j4];
+        if (4 * j4 + 1 < i) s -= r4.y * x[4 * j4 + 1];
+        if (4 * j4 + 2 < i) s -= r4.z * x[4 * j4 + 2];
+        if (4 * j4 + 3 < i) s -= r4.w * x[4 * j4 + 3];
+      }
+      x[i] = s;
+    }
+    float* dst = is_v ? a.u + (static_cast<long long>(bh) * a.n + c) * GC_C * a.dvp + col
+                      : a.w + (static_cast<long long>(bh) * a.n + c) * GC_C * GC_DK + (col - a.dvp);
+    const int ld = is_v ? a.dvp : GC_DK;
+#pragma unroll
+    for (int i = 0; i < GC_C; ++i) dst[static_cast<long long>(i) * ld] = x[i];
+  }
+}
+
 }  // namespace tyr
 
 // Causal depthwise conv1d (kernel taps K <= 4, zero history) + bias + SiLU on channels-last activations:
@@ -928,14 +1226,53 @@ extern "C" TYR_EXPORT int tyr_gdr_chunk_prepare(const void* q, const void* k, co
   return static_cast<int>(cudaGetLastError());
 }
 
+// Chunk-local quantities with a decay per key channel: a_raw bf16 [B * S, .] (channel hv * dk + d) and b_raw bf16 (channel hv) with row
+// strides strides[9] and strides[10]; log decay -exp(a_log[hv]) softplus(a_raw + dt_bias), write strength sigmoid(b_raw).  Outputs as
+// above with glast [B*Hv, n, 128].
+extern "C" TYR_EXPORT int tyr_gdr_chunk_prepare_channel(const void* q, const void* k, const void* v, const void* a_raw, const void* b_raw,
+                                                        const float* dt_bias, const float* a_log, float* u, float* w, float* qg, float* kd,
+                                                        float* intra, float* glast, const int* lens, const long long* strides, int B, int S,
+                                                        int Hk, int Hv, int dk, int dv, void* stream) {
+  using namespace tyr;
+  if (B <= 0 || S <= 0 || Hk <= 0 || Hv <= 0 || Hv % Hk || dk <= 0 || dk > GC_DK || (dk & 7) || dv <= 0 || dv > 128 || (dv & 7)) return -1;
+  for (int i = 0; i < 9; ++i)
+    if (strides[i] & 7) return -3;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v)) & 15) return -4;
+  GdrPrepChannelArgs a;
+  a.q = reinterpret_cast<const __nv_bfloat16*>(q);
+  a.k = reinterpret_cast<const __nv_bfloat16*>(k);
+  a.v = reinterpret_cast<const __nv_bfloat16*>(v);
+  a.a_raw = reinterpret_cast<const __nv_bfloat16*>(a_raw);
+  a.b_raw = reinterpret_cast<const __nv_bfloat16*>(b_raw);
+  a.dt_bias = dt_bias; a.a_log = a_log; a.u = u; a.w = w; a.qg = qg; a.kd = kd; a.intra = intra; a.glast = glast;
+  a.q_sb = strides[0]; a.q_ss = strides[1]; a.q_sh = strides[2];
+  a.k_sb = strides[3]; a.k_ss = strides[4]; a.k_sh = strides[5];
+  a.v_sb = strides[6]; a.v_ss = strides[7]; a.v_sh = strides[8];
+  a.a_ld = strides[9]; a.b_ld = strides[10];
+  a.S = S; a.n = (S + GC_C - 1) / GC_C; a.Hk = Hk; a.Hv = Hv; a.dk = dk; a.dv = dv; a.dvp = (dv + 63) & ~63;
+  a.lens = lens;
+  constexpr size_t smem = sizeof(GdrPrepChannelSmem);
+  static bool configured_dev[64] = {false};     // the attribute is per device
+  int cfg_dev = 0;
+  if (cudaGetDevice(&cfg_dev) != cudaSuccess || cfg_dev < 0 || cfg_dev >= 64) cfg_dev = 0;
+  bool& configured = configured_dev[cfg_dev];
+  if (!configured) {
+    cudaError_t e = cudaFuncSetAttribute(gdr_chunk_prepare_channel_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return 1000 + (int)e;
+    configured = true;
+  }
+  gdr_chunk_prepare_channel_kernel<<<dim3(a.n, B * Hv), 256, smem, reinterpret_cast<cudaStream_t>(stream)>>>(a);
+  return static_cast<int>(cudaGetLastError());
+}
+
 // Sequential chunk pass of the gated delta rule (chunk 64, dk <= 128, dv even), all tensors fp32 and contiguous:
 // u [BH, n, 64, dvp], w / qg / kd [BH, n, 64, 128], intra [BH, n, 64, 64], glast [BH, n] (= exp of the chunk's last cumulative
-// log decay), state_in [BH, dk, dv] (nullable = zeros), state_out [BH, dk, dv]; out: [B, S, Hv, dv] with BH = B * Hv and
+// log decay; `channel`: [BH, n, 128], one per key channel), state_in [BH, dk, dv] (nullable = zeros), state_out [BH, dk, dv]; out: [B, S, Hv, dv] with BH = B * Hv and
 // n = ceil(S / 64), bf16, or fp32 with `exact` (split TF32 products).
 extern "C" TYR_EXPORT int tyr_gdr_chunk_scan(const float* u, const float* w, const float* qg, const float* kd,
                                              const float* intra, const float* glast, const float* state_in,
                                              float* state_out, void* out, int BH, int n, int dk, int dv, int chunk, int S,
-                                             int Hv, int exact, void* stream) {
+                                             int Hv, int exact, int channel, void* stream) {
   using namespace tyr;
   if (BH <= 0 || n <= 0 || dk <= 0 || dk > GC_DK || chunk != GC_C || dv <= 0 || (dv & 7) || Hv <= 0 || BH % Hv || S <= 0 || S > n * GC_C) return -1;
   if ((reinterpret_cast<uintptr_t>(u) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(qg) |
@@ -955,12 +1292,13 @@ extern "C" TYR_EXPORT int tyr_gdr_chunk_scan(const float* u, const float* w, con
   }
   const int slices = (dv + GC_DVS - 1) / GC_DVS, dvp = slices * GC_DVS;
   const dim3 grid(slices, BH);
+  const int gl_ld = channel ? GC_DK : 1;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   if (exact)
-    gdr_chunk_scan_kernel<true, float><<<grid, 256, smem, st>>>(u, w, qg, kd, intra, glast, state_in, state_out, reinterpret_cast<float*>(out),
+    gdr_chunk_scan_kernel<true, float><<<grid, 256, smem, st>>>(u, w, qg, kd, intra, glast, gl_ld, state_in, state_out, reinterpret_cast<float*>(out),
                                                                 n, dk, dv, dvp, S, Hv);
   else
-    gdr_chunk_scan_kernel<false, __nv_bfloat16><<<grid, 256, smem, st>>>(u, w, qg, kd, intra, glast, state_in, state_out,
+    gdr_chunk_scan_kernel<false, __nv_bfloat16><<<grid, 256, smem, st>>>(u, w, qg, kd, intra, glast, gl_ld, state_in, state_out,
                                                                          reinterpret_cast<__nv_bfloat16*>(out), n, dk, dv, dvp, S, Hv);
   return static_cast<int>(cudaGetLastError());
 }
@@ -996,42 +1334,55 @@ extern "C" TYR_EXPORT int tyr_gdr_decode(const void* q, const void* k, const voi
 // dv == 128, dk 64 or 128, v / z rows 8-byte aligned (strides multiples of 4 elements): the shared-memory tile form of the
 // step (gdr_decode_tile_kernel); `z` / `norm_w` may be null (no gated RMSNorm); `round_o`: the norm sees the
 // read-out rounded to bf16 (else fp32).  `err`: the device error record.
+static int decode_tile_launch(const void* q, const void* k, const void* v, const float* g, const float* beta, float* state, void* out, int B,
+                              int Hk, int Hv, int dk, long long q_bstride, long long v_bstride, const void* z, long long z_bstride,
+                              const void* norm_w, float norm_eps, int round_o, long long out_bstride, const tyr::GdrChannelStep* channel,
+                              int* err, void* stream) {
+  using namespace tyr;
+  if (B <= 0 || Hk <= 0 || Hv <= 0 || Hv % Hk != 0 || (dk != 64 && dk != 128)) return -1;
+  if (z != nullptr && norm_w == nullptr) return -3;
+  if ((v_bstride & 3) || (out_bstride & 3) || (z != nullptr && (z_bstride & 3))) return -4;
+  if ((reinterpret_cast<uintptr_t>(v) | reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(out)) & 7) return -4;
+  if (reinterpret_cast<uintptr_t>(state) & 15) return -4;
+  const size_t smem = static_cast<size_t>(dk) * 128 * 4;
+  auto kernel = channel != nullptr ? (dk == 128 ? gdr_decode_tile_kernel<128, true> : gdr_decode_tile_kernel<64, true>)
+                                   : (dk == 128 ? gdr_decode_tile_kernel<128, false> : gdr_decode_tile_kernel<64, false>);
+  static bool configured[64][2][2] = {};
+  int dev = 0;
+  if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) dev = 0;
+  bool& done = configured[dev][dk == 128 ? 1 : 0][channel != nullptr ? 1 : 0];
+  if (!done) {
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return 1000 + static_cast<int>(e);
+    done = true;
+  }
+  const GdrChannelStep cs = channel != nullptr ? *channel : GdrChannelStep{};
+  return static_cast<int>(launch_dependent(kernel, dim3(B * Hv), dim3(256), smem, reinterpret_cast<cudaStream_t>(stream),
+                                           reinterpret_cast<const __nv_bfloat16*>(q), reinterpret_cast<const __nv_bfloat16*>(k),
+                                           reinterpret_cast<const __nv_bfloat16*>(v), g, beta, state, reinterpret_cast<__nv_bfloat16*>(out), Hk, Hv,
+                                           q_bstride, v_bstride, reinterpret_cast<const __nv_bfloat16*>(z), z_bstride,
+                                           reinterpret_cast<const __nv_bfloat16*>(norm_w), norm_eps, round_o, out_bstride, cs, err));
+}
+
 extern "C" TYR_EXPORT int tyr_gdr_decode_tile(const void* q, const void* k, const void* v, const float* g, const float* beta,
                                               float* state, void* out, int B, int Hk, int Hv, int dk,
                                               long long q_bstride, long long v_bstride, const void* z, long long z_bstride,
                                               const void* norm_w, float norm_eps, int round_o, int* err, void* stream) {
-  using namespace tyr;
-  if (B <= 0 || Hk <= 0 || Hv <= 0 || Hv % Hk != 0 || (dk != 64 && dk != 128)) return -1;
-  if (z != nullptr && norm_w == nullptr) return -3;
-  if ((v_bstride & 3) || (z != nullptr && (z_bstride & 3))) return -4;
-  if ((reinterpret_cast<uintptr_t>(v) | reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(out)) & 7) return -4;
-  if (reinterpret_cast<uintptr_t>(state) & 15) return -4;
-  const size_t smem = static_cast<size_t>(dk) * 128 * 4;
-  static bool configured[64][2] = {};
-  int dev = 0;
-  if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) dev = 0;
-  const int which = dk == 128 ? 1 : 0;
-  if (!configured[dev][which]) {
-    cudaError_t e = dk == 128 ? cudaFuncSetAttribute(gdr_decode_tile_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)
-                              : cudaFuncSetAttribute(gdr_decode_tile_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e != cudaSuccess) return 1000 + static_cast<int>(e);
-    configured[dev][which] = true;
-  }
-  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
-  auto* qq = reinterpret_cast<const __nv_bfloat16*>(q);
-  auto* kk = reinterpret_cast<const __nv_bfloat16*>(k);
-  auto* vv = reinterpret_cast<const __nv_bfloat16*>(v);
-  auto* zz = reinterpret_cast<const __nv_bfloat16*>(z);
-  auto* nw = reinterpret_cast<const __nv_bfloat16*>(norm_w);
-  auto* oo = reinterpret_cast<__nv_bfloat16*>(out);
-  cudaError_t e;
-  if (dk == 128)
-    e = launch_dependent(gdr_decode_tile_kernel<128>, dim3(B * Hv), dim3(256), smem, st, qq, kk, vv, g, beta, state, oo, Hk, Hv,
-                         q_bstride, v_bstride, zz, z_bstride, nw, norm_eps, round_o, err);
-  else
-    e = launch_dependent(gdr_decode_tile_kernel<64>, dim3(B * Hv), dim3(256), smem, st, qq, kk, vv, g, beta, state, oo, Hk, Hv,
-                         q_bstride, v_bstride, zz, z_bstride, nw, norm_eps, round_o, err);
-  return static_cast<int>(e);
+  return decode_tile_launch(q, k, v, g, beta, state, out, B, Hk, Hv, dk, q_bstride, v_bstride, z, z_bstride, norm_w, norm_eps, round_o,
+                            static_cast<long long>(Hv) * 128, nullptr, err, stream);
+}
+
+// A decay per key channel (a_raw / b_raw, dt_bias and a_log as in the chunk form), the norm of the fp32 read-out and a sigmoid gate z.
+// strides: batch strides of q / k, v, a_raw, b_raw, z, out.
+extern "C" TYR_EXPORT int tyr_gdr_decode_tile_channel(const void* q, const void* k, const void* v, const void* a_raw, const void* b_raw,
+                                                      const float* dt_bias, const float* a_log, float* state, void* out, const void* z,
+                                                      const void* norm_w, const long long* strides, int B, int Hk, int Hv, int dk,
+                                                      float norm_eps, int* err, void* stream) {
+  if (z == nullptr) return -3;
+  const tyr::GdrChannelStep cs{reinterpret_cast<const __nv_bfloat16*>(a_raw), reinterpret_cast<const __nv_bfloat16*>(b_raw), strides[2], strides[3],
+                               dt_bias, a_log};
+  return decode_tile_launch(q, k, v, nullptr, nullptr, state, out, B, Hk, Hv, dk, strides[0], strides[1], z, strides[4], norm_w, norm_eps, 0,
+                            strides[5], &cs, err, stream);
 }
 
 // The same step with the layer's gated RMSNorm in the epilogue when `z` (bf16 [B, Hv, dv], batch stride z_bstride) and

@@ -229,6 +229,7 @@ class DeltaMixer:
     a_log: torch.Tensor               # fp32
     dt_bias: torch.Tensor
     norm: torch.Tensor                # fp32 [vdim]
+    norm_lp: torch.Tensor             # the same in the compute dtype
 
 
 @dataclass
@@ -328,7 +329,7 @@ def build(cfg: KinetarConfig, get: Callable[[str], torch.Tensor], device="cpu", 
             rows = {n: take(p + n) for n in "qkvb"}
             rows["a1"], rows["g1"] = (F.pad(t, (0, 0, 0, w.shape[1] - t.shape[0])) for t, w in ((a1, w_a), (g1, w_g)))
             raw["rank"] = torch.tensor([a1.shape[0], g1.shape[0]])
-            mixer = (DeltaMixer({n: f32(f"{p}{n}.conv") for n in "qkv"}, w_a, w_g, f32(p + "A_log"), f32(p + "dt_bias"), f32(p + "norm")),)
+            mixer = (DeltaMixer({n: f32(f"{p}{n}.conv") for n in "qkv"}, w_a, w_g, f32(p + "A_log"), f32(p + "dt_bias"), f32(p + "norm"), take(p + "norm")),)
             act, outs = [("mix", m.value_dim)], {"mix": take(p + "o")}
         else:
             a, s = m.left, m.right
@@ -497,7 +498,7 @@ def channel_delta_mixer(s: ChannelDeltaSpec, l: Layer, h: torch.Tensor, act: tor
     args = (bufs["q"], bufs["k"], bufs["v"], a, y[..., l.cols["b"]])
     rec, out = state.lin[3].rec, act[..., l.act["mix"]]
     if t.step:
-        dr.channel_delta_decode(*args, z, m.dt_bias, m.a_log, m.norm, eps, rec, out)
+        dr.channel_delta_decode(*args, z, m.dt_bias, m.a_log, m.norm, m.norm_lp, eps, rec, out)
     else:
         dr.gated_norm(dr.channel_delta_prefill(*args, m.dt_bias, m.a_log, rec, t.lens), z, m.norm, eps, "sigmoid", out)
 

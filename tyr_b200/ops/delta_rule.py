@@ -36,7 +36,15 @@ def _sigs(lib_):
         fn.restype = ctypes.c_int
     fn = getattr(lib_, "tyr_gdr_chunk_scan", None)
     if fn is not None:
-        fn.argtypes = [P] * 9 + [I, I, I, I, I, I, I, I, P]
+        fn.argtypes = [P] * 9 + [I, I, I, I, I, I, I, I, I, P]
+        fn.restype = ctypes.c_int
+    fn = getattr(lib_, "tyr_gdr_chunk_prepare_channel", None)
+    if fn is not None:
+        fn.argtypes = [P] * 14 + [ctypes.POINTER(L), I, I, I, I, I, I, P]
+        fn.restype = ctypes.c_int
+    fn = getattr(lib_, "tyr_gdr_decode_tile_channel", None)
+    if fn is not None:
+        fn.argtypes = [P] * 11 + [ctypes.POINTER(L), I, I, I, I, ctypes.c_float, P, P]
         fn.restype = ctypes.c_int
     fn = getattr(lib_, "tyr_gdr_chunk_prepare", None)
     if fn is not None:
@@ -124,7 +132,7 @@ def chunk_gated_delta_rule_fused(q, k, v, g, beta, state: Optional[torch.Tensor]
     st_in = None if state is None else state.float().contiguous()
     st_out = f32(B, Hv, dk, dv) if state_out is None else state_out
     out = torch.empty((B, S, Hv, dv), dtype=torch.float32 if exact else torch.bfloat16, device=dev)   # the layer's layout, from the scan kernel
-    check(lib().tyr_gdr_chunk_scan(ptr(u), ptr(w), ptr(qg), ptr(kd), ptr(intra), ptr(glast), ptr(st_in), ptr(st_out), ptr(out), BH, n, dk, dv, 64, S, Hv, 1 if exact else 0, st),
+    check(lib().tyr_gdr_chunk_scan(ptr(u), ptr(w), ptr(qg), ptr(kd), ptr(intra), ptr(glast), ptr(st_in), ptr(st_out), ptr(out), BH, n, dk, dv, 64, S, Hv, 1 if exact else 0, 0, st),
           "gdr_chunk_scan")
     return out, st_out
 
@@ -413,12 +421,46 @@ def recurrent_channel_delta(q, k, v, a, b, dt_bias, a_log, state: torch.Tensor, 
     return out
 
 
+def chunk_channel_delta_fused(q, k, v, a, b, dt_bias, a_log, state: torch.Tensor, lens: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """The two chunk kernels with a decay per key channel, the exact form of the scan: fp32 read-out [B, S, Hv, dv] of fresh prompts;
+    ``state`` receives the state after each row's last token.  Operands of :func:`recurrent_channel_delta`, shapes of
+    :func:`chunk_kernels_supported`."""
+    import ctypes
+    B, S, Hk, dk = q.shape
+    Hv, dv = v.shape[2], v.shape[3]
+    n, BH, dev = (S + 63) // 64, B * Hv, q.device
+    f32 = lambda *shape: torch.empty(shape, dtype=torch.float32, device=dev)
+    u, w, qg, kd, intra, glast = f32(BH, n, 64, -(-dv // 64) * 64), f32(BH, n, 64, 128), f32(BH, n, 64, 128), f32(BH, n, 64, 128), f32(BH, n, 64, 64), f32(BH, n, 128)
+    assert a.dtype == b.dtype == q.dtype and dt_bias.dtype == a_log.dtype == torch.float32 and state.dtype == torch.float32 and state.is_contiguous()
+    strides = (ctypes.c_longlong * 11)(*[t.stride(i) for t in (q, k, v) for i in range(3)], row_stride(a), row_stride(b))
+    st = cur_stream(dev)
+    check(lib().tyr_gdr_chunk_prepare_channel(ptr(q), ptr(k), ptr(v), ptr(a), ptr(b), ptr(dt_bias), ptr(a_log), ptr(u), ptr(w), ptr(qg), ptr(kd), ptr(intra),
+                                              ptr(glast), ptr(lens), strides, B, S, Hk, Hv, dk, dv, st), "gdr_chunk_prepare_channel")
+    out = f32(B, S, Hv, dv)
+    check(lib().tyr_gdr_chunk_scan(ptr(u), ptr(w), ptr(qg), ptr(kd), ptr(intra), ptr(glast), None, ptr(state), ptr(out), BH, n, dk, dv, 64, S, Hv, 1, 1, st),
+          "gdr_chunk_scan")
+    return out
+
+
 def channel_delta_prefill(q, k, v, a, b, dt_bias, a_log, state: torch.Tensor, lens: Optional[torch.Tensor] = None) -> torch.Tensor:
     """:func:`delta_prefill` with a decay per key channel (operands of :func:`recurrent_channel_delta`)."""
+    if q.is_cuda and q.shape[1] > 1 and chunk_kernels_supported(q, k, v) and hasattr(lib(), "tyr_gdr_chunk_prepare_channel"):
+        return chunk_channel_delta_fused(q, k, v, a, b, dt_bias, a_log, state, lens)
     state.zero_()
     return recurrent_channel_delta(q, k, v, a, b, dt_bias, a_log, state, lens)
 
 
-def channel_delta_decode(q, k, v, a, b, z, dt_bias, a_log, norm_w: torch.Tensor, eps: float, state: torch.Tensor, out: torch.Tensor) -> None:
-    """One token per row: recurrence on ``state`` (in place), norm of the read-out and sigmoid gate ``z`` [B, 1, Hv * dv] -> ``out``."""
+def channel_delta_decode(q, k, v, a, b, z, dt_bias, a_log, norm_w: torch.Tensor, norm_lp: torch.Tensor, eps: float, state: torch.Tensor, out: torch.Tensor) -> None:
+    """One token per row: recurrence on ``state`` (in place), norm of the read-out and sigmoid gate ``z`` [B, 1, Hv * dv] -> ``out`` (rows
+    may be strided).  norm_w: fp32 [dv], norm_lp: the same in the activations' type."""
+    import ctypes
+    B, _, Hk, dk = q.shape
+    Hv, dv = v.shape[2], v.shape[3]
+    if (q.is_cuda and q.dtype == torch.bfloat16 and dk in (64, 128) and q.stride(0) == k.stride(0) and q.stride(2) == k.stride(2) == dk
+            and v.stride(2) == dv and _tile_ok(dv, v, z, B * Hv) and out.stride(0) % 4 == 0 and out.data_ptr() % 8 == 0
+            and hasattr(lib(), "tyr_gdr_decode_tile_channel")):
+        strides = (ctypes.c_longlong * 6)(q.stride(0), v.stride(0), a.stride(0), b.stride(0), z.stride(0), out.stride(0))
+        check(lib().tyr_gdr_decode_tile_channel(ptr(q), ptr(k), ptr(v), ptr(a), ptr(b), ptr(dt_bias), ptr(a_log), ptr(state), ptr(out), ptr(z), ptr(norm_lp),
+                                                strides, B, Hk, Hv, dk, eps, ptr(err_word(q.device)), cur_stream(q.device)), "gdr_decode_tile_channel")
+        return
     gated_norm(recurrent_channel_delta(q, k, v, a, b, dt_bias, a_log, state), z, norm_w, eps, "sigmoid", out)

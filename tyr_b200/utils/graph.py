@@ -3,9 +3,13 @@
 The step function must be free of host reads and host-dependent shapes: positions live in device tensors, stores are
 updated in place.  State that a step advances non-idempotently (position counters, recurrent states) is listed by the
 caller; it is saved before the warm-up runs and the capture, and restored after each of them, so capturing costs no step and
-every warm-up run writes the store slots of the step itself (a second position would overwrite the oldest key of a full ring)."""
+every warm-up run writes the store slots of the step itself (a second position would overwrite the oldest key of a full ring).
+
+Python's cycle collector is off during the capture: a finished session and its graph refer to each other, and destroying an old graph
+while a stream records invalidates the capture."""
 from __future__ import annotations
 
+import gc
 from typing import Callable, Optional, Sequence
 
 import torch
@@ -29,8 +33,14 @@ class GraphedStep:
         from ..ops import _common as opc
         self.graph = torch.cuda.CUDAGraph()
         before = opc.LAUNCH_COUNT[0]
-        with torch.no_grad(), torch.cuda.graph(self.graph):
-            self.static_out = fn(*self.static_in)
+        collecting = gc.isenabled()
+        gc.disable()
+        try:
+            with torch.no_grad(), torch.cuda.graph(self.graph):
+                self.static_out = fn(*self.static_in)
+        finally:
+            if collecting:
+                gc.enable()
         # launches of this library's kernels recorded into the graph: every replay runs them again
         self.kernel_launches_per_replay = opc.LAUNCH_COUNT[0] - before
         for t, s in zip(advancing_state, saved):
