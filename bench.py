@@ -46,8 +46,9 @@ def parse_args():
     ap.add_argument("--device-batch", type=int, default=32)
     ap.add_argument("--seq-len", type=int, default=2048)
     ap.add_argument("--vocab", type=int, default=65536)
-    ap.add_argument("--workload", default="nanochat", choices=["nanochat", "zatorax"],
-                    help="zatorax: prefill / decode throughput beside Qwen3.5 MoE at equal size on one GPU (benchmarks/zatorax_bench.py)")
+    ap.add_argument("--workload", default="nanochat", choices=["nanochat", "zatorax", "kinetar"],
+                    help="zatorax / kinetar: prefill / decode throughput beside Qwen3.5 MoE / Qwen3.5 at equal size on one GPU "
+                         "(benchmarks/zatorax_bench.py, benchmarks/kinetar_bench.py)")
     ap.add_argument("--no-e2e", action="store_true")
     ap.add_argument("--no-laguna", action="store_true", help="skip the Laguna MoE decode half of the metric")
     ap.add_argument("--laguna-steps", type=int, default=48)
@@ -239,11 +240,12 @@ def main():
     if args.impl == "reference":
         return reference_arm(args)
 
-    if args.workload == "zatorax":
-        from benchmarks import zatorax_bench
+    if args.workload != "nanochat":
+        import importlib
+        bench = importlib.import_module(f"benchmarks.{args.workload}_bench")
         sampler = ClockSampler(0)
         sampler.start()
-        out = zatorax_bench.run(args.warmup, args.steps)
+        out = bench.run(args.warmup, args.steps)
         out["clocks"] = sampler.stop()
         print(json.dumps(out))
         return 0
