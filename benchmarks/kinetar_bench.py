@@ -189,7 +189,7 @@ def kernels(only: str = "", warmup: int = 3, steps: int = 20, device="cuda") -> 
     for B, C in ((32, 4096), (64, 8192), (1, 4096)):
         x, dt, y, bc, o = mk(B, 1, C), mk(B, 1, C), mk(B, 1, 2 * C), mk(B, 1, 2 * STATES + 256), mk(B, 1, 2 * C)
         A, D, bias, state = -torch.rand(C, STATES, device=device) * 4 - 0.05, f32(C), f32(C) - 3.0, torch.zeros(B, C, STATES, device=device)
-        H = C // 128
+        H = max(1, C * STATES // 16384)                   # as many bytes of state
         rec, q, k, v = torch.zeros(B, H, 128, 128, device=device), mk(B, 1, H, 128), mk(B, 1, H, 128), mk(B, 1, H, 128)
         g, beta = -torch.rand(B, 1, H, device=device), torch.rand(B, 1, H, device=device)
         case(f"scan step batch {B}, {C} channels", lambda: ss.scan_step(x, dt, y[..., :C], bc[..., 256:256 + STATES], bc[..., 256 + STATES:], A, D, bias, state, o[..., :C]),
@@ -210,7 +210,8 @@ def kernels(only: str = "", warmup: int = 3, steps: int = 20, device="cuda") -> 
              lambda: rms_norm_weighted(x, gd, 1e-6, residual=r16, return_residual=True), gb(T * D * 8))
     for B, S, D in ((4, 2048, 2048), (32, 1, 2048)):
         ids, table, turns = torch.randint(0, VOCAB, (B, S), device=device), mk(VOCAB, D), position_turns(D, device=device)
-        case(f"embedding {B}x{S}, width {D}", lambda: embed_positions(ids, table, turns, 0.5), gb(B * S * D * 6),
+        pos = torch.full((B,), 1000, dtype=torch.int32, device=device) if S == 1 else None
+        case(f"embedding {B}x{S}, width {D}", lambda: embed_positions(ids, table, turns, 0.5, pos), gb(B * S * D * 6),
              lambda: torch.nn.functional.embedding(ids, table), gb(B * S * D * 4))
     return out
 

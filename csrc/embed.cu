@@ -71,29 +71,61 @@ embed_grad_sorted_kernel(const __nv_bfloat16* __restrict__ dy, const long long* 
 // Input rows of a decoder with sinusoidal positions: x[r, d] = table[ids[r], d] * scale + sin / cos(p * freq[d / 2]), fp32, channel 2i the
 // sine and 2i + 1 the cosine.  `turns` holds the frequencies over 2 pi in double, so that the angle is reduced to a fraction of a turn
 // before it is rounded and far positions keep their accuracy.  p = pos[r] (a decode step), else r % S.
+// A thread owns EP_PAIRS channel pairs of one position and walks the rows of the batch that share it (all of a prompt's; one of a step's).
+constexpr int EP_PAIRS = 4;
+__device__ __forceinline__ void ep_load(const __nv_bfloat16* p, float (&f)[8]) {
+  const uint4 u = *reinterpret_cast<const uint4*>(p);
+  const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    const float2 t = unpack_bf16x2(w[e]);
+    f[2 * e] = t.x; f[2 * e + 1] = t.y;
+  }
+}
+__device__ __forceinline__ void ep_load(const float* p, float (&f)[8]) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+
 template <typename T>
 __global__ void __launch_bounds__(256) embed_positions_kernel(const long long* __restrict__ ids, const T* __restrict__ table, const double* __restrict__ turns,
-                                                              const int* __restrict__ pos, float* __restrict__ x, long long rows, int S, int D,
-                                                              int vocab, float scale, int* err) {
+                                                              const int* __restrict__ pos, float* __restrict__ x, int B, int S, int D,
+                                                              int vocab, float scale, int vec, int* err) {
   pdl_entry();
-  const int half = (D + 1) / 2;
-  const long long total = rows * half;
-  for (long long i = blockIdx.x * 256LL + threadIdx.x; i < total; i += gridDim.x * 256LL) {
-    const long long r = i / half;
-    const int k = static_cast<int>(i % half);
-    const long long id = ids[r];
-    if (id < 0 || id >= vocab) {
-      if (k == 0) report_error(err, ERR_BOUNDS, static_cast<int>(id));
-      continue;
+  const int half = (D + 1) / 2, parts = (half + EP_PAIRS - 1) / EP_PAIRS;
+  const long long units = static_cast<long long>(pos ? B : S) * parts;
+  for (long long i = blockIdx.x * 256LL + threadIdx.x; i < units; i += gridDim.x * 256LL) {
+    const int u = static_cast<int>(i / parts), k0 = static_cast<int>(i % parts) * EP_PAIRS;
+    const int p = pos ? pos[u] : u;
+    float add[2 * EP_PAIRS];
+#pragma unroll
+    for (int j = 0; j < EP_PAIRS; ++j) {
+      const double t = k0 + j < half ? p * turns[k0 + j] : 0.0;
+      sincospif(2.f * static_cast<float>(t - rint(t)), &add[2 * j], &add[2 * j + 1]);
     }
-    const int p = pos ? pos[r] : static_cast<int>(r % S);
-    const double t = p * turns[k];
-    float sn, cs;
-    sincospif(2.f * static_cast<float>(t - rint(t)), &sn, &cs);
-    const T* e = table + id * D + 2 * k;
-    float* o = x + r * D + 2 * k;
-    o[0] = static_cast<float>(e[0]) * scale + sn;
-    if (2 * k + 1 < D) o[1] = static_cast<float>(e[1]) * scale + cs;
+    const long long stride = pos ? 1 : S;
+    for (int b = 0; b < (pos ? 1 : B); ++b) {
+      const long long r = u + b * stride;
+      const long long id = ids[r];
+      if (id < 0 || id >= vocab) {
+        if (k0 == 0) report_error(err, ERR_BOUNDS, static_cast<int>(id));
+        continue;
+      }
+      const T* e = table + id * D + 2 * k0;
+      float* o = x + r * D + 2 * k0;
+      if (vec) {
+        float f[8];
+        ep_load(e, f);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) f[j] = f[j] * scale + add[j];
+        reinterpret_cast<float4*>(o)[0] = make_float4(f[0], f[1], f[2], f[3]);
+        reinterpret_cast<float4*>(o)[1] = make_float4(f[4], f[5], f[6], f[7]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < 2 * EP_PAIRS; ++j)
+          if (2 * k0 + j < D) o[j] = static_cast<float>(e[j]) * scale + add[j];
+      }
+    }
   }
 }
 
@@ -111,19 +143,20 @@ extern "C" TYR_EXPORT int tyr_embed_grad_sorted(const void* dy, const long long*
   return static_cast<int>(cudaGetLastError());
 }
 
-// ids int64 [rows]; table [vocab, D] (dtype 0 = bf16, 1 = fp32); turns double [(D + 1) / 2]; pos int32 [rows] or null; x fp32 [rows, D].
+// ids int64 [B, S]; table [vocab, D] (dtype 0 = bf16, 1 = fp32); turns double [(D + 1) / 2]; pos int32 [B] (S == 1) or null; x fp32 [B, S, D].
 // An id outside the table is recorded in `err` and its row left alone.
-extern "C" TYR_EXPORT int tyr_embed_positions(const void* ids, const void* table, const double* turns, const int* pos, float* x, long long rows,
+extern "C" TYR_EXPORT int tyr_embed_positions(const void* ids, const void* table, const double* turns, const int* pos, float* x, int B,
                                               int S, int D, int vocab, float scale, int dtype, int* err, void* stream) {
   using namespace tyr;
-  if (rows <= 0 || S <= 0 || D <= 0 || vocab <= 0) return -1;
-  const long long want = (rows * ((D + 1) / 2) + 255) / 256;
+  if (B <= 0 || S <= 0 || D <= 0 || vocab <= 0 || (pos != nullptr && S != 1)) return -1;
+  const long long want = ((pos ? B : S) * static_cast<long long>(((D + 1) / 2 + EP_PAIRS - 1) / EP_PAIRS) + 255) / 256;
+  const int vec = (D & 7) == 0 && ((reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(x)) & 15) == 0;
   const dim3 grid(static_cast<unsigned>(want < 148LL * 32 ? want : 148LL * 32));
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   auto* id = static_cast<const long long*>(ids);
   if (dtype == 1)
-    return (int)launch_dependent(embed_positions_kernel<float>, grid, dim3(256), 0, st, id, static_cast<const float*>(table), turns, pos, x, rows, S, D,
-                                 vocab, scale, err);
+    return (int)launch_dependent(embed_positions_kernel<float>, grid, dim3(256), 0, st, id, static_cast<const float*>(table), turns, pos, x, B, S, D,
+                                 vocab, scale, vec, err);
   return (int)launch_dependent(embed_positions_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, id, static_cast<const __nv_bfloat16*>(table), turns, pos,
-                               x, rows, S, D, vocab, scale, err);
+                               x, B, S, D, vocab, scale, vec, err);
 }

@@ -137,60 +137,71 @@ __global__ void __launch_bounds__(256, 2) mix_vec_kernel(const __grid_constant__
 #pragma unroll
     for (int j = 0; j < 4; ++j) wt[e][j] = K == 0 ? (j == 3 ? 1.f : 0.f) : (j >= 4 - K ? s.w[(c + e) * K + j - (4 - K)] : 0.f);
   }
-  uint4 win[4];                                    // win[j] = x[t - 3 + j]
+  const int act = s.act, t1 = min(a.S, t0 + MC_TOK);
+  const bool temps = s.temp_every > 0.f;
+  __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(s.out) + (static_cast<long long>(b) * a.S + t0) * s.out_ld + c;
+  __nv_bfloat16* slot = s.store ? static_cast<__nv_bfloat16*>(s.store) + ((static_cast<long long>(b) * s.heads + head) * s.cap + t0) * s.store_d + d : nullptr;
+  const int keep = min(len, s.cap);                // tokens that go to the store
   auto load_row = [&](int t) {
     return t < 0 || t >= a.S ? make_uint4(0, 0, 0, 0) : *reinterpret_cast<const uint4*>(xb + t * a.x_ss);
   };
+  auto unpack = [](const uint4& u, float (&f)[8]) {
+    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
 #pragma unroll
-  for (int j = 0; j < 3; ++j) win[j] = load_row(t0 - 3 + j);
-  const int t1 = min(a.S, t0 + MC_TOK);
-  __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(s.out) + (static_cast<long long>(b) * a.S + t0) * s.out_ld + c;
-  __nv_bfloat16* slot = s.store ? static_cast<__nv_bfloat16*>(s.store) + ((static_cast<long long>(b) * s.heads + head) * s.cap + t0) * s.store_d + d : nullptr;
-#pragma unroll 2
-  for (int t = t0; t < t1; ++t) {
-    win[3] = load_row(t);
-    float acc[8];
+    for (int e = 0; e < 4; ++e) {
+      const float2 x = unpack_bf16x2(w[e]);
+      f[2 * e] = x.x; f[2 * e + 1] = x.y;
+    }
+  };
+  float win[4][8];                                 // x[t] in win[t % 4], counted from t0
 #pragma unroll
-    for (int e = 0; e < 8; ++e) acc[e] = bs[e];
+  for (int j = 0; j < 3; ++j) unpack(load_row(t0 - 3 + j), win[j + 1]);
+  uint4 next[4];
 #pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const uint32_t u[4] = {win[j].x, win[j].y, win[j].z, win[j].w};
+  for (int u = 0; u < 4; ++u) next[u] = load_row(t0 + u);
+#pragma unroll 1
+  for (int tb = t0; tb < t1; tb += 4) {
+    uint4 row[4];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const float2 f = unpack_bf16x2(u[e]);
-        acc[2 * e] += f.x * wt[2 * e][j];
-        acc[2 * e + 1] += f.y * wt[2 * e + 1][j];
+    for (int u = 0; u < 4; ++u) {
+      row[u] = next[u];
+      next[u] = load_row(tb + 4 + u < t1 ? tb + 4 + u : -1);
+    }
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      const int t = tb + u;
+      unpack(row[u], win[u]);
+      if (t < t1) {
+        float acc[8];
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          acc[e] = bs[e];
+#pragma unroll
+          for (int j = 0; j < 4; ++j) acc[e] += win[(u + 1 + j) & 3][e] * wt[e][j];
+          if (act == MC_SILU) acc[e] = __fdividef(acc[e], 1.f + __expf(-acc[e]));
+          if (act == MC_RELU2) acc[e] = fmaxf(acc[e], 0.f) * fmaxf(acc[e], 0.f);
+        }
+        if (temps) {
+          const float f = mc_temp(s, t);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) acc[e] *= f;
+        }
+        const uint4 r = make_uint4(pack_bf16x2(acc[0], acc[1]), pack_bf16x2(acc[2], acc[3]), pack_bf16x2(acc[4], acc[5]), pack_bf16x2(acc[6], acc[7]));
+        *reinterpret_cast<uint4*>(dst + u * s.out_ld) = r;
+        if (slot && t < keep) *reinterpret_cast<uint4*>(slot + u * s.store_d) = r;
       }
     }
-    const float temp = mc_temp(s, t);
+    dst += 4 * s.out_ld;
+    if (slot) slot += 4 * s.store_d;
+  }
+  if (K > 0 && s.window && len > t0 && len <= t0 + MC_TOK) {       // the row's last token lies here: its last K inputs
+    __nv_bfloat16* w = static_cast<__nv_bfloat16*>(s.window) + (static_cast<long long>(b) * C + c) * K;
+    for (int j = 0; j < K; ++j) {
+      float f[8];
+      unpack(load_row(len - K + j), f);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) {
-      if (s.act == MC_SILU) acc[e] = __fdividef(acc[e], 1.f + __expf(-acc[e]));
-      else acc[e] = mc_act(acc[e], s.act);
-      acc[e] *= temp;
+      for (int e = 0; e < 8; ++e) w[e * K + j] = __float2bfloat16(f[e]);
     }
-    const uint4 r = make_uint4(pack_bf16x2(acc[0], acc[1]), pack_bf16x2(acc[2], acc[3]), pack_bf16x2(acc[4], acc[5]), pack_bf16x2(acc[6], acc[7]));
-    *reinterpret_cast<uint4*>(dst) = r;
-    dst += s.out_ld;
-    if (slot) {
-      if (t < len && t < s.cap) *reinterpret_cast<uint4*>(slot) = r;
-      slot += s.store_d;
-    }
-    if (t == len - 1 && K > 0 && s.window) {
-      __nv_bfloat16* w = static_cast<__nv_bfloat16*>(s.window) + (static_cast<long long>(b) * C + c) * K;
-#pragma unroll
-      for (int j = 0; j < 4; ++j)
-        if (j >= 4 - K) {
-          const uint32_t u[4] = {win[j].x, win[j].y, win[j].z, win[j].w};
-#pragma unroll
-          for (int e = 0; e < 8; ++e) {
-            const float2 f = unpack_bf16x2(u[e >> 1]);
-            w[e * K + j - (4 - K)] = __float2bfloat16(e & 1 ? f.y : f.x);
-          }
-        }
-    }
-#pragma unroll
-    for (int j = 0; j < 3; ++j) win[j] = win[j + 1];
   }
 }
 

@@ -7,8 +7,7 @@
 // lanes share a channel, so the recurrence itself needs no communication; the sums over n are finished for LPC tokens at a time by
 // a transposing butterfly (LPC - 1 shuffles for LPC tokens).
 //
-//   * prompt: a CTA of 128 threads walks the tokens of 128 / LPC channels in tiles of 32; the inputs of the next tile are loaded into
-//     registers while this one runs, softplus and delta x are computed once per (token, channel) and kept in shared memory.
+//   * prompt: a CTA walks the tokens of 128 / LPC channels in tiles of 32, four warps on the recurrence and four on everything around it.
 //   * step: one token per row; bound by one read and one write of the state.
 //
 // EXACT (the fp32 mode): library exponentials and, close to 1, 1 + expm1: a one-ulp bias of exp, applied at every token, would add
@@ -21,8 +20,17 @@ __device__ __forceinline__ float ss_load(const float* p) { return *p; }
 __device__ __forceinline__ float ss_load(const __nv_bfloat16* p) { return __bfloat162float(*p); }
 __device__ __forceinline__ void ss_store(float* p, float v) { *p = v; }
 __device__ __forceinline__ void ss_store(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
-__device__ __forceinline__ float ss_softplus(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
-__device__ __forceinline__ float ss_silu(float v) { return v / (1.f + expf(-v)); }
+template <bool EXACT>
+__device__ __forceinline__ float ss_softplus(float v) {
+  if constexpr (EXACT) return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v)));
+  const float e = __expf(-fabsf(v));             // ln(1 + e): the logarithm, or its series where 1 + e would lose digits of e
+  return fmaxf(v, 0.f) + (e > 0.0625f ? __logf(1.f + e) : e * (1.f - e * (0.5f - e * (0.33333333f - e * 0.25f))));
+}
+template <bool EXACT>
+__device__ __forceinline__ float ss_silu(float v) {
+  if constexpr (EXACT) return v / (1.f + expf(-v));
+  return __fdividef(v, 1.f + __expf(-v));        // far below 0 the divisor is huge or infinite, and the quotient 0
+}
 
 // exp(delta a): `a` comes premultiplied by log2(e) unless EXACT
 template <bool EXACT>
@@ -50,33 +58,49 @@ struct ScanArgs {
 
 constexpr int SS_THREADS = 128;
 
-// eight consecutive elements at p (those at index >= n are zero)
-__device__ __forceinline__ void ss_load8(const __nv_bfloat16* p, int n, bool vec, float (&f)[8]) {
-  if (vec && n >= 8) {
-    const uint4 u = *reinterpret_cast<const uint4*>(p);
+// eight consecutive elements at p (those at index >= n are zero), kept raw so that the loads stay in flight until they are used
+template <typename T>
+struct Raw8;
+template <>
+struct Raw8<__nv_bfloat16> {
+  uint4 u;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p, int n, bool vec) {
+    u = make_uint4(0, 0, 0, 0);
+    if (vec) {
+      if (n >= 8) u = *reinterpret_cast<const uint4*>(p);
+    } else {
+      uint32_t w[4] = {0, 0, 0, 0};
+#pragma unroll
+      for (int e = 0; e < 8; ++e)
+        if (e < n) w[e >> 1] |= static_cast<uint32_t>(__bfloat16_as_ushort(p[e])) << (16 * (e & 1));
+      u = make_uint4(w[0], w[1], w[2], w[3]);
+    }
+  }
+  __device__ __forceinline__ void get(float (&f)[8]) const {
     const uint32_t w[4] = {u.x, u.y, u.z, u.w};
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const float2 t = unpack_bf16x2(w[e]);
       f[2 * e] = t.x; f[2 * e + 1] = t.y;
     }
-  } else {
-#pragma unroll
-    for (int e = 0; e < 8; ++e) f[e] = e < n ? __bfloat162float(p[e]) : 0.f;
   }
-}
-__device__ __forceinline__ void ss_load8(const float* p, int n, bool vec, float (&f)[8]) {
-  if (vec && n >= 8) {
-    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
-    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
-  } else {
+};
+template <>
+struct Raw8<float> {
+  float v[8];
+  __device__ __forceinline__ void load(const float* p, int n, bool vec) {
 #pragma unroll
-    for (int e = 0; e < 8; ++e) f[e] = e < n ? p[e] : 0.f;
+    for (int e = 0; e < 8; ++e) v[e] = e < n ? p[e] : 0.f;
   }
-}
+  __device__ __forceinline__ void get(float (&f)[8]) const {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) f[e] = v[e];
+  }
+};
 __device__ __forceinline__ void ss_store8(__nv_bfloat16* p, int n, bool vec, const float (&f)[8]) {
-  if (vec && n >= 8) {
-    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7]));
+  if (vec) {
+    if (n >= 8)
+      *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7]));
   } else {
 #pragma unroll
     for (int e = 0; e < 8; ++e)
@@ -84,38 +108,142 @@ __device__ __forceinline__ void ss_store8(__nv_bfloat16* p, int n, bool vec, con
   }
 }
 __device__ __forceinline__ void ss_store8(float* p, int n, bool vec, const float (&f)[8]) {
-  if (vec && n >= 8) {
-    reinterpret_cast<float4*>(p)[0] = make_float4(f[0], f[1], f[2], f[3]);
-    reinterpret_cast<float4*>(p)[1] = make_float4(f[4], f[5], f[6], f[7]);
-  } else {
 #pragma unroll
-    for (int e = 0; e < 8; ++e)
-      if (e < n) p[e] = f[e];
-  }
+  for (int e = 0; e < 8; ++e)
+    if (e < n) p[e] = f[e];
 }
 
+template <int SPT, int LPC>
+struct ScanShape {
+  static constexpr int CH = SS_THREADS / LPC;            // channels of a CTA
+  static constexpr int NP = SPT * LPC;                   // states, padded
+  static constexpr int TOK = NP >= 128 ? 16 : 32;        // tokens of a tile
+  static constexpr int CL = CH + 1;                      // row length that spreads the banks
+};
+template <int SPT, int LPC>
+struct __align__(16) ScanTile {
+  using H = ScanShape<SPT, LPC>;
+  float b[H::TOK][H::NP], c[H::TOK][H::NP];
+  float2 d[H::TOK][H::CL];                               // {delta, delta x}
+  float y[H::TOK][H::CL];                                // sum_n S C
+};
+
+// 256 threads: warps 0 - 3 run the recurrence of tile i, warps 4 - 7 meanwhile prepare tile i + 1 (softplus, delta x), finish and write
+// tile i - 1 (skip, gate) and keep the loads of tile i + 2 in flight.  One barrier per tile; the tiles alternate between two buffers.
 template <typename T, int SPT, int LPC>
-__global__ void __launch_bounds__(SS_THREADS) scan_prompt_kernel(ScanArgs a, int vec) {
+__global__ void __launch_bounds__(2 * SS_THREADS, (sizeof(T) == 2 && SPT == 4 && LPC == 4) ? 4 : (SPT == 16 ? 1 : 2)) scan_prompt_kernel(ScanArgs a, int vec) {
+  using H = ScanShape<SPT, LPC>;
   constexpr bool EXACT = sizeof(T) == 4;
-  constexpr int CH = SS_THREADS / LPC;                  // channels of the CTA
-  constexpr int NP = SPT * LPC;                         // states, padded
-  constexpr int SS_TOK = NP > 128 ? 16 : 32;            // tokens of a tile
-  constexpr int CL = CH + 1;                            // row lengths that spread the banks
-  constexpr int V8 = (CH + 7) / 8;                      // vectors of 8 channels per token
-  constexpr int PER = (SS_TOK * V8 + SS_THREADS - 1) / SS_THREADS;      // vectors per thread and tile
-  constexpr int BPT = (SS_TOK * NP + SS_THREADS - 1) / SS_THREADS;      // B (and C) values per thread and tile
-  __shared__ float2 s_d[SS_TOK][CL];                    // {delta, delta x}
-  __shared__ float s_y[SS_TOK][CL];
-  __shared__ __align__(16) float s_b[SS_TOK][NP], s_c[SS_TOK][NP];
+  constexpr int CH = H::CH, NP = H::NP, TOK = H::TOK;
+  constexpr int V8 = (CH + 7) / 8;                       // vectors of 8 channels per token
+  constexpr int PER = (TOK * V8 + SS_THREADS - 1) / SS_THREADS;      // vectors per helper thread and tile
+  constexpr int BPT = (TOK * NP + SS_THREADS - 1) / SS_THREADS;      // B (and C) values per helper thread and tile
+  extern __shared__ __align__(16) uint8_t ss_smem[];
+  ScanTile<SPT, LPC>* const tile = reinterpret_cast<ScanTile<SPT, LPC>*>(ss_smem);
   pdl_entry();
-  const int b = blockIdx.y, c0 = blockIdx.x * CH, tid = threadIdx.x;
-  const int ch = tid / LPC, l = tid % LPC, c = c0 + ch;
+  const int b = blockIdx.y, c0 = blockIdx.x * CH;
   const int n = a.lens ? min(a.lens[b], a.S) : a.S;
+  const int tiles = (n + TOK - 1) / TOK;
   const long long row0 = static_cast<long long>(b) * a.S;
-  const T *xp = static_cast<const T*>(a.x) + row0 * a.x_ld + c0, *dtp = static_cast<const T*>(a.dt) + row0 * a.dt_ld + c0;
-  const T *zp = static_cast<const T*>(a.z) + row0 * a.z_ld + c0;
-  const T *bp = static_cast<const T*>(a.bm) + row0 * a.bc_ld, *cp = static_cast<const T*>(a.cm) + row0 * a.bc_ld;
-  T* op = static_cast<T*>(a.out) + row0 * a.out_ld + c0;
+  if (threadIdx.x >= SS_THREADS) {
+    // ------------------------------------------------------------------ helpers
+    const int tid = threadIdx.x - SS_THREADS;
+    const T *xp = static_cast<const T*>(a.x) + row0 * a.x_ld + c0, *dtp = static_cast<const T*>(a.dt) + row0 * a.dt_ld + c0;
+    const T *zp = static_cast<const T*>(a.z) + row0 * a.z_ld + c0;
+    const T *bp = static_cast<const T*>(a.bm) + row0 * a.bc_ld, *cp = static_cast<const T*>(a.cm) + row0 * a.bc_ld;
+    T* op = static_cast<T*>(a.out) + row0 * a.out_ld + c0;
+    const int live = min(a.C - c0, CH);
+    // vector j of this thread: token i / V8, channels 8 (i % V8) .. of the tile, i = tid + j SS_THREADS
+    auto left = [&](int j, int t0, int& t, int& k) {
+      const int i = tid + j * SS_THREADS;
+      t = i / V8; k = (i % V8) * 8;
+      return (i < TOK * V8 && t0 + t < n) ? live - k : 0;
+    };
+    Raw8<T> rx[PER], rd[PER], px[PER], pz[PER];
+    T rb[BPT], rc[BPT];
+    auto fetch = [&](int t0) {
+#pragma unroll
+      for (int j = 0; j < PER; ++j) {
+        int t, k;
+        const int m = left(j, t0, t, k);
+        rx[j].load(xp + (t0 + t) * a.x_ld + k, m, vec);
+        rd[j].load(dtp + (t0 + t) * a.dt_ld + k, m, vec);
+      }
+#pragma unroll
+      for (int j = 0; j < BPT; ++j) {
+        const int i = tid + j * SS_THREADS, t = t0 + i / NP, k = i % NP;
+        const bool ok = i < TOK * NP && t < n && k < a.N;
+        rb[j] = ok ? bp[t * a.bc_ld + k] : T(0.f);
+        rc[j] = ok ? cp[t * a.bc_ld + k] : T(0.f);
+      }
+    };
+    auto prepare = [&](int t0, ScanTile<SPT, LPC>& o) {
+#pragma unroll
+      for (int j = 0; j < PER; ++j) {
+        int t, k;
+        const int m = left(j, t0, t, k);
+        if (tid + j * SS_THREADS >= TOK * V8) continue;
+        float fx[8], fd[8];
+        rx[j].get(fx);
+        rd[j].get(fd);
+#pragma unroll
+        for (int e = 0; e < 8; ++e)
+          if (k + e < CH) {
+            const float delta = e < m ? ss_softplus<EXACT>(fd[e] + a.dt_bias[c0 + k + e]) : 0.f;      // 0: the state stays
+            o.d[t][k + e] = make_float2(delta, delta * fx[e]);
+          }
+      }
+#pragma unroll
+      for (int j = 0; j < BPT; ++j) {
+        const int i = tid + j * SS_THREADS;
+        if (i < TOK * NP) {
+          o.b[i / NP][i % NP] = ss_load(&rb[j]);
+          o.c[i / NP][i % NP] = ss_load(&rc[j]);
+        }
+      }
+    };
+    auto finish = [&](int t0, const ScanTile<SPT, LPC>& o) {
+#pragma unroll
+      for (int j = 0; j < PER; ++j) {
+        int t, k;
+        const int m = left(j, t0, t, k);
+        if (m <= 0) continue;
+        float fx[8], fz[8], r[8];
+        px[j].get(fx);
+        pz[j].get(fz);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) r[e] = e < m && k + e < CH ? a.scale * ((o.y[t][k + e] + a.d[c0 + k + e] * fx[e]) * ss_silu<EXACT>(fz[e])) : 0.f;
+        ss_store8(op + (t0 + t) * a.out_ld + k, m, vec, r);
+      }
+    };
+    if (tiles > 0) {
+      fetch(0);
+      prepare(0, tile[0]);
+      fetch(TOK);
+    }
+    __syncthreads();
+    for (int i = 0; i <= tiles; ++i) {
+      if (i > 0) finish((i - 1) * TOK, tile[(i - 1) & 1]);
+      if (i < tiles) {
+#pragma unroll
+        for (int j = 0; j < PER; ++j) {
+          int t, k;
+          const int m = left(j, i * TOK, t, k);
+          px[j].load(xp + (i * TOK + t) * a.x_ld + k, m, vec);
+          pz[j].load(zp + (i * TOK + t) * a.z_ld + k, m, vec);
+        }
+        prepare((i + 1) * TOK, tile[(i + 1) & 1]);
+        fetch((i + 2) * TOK);
+        __syncthreads();
+      }
+    }
+    // rows of a padded batch: nothing reads them, but they must hold numbers
+    for (int i = tid; i < (a.S - n) * CH; i += SS_THREADS)
+      if (c0 + i % CH < a.C) ss_store(op + (n + i / CH) * a.out_ld + i % CH, 0.f);
+    return;
+  }
+  // -------------------------------------------------------------------- recurrence
+  const int ch = threadIdx.x / LPC, l = threadIdx.x % LPC, c = c0 + ch;
   float A[SPT], S[SPT];
   float* st = a.state + (static_cast<long long>(b) * a.C + c) * a.N;
 #pragma unroll
@@ -125,76 +253,38 @@ __global__ void __launch_bounds__(SS_THREADS) scan_prompt_kernel(ScanArgs a, int
     A[i] = ok ? a.a[static_cast<long long>(c) * a.N + k] * (EXACT ? 1.f : 1.4426950408889634f) : 0.f;
     S[i] = ok && !a.fresh ? st[k] : 0.f;
   }
-  // the inputs of a tile: PER vectors of 8 channels (token i / V8, channels 8 (i % V8)) and BPT values of B and C
-  float fx[PER][8], fd[PER][8];
-  T rb[BPT], rc[BPT];
-  auto fetch = [&](int t0) {
-#pragma unroll
-    for (int j = 0; j < PER; ++j) {
-      const int i = tid + j * SS_THREADS, t = t0 + i / V8, k = (i % V8) * 8;
-      const int left = (i < SS_TOK * V8 && t < n) ? min(a.C - c0, CH) - k : 0;
-      ss_load8(xp + t * a.x_ld + k, left, vec, fx[j]);
-      ss_load8(dtp + t * a.dt_ld + k, left, vec, fd[j]);
-    }
-#pragma unroll
-    for (int j = 0; j < BPT; ++j) {
-      const int i = tid + j * SS_THREADS, t = t0 + i / NP, k = i % NP;
-      const bool ok = i < SS_TOK * NP && t < n && k < a.N;
-      rb[j] = ok ? bp[t * a.bc_ld + k] : T(0.f);
-      rc[j] = ok ? cp[t * a.bc_ld + k] : T(0.f);
-    }
-  };
-  if (n > 0) fetch(0);
-  for (int t0 = 0; t0 < n; t0 += SS_TOK) {
-    float hx[PER][8];
-#pragma unroll
-    for (int j = 0; j < PER; ++j) {
-      const int i = tid + j * SS_THREADS, t = i / V8, k = (i % V8) * 8;
-#pragma unroll
-      for (int e = 0; e < 8; ++e) hx[j][e] = fx[j][e];
-      if (i < SS_TOK * V8) {
-#pragma unroll
-        for (int e = 0; e < 8; ++e)
-          if (k + e < CH) {
-            const bool ok = t0 + t < n && c0 + k + e < a.C;
-            const float delta = ok ? ss_softplus(fd[j][e] + a.dt_bias[c0 + k + e]) : 0.f;      // 0: the state stays
-            s_d[t][k + e] = make_float2(delta, delta * fx[j][e]);
-          }
-      }
-    }
-#pragma unroll
-    for (int j = 0; j < BPT; ++j) {
-      const int i = tid + j * SS_THREADS;
-      if (i < SS_TOK * NP) {
-        s_b[i / NP][i % NP] = ss_load(&rb[j]);
-        s_c[i / NP][i % NP] = ss_load(&rc[j]);
-      }
-    }
-    __syncthreads();
-    float fz[PER][8];
-#pragma unroll
-    for (int j = 0; j < PER; ++j) {
-      const int i = tid + j * SS_THREADS, t = t0 + i / V8, k = (i % V8) * 8;
-      ss_load8(zp + t * a.z_ld + k, (i < SS_TOK * V8 && t < n) ? min(a.C - c0, CH) - k : 0, vec, fz[j]);
-    }
-    if (t0 + SS_TOK < n) fetch(t0 + SS_TOK);
-    // ---- the recurrence, G tokens at a time
-    constexpr int G = LPC < 4 ? 4 : LPC;
-#pragma unroll 1
-    for (int tg = 0; tg < SS_TOK; tg += G) {
+  __syncthreads();
+  constexpr int G = LPC < 4 ? 4 : LPC;                   // tokens whose sums are finished together
+  for (int ti = 0; ti < tiles; ++ti) {
+    ScanTile<SPT, LPC>& o = tile[ti & 1];
+#pragma unroll 2
+    for (int tg = 0; tg < TOK; tg += G) {
       float y[G];
 #pragma unroll
       for (int u = 0; u < G; ++u) {
         const int t = tg + u;
-        const float2 dd = s_d[t][ch];
+        const float2 dd = o.d[t][ch];
+        float bv[SPT], cv[SPT];
+        if constexpr (SPT % 4 == 0) {
+#pragma unroll
+          for (int i = 0; i < SPT; i += 4) {
+            const float4 b4 = *reinterpret_cast<const float4*>(&o.b[t][l * SPT + i]), c4 = *reinterpret_cast<const float4*>(&o.c[t][l * SPT + i]);
+            bv[i] = b4.x; bv[i + 1] = b4.y; bv[i + 2] = b4.z; bv[i + 3] = b4.w;
+            cv[i] = c4.x; cv[i + 1] = c4.y; cv[i + 2] = c4.z; cv[i + 3] = c4.w;
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < SPT; i += 2) {
+            const float2 b2 = *reinterpret_cast<const float2*>(&o.b[t][l * SPT + i]), c2 = *reinterpret_cast<const float2*>(&o.c[t][l * SPT + i]);
+            bv[i] = b2.x; bv[i + 1] = b2.y;
+            cv[i] = c2.x; cv[i + 1] = c2.y;
+          }
+        }
         float acc = 0.f;
 #pragma unroll
-        for (int i = 0; i < SPT; i += 2) {
-          const float2 bv = *reinterpret_cast<const float2*>(&s_b[t][l * SPT + i]), cv = *reinterpret_cast<const float2*>(&s_c[t][l * SPT + i]);
-          S[i] = ss_decay<EXACT>(dd.x, A[i]) * S[i] + dd.y * bv.x;
-          S[i + 1] = ss_decay<EXACT>(dd.x, A[i + 1]) * S[i + 1] + dd.y * bv.y;
-          acc += S[i] * cv.x;
-          acc += S[i + 1] * cv.y;
+        for (int i = 0; i < SPT; ++i) {
+          S[i] = ss_decay<EXACT>(dd.x, A[i]) * S[i] + dd.y * bv[i];
+          acc += S[i] * cv[i];
         }
         y[u] = acc;
       }
@@ -202,7 +292,7 @@ __global__ void __launch_bounds__(SS_THREADS) scan_prompt_kernel(ScanArgs a, int
 #pragma unroll
         for (int u = 0; u < G; ++u) {
           if constexpr (LPC == 2) y[u] += __shfl_xor_sync(0xffffffffu, y[u], 1);
-          if (l == 0) s_y[tg + u][ch] = y[u];
+          if (l == 0) o.y[tg + u][ch] = y[u];
         }
       } else {
         // butterfly: after the round over bit h, a lane keeps the tokens whose bit h equals its own
@@ -215,27 +305,11 @@ __global__ void __launch_bounds__(SS_THREADS) scan_prompt_kernel(ScanArgs a, int
             y[u] = keep + __shfl_xor_sync(0xffffffffu, give, h);
           }
         }
-        s_y[tg + l][ch] = y[0];
+        o.y[tg + l][ch] = y[0];
       }
     }
     __syncthreads();
-#pragma unroll
-    for (int j = 0; j < PER; ++j) {
-      const int i = tid + j * SS_THREADS, t = i / V8, k = (i % V8) * 8;
-      if (i < SS_TOK * V8 && t0 + t < n) {
-        float r[8];
-#pragma unroll
-        for (int e = 0; e < 8; ++e)
-          r[e] = (k + e < CH && c0 + k + e < a.C) ? a.scale * ((s_y[t][k + e] + a.d[c0 + k + e] * hx[j][e]) * ss_silu(fz[j][e])) : 0.f;
-        ss_store8(op + (t0 + t) * a.out_ld + k, min(a.C - c0, CH) - k, vec, r);
-      }
-    }
-    // the next tile writes s_d / s_b / s_c, which every thread has finished reading before the barrier above; s_y is written again
-    // only after the next tile's first barrier
   }
-  // rows of a padded batch: nothing reads them, but they must hold numbers
-  for (int i = tid; i < (a.S - n) * CH; i += SS_THREADS)
-    if (c0 + i % CH < a.C) ss_store(op + (n + i / CH) * a.out_ld + i % CH, 0.f);
 #pragma unroll
   for (int i = 0; i < SPT; ++i) {
     const int k = l * SPT + i;
@@ -243,6 +317,7 @@ __global__ void __launch_bounds__(SS_THREADS) scan_prompt_kernel(ScanArgs a, int
   }
 }
 
+// vec: elements of a state vector access (4, 2 or 1), which divide SPT and N
 template <typename T, int SPT, int LPC>
 __global__ void __launch_bounds__(SS_THREADS) scan_step_kernel(ScanArgs a, int vec) {
   constexpr bool EXACT = sizeof(T) == 4;
@@ -251,13 +326,19 @@ __global__ void __launch_bounds__(SS_THREADS) scan_step_kernel(ScanArgs a, int v
   const bool live = c < a.C;
   float* st = a.state + (static_cast<long long>(b) * a.C + (live ? c : 0)) * a.N + l * SPT;
   const float* ap = a.a + static_cast<long long>(live ? c : 0) * a.N + l * SPT;
+  if (live && l * SPT < a.N) asm volatile("prefetch.global.L2 [%0];" ::"l"(st));      // written a whole step earlier
   float A[SPT], S[SPT];
-  // constants, and the state, which was last written a whole step earlier
 #pragma unroll
   for (int i = 0; i < SPT; ++i) A[i] = live && l * SPT + i < a.N ? ap[i] * (EXACT ? 1.f : 1.4426950408889634f) : 0.f;
   const float dskip = live ? a.d[c] : 0.f, bias = live ? a.dt_bias[c] : 0.f;
   pdl_wait();
-  if (vec) {
+  if (SPT % 4 == 0 && vec == 4) {
+#pragma unroll
+    for (int i = 0; i + 3 < SPT; i += 4) {
+      const float4 v = live && l * SPT + i < a.N ? *reinterpret_cast<const float4*>(st + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      S[i] = v.x; S[i + 1] = v.y; S[i + 2] = v.z; S[i + 3] = v.w;
+    }
+  } else if (vec >= 2) {
 #pragma unroll
     for (int i = 0; i < SPT; i += 2) {
       const float2 v = live && l * SPT + i < a.N ? *reinterpret_cast<const float2*>(st + i) : make_float2(0.f, 0.f);
@@ -270,7 +351,7 @@ __global__ void __launch_bounds__(SS_THREADS) scan_step_kernel(ScanArgs a, int v
   const T *bp = static_cast<const T*>(a.bm) + b * a.bc_ld + l * SPT, *cp = static_cast<const T*>(a.cm) + b * a.bc_ld + l * SPT;
   const float x = live ? ss_load(static_cast<const T*>(a.x) + b * a.x_ld + c) : 0.f;
   const float z = live ? ss_load(static_cast<const T*>(a.z) + b * a.z_ld + c) : 0.f;
-  const float delta = live ? ss_softplus(ss_load(static_cast<const T*>(a.dt) + b * a.dt_ld + c) + bias) : 0.f;
+  const float delta = live ? ss_softplus<EXACT>(ss_load(static_cast<const T*>(a.dt) + b * a.dt_ld + c) + bias) : 0.f;
   float acc = 0.f;
 #pragma unroll
   for (int i = 0; i < SPT; ++i) {
@@ -281,8 +362,12 @@ __global__ void __launch_bounds__(SS_THREADS) scan_step_kernel(ScanArgs a, int v
 #pragma unroll
   for (int h = LPC / 2; h >= 1; h >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, h);
   if (!live) return;
-  if (l == 0) ss_store(static_cast<T*>(a.out) + b * a.out_ld + c, a.scale * ((acc + dskip * x) * ss_silu(z)));
-  if (vec) {
+  if (l == 0) ss_store(static_cast<T*>(a.out) + b * a.out_ld + c, a.scale * ((acc + dskip * x) * ss_silu<EXACT>(z)));
+  if (SPT % 4 == 0 && vec == 4) {
+#pragma unroll
+    for (int i = 0; i + 3 < SPT; i += 4)
+      if (l * SPT + i < a.N) *reinterpret_cast<float4*>(st + i) = make_float4(S[i], S[i + 1], S[i + 2], S[i + 3]);
+  } else if (vec >= 2) {
 #pragma unroll
     for (int i = 0; i < SPT; i += 2)
       if (l * SPT + i < a.N) *reinterpret_cast<float2*>(st + i) = make_float2(S[i], S[i + 1]);
@@ -291,6 +376,24 @@ __global__ void __launch_bounds__(SS_THREADS) scan_step_kernel(ScanArgs a, int v
     for (int i = 0; i < SPT; ++i)
       if (l * SPT + i < a.N) st[i] = S[i];
   }
+}
+
+template <typename T, int SPT, int LPC>
+static int scan_launch(const ScanArgs& a, int step, int vec, cudaStream_t st) {
+  const dim3 grid((a.C + SS_THREADS / LPC - 1) / (SS_THREADS / LPC), a.B);
+  if (step) return (int)launch_dependent(scan_step_kernel<T, SPT, LPC>, grid, dim3(SS_THREADS), 0, st, a, vec);
+  constexpr size_t smem = 2 * sizeof(ScanTile<SPT, LPC>);
+  if (smem > 48 * 1024) {
+    static bool configured[64] = {};            // the attribute is per device
+    int dev = 0;
+    if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) dev = 0;
+    if (!configured[dev]) {
+      const cudaError_t e = cudaFuncSetAttribute(scan_prompt_kernel<T, SPT, LPC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      if (e != cudaSuccess) return 1000 + (int)e;
+      configured[dev] = true;
+    }
+  }
+  return (int)launch_dependent(scan_prompt_kernel<T, SPT, LPC>, grid, dim3(2 * SS_THREADS), smem, st, a, vec);
 }
 
 }  // namespace tyr
@@ -310,18 +413,10 @@ extern "C" TYR_EXPORT int tyr_selective_scan(const void* x, const void* dt, cons
   a.a = A; a.d = D; a.dt_bias = dt_bias; a.state = state; a.out = out; a.lens = lens;
   a.B = B; a.S = S; a.C = C; a.N = N; a.fresh = fresh; a.scale = scale;
   const uintptr_t al = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(dt) | reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(out);
-  const int vec = step ? ((N & 1) == 0 && (reinterpret_cast<uintptr_t>(state) & 7) == 0)
+  const int vec = step ? ((reinterpret_cast<uintptr_t>(state) & 15) || (N & 1) ? 1 : (N & 3) ? 2 : 4)
                        : ((al & 15) == 0 && ((ld[0] | ld[1] | ld[2] | ld[4] | C) & 7) == 0);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-#define TYR_SS(SPT_, LPC_)                                                                                                        \
-  {                                                                                                                               \
-    const dim3 grid((C + SS_THREADS / LPC_ - 1) / (SS_THREADS / LPC_), B), block(SS_THREADS);                                     \
-    if (dtype == 1)                                                                                                               \
-      return (int)(step ? launch_dependent(scan_step_kernel<float, SPT_, LPC_>, grid, block, 0, st, a, vec)                       \
-                        : launch_dependent(scan_prompt_kernel<float, SPT_, LPC_>, grid, block, 0, st, a, vec));                   \
-    return (int)(step ? launch_dependent(scan_step_kernel<__nv_bfloat16, SPT_, LPC_>, grid, block, 0, st, a, vec)                 \
-                      : launch_dependent(scan_prompt_kernel<__nv_bfloat16, SPT_, LPC_>, grid, block, 0, st, a, vec));             \
-  }
+#define TYR_SS(SPT_, LPC_) return dtype == 1 ? scan_launch<float, SPT_, LPC_>(a, step, vec, st) : scan_launch<__nv_bfloat16, SPT_, LPC_>(a, step, vec, st);
   if (N <= 8) TYR_SS(4, 2)
   if (N <= 16) TYR_SS(4, 4)
   if (N <= 24) TYR_SS(6, 4)

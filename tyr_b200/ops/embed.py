@@ -20,7 +20,7 @@ def _sigs(lib_):
         fn.restype = I
     fn = getattr(lib_, "tyr_embed_positions", None)
     if fn is not None:
-        fn.argtypes = [P, P, P, P, P, L, I, I, I, ctypes.c_float, I, P, P]
+        fn.argtypes = [P, P, P, P, P, I, I, I, I, ctypes.c_float, I, P, P]
         fn.restype = I
 
 
@@ -66,6 +66,6 @@ def embed_positions(ids: torch.Tensor, table: torch.Tensor, turns: torch.Tensor,
     assert pos is None or (S == 1 and pos.dtype == torch.int32 and pos.numel() == B)
     x = torch.empty((B, S, D), dtype=torch.float32, device=ids.device)
     kind = {torch.bfloat16: 0, torch.float32: 1}[table.dtype]
-    check(lib().tyr_embed_positions(ptr(ids.contiguous()), ptr(table), ptr(turns), ptr(pos), ptr(x), B * S, S, D, V, scale, kind, ptr(err_word(ids.device)),
+    check(lib().tyr_embed_positions(ptr(ids.contiguous()), ptr(table), ptr(turns), ptr(pos), ptr(x), B, S, D, V, scale, kind, ptr(err_word(ids.device)),
                                     cur_stream(ids.device)), "embed_positions")
     return x
