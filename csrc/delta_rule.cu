@@ -830,6 +830,12 @@ __global__ void __launch_bounds__(256, 2) gdr_chunk_prepare_kernel(GdrPrepArgs a
 // ------------------------------------------------------------------------------------------------------------------
 constexpr float GP_STEEP = -60.f;
 
+// ln(1 + e^z): the logarithm of 1 + e, or its series where 1 + e would lose digits of e = e^-|z|
+__device__ __forceinline__ float softplus_fast(float z) {
+  const float e = __expf(-fabsf(z));
+  return fmaxf(z, 0.f) + (e > 0.0625f ? __logf(1.f + e) : e * (1.f - e * (0.5f - e * (0.33333333f - e * 0.25f))));
+}
+
 struct GdrPrepChannelSmem {
   float k[GC_C * GC_LDW];            // raw, then kh
   float q[GC_C * GC_LDW];            // raw, then q exp(gl); then the matrix of the triangular solve [64][GP_LDA]
@@ -899,7 +905,7 @@ __global__ void __launch_bounds__(256, 2) gdr_chunk_prepare_channel_kernel(GdrPr
 #pragma unroll
       for (int t = 0; t < 16; ++t) {
         const float z = gl[h][t];
-        run += rate * (z == -INFINITY ? 0.f : fmaxf(z, 0.f) + log1pf(__expf(-fabsf(z))));
+        run += rate * (z == -INFINITY ? 0.f : softplus_fast(z));
         gl[h][t] = run;
       }
     }

@@ -6,7 +6,7 @@
 //   * prompt: whole prompts [B, S, columns], rows of unequal length; leaves the last `taps` inputs of every row as the window.
 //   * step:   one token per row; windows shifted in place.
 //
-// The vector form of the prompt kernel keeps the taps and a sliding window of 8 channels in registers, so that an input row is
+// The vector form of the prompt kernel keeps the taps and a sliding window of 2 channels in registers, so that an input row is
 // loaded once; the plain form takes any size, any number of taps and fp32.  Compiled without fast math.
 #include "common.cuh"
 
@@ -33,7 +33,7 @@ struct MixArgs {
   long long x_sb, x_ss;
   const int* lens;               // prompt: tokens of each row (nullable: S)
   const int* pos;                // step: position of the new token of each row
-  int B, S, n_seg, groups;       // groups: channels (or vectors of 8) of all segments' outputs
+  int B, S, n_seg, groups;       // groups: channels (or pairs) of all segments' outputs
   MixSegment seg[MC_SEGS];
 };
 
@@ -49,6 +49,14 @@ __device__ __forceinline__ float mc_act(float v, int act) {
 __device__ __forceinline__ float mc_temp(const MixSegment& s, int p) {
   return s.temp_every > 0.f ? 1.f + s.temp_coef * logf(floorf(static_cast<float>(p + 1) / s.temp_every) + 1.f) : 1.f;
 }
+// the same for 16-bit results: approximate quotient, put right against its neighbours before the floor matters
+__device__ __forceinline__ float mc_temp_fast(float coef, float every, int p) {
+  const float n = static_cast<float>(p + 1);
+  float q = floorf(__fdividef(n, every));
+  if ((q + 1.f) * every <= n) q += 1.f;
+  if (q * every > n) q -= 1.f;
+  return 1.f + coef * __logf(q + 1.f);
+}
 
 // Output channel `o` of all segments -> its segment; `o` becomes the channel inside it.
 __device__ __forceinline__ int mc_find(const MixArgs& a, int& o, int per) {
@@ -61,18 +69,19 @@ __device__ __forceinline__ int mc_find(const MixArgs& a, int& o, int per) {
   return i;
 }
 
+// One thread per (token, output channel); blockIdx.y walks the tokens of the batch.
 template <typename T, bool STEP>
 __global__ void __launch_bounds__(256) mix_plain_kernel(const __grid_constant__ MixArgs a) {
+  int o = static_cast<int>(blockIdx.x * 256 + threadIdx.x);
+  const bool live = o < a.groups;
+  const MixSegment& s = a.seg[mc_find(a, o, 1)];
+  const int head = s.d_in == s.d_out ? 0 : o / s.d_out, d = s.d_in == s.d_out ? o : o % s.d_out;     // unpadded heads: one wide head
   pdl_entry();
-  const long long total = static_cast<long long>(a.B) * a.S * a.groups;
-  for (long long i = blockIdx.x * 256LL + threadIdx.x; i < total; i += gridDim.x * 256LL) {
-    int o = static_cast<int>(i % a.groups);
-    const long long row = i / a.groups;
-    const int b = static_cast<int>(row / a.S), t = static_cast<int>(row % a.S);
-    const MixSegment& s = a.seg[mc_find(a, o, 1)];
-    const int head = o / s.d_out, d = o % s.d_out;
+  if (!live) return;
+  for (long long row = blockIdx.y; row < static_cast<long long>(a.B) * a.S; row += gridDim.y) {
+    const int b = STEP ? static_cast<int>(row) : static_cast<int>(row / a.S), t = STEP ? 0 : static_cast<int>(row % a.S);
     T* dst = static_cast<T*>(s.out) + row * s.out_ld + o;
-    if (d >= s.d_in) {                                  // padded channel of a head
+    if (d >= s.d_in && s.d_in != s.d_out) {             // padded channel of a head
       mc_store(dst, 0.f);
       continue;
     }
@@ -86,7 +95,28 @@ __global__ void __launch_bounds__(256) mix_plain_kernel(const __grid_constant__ 
       acc = s.bias ? s.bias[c] : 0.f;
       const float* w = s.w + static_cast<long long>(c) * K;
       T* win = s.window ? static_cast<T*>(s.window) + (static_cast<long long>(b) * C + c) * K : nullptr;
-      if constexpr (STEP) {
+      if constexpr (STEP && sizeof(T) == 2) {
+        if (K == 4) {                                   // the window in one access
+          uint2 v = *reinterpret_cast<const uint2*>(win);
+          v.x = __byte_perm(v.x, v.y, 0x5432);
+          v.y = __byte_perm(v.y, __bfloat16_as_ushort(*xb), 0x5432);
+          *reinterpret_cast<uint2*>(win) = v;
+          const float2 u0 = unpack_bf16x2(v.x), u1 = unpack_bf16x2(v.y);
+          acc += u0.x * w[0];
+          acc += u0.y * w[1];
+          acc += u1.x * w[2];
+          acc += u1.y * w[3];
+        } else {
+          for (int j = 0; j + 1 < K; ++j) {
+            const T v = win[j + 1];
+            win[j] = v;
+            acc += mc_load(&v) * w[j];
+          }
+          const T v = *xb;
+          win[K - 1] = v;
+          acc += mc_load(&v) * w[K - 1];
+        }
+      } else if constexpr (STEP) {
         for (int j = 0; j + 1 < K; ++j) {
           const T v = win[j + 1];
           win[j] = v;
@@ -110,97 +140,108 @@ __global__ void __launch_bounds__(256) mix_plain_kernel(const __grid_constant__ 
     acc = mc_act(acc, s.act) * mc_temp(s, STEP ? a.pos[b] : t);
     mc_store(dst, acc);
     if (!STEP && s.store && t < len && t < s.cap)
-      mc_store(static_cast<T*>(s.store) + ((static_cast<long long>(b) * s.heads + head) * s.cap + t) * s.store_d + d, acc);
+      mc_store(static_cast<T*>(s.store) + ((static_cast<long long>(b) * s.heads + c / s.d_in) * s.cap + t) * s.store_d + c % s.d_in, acc);
   }
 }
 
-// bf16, at most 4 taps, d_in a multiple of 8 and equal to d_out, 16-byte aligned rows.  A thread owns 8 channels x MC_TOK tokens.
-constexpr int MC_TOK = 32;
-__global__ void __launch_bounds__(256, 2) mix_vec_kernel(const __grid_constant__ MixArgs a) {
+// bf16, at most 4 taps, d_in even and equal to d_out, 4-byte aligned rows.  A thread owns 2 channels x MC_TOK tokens (few registers, so
+// that many warps fit an SM: the kernel lives on loads in flight); the rows of its next eight tokens are on their way while it works
+// on these.
+constexpr int MC_TOK = 64, MC_VEC = 256;
+__global__ void __launch_bounds__(MC_VEC, 4) mix_vec_kernel(const __grid_constant__ MixArgs a) {
   pdl_entry();
   const int nblk = (a.S + MC_TOK - 1) / MC_TOK;
   const long long total = static_cast<long long>(a.B) * nblk * a.groups;
-  const long long i = blockIdx.x * 256LL + threadIdx.x;
+  const long long i = blockIdx.x * static_cast<long long>(MC_VEC) + threadIdx.x;
   if (i >= total) return;
   int o = static_cast<int>(i % a.groups);
   const long long bt = i / a.groups;
   const int t0 = static_cast<int>(bt % nblk) * MC_TOK, b = static_cast<int>(bt / nblk);
-  const MixSegment& s = a.seg[mc_find(a, o, 8)];
-  const int c = o * 8, K = s.taps, C = s.heads * s.d_in;
-  const int head = c / s.d_in, d = c % s.d_in;
-  const __nv_bfloat16* xb = static_cast<const __nv_bfloat16*>(a.x) + b * a.x_sb + s.col + c;
+  const MixSegment& s = a.seg[mc_find(a, o, 2)];
+  const int c = o * 2, K = s.taps;
   const int len = a.lens ? a.lens[b] : a.S;
-  float wt[8][4], bs[8];                           // fewer than 4 taps: leading zeros
+  float wt[2][4], bs[2];                           // fewer than 4 taps: leading zeros
+  const bool quad = K == 4 && (reinterpret_cast<uintptr_t>(s.w) & 15) == 0;
 #pragma unroll
-  for (int e = 0; e < 8; ++e) {
+  for (int e = 0; e < 2; ++e) {
     bs[e] = K > 0 && s.bias ? s.bias[c + e] : 0.f;
+    if (quad) {
+      const float4 w4 = *reinterpret_cast<const float4*>(s.w + (c + e) * 4);
+      wt[e][0] = w4.x; wt[e][1] = w4.y; wt[e][2] = w4.z; wt[e][3] = w4.w;
+      continue;
+    }
 #pragma unroll
     for (int j = 0; j < 4; ++j) wt[e][j] = K == 0 ? (j == 3 ? 1.f : 0.f) : (j >= 4 - K ? s.w[(c + e) * K + j - (4 - K)] : 0.f);
   }
-  const int act = s.act, t1 = min(a.S, t0 + MC_TOK);
-  const bool temps = s.temp_every > 0.f;
-  __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(s.out) + (static_cast<long long>(b) * a.S + t0) * s.out_ld + c;
-  __nv_bfloat16* slot = s.store ? static_cast<__nv_bfloat16*>(s.store) + ((static_cast<long long>(b) * s.heads + head) * s.cap + t0) * s.store_d + d : nullptr;
-  const int keep = min(len, s.cap);                // tokens that go to the store
-  auto load_row = [&](int t) {
-    return t < 0 || t >= a.S ? make_uint4(0, 0, 0, 0) : *reinterpret_cast<const uint4*>(xb + t * a.x_ss);
-  };
-  auto unpack = [](const uint4& u, float (&f)[8]) {
-    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+  const int act = s.act;
+  const float coef = s.temp_coef, every = s.temp_every;
+  const long long x_ss = a.x_ss, out_ld = s.out_ld;
+  const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(a.x) + b * a.x_sb + s.col + c + t0 * x_ss;
+  __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(s.out) + (static_cast<long long>(b) * a.S + t0) * out_ld + c;
+  __nv_bfloat16* slot = s.store ? static_cast<__nv_bfloat16*>(s.store) + ((static_cast<long long>(b) * s.heads + c / s.d_in) * s.cap + t0) * s.store_d + c % s.d_in : nullptr;
+  const int store_d = s.store_d, keep = min(len, s.cap);      // keep: tokens that go to the store
+  auto row = [&](int u) { return *reinterpret_cast<const uint32_t*>(src + u * x_ss); };
+  float2 win[4];                                   // x[t] in win[(t - t0) % 4]
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const float2 x = unpack_bf16x2(w[e]);
-      f[2 * e] = x.x; f[2 * e + 1] = x.y;
+  for (int j = 0; j < 3; ++j) win[j + 1] = unpack_bf16x2(t0 > 0 ? row(j - 3) : 0u);      // before the start: zeros (MC_TOK >= 3)
+  auto one = [&](int t, int u, uint32_t raw) {
+    win[u] = unpack_bf16x2(raw);
+    float a0 = bs[0], a1 = bs[1];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      a0 += win[(u + 1 + j) & 3].x * wt[0][j];
+      a1 += win[(u + 1 + j) & 3].y * wt[1][j];
+    }
+    if (act == MC_SILU) {
+      a0 = __fdividef(a0, 1.f + __expf(-a0));
+      a1 = __fdividef(a1, 1.f + __expf(-a1));
+    } else if (act == MC_RELU2) {
+      a0 = fmaxf(a0, 0.f) * fmaxf(a0, 0.f);
+      a1 = fmaxf(a1, 0.f) * fmaxf(a1, 0.f);
+    }
+    if (every > 0.f) {
+      const float f = mc_temp_fast(coef, every, t);
+      a0 *= f; a1 *= f;
+    }
+    const uint32_t r = pack_bf16x2(a0, a1);
+    *reinterpret_cast<uint32_t*>(dst) = r;
+    dst += out_ld;
+    if (slot) {
+      if (t < keep) *reinterpret_cast<uint32_t*>(slot) = r;
+      slot += store_d;
     }
   };
-  float win[4][8];                                 // x[t] in win[t % 4], counted from t0
+  if (t0 + MC_TOK <= a.S) {                        // a whole block
+    uint32_t next[8];
 #pragma unroll
-  for (int j = 0; j < 3; ++j) unpack(load_row(t0 - 3 + j), win[j + 1]);
-  uint4 next[4];
-#pragma unroll
-  for (int u = 0; u < 4; ++u) next[u] = load_row(t0 + u);
+    for (int u = 0; u < 8; ++u) next[u] = row(u);
 #pragma unroll 1
-  for (int tb = t0; tb < t1; tb += 4) {
-    uint4 row[4];
+    for (int t = t0; t < t0 + MC_TOK; t += 8) {
+      src += 8 * x_ss;
+      const bool more = t + 8 < t0 + MC_TOK;
 #pragma unroll
-    for (int u = 0; u < 4; ++u) {
-      row[u] = next[u];
-      next[u] = load_row(tb + 4 + u < t1 ? tb + 4 + u : -1);
-    }
-#pragma unroll
-    for (int u = 0; u < 4; ++u) {
-      const int t = tb + u;
-      unpack(row[u], win[u]);
-      if (t < t1) {
-        float acc[8];
-#pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          acc[e] = bs[e];
-#pragma unroll
-          for (int j = 0; j < 4; ++j) acc[e] += win[(u + 1 + j) & 3][e] * wt[e][j];
-          if (act == MC_SILU) acc[e] = __fdividef(acc[e], 1.f + __expf(-acc[e]));
-          if (act == MC_RELU2) acc[e] = fmaxf(acc[e], 0.f) * fmaxf(acc[e], 0.f);
-        }
-        if (temps) {
-          const float f = mc_temp(s, t);
-#pragma unroll
-          for (int e = 0; e < 8; ++e) acc[e] *= f;
-        }
-        const uint4 r = make_uint4(pack_bf16x2(acc[0], acc[1]), pack_bf16x2(acc[2], acc[3]), pack_bf16x2(acc[4], acc[5]), pack_bf16x2(acc[6], acc[7]));
-        *reinterpret_cast<uint4*>(dst + u * s.out_ld) = r;
-        if (slot && t < keep) *reinterpret_cast<uint4*>(slot + u * s.store_d) = r;
+      for (int u = 0; u < 8; ++u) {
+        const uint32_t raw = next[u];
+        if (more) next[u] = row(u);
+        one(t + u, u & 3, raw);
       }
     }
-    dst += 4 * s.out_ld;
-    if (slot) slot += 4 * s.store_d;
+  } else {
+#pragma unroll 1
+    for (int t = t0; t < a.S; t += 4) {
+#pragma unroll
+      for (int u = 0; u < 4; ++u)
+        if (t + u < a.S) one(t + u, u, row(u));
+      src += 4 * x_ss;
+    }
   }
   if (K > 0 && s.window && len > t0 && len <= t0 + MC_TOK) {       // the row's last token lies here: its last K inputs
-    __nv_bfloat16* w = static_cast<__nv_bfloat16*>(s.window) + (static_cast<long long>(b) * C + c) * K;
+    const __nv_bfloat16* xb = static_cast<const __nv_bfloat16*>(a.x) + b * a.x_sb + s.col + c;
+    __nv_bfloat16* w = static_cast<__nv_bfloat16*>(s.window) + (static_cast<long long>(b) * s.heads * s.d_in + c) * K;
     for (int j = 0; j < K; ++j) {
-      float f[8];
-      unpack(load_row(len - K + j), f);
-#pragma unroll
-      for (int e = 0; e < 8; ++e) w[e * K + j] = __float2bfloat16(f[e]);
+      const int t = len - K + j;
+      w[j] = t < 0 ? __float2bfloat16(0.f) : xb[t * x_ss];
+      w[K + j] = t < 0 ? __float2bfloat16(0.f) : xb[t * x_ss + 1];
     }
   }
 }
@@ -214,26 +255,27 @@ using namespace tyr;
 extern "C" TYR_EXPORT int tyr_mix_conv(const MixArgs* args, int step, int dtype, void* stream) {
   MixArgs a = *args;
   if (a.B <= 0 || a.S <= 0 || a.n_seg <= 0 || a.n_seg > MC_SEGS || (step && (a.S != 1 || a.pos == nullptr))) return -1;
-  bool vec = !step && dtype == 0 && (a.x_sb & 7) == 0 && (a.x_ss & 7) == 0 && (reinterpret_cast<uintptr_t>(a.x) & 15) == 0;
+  bool vec = !step && dtype == 0 && ((a.x_sb | a.x_ss) & 1) == 0 && (reinterpret_cast<uintptr_t>(a.x) & 3) == 0;
   long long channels = 0;
   for (int i = 0; i < a.n_seg; ++i) {
     const MixSegment& s = a.seg[i];
     if (s.heads <= 0 || s.d_in <= 0 || s.d_out < s.d_in || s.taps < 0 || s.out == nullptr || (s.taps > 0 && s.w == nullptr)) return -2;
     if (step && ((s.taps > 0 && s.window == nullptr) || s.store != nullptr)) return -3;
+    if (reinterpret_cast<uintptr_t>(s.window) & 7) return -3;
     if (s.store != nullptr && (s.cap <= 0 || s.store_d < s.d_in)) return -4;
     channels += static_cast<long long>(s.heads) * s.d_out;
-    vec = vec && s.taps <= 4 && s.d_in == s.d_out && (s.d_in & 7) == 0 && (s.col & 7) == 0 && (s.out_ld & 7) == 0 && (s.store_d & 7) == 0 &&
-          ((reinterpret_cast<uintptr_t>(s.out) | reinterpret_cast<uintptr_t>(s.store)) & 15) == 0;
+    vec = vec && s.taps <= 4 && s.d_in == s.d_out && ((s.d_in | s.col | s.out_ld | s.store_d) & 1) == 0 &&
+          ((reinterpret_cast<uintptr_t>(s.out) | reinterpret_cast<uintptr_t>(s.store)) & 3) == 0;
   }
   if (channels > 0x7fffffffLL) return -1;
-  a.groups = static_cast<int>(vec ? channels / 8 : channels);
+  a.groups = static_cast<int>(vec ? channels / 2 : channels);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (vec) {
     const long long total = static_cast<long long>(a.B) * ((a.S + MC_TOK - 1) / MC_TOK) * a.groups;
-    return (int)launch_dependent(mix_vec_kernel, dim3(static_cast<unsigned>((total + 255) / 256)), dim3(256), 0, st, a);
+    return (int)launch_dependent(mix_vec_kernel, dim3(static_cast<unsigned>((total + MC_VEC - 1) / MC_VEC)), dim3(MC_VEC), 0, st, a);
   }
-  const long long want = (static_cast<long long>(a.B) * a.S * a.groups + 255) / 256;
-  const dim3 grid(static_cast<unsigned>(want < 148LL * 64 ? want : 148LL * 64));
+  const long long rows = static_cast<long long>(a.B) * a.S;
+  const dim3 grid(static_cast<unsigned>((a.groups + 255) / 256), static_cast<unsigned>(rows < 65535 ? rows : 65535));
   if (step)
     return (int)(dtype == 1 ? launch_dependent(mix_plain_kernel<float, true>, grid, dim3(256), 0, st, a)
                             : launch_dependent(mix_plain_kernel<__nv_bfloat16, true>, grid, dim3(256), 0, st, a));

@@ -4,10 +4,11 @@
 //   out = scale * y * silu(z),
 //
 // with the state and everything that enters it in fp32.  A thread keeps SPT states of one channel in registers and LPC adjacent
-// lanes share a channel, so the recurrence itself needs no communication; the sums over n are finished for LPC tokens at a time by
-// a transposing butterfly (LPC - 1 shuffles for LPC tokens).
+// lanes share a channel, so the recurrence itself needs no communication; the sums over n are finished for LPC tokens at a time by a
+// transposing butterfly.  With SPT = 8 the reads of B and C are nearly warp-wide broadcasts, and the kernel is bound by one ex2 per
+// (token, channel, state); pairs of states share packed fp32 instructions.
 //
-//   * prompt: a CTA walks the tokens of 128 / LPC channels in tiles of 32, four warps on the recurrence and four on everything around it.
+//   * prompt: a CTA walks the tokens of its channels in tiles of 32, two warps on the recurrence and four on everything around it.
 //   * step: one token per row; bound by one read and one write of the state.
 //
 // EXACT (the fp32 mode): library exponentials and, close to 1, 1 + expm1: a one-ulp bias of exp, applied at every token, would add
@@ -32,7 +33,7 @@ __device__ __forceinline__ float ss_silu(float v) {
   return __fdividef(v, 1.f + __expf(-v));        // far below 0 the divisor is huge or infinite, and the quotient 0
 }
 
-// exp(delta a): `a` comes premultiplied by log2(e) unless EXACT
+// The decay exp(delta a).  EXACT: of a; otherwise of the product delta a log2(e).
 template <bool EXACT>
 __device__ __forceinline__ float ss_decay(float delta, float a) {
   if constexpr (EXACT) {
@@ -40,9 +41,27 @@ __device__ __forceinline__ float ss_decay(float delta, float a) {
     return g > -0.5f ? 1.f + expm1f(g) : expf(g);
   } else {
     float r;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(delta * a));
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(a));
     return r;
   }
+}
+
+// packed pairs of fp32
+__device__ __forceinline__ uint64_t pack2(float x, float y) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(x), "f"(y));
+  return r;
+}
+__device__ __forceinline__ void unpack2(uint64_t v, float& x, float& y) { asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(v)); }
+__device__ __forceinline__ uint64_t mul2(uint64_t x, uint64_t y) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(x), "l"(y));
+  return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t x, uint64_t y, uint64_t z) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(x), "l"(y), "l"(z));
+  return r;
 }
 
 struct ScanArgs {
@@ -56,7 +75,9 @@ struct ScanArgs {
   float scale;
 };
 
-constexpr int SS_THREADS = 128;
+constexpr int SS_REC = 64;             // threads of a prompt CTA on the recurrence
+constexpr int SS_HELP = 128;           // ... and on the rest
+constexpr int SS_STEP = 128;           // threads of a step CTA
 
 // eight consecutive elements at p (those at index >= n are zero), kept raw so that the loads stay in flight until they are used
 template <typename T>
@@ -115,7 +136,7 @@ __device__ __forceinline__ void ss_store8(float* p, int n, bool vec, const float
 
 template <int SPT, int LPC>
 struct ScanShape {
-  static constexpr int CH = SS_THREADS / LPC;            // channels of a CTA
+  static constexpr int CH = SS_REC / LPC;                // channels of a CTA
   static constexpr int NP = SPT * LPC;                   // states, padded
   static constexpr int TOK = NP >= 128 ? 16 : 32;        // tokens of a tile
   static constexpr int CL = CH + 1;                      // row length that spreads the banks
@@ -127,93 +148,138 @@ struct __align__(16) ScanTile {
   float2 d[H::TOK][H::CL];                               // {delta, delta x}
   float y[H::TOK][H::CL];                                // sum_n S C
 };
+template <int SPT, int LPC>
+struct __align__(16) ScanSmem {
+  ScanTile<SPT, LPC> tile[2];
+  float bias[ScanShape<SPT, LPC>::CH], skip[ScanShape<SPT, LPC>::CH];
+};
 
-// 256 threads: warps 0 - 3 run the recurrence of tile i, warps 4 - 7 meanwhile prepare tile i + 1 (softplus, delta x), finish and write
-// tile i - 1 (skip, gate) and keep the loads of tile i + 2 in flight.  One barrier per tile; the tiles alternate between two buffers.
+// SS_REC threads run the recurrence of tile i; the helpers meanwhile prepare tile i + 1 (softplus, delta x), finish and write tile
+// i - 1 (skip, gate) and keep the loads of tile i + 2 in flight.  One barrier per tile; the tiles alternate between two buffers.
 template <typename T, int SPT, int LPC>
-__global__ void __launch_bounds__(2 * SS_THREADS, (sizeof(T) == 2 && SPT == 4 && LPC == 4) ? 4 : (SPT == 16 ? 1 : 2)) scan_prompt_kernel(ScanArgs a, int vec) {
+__global__ void __launch_bounds__(SS_REC + SS_HELP, (sizeof(T) == 2 && SPT <= 8) ? 4 : 2) scan_prompt_kernel(ScanArgs a, int vec) {
   using H = ScanShape<SPT, LPC>;
   constexpr bool EXACT = sizeof(T) == 4;
   constexpr int CH = H::CH, NP = H::NP, TOK = H::TOK;
   constexpr int V8 = (CH + 7) / 8;                       // vectors of 8 channels per token
-  constexpr int PER = (TOK * V8 + SS_THREADS - 1) / SS_THREADS;      // vectors per helper thread and tile
-  constexpr int BPT = (TOK * NP + SS_THREADS - 1) / SS_THREADS;      // B (and C) values per helper thread and tile
+  constexpr int PER = (TOK * V8 + SS_HELP - 1) / SS_HELP;      // vectors per helper thread and tile
+  constexpr int BPT = (TOK * NP + SS_HELP - 1) / SS_HELP;      // B (and C) values per helper thread and tile
   extern __shared__ __align__(16) uint8_t ss_smem[];
-  ScanTile<SPT, LPC>* const tile = reinterpret_cast<ScanTile<SPT, LPC>*>(ss_smem);
+  if (CH % 8 != 0) vec = 0;
+  ScanSmem<SPT, LPC>& sm = *reinterpret_cast<ScanSmem<SPT, LPC>*>(ss_smem);
+  ScanTile<SPT, LPC>* const tile = sm.tile;
   pdl_entry();
   const int b = blockIdx.y, c0 = blockIdx.x * CH;
   const int n = a.lens ? min(a.lens[b], a.S) : a.S;
   const int tiles = (n + TOK - 1) / TOK;
   const long long row0 = static_cast<long long>(b) * a.S;
-  if (threadIdx.x >= SS_THREADS) {
+  if (threadIdx.x >= SS_REC) {
     // ------------------------------------------------------------------ helpers
-    const int tid = threadIdx.x - SS_THREADS;
+    const int tid = threadIdx.x - SS_REC;
     const T *xp = static_cast<const T*>(a.x) + row0 * a.x_ld + c0, *dtp = static_cast<const T*>(a.dt) + row0 * a.dt_ld + c0;
     const T *zp = static_cast<const T*>(a.z) + row0 * a.z_ld + c0;
     const T *bp = static_cast<const T*>(a.bm) + row0 * a.bc_ld, *cp = static_cast<const T*>(a.cm) + row0 * a.bc_ld;
     T* op = static_cast<T*>(a.out) + row0 * a.out_ld + c0;
     const int live = min(a.C - c0, CH);
-    // vector j of this thread: token i / V8, channels 8 (i % V8) .. of the tile, i = tid + j SS_THREADS
-    auto left = [&](int j, int t0, int& t, int& k) {
-      const int i = tid + j * SS_THREADS;
-      t = i / V8; k = (i % V8) * 8;
-      return (i < TOK * V8 && t0 + t < n) ? live - k : 0;
+    for (int i = tid; i < CH; i += SS_HELP) {
+      sm.bias[i] = i < live ? a.dt_bias[c0 + i] : 0.f;
+      sm.skip[i] = i < live ? a.d[c0 + i] : 0.f;
+    }
+    asm volatile("bar.sync 1, %0;" ::"n"(SS_HELP) : "memory");      // the helpers alone
+    // vector j of this thread: token i / V8, channels 8 (i % V8) .. of the tile, i = tid + j SS_HELP.  FULL: the tile lies inside the
+    // sequence and the channels, and vectors are aligned.
+    const bool full_ch = vec && live == CH && CH % 8 == 0 && a.N == NP;
+    auto full = [&](int t0) { return full_ch && t0 + TOK <= n; };
+    auto left = [&](int j, int t0) {
+      const int i = tid + j * SS_HELP;
+      return (i < TOK * V8 && t0 + i / V8 < n) ? live - (i % V8) * 8 : 0;
     };
+    const int tv = tid / V8, kv = (tid % V8) * 8;                        // vector 0; the others are SS_HELP / V8 tokens further each
+    constexpr int DT = SS_HELP / V8;
+    static_assert(SS_HELP % V8 == 0, "vectors of a token belong to one round");
+    const T *x0 = xp + static_cast<long long>(tv) * a.x_ld + kv, *d0 = dtp + static_cast<long long>(tv) * a.dt_ld + kv, *z0 = zp + static_cast<long long>(tv) * a.z_ld + kv;
+    T* o0 = op + static_cast<long long>(tv) * a.out_ld + kv;
+    const T *b0 = bp + static_cast<long long>(tid / NP) * a.bc_ld + tid % NP, *cc0 = cp + static_cast<long long>(tid / NP) * a.bc_ld + tid % NP;
     Raw8<T> rx[PER], rd[PER], px[PER], pz[PER];
     T rb[BPT], rc[BPT];
     auto fetch = [&](int t0) {
+      const bool f = full(t0);
 #pragma unroll
       for (int j = 0; j < PER; ++j) {
-        int t, k;
-        const int m = left(j, t0, t, k);
-        rx[j].load(xp + (t0 + t) * a.x_ld + k, m, vec);
-        rd[j].load(dtp + (t0 + t) * a.dt_ld + k, m, vec);
+        const int m = f && TOK * V8 % SS_HELP == 0 ? 8 : left(j, t0);
+        rx[j].load(x0 + (t0 + j * DT) * a.x_ld, m, vec);
+        rd[j].load(d0 + (t0 + j * DT) * a.dt_ld, m, vec);
       }
+      if constexpr (NP <= SS_HELP && SS_HELP % NP == 0) {
 #pragma unroll
-      for (int j = 0; j < BPT; ++j) {
-        const int i = tid + j * SS_THREADS, t = t0 + i / NP, k = i % NP;
-        const bool ok = i < TOK * NP && t < n && k < a.N;
-        rb[j] = ok ? bp[t * a.bc_ld + k] : T(0.f);
-        rc[j] = ok ? cp[t * a.bc_ld + k] : T(0.f);
+        for (int j = 0; j < BPT; ++j) {
+          const int dt = j * (SS_HELP / NP);
+          const bool ok = f || (tid / NP + dt < TOK && t0 + tid / NP + dt < n && tid % NP < a.N);
+          rb[j] = ok ? b0[(t0 + dt) * a.bc_ld] : T(0.f);
+          rc[j] = ok ? cc0[(t0 + dt) * a.bc_ld] : T(0.f);
+        }
+      } else {
+#pragma unroll
+        for (int j = 0; j < BPT; ++j) {
+          const int i = tid + j * SS_HELP, t = t0 + i / NP, k = i % NP;
+          const bool ok = i < TOK * NP && t < n && k < a.N;
+          rb[j] = ok ? bp[t * a.bc_ld + k] : T(0.f);
+          rc[j] = ok ? cp[t * a.bc_ld + k] : T(0.f);
+        }
       }
     };
     auto prepare = [&](int t0, ScanTile<SPT, LPC>& o) {
+      const bool f = full(t0);
 #pragma unroll
       for (int j = 0; j < PER; ++j) {
-        int t, k;
-        const int m = left(j, t0, t, k);
-        if (tid + j * SS_THREADS >= TOK * V8) continue;
+        if (TOK * V8 % SS_HELP != 0 && tid + j * SS_HELP >= TOK * V8) continue;
         float fx[8], fd[8];
         rx[j].get(fx);
         rd[j].get(fd);
+        float2* row = &o.d[tv + j * DT][kv];
+        if (f) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e)
-          if (k + e < CH) {
-            const float delta = e < m ? ss_softplus<EXACT>(fd[e] + a.dt_bias[c0 + k + e]) : 0.f;      // 0: the state stays
-            o.d[t][k + e] = make_float2(delta, delta * fx[e]);
+          for (int e = 0; e < 8; ++e) {
+            const float delta = ss_softplus<EXACT>(fd[e] + sm.bias[kv + e]);
+            row[e] = make_float2(delta, delta * fx[e]);
           }
+        } else {
+          const int m = left(j, t0);
+#pragma unroll
+          for (int e = 0; e < 8; ++e)
+            if (kv + e < CH) {
+              const float delta = e < m ? ss_softplus<EXACT>(fd[e] + sm.bias[kv + e]) : 0.f;      // 0: the state stays
+              row[e] = make_float2(delta, delta * fx[e]);
+            }
+        }
       }
 #pragma unroll
       for (int j = 0; j < BPT; ++j) {
-        const int i = tid + j * SS_THREADS;
-        if (i < TOK * NP) {
-          o.b[i / NP][i % NP] = ss_load(&rb[j]);
-          o.c[i / NP][i % NP] = ss_load(&rc[j]);
+        const int i = tid + j * SS_HELP;
+        if (TOK * NP % SS_HELP == 0 || i < TOK * NP) {
+          (&o.b[0][0])[i] = ss_load(&rb[j]);
+          (&o.c[0][0])[i] = ss_load(&rc[j]);
         }
       }
     };
     auto finish = [&](int t0, const ScanTile<SPT, LPC>& o) {
+      const bool f = full(t0);
 #pragma unroll
       for (int j = 0; j < PER; ++j) {
-        int t, k;
-        const int m = left(j, t0, t, k);
+        const int m = left(j, t0);
         if (m <= 0) continue;
         float fx[8], fz[8], r[8];
         px[j].get(fx);
         pz[j].get(fz);
+        const float* row = &o.y[tv + j * DT][kv];
+        if (f) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) r[e] = e < m && k + e < CH ? a.scale * ((o.y[t][k + e] + a.d[c0 + k + e] * fx[e]) * ss_silu<EXACT>(fz[e])) : 0.f;
-        ss_store8(op + (t0 + t) * a.out_ld + k, m, vec, r);
+          for (int e = 0; e < 8; ++e) r[e] = (row[e] + sm.skip[kv + e] * fx[e]) * (a.scale * ss_silu<EXACT>(fz[e]));
+        } else {
+#pragma unroll
+          for (int e = 0; e < 8; ++e) r[e] = e < m && kv + e < CH ? (row[e] + sm.skip[kv + e] * fx[e]) * (a.scale * ss_silu<EXACT>(fz[e])) : 0.f;
+        }
+        ss_store8(o0 + (t0 + j * DT) * a.out_ld, m, vec, r);
       }
     };
     if (tiles > 0) {
@@ -227,10 +293,9 @@ __global__ void __launch_bounds__(2 * SS_THREADS, (sizeof(T) == 2 && SPT == 4 &&
       if (i < tiles) {
 #pragma unroll
         for (int j = 0; j < PER; ++j) {
-          int t, k;
-          const int m = left(j, i * TOK, t, k);
-          px[j].load(xp + (i * TOK + t) * a.x_ld + k, m, vec);
-          pz[j].load(zp + (i * TOK + t) * a.z_ld + k, m, vec);
+          const int m = left(j, i * TOK);
+          px[j].load(x0 + (i * TOK + j * DT) * a.x_ld, m, vec);
+          pz[j].load(z0 + (i * TOK + j * DT) * a.z_ld, m, vec);
         }
         prepare((i + 1) * TOK, tile[(i + 1) & 1]);
         fetch((i + 2) * TOK);
@@ -238,62 +303,81 @@ __global__ void __launch_bounds__(2 * SS_THREADS, (sizeof(T) == 2 && SPT == 4 &&
       }
     }
     // rows of a padded batch: nothing reads them, but they must hold numbers
-    for (int i = tid; i < (a.S - n) * CH; i += SS_THREADS)
+    for (int i = tid; i < (a.S - n) * CH; i += SS_HELP)
       if (c0 + i % CH < a.C) ss_store(op + (n + i / CH) * a.out_ld + i % CH, 0.f);
     return;
   }
   // -------------------------------------------------------------------- recurrence
   const int ch = threadIdx.x / LPC, l = threadIdx.x % LPC, c = c0 + ch;
-  float A[SPT], S[SPT];
   float* st = a.state + (static_cast<long long>(b) * a.C + c) * a.N;
+  uint64_t A[SPT / 2], S[SPT / 2];                       // pairs of states
 #pragma unroll
-  for (int i = 0; i < SPT; ++i) {
-    const int k = l * SPT + i;
-    const bool ok = c < a.C && k < a.N;
-    A[i] = ok ? a.a[static_cast<long long>(c) * a.N + k] * (EXACT ? 1.f : 1.4426950408889634f) : 0.f;
-    S[i] = ok && !a.fresh ? st[k] : 0.f;
+  for (int i = 0; i < SPT; i += 2) {
+    float av[2], sv[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int k = l * SPT + i + e;
+      const bool ok = c < a.C && k < a.N;
+      av[e] = ok ? a.a[static_cast<long long>(c) * a.N + k] * (EXACT ? 1.f : 1.4426950408889634f) : 0.f;
+      sv[e] = ok && !a.fresh ? st[k] : 0.f;
+    }
+    A[i / 2] = pack2(av[0], av[1]);
+    S[i / 2] = pack2(sv[0], sv[1]);
   }
   __syncthreads();
-  constexpr int G = LPC < 4 ? 4 : LPC;                   // tokens whose sums are finished together
+  constexpr int G = LPC < 2 ? 2 : LPC;                   // tokens whose sums are finished together
+  constexpr int U = SPT > 8 ? 1 : 2;                     // tokens whose operands are loaded together
+  uint64_t bv[U][SPT / 2], cv[U][SPT / 2];
+  float2 dd[U];                                          // {delta, delta x}
+  auto load = [&](const ScanTile<SPT, LPC>& o, int t0) {
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int t = t0 + u;
+      dd[u] = o.d[t][ch];
+#pragma unroll
+      for (int i = 0; i < SPT / 2; i += SPT % 4 == 0 ? 2 : 1) {
+        if constexpr (SPT % 4 == 0) {
+          const ulonglong2 b4 = *reinterpret_cast<const ulonglong2*>(&o.b[t][l * SPT + 2 * i]), c4 = *reinterpret_cast<const ulonglong2*>(&o.c[t][l * SPT + 2 * i]);
+          bv[u][i] = b4.x; bv[u][i + 1] = b4.y;
+          cv[u][i] = c4.x; cv[u][i + 1] = c4.y;
+        } else {
+          bv[u][i] = *reinterpret_cast<const uint64_t*>(&o.b[t][l * SPT + 2 * i]);
+          cv[u][i] = *reinterpret_cast<const uint64_t*>(&o.c[t][l * SPT + 2 * i]);
+        }
+      }
+    }
+  };
   for (int ti = 0; ti < tiles; ++ti) {
     ScanTile<SPT, LPC>& o = tile[ti & 1];
+    load(o, 0);
 #pragma unroll 2
     for (int tg = 0; tg < TOK; tg += G) {
       float y[G];
 #pragma unroll
-      for (int u = 0; u < G; ++u) {
-        const int t = tg + u;
-        const float2 dd = o.d[t][ch];
-        float bv[SPT], cv[SPT];
-        if constexpr (SPT % 4 == 0) {
+      for (int g0 = 0; g0 < G; g0 += U) {
 #pragma unroll
-          for (int i = 0; i < SPT; i += 4) {
-            const float4 b4 = *reinterpret_cast<const float4*>(&o.b[t][l * SPT + i]), c4 = *reinterpret_cast<const float4*>(&o.c[t][l * SPT + i]);
-            bv[i] = b4.x; bv[i + 1] = b4.y; bv[i + 2] = b4.z; bv[i + 3] = b4.w;
-            cv[i] = c4.x; cv[i + 1] = c4.y; cv[i + 2] = c4.z; cv[i + 3] = c4.w;
+        for (int u = 0; u < U; ++u) {
+          const uint64_t delta = pack2(dd[u].x, dd[u].x), dx = pack2(dd[u].y, dd[u].y);
+          uint64_t acc = 0;
+#pragma unroll
+          for (int i = 0; i < SPT / 2; ++i) {
+            float a0, a1;
+            unpack2(EXACT ? A[i] : mul2(delta, A[i]), a0, a1);
+            a0 = ss_decay<EXACT>(dd[u].x, a0);
+            a1 = ss_decay<EXACT>(dd[u].x, a1);
+            S[i] = fma2(pack2(a0, a1), S[i], mul2(dx, bv[u][i]));
+            acc = fma2(S[i], cv[u][i], acc);
           }
-        } else {
-#pragma unroll
-          for (int i = 0; i < SPT; i += 2) {
-            const float2 b2 = *reinterpret_cast<const float2*>(&o.b[t][l * SPT + i]), c2 = *reinterpret_cast<const float2*>(&o.c[t][l * SPT + i]);
-            bv[i] = b2.x; bv[i + 1] = b2.y;
-            cv[i] = c2.x; cv[i + 1] = c2.y;
-          }
+          float y0, y1;
+          unpack2(acc, y0, y1);
+          y[g0 + u] = y0 + y1;
         }
-        float acc = 0.f;
-#pragma unroll
-        for (int i = 0; i < SPT; ++i) {
-          S[i] = ss_decay<EXACT>(dd.x, A[i]) * S[i] + dd.y * bv[i];
-          acc += S[i] * cv[i];
-        }
-        y[u] = acc;
+        // the next operands are on their way while the sums below are finished (past the tile's end: its last tokens again, unused)
+        load(o, min(tg + g0 + U, TOK - U));
       }
-      if constexpr (LPC <= 2) {
+      if constexpr (LPC == 1) {
 #pragma unroll
-        for (int u = 0; u < G; ++u) {
-          if constexpr (LPC == 2) y[u] += __shfl_xor_sync(0xffffffffu, y[u], 1);
-          if (l == 0) o.y[tg + u][ch] = y[u];
-        }
+        for (int u = 0; u < G; ++u) o.y[tg + u][ch] = y[u];
       } else {
         // butterfly: after the round over bit h, a lane keeps the tokens whose bit h equals its own
 #pragma unroll
@@ -311,18 +395,23 @@ __global__ void __launch_bounds__(2 * SS_THREADS, (sizeof(T) == 2 && SPT == 4 &&
     __syncthreads();
   }
 #pragma unroll
-  for (int i = 0; i < SPT; ++i) {
-    const int k = l * SPT + i;
-    if (c < a.C && k < a.N) st[k] = S[i];
+  for (int i = 0; i < SPT; i += 2) {
+    float sv[2];
+    unpack2(S[i / 2], sv[0], sv[1]);
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int k = l * SPT + i + e;
+      if (c < a.C && k < a.N) st[k] = sv[e];
+    }
   }
 }
 
 // vec: elements of a state vector access (4, 2 or 1), which divide SPT and N
 template <typename T, int SPT, int LPC>
-__global__ void __launch_bounds__(SS_THREADS) scan_step_kernel(ScanArgs a, int vec) {
+__global__ void __launch_bounds__(SS_STEP) scan_step_kernel(ScanArgs a, int vec) {
   constexpr bool EXACT = sizeof(T) == 4;
   pdl_trigger();
-  const int b = blockIdx.y, l = threadIdx.x % LPC, c = blockIdx.x * (SS_THREADS / LPC) + threadIdx.x / LPC;
+  const int b = blockIdx.y, l = threadIdx.x % LPC, c = blockIdx.x * (SS_STEP / LPC) + threadIdx.x / LPC;
   const bool live = c < a.C;
   float* st = a.state + (static_cast<long long>(b) * a.C + (live ? c : 0)) * a.N + l * SPT;
   const float* ap = a.a + static_cast<long long>(live ? c : 0) * a.N + l * SPT;
@@ -356,7 +445,7 @@ __global__ void __launch_bounds__(SS_THREADS) scan_step_kernel(ScanArgs a, int v
 #pragma unroll
   for (int i = 0; i < SPT; ++i) {
     const bool ok = l * SPT + i < a.N;
-    S[i] = ss_decay<EXACT>(delta, A[i]) * S[i] + delta * x * (ok ? ss_load(bp + i) : 0.f);
+    S[i] = ss_decay<EXACT>(delta, EXACT ? A[i] : delta * A[i]) * S[i] + delta * x * (ok ? ss_load(bp + i) : 0.f);
     acc += S[i] * (ok ? ss_load(cp + i) : 0.f);
   }
 #pragma unroll
@@ -379,10 +468,16 @@ __global__ void __launch_bounds__(SS_THREADS) scan_step_kernel(ScanArgs a, int v
 }
 
 template <typename T, int SPT, int LPC>
-static int scan_launch(const ScanArgs& a, int step, int vec, cudaStream_t st) {
-  const dim3 grid((a.C + SS_THREADS / LPC - 1) / (SS_THREADS / LPC), a.B);
-  if (step) return (int)launch_dependent(scan_step_kernel<T, SPT, LPC>, grid, dim3(SS_THREADS), 0, st, a, vec);
-  constexpr size_t smem = 2 * sizeof(ScanTile<SPT, LPC>);
+static int step_launch(const ScanArgs& a, int vec, cudaStream_t st) {
+  const dim3 grid((a.C + SS_STEP / LPC - 1) / (SS_STEP / LPC), a.B);
+  return (int)launch_dependent(scan_step_kernel<T, SPT, LPC>, grid, dim3(SS_STEP), 0, st, a, vec);
+}
+
+template <typename T, int SPT, int LPC>
+static int prompt_launch(const ScanArgs& a, int vec, cudaStream_t st) {
+  constexpr int CH = ScanShape<SPT, LPC>::CH;
+  const dim3 grid((a.C + CH - 1) / CH, a.B);
+  constexpr size_t smem = sizeof(ScanSmem<SPT, LPC>);
   if (smem > 48 * 1024) {
     static bool configured[64] = {};            // the attribute is per device
     int dev = 0;
@@ -393,7 +488,7 @@ static int scan_launch(const ScanArgs& a, int step, int vec, cudaStream_t st) {
       configured[dev] = true;
     }
   }
-  return (int)launch_dependent(scan_prompt_kernel<T, SPT, LPC>, grid, dim3(2 * SS_THREADS), smem, st, a, vec);
+  return (int)launch_dependent(scan_prompt_kernel<T, SPT, LPC>, grid, dim3(SS_REC + SS_HELP), smem, st, a, vec);
 }
 
 }  // namespace tyr
@@ -416,13 +511,21 @@ extern "C" TYR_EXPORT int tyr_selective_scan(const void* x, const void* dt, cons
   const int vec = step ? ((reinterpret_cast<uintptr_t>(state) & 15) || (N & 1) ? 1 : (N & 3) ? 2 : 4)
                        : ((al & 15) == 0 && ((ld[0] | ld[1] | ld[2] | ld[4] | C) & 7) == 0);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-#define TYR_SS(SPT_, LPC_) return dtype == 1 ? scan_launch<float, SPT_, LPC_>(a, step, vec, st) : scan_launch<__nv_bfloat16, SPT_, LPC_>(a, step, vec, st);
-  if (N <= 8) TYR_SS(4, 2)
-  if (N <= 16) TYR_SS(4, 4)
-  if (N <= 24) TYR_SS(6, 4)
-  if (N <= 32) TYR_SS(8, 4)
-  if (N <= 64) TYR_SS(8, 8)
-  if (N <= 128) TYR_SS(8, 16)
-  TYR_SS(16, 16)
+#define TYR_SS(kind, SPT_, LPC_) return dtype == 1 ? kind##_launch<float, SPT_, LPC_>(a, vec, st) : kind##_launch<__nv_bfloat16, SPT_, LPC_>(a, vec, st);
+  if (step) {                                   // few states per thread: enough threads to keep the memory busy
+    if (N <= 8) TYR_SS(step, 4, 2)
+    if (N <= 16) TYR_SS(step, 4, 4)
+    if (N <= 32) TYR_SS(step, 4, 8)
+    if (N <= 64) TYR_SS(step, 8, 8)
+    if (N <= 128) TYR_SS(step, 8, 16)
+    TYR_SS(step, 16, 16)
+  }
+  if (N <= 8) TYR_SS(prompt, 8, 1)
+  if (N <= 16) TYR_SS(prompt, 8, 2)
+  if (N <= 24) TYR_SS(prompt, 6, 4)
+  if (N <= 32) TYR_SS(prompt, 8, 4)
+  if (N <= 64) TYR_SS(prompt, 8, 8)
+  if (N <= 128) TYR_SS(prompt, 8, 16)
+  TYR_SS(prompt, 16, 16)
 #undef TYR_SS
 }

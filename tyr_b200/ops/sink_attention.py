@@ -78,6 +78,12 @@ def store_dim(H: int, G: int, d: int, dtype, device) -> int:
     return 64 if d <= 64 else 128
 
 
+def pick_splits(B: int, G: int, keys: int) -> int:
+    """Slices of the keys for one (row, K/V head): two to three CTAs per SM, at least 128 keys per slice (measured: more slices cost
+    more in the merge than they hide)."""
+    return max(2 if keys >= 512 else 1, min(-(-384 // max(1, B * G)), 32, -(-keys // 128)))
+
+
 def step_fused(q, G: int, store) -> bool:
     """The split-KV kernel takes this step: bf16 stores of 64 or 128 channels."""
     H, d = q.shape[2], q.shape[3]
@@ -94,7 +100,7 @@ def step_attention(q, k_new, v_new, store, pos: torch.Tensor, dv: int, *, scale:
     if out is None:
         out = torch.empty((B, 1, H * dv), dtype=q.dtype, device=q.device)
     if step_fused(q, G, store):
-        splits = da.pick_splits(B, G, cap)
+        splits = pick_splits(B, G, cap)
         key = (q.device.index, B, H, G, dkp, splits)
         ws = da._workspaces.get(key)
         if ws is None:
