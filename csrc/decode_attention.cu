@@ -102,6 +102,67 @@ __device__ __forceinline__ uint32_t prmt(uint32_t a, uint32_t b, uint32_t sel) {
   return r;
 }
 
+// The end of both kernels: combine the four warps' states {s_m, s_l, acc} (acc_warp: floats between two warps' accumulators), write the
+// result of a single slice, or leave the partial and let the last CTA of this (batch, K/V head) merge all slices.
+template <int DV, int GM>
+__device__ __forceinline__ void decode_combine(const DecodeAttnArgs& a, int b, int hkv, int split, const float (*s_m)[GM], const float (*s_l)[GM],
+                                               const float (*acc)[DV], int acc_warp, int* ticket) {
+  const int tid = threadIdx.x, G = a.Hq / a.Hkv;
+  // ---- combine the four warps -------------------------------------------------------------------------------
+  __syncthreads();
+  const int hq0 = hkv * G;
+  for (int i = tid; i < G * DV; i += kDecWarps * 32) {
+    const int g = i / DV, d = i - g * DV;
+    float M = -INFINITY;
+#pragma unroll
+    for (int w = 0; w < kDecWarps; ++w) M = fmaxf(M, s_m[w][g]);
+    float L = 0.f, A = 0.f;
+    if (M > -INFINITY) {
+#pragma unroll
+      for (int w = 0; w < kDecWarps; ++w) {
+        const float f = exp2f(s_m[w][g] - M);
+        L += s_l[w][g] * f;
+        A += acc[w * (acc_warp / DV) + g][d] * f;
+      }
+    }
+    const long long row = static_cast<long long>(b) * a.Hq + hq0 + g;
+    if (a.splits == 1) {
+      decode_write(a, b, hq0 + g, d, M, L, A);
+    } else {
+      a.part_acc[(row * a.splits + split) * DV + d] = A;
+      if (d == 0) {
+        a.part_ml[(row * a.splits + split) * 2] = M;
+        a.part_ml[(row * a.splits + split) * 2 + 1] = L;
+      }
+    }
+  }
+  if (a.splits == 1) return;
+
+  // ---- last CTA of this (batch, K/V head) merges the splits ---------------------------------------------------
+  __threadfence();
+  __syncthreads();
+  if (tid == 0) *ticket = atomicAdd(&a.counters[b * a.Hkv + hkv], 1);
+  __syncthreads();
+  if (*ticket != a.splits - 1) return;
+  __threadfence();
+  for (int i = tid; i < G * DV; i += kDecWarps * 32) {
+    const int g = i / DV, d = i - g * DV;
+    const long long row = static_cast<long long>(b) * a.Hq + hq0 + g;
+    float M = -INFINITY;
+    for (int sp = 0; sp < a.splits; ++sp) M = fmaxf(M, __ldcg(&a.part_ml[(row * a.splits + sp) * 2]));
+    float L = 0.f, A = 0.f;
+    if (M > -INFINITY) {
+      for (int sp = 0; sp < a.splits; ++sp) {
+        const float f = exp2f(__ldcg(&a.part_ml[(row * a.splits + sp) * 2]) - M);
+        L += __ldcg(&a.part_ml[(row * a.splits + sp) * 2 + 1]) * f;
+        A += __ldcg(&a.part_acc[(row * a.splits + sp) * DV + d]) * f;
+      }
+    }
+    decode_write(a, b, hq0 + g, d, M, L, A);
+  }
+  if (tid == 0) a.counters[b * a.Hkv + hkv] = 0;
+}
+
 // Tensor-core formulation (mma.sync m16n8k16, bf16 in, fp32 accumulate); one warp consumes 16 keys per step.
 //   S = Q K^T : M = query heads of the group (<= 8 real rows), N = 8 keys, K = 16 channels.  The reduction over channels
 //   is order-free, so lane (g, t) feeds the B fragment straight from one 16-byte load of key row g (channels
@@ -293,59 +354,138 @@ __global__ void __launch_bounds__(kDecWarps * 32) decode_attention_kernel(Decode
     }
   }
 
-  // ---- combine the four warps -------------------------------------------------------------------------------
-  __syncthreads();
-  const int hq0 = hkv * G;
-  for (int i = tid; i < G * DV; i += kDecWarps * 32) {
-    const int g = i / DV, d = i - g * DV;
-    float M = -INFINITY;
-#pragma unroll
-    for (int w = 0; w < kDecWarps; ++w) M = fmaxf(M, s_m[w][g]);
-    float L = 0.f, A = 0.f;
-    if (M > -INFINITY) {
-#pragma unroll
-      for (int w = 0; w < kDecWarps; ++w) {
-        const float f = exp2f(s_m[w][g] - M);
-        L += s_l[w][g] * f;
-        A += s_acc[w][g][d] * f;
-      }
-    }
-    const long long row = static_cast<long long>(b) * a.Hq + hq0 + g;
-    if (a.splits == 1) {
-      decode_write(a, b, hq0 + g, d, M, L, A);
-    } else {
-      a.part_acc[(row * a.splits + split) * DV + d] = A;
-      if (d == 0) {
-        a.part_ml[(row * a.splits + split) * 2] = M;
-        a.part_ml[(row * a.splits + split) * 2 + 1] = L;
-      }
-    }
-  }
-  if (a.splits == 1) return;
+  decode_combine<DV, GM>(a, b, hkv, split, s_m, s_l, s_acc[0], GM * DV, &s_ticket);
+}
 
-  // ---- last CTA of this (batch, K/V head) merges the splits ---------------------------------------------------
-  __threadfence();
-  __syncthreads();
-  if (tid == 0) s_ticket = atomicAdd(&a.counters[b * a.Hkv + hkv], 1);
-  __syncthreads();
-  if (s_ticket != a.splits - 1) return;
-  __threadfence();
-  for (int i = tid; i < G * DV; i += kDecWarps * 32) {
-    const int g = i / DV, d = i - g * DV;
-    const long long row = static_cast<long long>(b) * a.Hq + hq0 + g;
-    float M = -INFINITY;
-    for (int sp = 0; sp < a.splits; ++sp) M = fmaxf(M, __ldcg(&a.part_ml[(row * a.splits + sp) * 2]));
-    float L = 0.f, A = 0.f;
-    if (M > -INFINITY) {
-      for (int sp = 0; sp < a.splits; ++sp) {
-        const float f = exp2f(__ldcg(&a.part_ml[(row * a.splits + sp) * 2]) - M);
-        L += __ldcg(&a.part_ml[(row * a.splits + sp) * 2 + 1]) * f;
-        A += __ldcg(&a.part_acc[(row * a.splits + sp) * DV + d]) * f;
+// The values are the keys (one store), at most 8 query heads per K/V head.  Every warp brings its 16-key tiles into a ring of its own in
+// shared memory with cp.async, several tiles ahead, and takes the operands of both products from there: each row is read from memory
+// once, and the bytes in flight do not depend on registers.  Rows of D channels are chunks of 16 bytes at position chunk ^ (row & 7).
+constexpr int kRing = 4;
+
+__device__ __forceinline__ void da_cp_async16(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
+
+template <int D>
+__global__ void __launch_bounds__(kDecWarps * 32, 3) decode_attention_shared_kernel(DecodeAttnArgs a) {
+  constexpr int NJ = D / 32, NC = D / 64, GM = 8, CPR = D / 8;      // CPR: 16-byte chunks of a row
+  constexpr int kTile = 16 * D * 2;
+  extern __shared__ __align__(128) uint8_t da_ring[];
+  __shared__ float s_m[kDecWarps][GM], s_l[kDecWarps][GM];
+  __shared__ int s_ticket;
+  const int split = blockIdx.x, hkv = blockIdx.y, b = blockIdx.z;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int g = lane >> 2, t = lane & 3;
+  const int G = a.Hq / a.Hkv;
+  uint8_t* const ring = da_ring + warp * kRing * kTile;
+  const uint32_t ring_u = smem_u32(ring);
+  pdl_entry();
+  const int pos = a.pos[b * a.pos_stride];
+  if (pos < 0 || pos >= a.cap) {                 // position outside the store: report, leave the output untouched
+    if (tid == 0) report_error(a.err, ERR_BOUNDS, pos);
+    return;
+  }
+  const int n_keys = pos + 1;
+  int chunk = (n_keys + a.splits - 1) / a.splits;
+  chunk = (chunk + 63) & ~63;
+  const int lo = split * chunk, hi = min(lo + chunk, n_keys);
+  __nv_bfloat16* kc = a.k_cache + (static_cast<long long>(b) * a.Hkv + hkv) * a.cap * D;
+  const __nv_bfloat16* kn = a.k_new + b * a.kn_bs + static_cast<long long>(hkv) * D;
+  const int first = lo + warp * 16;
+  auto fetch = [&](int base, int stage) {        // 16 rows, a row's chunks by adjacent lanes
+    if (base < hi) {
+#pragma unroll
+      for (int i = 0; i < 16 * CPR / 32; ++i) {
+        const int x = lane + 32 * i, r = x / CPR, c = x % CPR;
+        const int row = min(base + r, hi - 1);   // clamped rows are masked below
+        const __nv_bfloat16* src = row == n_keys - 1 ? kn : kc + static_cast<long long>(row) * D;
+        da_cp_async16(ring_u + stage * kTile + (r * CPR + (c ^ (r & 7))) * 16, src + c * 8);
       }
     }
-    decode_write(a, b, hq0 + g, d, M, L, A);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+#pragma unroll
+  for (int i = 0; i < kRing - 1; ++i) fetch(first + i * kDecWarps * 16, i);
+  if (a.append && split == 0)                    // fused append; nobody reads this slot from the store in this launch
+    for (int i = tid; i < CPR; i += kDecWarps * 32) reinterpret_cast<uint4*>(kc + static_cast<long long>(pos) * D)[i] = reinterpret_cast<const uint4*>(kn)[i];
+  uint4 qf[NJ];                                  // A fragments of head g; zero rows beyond G
+  {
+    const __nv_bfloat16* qrow = a.q + b * a.q_bs + static_cast<long long>(hkv * G + (g < G ? g : 0)) * D;
+#pragma unroll
+    for (int j = 0; j < NJ; ++j) qf[j] = g < G ? *reinterpret_cast<const uint4*>(qrow + 32 * j + 8 * t) : make_uint4(0u, 0u, 0u, 0u);
   }
-  if (tid == 0) a.counters[b * a.Hkv + hkv] = 0;
+  float m = -INFINITY, l = 0.f, o[NC][8][2];
+#pragma unroll
+  for (int c = 0; c < NC; ++c)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) o[c][e][0] = o[c][e][1] = 0.f;
+  int stage = 0;
+#pragma unroll 1
+  for (int base = first; base < hi; base += kDecWarps * 16) {
+    asm volatile("cp.async.wait_group %0;" ::"n"(kRing - 2) : "memory");
+    __syncwarp();                                // every lane's part of the tile has landed, and the stage fetched next is free
+    fetch(base + (kRing - 1) * kDecWarps * 16, stage == 0 ? kRing - 1 : stage - 1);
+    const uint8_t* kt = ring + stage * kTile;
+    stage = stage + 1 == kRing ? 0 : stage + 1;
+    auto chunk_at = [&](int r, int c) { return *reinterpret_cast<const uint4*>(kt + (r * CPR + (c ^ (r & 7))) * 16); };
+    float s[2][2], none[2] = {0.f, 0.f};
+#pragma unroll
+    for (int tile = 0; tile < 2; ++tile) {
+      float c_lo[2] = {0.f, 0.f};
+#pragma unroll
+      for (int j = 0; j < NJ; ++j) {
+        const uint4 kf = chunk_at(8 * tile + g, 4 * j + t);
+        mma_bf16_16816<false>(c_lo, none, qf[j].x, qf[j].y, 0u, 0u, kf.x, kf.y);
+        mma_bf16_16816<false>(c_lo, none, qf[j].z, qf[j].w, 0u, 0u, kf.z, kf.w);
+      }
+      const int key0 = base + 8 * tile + 2 * t;
+      s[tile][0] = key0 < hi ? c_lo[0] * a.scale_log2 : -INFINITY;
+      s[tile][1] = key0 + 1 < hi ? c_lo[1] * a.scale_log2 : -INFINITY;
+    }
+    float mx = fmaxf(fmaxf(s[0][0], s[0][1]), fmaxf(s[1][0], s[1][1]));
+    mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+    mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
+    const float m_new = fmaxf(m, mx);            // finite: key `base` is always in range
+    const float p00 = exp2f(s[0][0] - m_new), p01 = exp2f(s[0][1] - m_new), p10 = exp2f(s[1][0] - m_new), p11 = exp2f(s[1][1] - m_new);
+    if (__any_sync(0xffffffffu, m_new > m)) {
+      const float alpha = exp2f(m - m_new);
+      l *= alpha;
+#pragma unroll
+      for (int c = 0; c < NC; ++c)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) { o[c][e][0] *= alpha; o[c][e][1] *= alpha; }
+      m = m_new;
+    }
+    l += (p00 + p01) + (p10 + p11);
+    const uint32_t pa0 = pack_bf16x2(p00, p01), pa2 = pack_bf16x2(p10, p11);
+#pragma unroll
+    for (int c = 0; c < NC; ++c) {
+      const uint4 q0 = chunk_at(2 * t, 8 * c + g), q1 = chunk_at(2 * t + 1, 8 * c + g), q2 = chunk_at(2 * t + 8, 8 * c + g), q3 = chunk_at(2 * t + 9, 8 * c + g);
+      const uint32_t v0[4] = {q0.x, q0.y, q0.z, q0.w}, v1[4] = {q1.x, q1.y, q1.z, q1.w}, v2[4] = {q2.x, q2.y, q2.z, q2.w}, v3[4] = {q3.x, q3.y, q3.z, q3.w};
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        const uint32_t sel = (e & 1) ? 0x7632u : 0x5410u;
+        mma_bf16_16816<false>(o[c][e], none, pa0, pa2, 0u, 0u, prmt(v0[e >> 1], v1[e >> 1], sel), prmt(v2[e >> 1], v3[e >> 1], sel));
+      }
+    }
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncwarp();
+  // this warp's state: the accumulators go over its own ring
+  float* acc = reinterpret_cast<float*>(ring);
+  l += __shfl_xor_sync(0xffffffffu, l, 1);
+  l += __shfl_xor_sync(0xffffffffu, l, 2);
+  if (g < G) {
+    if (t == 0) { s_m[warp][g] = m; s_l[warp][g] = l; }
+#pragma unroll
+    for (int c = 0; c < NC; ++c)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        acc[g * D + 64 * c + 16 * t + e] = o[c][e][0];
+        acc[g * D + 64 * c + 16 * t + 8 + e] = o[c][e][1];
+      }
+  }
+  decode_combine<D, GM>(a, b, hkv, split, s_m, s_l, reinterpret_cast<float(*)[D]>(da_ring), kRing * kTile / 4, &s_ticket);
 }
 
 }  // namespace tyr
@@ -386,6 +526,20 @@ static int decode_attention_launch(const void* q, const void* k_new, const void*
   const dim3 grid(splits, Hkv, B);
   const cudaStream_t st = (cudaStream_t)stream;
   const dim3 block(kDecWarps * 32);
+  if (k_cache == v_cache && k_new == v_new && DK == DV && (DK == 64 || DK == 128) && !wide && r1 == nullptr && !ring && window == 0) {
+    const size_t smem = static_cast<size_t>(kDecWarps) * kRing * 16 * DK * 2;
+    auto kernel = DK == 64 ? decode_attention_shared_kernel<64> : decode_attention_shared_kernel<128>;
+    static bool configured[64][2] = {};          // the attribute is per device
+    int dev = 0;
+    if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) dev = 0;
+    bool& done = configured[dev][DK == 128 ? 1 : 0];
+    if (!done) {
+      const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      if (e != cudaSuccess) return 1000 + (int)e;
+      done = true;
+    }
+    return (int)launch_dependent(kernel, grid, block, smem, st, a);
+  }
   const bool bias = r1 != nullptr;
 #define TYR_DEC(DK_, DV_, WIDE_, BIAS_)                                  \
   if (DK == DK_ && DV == DV_ && wide == WIDE_ && bias == BIAS_)         \

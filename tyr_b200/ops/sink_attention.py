@@ -79,9 +79,10 @@ def store_dim(H: int, G: int, d: int, dtype, device) -> int:
 
 
 def pick_splits(B: int, G: int, keys: int) -> int:
-    """Slices of the keys for one (row, K/V head): two to three CTAs per SM, at least 128 keys per slice (measured: more slices cost
-    more in the merge than they hide)."""
-    return max(2 if keys >= 512 else 1, min(-(-384 // max(1, B * G)), 32, -(-keys // 128)))
+    """Slices of the keys for one (row, K/V head).  The merge costs about as much as 512 keys, so slices are no shorter and one per (row,
+    head) is best once those fill the SMs; far beyond that, three even out the last wave (measured)."""
+    want = max(1, 192 // (B * G)) if B * G <= 192 else 3
+    return max(1, min(want, -(-keys // 512), 32))
 
 
 def step_fused(q, G: int, store) -> bool:
