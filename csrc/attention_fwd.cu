@@ -32,7 +32,7 @@
 // table is the mask of the second pass too); BIAS 2 evaluates the logarithm per score.  These forms also take head sizes below
 // 128 (a multiple of 8): TMA fills the missing channels with zeros and the Q K^T loop stops at the last real one.
 //
-// Sink and gate (BIAS 3): the same head sizes without a penalty; the softmax denominator also holds exp(sink_h), and the output is
+// Sink and gate (BIAS 3): the same head sizes without a penalty, with an optional window; the softmax denominator also holds exp(sink_h), and the output is
 // multiplied by out_scale * sigmoid(gate), both in the epilogue.
 //
 // The reference calls at::scaled_dot_product_attention, or a query-chunked masked-math fallback
@@ -654,12 +654,12 @@ extern "C" TYR_EXPORT int tyr_flash_fwd_biased(const void* q, const void* k, con
 }
 
 // Causal attention with a sink per head (nullable) in the softmax denominator and the output multiplied by out_scale * sigmoid(gate)
-// (gate nullable); sizes as above.  strides: (batch, row, head) of q, k, v, o, gate.  v may be k.
+// (gate nullable) and an optional sliding window (0: none); sizes as above.  strides: (batch, row, head) of q, k, v, o, gate.  v may be k.
 extern "C" TYR_EXPORT int tyr_flash_fwd_sink(const void* q, const void* k, const void* v, void* o, const float* sink, const void* gate, int B,
-                                             int Hq, int Hkv, int T, int dk, int dv, const long long* strides, float scale, float out_scale,
-                                             int* err, void* stream) {
-  if (dk <= 0 || dv <= 0 || dk > ATT_D || dv > ATT_D || (dk & 7) || (dv & 7) || scale <= 0.f) return -1;
+                                             int Hq, int Hkv, int T, int dk, int dv, const long long* strides, int window, float scale,
+                                             float out_scale, int* err, void* stream) {
+  if (dk <= 0 || dv <= 0 || dk > ATT_D || dv > ATT_D || (dk & 7) || (dv & 7) || window < 0 || scale <= 0.f) return -1;
   if (gate != nullptr && (((strides[12] | strides[13] | strides[14]) & 7) || (reinterpret_cast<uintptr_t>(gate) & 15))) return -3;
   const FlashExtra ex{sink, gate, strides + 12, out_scale};
-  return flash_fwd_launch(q, k, v, o, nullptr, B, Hq, Hkv, T, T, dk, dv, strides, 1, 0, 0, scale, nullptr, nullptr, err, stream, &ex);
+  return flash_fwd_launch(q, k, v, o, nullptr, B, Hq, Hkv, T, T, dk, dv, strides, 1, window, 0, scale, nullptr, nullptr, err, stream, &ex);
 }

@@ -4,7 +4,7 @@
 //
 // a sink (the softmax denominator also holds exp(sink_h)) and an output gate (element by element, out_scale sigmoid(gate)).
 //
-//   * qk_norm_store: per-head RMSNorm of q and k (no rotation), v copied, rows of the padded batch written to the K/V store at
+//   * qk_norm_store: per-head RMSNorm of q and k (no rotation; weights and projection biases optional), v copied, rows of the padded batch written to the K/V store at
 //                    their own positions (plain or ring).
 //   * general:       one warp per (query, head), online softmax in fp32; reads keys from the prompt's own rows or from the store.
 //
@@ -22,7 +22,8 @@ __device__ __forceinline__ void ag_store(__nv_bfloat16* p, float v) { *p = __flo
 struct QkNormArgs {
   const void* y;               // [B * S, ld]: q (H * dk) | k (G * dk) | v (G * dv); G = 0 when the layer has no keys of its own
   long long ld;
-  const float *q_w, *k_w;      // [dk] (k_w unused when G == 0)
+  const float *q_w, *k_w;      // [dk] (k_w unused when G == 0); null: ones
+  const float* bias;           // [(H + G) dk + G dv] added to the columns of y (nullable)
   void* q_out;                 // [B * S, H, dkp]
   void* k_out;                 // [B * S, G, dkp]
   void* v_out;                 // [B * S, G, dvp] or null
@@ -48,7 +49,9 @@ __global__ void __launch_bounds__(256) qk_norm_store_kernel(QkNormArgs a) {
     const bool is_q = hd < a.H, is_v = hd >= a.H + a.G;
     const int g = is_q ? hd : (is_v ? hd - a.H - a.G : hd - a.H);
     const int d_in = is_v ? a.dv : a.dk, d_out = is_v ? a.dvp : a.dkp;
-    src += is_v ? static_cast<long long>(a.H + a.G) * a.dk + static_cast<long long>(g) * a.dv : static_cast<long long>(hd) * a.dk;
+    const int col = is_v ? (a.H + a.G) * a.dk + g * a.dv : hd * a.dk;
+    src += col;
+    const float* bias = a.bias ? a.bias + col : nullptr;
     T* dst = is_q ? static_cast<T*>(a.q_out) + (row * a.H + g) * d_out
                   : (is_v ? (a.v_out ? static_cast<T*>(a.v_out) + (row * a.G + g) * d_out : nullptr)
                           : static_cast<T*>(a.k_out) + (row * a.G + g) * d_out);
@@ -65,15 +68,15 @@ __global__ void __launch_bounds__(256) qk_norm_store_kernel(QkNormArgs a) {
     if (!is_v) {
       float ss = 0.f;
       for (int d = lane; d < d_in; d += 32) {
-        const float v = ag_load(src + d);
+        const float v = ag_load(src + d) + (bias ? bias[d] : 0.f);
         ss += v * v;
       }
       rstd = 1.f / sqrtf(warp_sum(ss) / d_in + a.eps);
     }
     const float* w = is_q ? a.q_w : a.k_w;
     for (int d = lane; d < d_out; d += 32) {
-      float v = d < d_in ? ag_load(src + d) : 0.f;
-      if (!is_v && d < d_in) v = v * rstd * w[d];
+      float v = d < d_in ? ag_load(src + d) + (bias ? bias[d] : 0.f) : 0.f;
+      if (!is_v && d < d_in) v = v * rstd * (w ? w[d] : 1.f);
       if (dst) ag_store(dst + d, v);
       if (slot) ag_store(slot + d, v);
     }
@@ -165,13 +168,13 @@ __global__ void __launch_bounds__(GA_WARPS * 32) general_attention_kernel(Genera
 
 using namespace tyr;
 
-extern "C" TYR_EXPORT int tyr_qk_norm_store(const void* y, long long ld, const float* q_w, const float* k_w, void* q_out, void* k_out,
+extern "C" TYR_EXPORT int tyr_qk_norm_store(const void* y, long long ld, const float* q_w, const float* k_w, const float* bias, void* q_out, void* k_out,
                                             void* v_out, void* k_store, void* v_store, const int* pos, const int* lens, int B, int S,
                                             int H, int G, int dk, int dv, int dkp, int dvp, int cap, int ring, float eps, int dtype,
                                             void* stream) {
   if (B <= 0 || S <= 0 || H <= 0 || G < 0 || dk <= 0 || dkp < dk || dvp < dv || (G > 0 && dv <= 0)) return -1;
   if ((k_store != nullptr) != (v_store != nullptr) || (k_store != nullptr && cap <= 0)) return -2;
-  QkNormArgs a{y, ld, q_w, k_w, q_out, k_out, v_out, k_store, v_store, pos, lens, B, S, H, G, dk, dv, dkp, dvp, cap, ring, eps};
+  QkNormArgs a{y, ld, q_w, k_w, bias, q_out, k_out, v_out, k_store, v_store, pos, lens, B, S, H, G, dk, dv, dkp, dvp, cap, ring, eps};
   const long long want = (static_cast<long long>(B) * S * (H + 2 * G) + 7) / 8;
   const dim3 grid(static_cast<unsigned>(want < 148LL * 32 ? want : 148LL * 32));
   return (int)(dtype == 1 ? launch_dependent(qk_norm_store_kernel<float>, grid, dim3(256), 0, (cudaStream_t)stream, a)

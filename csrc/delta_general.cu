@@ -258,6 +258,56 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(const float* __restrict
   }
 }
 
+// The same for wide heads (all of a layer's channels normed together): one CTA per (row, head).
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256) gated_norm_wide_kernel(const float* __restrict__ o, const T* __restrict__ z, long long ld_z,
+                                                              const float* __restrict__ w, T* __restrict__ y, long long ld_y, int Hv, int dv,
+                                                              float eps, int act) {
+  __shared__ float red[8];
+  pdl_entry();
+  const int tid = threadIdx.x;
+  const long long i = blockIdx.x;
+  const float* op = o + i * dv;
+  const T* zp = z + (i / Hv) * ld_z + (i % Hv) * dv;
+  T* yp = y + (i / Hv) * ld_y + (i % Hv) * dv;
+  constexpr int NV = 4;                  // float4 vectors of a thread kept between the reduction and the write
+  float4 v[NV];
+  float ss = 0.f;
+  if constexpr (VEC) {
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+      const int d = 4 * (tid + 256 * j);
+      v[j] = d < dv ? *reinterpret_cast<const float4*>(op + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+      ss += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
+    }
+  } else {
+    for (int d = tid; d < dv; d += 256) ss += op[d] * op[d];
+  }
+  ss = warp_sum(ss);
+  if ((tid & 31) == 0) red[tid >> 5] = ss;
+  __syncthreads();
+  float tot = 0.f;
+#pragma unroll
+  for (int k = 0; k < 8; ++k) tot += red[k];
+  const float rstd = 1.f / sqrtf(tot / dv + eps);
+  if constexpr (VEC) {
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+      const int d = 4 * (tid + 256 * j);
+      if (d >= dv) continue;
+      const uint2 zu = *reinterpret_cast<const uint2*>(reinterpret_cast<const char*>(zp + d));
+      const float2 z0 = unpack_bf16x2(zu.x), z1 = unpack_bf16x2(zu.y);
+      const float4 wv = *reinterpret_cast<const float4*>(w + d);
+      uint2 r;
+      r.x = pack_bf16x2(v[j].x * rstd * wv.x * dg_gate(z0.x, act), v[j].y * rstd * wv.y * dg_gate(z0.y, act));
+      r.y = pack_bf16x2(v[j].z * rstd * wv.z * dg_gate(z1.x, act), v[j].w * rstd * wv.w * dg_gate(z1.y, act));
+      *reinterpret_cast<uint2*>(reinterpret_cast<char*>(yp + d)) = r;
+    }
+  } else {
+    for (int d = tid; d < dv; d += 256) dg_store(yp + d, op[d] * rstd * w[d] * dg_gate(dg_load(zp + d), act));
+  }
+}
+
 }  // namespace tyr
 
 using namespace tyr;
@@ -354,6 +404,16 @@ extern "C" TYR_EXPORT int tyr_gated_norm(const float* o, const void* z, long lon
   const long long want = (rows * Hv + 7) / 8;
   const dim3 grid(static_cast<unsigned>(want < 148LL * 32 ? want : 148LL * 32));
   cudaStream_t st = (cudaStream_t)stream;
+  if (dv > 256) {
+    const dim3 wide(static_cast<unsigned>(rows * Hv));
+    if (dtype == 1)
+      return (int)launch_dependent(gated_norm_wide_kernel<float, false>, wide, dim3(256), 0, st, o, (const float*)z, ld_z, w, (float*)y, ld_y, Hv, dv, eps, act);
+    const bool vec = (dv & 3) == 0 && dv <= 4096 && ((ld_z | ld_y) & 3) == 0 && ((reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(y)) & 7) == 0;
+    return (int)(vec ? launch_dependent(gated_norm_wide_kernel<__nv_bfloat16, true>, wide, dim3(256), 0, st, o, (const __nv_bfloat16*)z, ld_z, w,
+                                        (__nv_bfloat16*)y, ld_y, Hv, dv, eps, act)
+                     : launch_dependent(gated_norm_wide_kernel<__nv_bfloat16, false>, wide, dim3(256), 0, st, o, (const __nv_bfloat16*)z, ld_z, w,
+                                        (__nv_bfloat16*)y, ld_y, Hv, dv, eps, act));
+  }
   if (dtype == 1)
     return (int)launch_dependent(gated_norm_kernel<float>, grid, dim3(256), 0, st, o, (const float*)z, ld_z, w, (float*)y, ld_y, rows, Hv, dv, eps, act);
   return (int)launch_dependent(gated_norm_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, o, (const __nv_bfloat16*)z, ld_z, w, (__nv_bfloat16*)y, ld_y,

@@ -110,12 +110,19 @@ __device__ __forceinline__ float apply_act(float v, int act) {
 // One 32-column chunk of the epilogue with the activation fixed at compile time (no per-element branches):
 //   ACT 0: v = alpha * acc (+ beta * aux)      1: alpha * relu(acc)^2 (+ ...)      2: alpha * relu(acc) (+ ...)
 //   ACT 3: v = alpha * acc * 2 * sqrt(aux)     (gradient of y = relu(z)^2 given aux = y)
+//   ACT 6: xIELU of acc: alpha z^2 + z / 2 above zero, beta (e^z - 1 - z) + z / 2 below (no aux)
 template <int ACT>
 __device__ __forceinline__ void epi_chunk(const uint32_t (&r)[32], const float (&ax)[32], bool use_aux, float alpha,
                                           float beta, float (&v)[32]) {
   if constexpr (ACT == 3) {
 #pragma unroll
     for (int j = 0; j < 32; ++j) v[j] = alpha * __uint_as_float(r[j]) * 2.f * sqrtf(fmaxf(ax[j], 0.f));
+  } else if constexpr (ACT == 6) {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) {
+      const float z = __uint_as_float(r[j]);
+      v[j] = fmaf(0.5f, z, z > 0.f ? alpha * z * z : beta * (__expf(z) - 1.f - z));
+    }
   } else {
 #pragma unroll
     for (int j = 0; j < 32; ++j) {
@@ -638,6 +645,7 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA,
         if (p.act == 0) epi_chunk<0>(r, ax, use_aux, p.alpha, p.beta, v);
         else if (p.act == 1) epi_chunk<1>(r, ax, use_aux, p.alpha, p.beta, v);
         else if (p.act == 2) epi_chunk<2>(r, ax, use_aux, p.alpha, p.beta, v);
+        else if (p.act == 6) epi_chunk<6>(r, ax, use_aux, p.alpha, p.beta, v);
         else epi_chunk<3>(r, ax, use_aux, p.alpha, p.beta, v);
         if (tma_out) {
           uint8_t* st = s.out_stage[epi][n_stores % EPI_BUFS] + lane * 128;

@@ -1,6 +1,6 @@
 // What lies between a layer's input projection and its mixers, in one launch: the columns of the projection are cut into segments,
 // and each segment takes an optional causal depthwise convolution over time (any number of taps, bias), an optional activation
-// (SiLU or squared ReLU), an optional factor that depends on the position alone (query temperature
+// (SiLU, squared ReLU or xIELU), an optional factor that depends on the position alone (query temperature
 // 1 + coef ln(floor((p + 1) / every) + 1)), and a destination of its own: rows of heads that may be padded, and a K/V store.
 //
 //   * prompt: whole prompts [B, S, columns], rows of unequal length; leaves the last `taps` inputs of every row as the window.
@@ -13,7 +13,7 @@
 namespace tyr {
 
 constexpr int MC_SEGS = 6;
-enum MixAct : int { MC_NONE = 0, MC_SILU = 1, MC_RELU2 = 2 };
+enum MixAct : int { MC_NONE = 0, MC_SILU = 1, MC_RELU2 = 2, MC_XIELU = 3 };
 
 struct MixSegment {
   int col, heads, d_in, d_out;   // source columns [col, col + heads * d_in); a head's d_in channels go to the first of d_out
@@ -26,6 +26,7 @@ struct MixSegment {
   void* store;                   // [B, heads, cap, store_d] by position (nullable; prompt only)
   int cap, store_d;
   float temp_coef, temp_every;   // temp_every 0: no factor
+  float act_a, act_b;            // xIELU: a z^2 + z / 2 above zero, b (e^z - 1 - z) + z / 2 below
 };
 
 struct MixArgs {
@@ -41,9 +42,12 @@ __device__ __forceinline__ float mc_load(const float* p) { return *p; }
 __device__ __forceinline__ float mc_load(const __nv_bfloat16* p) { return __bfloat162float(*p); }
 __device__ __forceinline__ void mc_store(float* p, float v) { *p = v; }
 __device__ __forceinline__ void mc_store(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
-__device__ __forceinline__ float mc_act(float v, int act) {
+__device__ __forceinline__ float mc_xielu(float v, float a, float b) { return (v > 0.f ? a * v * v : b * (expm1f(v) - v)) + 0.5f * v; }
+__device__ __forceinline__ float mc_act(float v, const MixSegment& s) {
+  const int act = s.act;
   if (act == MC_SILU) return v / (1.f + expf(-v));
   if (act == MC_RELU2) { const float r = fmaxf(v, 0.f); return r * r; }
+  if (act == MC_XIELU) return mc_xielu(v, s.act_a, s.act_b);
   return v;
 }
 __device__ __forceinline__ float mc_temp(const MixSegment& s, int p) {
@@ -137,7 +141,7 @@ __global__ void __launch_bounds__(256) mix_plain_kernel(const __grid_constant__ 
           }
       }
     }
-    acc = mc_act(acc, s.act) * mc_temp(s, STEP ? a.pos[b] : t);
+    acc = mc_act(acc, s) * mc_temp(s, STEP ? a.pos[b] : t);
     mc_store(dst, acc);
     if (!STEP && s.store && t < len && t < s.cap)
       mc_store(static_cast<T*>(s.store) + ((static_cast<long long>(b) * s.heads + c / s.d_in) * s.cap + t) * s.store_d + c % s.d_in, acc);
@@ -174,7 +178,7 @@ __global__ void __launch_bounds__(MC_VEC, 4) mix_vec_kernel(const __grid_constan
     for (int j = 0; j < 4; ++j) wt[e][j] = K == 0 ? (j == 3 ? 1.f : 0.f) : (j >= 4 - K ? s.w[(c + e) * K + j - (4 - K)] : 0.f);
   }
   const int act = s.act;
-  const float coef = s.temp_coef, every = s.temp_every;
+  const float coef = s.temp_coef, every = s.temp_every, act_a = s.act_a, act_b = s.act_b;
   const long long x_ss = a.x_ss, out_ld = s.out_ld;
   const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(a.x) + b * a.x_sb + s.col + c + t0 * x_ss;
   __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(s.out) + (static_cast<long long>(b) * a.S + t0) * out_ld + c;
@@ -198,6 +202,9 @@ __global__ void __launch_bounds__(MC_VEC, 4) mix_vec_kernel(const __grid_constan
     } else if (act == MC_RELU2) {
       a0 = fmaxf(a0, 0.f) * fmaxf(a0, 0.f);
       a1 = fmaxf(a1, 0.f) * fmaxf(a1, 0.f);
+    } else if (act == MC_XIELU) {
+      a0 = mc_xielu(a0, act_a, act_b);
+      a1 = mc_xielu(a1, act_a, act_b);
     }
     if (every > 0.f) {
       const float f = mc_temp_fast(coef, every, t);

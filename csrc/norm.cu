@@ -514,6 +514,111 @@ __global__ void __launch_bounds__(256) add_norm_kernel(AddNormArgs a) {
   }
 }
 
+// A sublayer with a norm on either side of it: its output joins an fp32 stream and the next sublayer reads the norm of the sum.
+//   t = x + bias;   t <- norm(t) * post;   r = resid + t (replace: r = t);   resid_out = r;   y = norm(r) * gain (no gain: y = r).
+struct SandwichNormArgs {
+  const void* x;           // [rows, D] (TX)
+  const float* bias;       // [D], nullable
+  const float* post;       // [D], nullable: x joins as it is
+  const float* gain;       // [D], nullable
+  float* resid;            // [rows, D], in place
+  void* y;                 // [rows, D] (TY)
+  long long x_stride, y_stride;      // elements between rows
+  int D, replace;
+  float eps;
+};
+
+__device__ __forceinline__ float pn_block_sum(float v, float* red, int tid, int nw) {
+  v = warp_sum(v);
+  if ((tid & 31) == 0) red[tid >> 5] = v;
+  __syncthreads();
+  float tot = 0.f;
+  for (int i = 0; i < nw; ++i) tot += red[i];
+  return tot;
+}
+
+template <typename TX, typename TY, bool VEC>
+__global__ void __launch_bounds__(256) sandwich_norm_kernel(SandwichNormArgs a) {
+  __shared__ float red[2][8];
+  const long long row = blockIdx.x;
+  const int tid = threadIdx.x, nw = blockDim.x >> 5;
+  const TX* x = static_cast<const TX*>(a.x) + row * a.x_stride;
+  float* resid = a.resid + row * a.D;
+  TY* y = static_cast<TY*>(a.y) + row * a.y_stride;
+  pdl_entry();
+  float f[kPnVecs][8], ss = 0.f;
+  if constexpr (VEC) {
+#pragma unroll
+    for (int j = 0; j < kPnVecs; ++j) {
+      const int v = (tid + j * blockDim.x) * 8;
+      if (v >= a.D) continue;
+      pn_load8(x + v, f[j]);
+      if (a.bias) {
+        float b[8];
+        pn_load8(a.bias + v, b);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[j][e] += b[e];
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss += f[j][e] * f[j][e];
+    }
+  } else {
+    for (int d = tid; d < a.D; d += blockDim.x) {
+      const float t = pn_get(x + d) + (a.bias ? a.bias[d] : 0.f);
+      ss += t * t;
+    }
+  }
+  const float inner = a.post ? rsqrtf(pn_block_sum(ss, red[0], tid, nw) / a.D + a.eps) : 1.f;
+  ss = 0.f;
+  if constexpr (VEC) {
+#pragma unroll
+    for (int j = 0; j < kPnVecs; ++j) {
+      const int v = (tid + j * blockDim.x) * 8;
+      if (v >= a.D) continue;
+      if (a.post) {
+        float w[8];
+        pn_load8(a.post + v, w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[j][e] *= inner * w[e];
+      }
+      if (!a.replace) {
+        float r[8];
+        pn_load8(resid + v, r);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[j][e] += r[e];
+      }
+      pn_store8(resid + v, f[j]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss += f[j][e] * f[j][e];
+    }
+  } else {
+    for (int d = tid; d < a.D; d += blockDim.x) {
+      float t = pn_get(x + d) + (a.bias ? a.bias[d] : 0.f);
+      if (a.post) t *= inner * a.post[d];
+      if (!a.replace) t += resid[d];
+      resid[d] = t;
+      ss += t * t;
+    }
+  }
+  const float outer = a.gain ? rsqrtf(pn_block_sum(ss, red[1], tid, nw) / a.D + a.eps) : 1.f;
+  if constexpr (VEC) {
+#pragma unroll
+    for (int j = 0; j < kPnVecs; ++j) {
+      const int v = (tid + j * blockDim.x) * 8;
+      if (v >= a.D) continue;
+      if (a.gain) {
+        float w[8];
+        pn_load8(a.gain + v, w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[j][e] *= outer * w[e];
+      }
+      pn_store8(y + v, f[j]);
+    }
+  } else {
+    for (int d = tid; d < a.D; d += blockDim.x) pn_put(y + d, a.gain ? resid[d] * outer * a.gain[d] : resid[d]);
+  }
+}
+
 static int grid_for_rows(long long rows, int warps_per_block) {
   long long blocks = (rows + warps_per_block - 1) / warps_per_block;
   const long long cap = 148LL * 16;
@@ -622,4 +727,24 @@ extern "C" TYR_EXPORT int tyr_add_norm(const void* x, long long x_stride, const 
   if (x_dtype == 0) return (int)(y_dtype == 0 ? TYR_AN(__nv_bfloat16, __nv_bfloat16) : TYR_AN(__nv_bfloat16, float));
   return (int)(y_dtype == 0 ? TYR_AN(float, __nv_bfloat16) : TYR_AN(float, float));
 #undef TYR_AN
+}
+
+// bias, post, gain fp32 [D], each nullable; resid fp32 [rows, D] contiguous, in place; y rows of y_stride elements.
+extern "C" TYR_EXPORT int tyr_sandwich_norm(const void* x, long long x_stride, const float* bias, const float* post, const float* gain, float* resid,
+                                            void* y, long long y_stride, long long rows, int D, int replace, float eps, int x_dtype, int y_dtype,
+                                            void* stream) {
+  if (rows <= 0 || D <= 0 || x == nullptr || resid == nullptr || y == nullptr) return -1;
+  SandwichNormArgs a{x, bias, post, gain, resid, y, x_stride, y_stride, D, replace, eps};
+  const uintptr_t al = reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(bias) | reinterpret_cast<uintptr_t>(post) |
+                       reinterpret_cast<uintptr_t>(gain) | reinterpret_cast<uintptr_t>(resid) | reinterpret_cast<uintptr_t>(y);
+  const bool vec = (D & 7) == 0 && (x_stride & 7) == 0 && (y_stride & 7) == 0 && (al & 15) == 0 && D <= 256 * 8 * kPnVecs;
+  int threads = 256;
+  while (threads > 32 && threads * 4 >= D) threads >>= 1;       // narrow rows: no idle warps
+  const dim3 grid(static_cast<unsigned>(rows)), block(threads);
+  cudaStream_t st = (cudaStream_t)stream;
+#define TYR_SN(TX, TY) (vec ? launch_dependent(sandwich_norm_kernel<TX, TY, true>, grid, block, 0, st, a) \
+                            : launch_dependent(sandwich_norm_kernel<TX, TY, false>, grid, block, 0, st, a))
+  if (x_dtype == 0) return (int)(y_dtype == 0 ? TYR_SN(__nv_bfloat16, __nv_bfloat16) : TYR_SN(__nv_bfloat16, float));
+  return (int)(y_dtype == 0 ? TYR_SN(float, __nv_bfloat16) : TYR_SN(float, float));
+#undef TYR_SN
 }

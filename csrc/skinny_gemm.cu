@@ -24,7 +24,14 @@ struct SkinnyArgs {
   float* ws;                   // [M, N] fp32, zero on entry and exit; used when the reduction is split over gridDim.y CTAs
   long long ldx, ldw, ldy;
   int M, N, K;
+  long long hx, hw, hy;        // per-head form: elements from head to head (gridDim.z heads)
+  int act;                     // 6: xIELU with factors act_a, act_b, as in csrc/gemm_tcgen05.cu; 0: none
+  float act_a, act_b;
 };
+
+__device__ __forceinline__ float sk_act(float z, const SkinnyArgs& a) {
+  return a.act == 6 ? fmaf(0.5f, z, z > 0.f ? a.act_a * z * z : a.act_b * (__expf(z) - 1.f - z)) : z;
+}
 
 __device__ __forceinline__ void mma_16816(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
@@ -40,6 +47,9 @@ __global__ void __launch_bounds__(kSkWarps * 32) skinny_gemm_kernel(SkinnyArgs a
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int g = lane >> 2, t = lane & 3;
   const int row0 = blockIdx.x * 16;
+  a.w += blockIdx.z * a.hw;
+  a.x += blockIdx.z * a.hx;
+  a.y += blockIdx.z * a.hy;
   // The weights are constants: while the kernel that produces `x` still runs (this one may already be resident, see
   // launch_dependent), pull the head of every weight row of this CTA into the L2.  The whole grid asks for at most
   // kSkPrefetchBytes, so what it brings in is still there when the loop below reads it.
@@ -49,7 +59,7 @@ __global__ void __launch_bounds__(kSkWarps * 32) skinny_gemm_kernel(SkinnyArgs a
     const int chunks = a.K >> 5;
     const int c0 = static_cast<int>(static_cast<long long>(chunks) * blockIdx.y / gridDim.y);
     const int c1 = static_cast<int>(static_cast<long long>(chunks) * (blockIdx.y + 1) / gridDim.y);
-    long long per_row = kSkPrefetchBytes / (static_cast<long long>(gridDim.x) * gridDim.y * (GATED ? 32 : 16));
+    long long per_row = kSkPrefetchBytes / (static_cast<long long>(gridDim.x) * gridDim.y * gridDim.z * (GATED ? 32 : 16));
     per_row = min(per_row & ~127LL, static_cast<long long>(c1 - c0) * 64);
     if (r < a.N && per_row >= 128)
       bulk_prefetch_l2((tid < 16 ? a.w : a.w2) + static_cast<long long>(r) * a.ldw + 32LL * c0, static_cast<uint32_t>(per_row));
@@ -128,7 +138,7 @@ __global__ void __launch_bounds__(kSkWarps * 32) skinny_gemm_kernel(SkinnyArgs a
         a.y[tok * a.ldy + row] = __float2bfloat16(s / (1.f + __expf(-s)) * u);
       } else if (gridDim.y == 1) {
         if (a.bias) s += __bfloat162float(a.bias[row]);
-        a.y[tok * a.ldy + row] = __float2bfloat16(s);
+        a.y[tok * a.ldy + row] = __float2bfloat16(sk_act(s, a));
       } else {
         atomicAdd(a.ws + static_cast<long long>(tok) * a.N + row, s);
       }
@@ -145,7 +155,7 @@ __global__ void __launch_bounds__(256) skinny_finish_kernel(SkinnyArgs a) {
     float s = a.ws[i];
     a.ws[i] = 0.f;
     if (a.bias) s += __bfloat162float(a.bias[row]);
-    a.y[tok * a.ldy + row] = __float2bfloat16(s);
+    a.y[tok * a.ldy + row] = __float2bfloat16(sk_act(s, a));
   }
 }
 
@@ -193,13 +203,15 @@ extern "C" TYR_EXPORT int tyr_skinny_gemm_splits(int N, int K) {
   return splits < 1 ? 1 : splits;
 }
 
-extern "C" TYR_EXPORT int tyr_skinny_gemm_bf16(const void* x, const void* w, const void* bias, void* y, void* ws, long long ldx,
-                                               long long ldw, long long ldy, int M, int N, int K, void* stream) {
+static int skinny_launch(const void* x, const void* w, const void* bias, void* y, void* ws, long long ldx, long long ldw, long long ldy, int M,
+                         int N, int K, int act, float act_a, float act_b, void* stream) {
   using namespace tyr;
+  if (act != 0 && act != 6) return -4;
   if (M < 1 || M > 32 || N < 1 || K < 32 || (K & 31)) return -1;
   if ((ldx | ldw) & 7) return -2;                                    // 16-byte loads
   if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) return -3;
-  SkinnyArgs a{(const __nv_bfloat16*)x, (const __nv_bfloat16*)w, nullptr, (const __nv_bfloat16*)bias, (__nv_bfloat16*)y, (float*)ws, ldx, ldw, ldy, M, N, K};
+  SkinnyArgs a{(const __nv_bfloat16*)x, (const __nv_bfloat16*)w, nullptr, (const __nv_bfloat16*)bias, (__nv_bfloat16*)y, (float*)ws, ldx, ldw, ldy, M, N, K,
+               0, 0, 0, act, act_a, act_b};
   const int splits = ws != nullptr ? tyr_skinny_gemm_splits(N, K) : 1;
   const dim3 grid((N + 15) / 16, splits);
   skinny_prefer_l1();
@@ -212,6 +224,34 @@ extern "C" TYR_EXPORT int tyr_skinny_gemm_bf16(const void* x, const void* w, con
     launch_dependent(skinny_finish_kernel, dim3((int)blocks), dim3(256), 0, (cudaStream_t)stream, a);
   }
   return (int)cudaGetLastError();
+}
+
+extern "C" TYR_EXPORT int tyr_skinny_gemm_bf16(const void* x, const void* w, const void* bias, void* y, void* ws, long long ldx,
+                                               long long ldw, long long ldy, int M, int N, int K, void* stream) {
+  return skinny_launch(x, w, bias, y, ws, ldx, ldw, ldy, M, N, K, 0, 0.f, 0.f, stream);
+}
+
+// The same with an activation in the epilogue (6: xIELU, factors act_a above zero and act_b below).
+extern "C" TYR_EXPORT int tyr_skinny_gemm_act_bf16(const void* x, const void* w, const void* bias, void* y, void* ws, long long ldx, long long ldw,
+                                                   long long ldy, int M, int N, int K, int act, float act_a, float act_b, void* stream) {
+  return skinny_launch(x, w, bias, y, ws, ldx, ldw, ldy, M, N, K, act, act_a, act_b, stream);
+}
+
+// A product of its own for each head: y[m, h, :N] = x[m, h, :K] @ W[h]^T for `heads` heads, rows (ldx, ldy) and heads (hx, hw, hy) apart
+// by element strides.
+extern "C" TYR_EXPORT int tyr_skinny_heads_bf16(const void* x, const void* w, void* y, long long ldx, long long hx, long long hw, long long ldw,
+                                                long long ldy, long long hy, int heads, int M, int N, int K, void* stream) {
+  using namespace tyr;
+  if (M < 1 || M > 32 || N < 1 || K < 32 || (K & 31) || heads < 1 || heads > 65535) return -1;
+  if ((ldx | ldw | hx | hw) & 7) return -2;
+  if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) return -3;
+  SkinnyArgs a{(const __nv_bfloat16*)x, (const __nv_bfloat16*)w, nullptr, nullptr, (__nv_bfloat16*)y, nullptr, ldx, ldw, ldy, M, N, K, hx, hw, hy, 0, 0.f, 0.f};
+  const dim3 grid((N + 15) / 16, 1, heads), block(kSkWarps * 32);
+  skinny_prefer_l1();
+  const cudaStream_t st = (cudaStream_t)stream;
+  return (int)(M <= 8 ? launch_dependent(skinny_gemm_kernel<1, false>, grid, block, 0, st, a)
+                      : M <= 16 ? launch_dependent(skinny_gemm_kernel<2, false>, grid, block, 0, st, a)
+                                : launch_dependent(skinny_gemm_kernel<4, false>, grid, block, 0, st, a));
 }
 
 // y[M, N] = silu(x wg^T) * (x wu^T): the gate and up projections of a SwiGLU MLP for decode-sized M in one pass over both

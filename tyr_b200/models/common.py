@@ -20,6 +20,7 @@ from ..ops.gemm import gemm as _gemm
 from ..ops import decode_gemm as _decode_gemm
 from ..ops import skinny as _skinny
 from ..ops.attention import attention
+from ..ops.mix_conv import activate
 from ..ops.norm import rms_norm_weighted
 
 TCGEN05_MIN_ROWS = 128
@@ -83,6 +84,18 @@ def swiglu_mlp(x, gate_w, up_w, down_w):
         if _skinny.swiglu_supported(x2, gate_w, up_w):          # decode: gate and up in one pass, SwiGLU in the epilogue
             return lin(_skinny.skinny_swiglu(x2, gate_w, up_w).reshape(*x.shape[:-1], gate_w.shape[0]), down_w)
     return lin(F.silu(lin(x, gate_w)) * lin(x, up_w), down_w)
+
+
+def xielu_mlp(x, up_w, down_w, a: float, b: float):
+    """``down xIELU(up x)``; the activation (factors ``a`` above zero, ``b`` below) is taken in the up product's epilogue where one applies."""
+    rows = x.numel() // x.shape[-1]
+    x2 = x.reshape(rows, -1)
+    if x.is_cuda and not torch.is_grad_enabled():
+        if (rows >= TCGEN05_MIN_ROWS and x.dtype == up_w.dtype == torch.bfloat16 and up_w.shape[0] % 8 == 0 and up_w.shape[1] % 8 == 0 and up_w.is_contiguous()):
+            return lin(_gemm(x2.contiguous(), up_w, act="xielu", alpha=a, beta=b).reshape(*x.shape[:-1], -1), down_w)
+        if _skinny.supported(x2, up_w):
+            return lin(_skinny.skinny_xielu(x2, up_w, a, b).reshape(*x.shape[:-1], -1), down_w)
+    return lin(activate(lin(x, up_w), "xielu", (a, b)), down_w)
 
 
 def norm_w(x, w, eps, one_plus_w: bool = False, residual=None, return_residual: bool = False):

@@ -24,7 +24,7 @@ MAX_HEAD = 256
 @register_signatures
 def _sigs(lib_):
     P, I, L, F = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong, ctypes.c_float
-    for name, args in (("tyr_qk_norm_store", [P, L] + [P] * 9 + [I] * 10 + [F, I, P]),
+    for name, args in (("tyr_qk_norm_store", [P, L] + [P] * 10 + [I] * 10 + [F, I, P]),
                        ("tyr_general_attention", [P] * 7 + [ctypes.POINTER(L)] + [I] * 10 + [F, I, P, P])):
         fn = getattr(lib_, name, None)
         if fn is not None:
@@ -52,21 +52,23 @@ def penalty(r1: torch.Tensor, r2: torch.Tensor, dist: torch.Tensor) -> torch.Ten
     return r1.reshape(shape) * torch.log1p(r2.reshape(shape) * dist.float())
 
 
-def qk_norm_store(y: torch.Tensor, q_w: torch.Tensor, k_w: Optional[torch.Tensor], H: int, G: int, dk: int, dv: int, eps: float, *,
+def qk_norm_store(y: torch.Tensor, q_w: Optional[torch.Tensor], k_w: Optional[torch.Tensor], H: int, G: int, dk: int, dv: int, eps: float, *,
                   dkp: int, dvp: int, store=None, pos: Optional[torch.Tensor] = None, lens: Optional[torch.Tensor] = None,
-                  want_v: bool = True):
-    """y: [B, S, >= (H + G) dk + G dv] rows q | k | v (G = 0: q alone).  Per-head RMSNorm of q and k with the fp32 weights;
+                  want_v: bool = True, bias: Optional[torch.Tensor] = None):
+    """y: [B, S, >= (H + G) dk + G dv] rows q | k | v (G = 0: q alone), to which ``bias`` (fp32, one per column) is
+    added.  Per-head RMSNorm of q and k with the fp32 weights (None: no weight);
     returns (q [B, S, H, dkp], k [B, S, G, dkp], v [B, S, G, dvp]) with zeros in the padded channels.  ``store`` (a ``KVCache``)
     receives k and v of the first ``lens[b]`` tokens of every row at positions ``pos[b]`` + s (a ring store: its last ``cap``)."""
     B, S, _ = y.shape
     F_ = torch.nn.functional
     if not y.is_cuda:
-        norm = lambda t, w: (t.float() * torch.rsqrt(t.float().pow(2).mean(-1, keepdim=True) + eps) * w).to(y.dtype)
+        dt, y = y.dtype, y[..., :(H + G) * dk + G * dv].float() + (0.0 if bias is None else bias)
+        norm = lambda t, w: (t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) * (1.0 if w is None else w)).to(dt)
         q = F_.pad(norm(y[..., :H * dk].reshape(B, S, H, dk), q_w), (0, dkp - dk))
         if G == 0:
             return q, None, None
         k = F_.pad(norm(y[..., H * dk:(H + G) * dk].reshape(B, S, G, dk), k_w), (0, dkp - dk))
-        v = F_.pad(y[..., (H + G) * dk:(H + G) * dk + G * dv].reshape(B, S, G, dv), (0, dvp - dv))
+        v = F_.pad(y[..., (H + G) * dk:(H + G) * dk + G * dv].reshape(B, S, G, dv), (0, dvp - dv)).to(dt)
         if store is not None:
             for b in range(B):
                 n, p0 = S if lens is None else int(lens[b]), 0 if pos is None else int(pos[b])
@@ -78,7 +80,7 @@ def qk_norm_store(y: torch.Tensor, q_w: torch.Tensor, k_w: Optional[torch.Tensor
     q = torch.empty((B, S, H, dkp), dtype=y.dtype, device=y.device)
     k = torch.empty((B, S, G, dkp), dtype=y.dtype, device=y.device) if G else None
     v = torch.empty((B, S, G, dvp), dtype=y.dtype, device=y.device) if G and want_v else None
-    check(lib().tyr_qk_norm_store(ptr(y), row_stride(y), ptr(q_w), ptr(k_w), ptr(q), ptr(k), ptr(v), ptr(store.k) if store is not None else None,
+    check(lib().tyr_qk_norm_store(ptr(y), row_stride(y), ptr(q_w), ptr(k_w), ptr(bias), ptr(q), ptr(k), ptr(v), ptr(store.k) if store is not None else None,
                                   ptr(store.v) if store is not None else None, ptr(pos), ptr(lens), B, S, H, G, dk, dv, dkp, dvp,
                                   store.cap if store is not None else 0, 1 if store is not None and store.ring else 0, eps, _dt(y),
                                   cur_stream(y.device)), "qk_norm_store")

@@ -37,7 +37,7 @@ def _sigs(lib_):
         fn.restype = ctypes.c_int
     fn = getattr(lib_, "tyr_flash_fwd_sink", None)
     if fn is not None:
-        fn.argtypes = [P, P, P, P, P, P, I, I, I, I, I, I, ctypes.POINTER(L), F, F, P, P]
+        fn.argtypes = [P, P, P, P, P, P, I, I, I, I, I, I, ctypes.POINTER(L), I, F, F, P, P]
         fn.restype = ctypes.c_int
     fn = getattr(lib_, "tyr_flash_bwd_workspace_bytes", None)
     if fn is not None:
@@ -182,9 +182,10 @@ def sink_supported(q, k, v, gate, out) -> bool:
     return biased_supported(q, k, v) and hasattr(lib(), "tyr_flash_fwd_sink") and rows(gate) and rows(out)
 
 
-def flash_fwd_sink(q, k, v, *, scale: float, sink=None, gate=None, out_scale: float = 1.0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+def flash_fwd_sink(q, k, v, *, scale: float, sink=None, gate=None, out_scale: float = 1.0, out: Optional[torch.Tensor] = None,
+                   window: Optional[int] = None) -> torch.Tensor:
     """Causal attention of whole prompts with ``exp(sink[h])`` in the softmax denominator and the output multiplied by
-    ``out_scale * sigmoid(gate)``.  q: [B, T, Hq, dk], k: [B, T, Hkv, dk], v: [B, T, Hkv, dv] (views), sink fp32 [Hq], gate
+    ``out_scale * sigmoid(gate)``; ``window`` keys each when given.  q: [B, T, Hq, dk], k: [B, T, Hkv, dk], v: [B, T, Hkv, dv] (views), sink fp32 [Hq], gate
     [B, T, Hq * dv] -> [B, T, Hq * dv]."""
     import ctypes
     B, T, Hq, dk = q.shape
@@ -194,6 +195,6 @@ def flash_fwd_sink(q, k, v, *, scale: float, sink=None, gate=None, out_scale: fl
     o4 = out.unflatten(2, (Hq, dv))
     strides = (ctypes.c_longlong * 15)(*[x for t in (q, k, v, o4) for x in _bthd_strides(t)],
                                        *((0, 0, 0) if gate is None else _bthd_strides(gate.unflatten(2, (Hq, dv)))))
-    check(lib().tyr_flash_fwd_sink(ptr(q), ptr(k), ptr(v), ptr(out), ptr(sink), ptr(gate), B, Hq, Hkv, T, dk, dv, strides, scale, out_scale,
+    check(lib().tyr_flash_fwd_sink(ptr(q), ptr(k), ptr(v), ptr(out), ptr(sink), ptr(gate), B, Hq, Hkv, T, dk, dv, strides, int(window or 0), scale, out_scale,
                                    ptr(err_word(q.device)), cur_stream(q.device)), "flash_fwd_sink")
     return out

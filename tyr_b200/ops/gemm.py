@@ -8,7 +8,8 @@ Operand layouts (no transposes are ever materialised):
 * ``b_layout='K'``  : ``b`` has shape ``[..., N, K]``
 * ``b_layout='MN'`` : ``b`` has shape ``[..., K, N]``
 
-``out = alpha * act(A @ B) + beta * aux`` (``act='relu2_grad'``: ``alpha * (A @ B) * 2*sqrt(aux)``); ``out_dtype`` bf16 or fp32; ``accumulate=True`` adds
+``out = alpha * act(A @ B) + beta * aux`` (``act='relu2_grad'``: ``alpha * (A @ B) * 2*sqrt(aux)``; ``act='xielu'``: xIELU of A @ B with
+factors ``alpha`` above zero and ``beta`` below, no ``aux``); ``out_dtype`` bf16 or fp32; ``accumulate=True`` adds
 into an existing fp32 ``out`` with an even stream-K split (used for weight gradients).
 
 The reference reaches cuBLAS for these products (cc/src/tyr.cpp:1003-1036, 1267-1300) and runs
@@ -24,7 +25,7 @@ import torch
 from .._native import GemmArgs
 from ._common import check, cur_stream, err_word, lib
 
-_ACT = {None: 0, "none": 0, "relu2": 1, "relu": 2, "relu2_grad": 3, "swiglu": 4, "geglu": 5}
+_ACT = {None: 0, "none": 0, "relu2": 1, "relu": 2, "relu2_grad": 3, "swiglu": 4, "geglu": 5, "xielu": 6}
 
 
 def _dims(t, layout, is_a):
@@ -64,6 +65,9 @@ def _reference(a, b, a_layout, b_layout, aux, alpha, beta, act, out_dtype):
     elif act == "relu2_grad":
         # aux holds y = relu(z)^2 of the forward pass: d/dz = 2*relu(z) = 2*sqrt(y)
         return (alpha * acc * 2.0 * torch.sqrt(aux.float().clamp_min(0))).to(out_dtype)
+    elif act == "xielu":
+        low = acc.clamp_max(0.0)
+        return (torch.where(acc > 0, alpha * acc * acc, beta * (torch.expm1(low) - low)) + 0.5 * acc).to(out_dtype)
     acc = alpha * acc
     if aux is not None and beta != 0.0:
         acc = acc + beta * aux.float()

@@ -1,0 +1,134 @@
+"""Causal attention in which all heads of a query are worked on together (csrc/joint_attention.cu):
+
+    s_g(i, j) = softcap tanh(scale temp_g q_g . k_j / softcap) + rel[bucket(i - j), g]
+    score_h   = sum_g talk[h, g] s_g,    0 <= i - j < window
+
+``talking_prompt`` / ``talking_step`` mix the heads' scores before the softmax (``Talk``); ``latent_step`` lets every head read one
+shared row per position whose first channels are its value.  The steps read a ``KVCache`` that already holds the new token.  Plain
+PyTorch computes the same off the GPU."""
+from __future__ import annotations
+
+import ctypes
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+
+from .._native import register_signatures
+from ._common import check, cur_stream, err_word, lib, ptr
+
+
+class _Scores(ctypes.Structure):
+    _fields_ = [("temp", ctypes.c_void_p), ("rel", ctypes.c_void_p), ("bucket", ctypes.c_void_p), ("talk", ctypes.c_void_p),
+                ("reach", ctypes.c_int), ("scale", ctypes.c_float), ("softcap", ctypes.c_float)]
+
+
+@register_signatures
+def _sigs(lib_):
+    P, I, L = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong
+    for name, args in (("tyr_joint_attention", [P, P, P, P, P, ctypes.POINTER(_Scores), ctypes.POINTER(L)] + [I] * 11 + [P, P]),):
+        fn = getattr(lib_, name, None)
+        if fn is not None:
+            fn.argtypes, fn.restype = args, I
+
+
+def distance_buckets(rows: int, reach: int) -> torch.Tensor:
+    """int32 [reach + 1]: the row of a table of ``rows`` for the distances 0 .. reach; every distance from ``reach`` on has the last row.
+    Half of the rows stand for one distance each, the others for logarithmic steps up to ``reach``."""
+    half = rows // 2
+    if half < 1 or reach <= half:
+        raise ValueError(f"a distance table needs at least 2 rows and a reach beyond half of them, got {rows} and {reach}")
+    steps, out, x = rows - half, [], 0
+    for n in range(reach + 1):
+        # floor(steps ln(n / half) / ln(reach / half)), decided in whole numbers: x + 1 is reached when (n / half)^steps >= (reach / half)^(x + 1)
+        while x < steps - 1 and n > half and n ** steps * half ** (x + 1) >= reach ** (x + 1) * half ** steps:
+            x += 1
+        out.append(n if n < half else half + x)
+    return torch.tensor(out, dtype=torch.int32)
+
+
+@dataclass
+class Talk:
+    """What happens to the scores of one layer before the softmax."""
+    temp: torch.Tensor            # fp32 [H]
+    rel: torch.Tensor             # fp32 [rows, H]
+    bucket: torch.Tensor          # int32 [reach + 1]: row of rel for a distance
+    mix: torch.Tensor             # fp32 [H, H]
+    softcap: float
+
+    def scores(self, dots: torch.Tensor, dist: torch.Tensor) -> torch.Tensor:
+        """dots: scaled products [..., H, i, j], dist: [i, j] -> mixed scores."""
+        s = self.softcap * torch.tanh(dots * self.temp[:, None, None] / self.softcap)
+        s = s + self.rel[self.bucket[dist.clamp(0, self.bucket.numel() - 1).long()].long()].permute(2, 0, 1)
+        return torch.einsum("hg,...gij->...hij", self.mix, s)
+
+    def args(self, scale: float) -> _Scores:
+        assert all(t.dtype == torch.float32 and t.is_contiguous() for t in (self.temp, self.rel, self.mix)) and self.bucket.dtype == torch.int32
+        a = _Scores(scale=scale, softcap=self.softcap, reach=self.bucket.numel() - 1)
+        a.temp, a.rel, a.bucket, a.talk = (t.data_ptr() for t in (self.temp, self.rel, self.bucket, self.mix))
+        return a
+
+
+def store_dims(dk: int, dv: int, dtype, device) -> tuple:
+    """Row lengths of the K and V stores (and of the queries and new keys)."""
+    return dk, dv
+
+
+def _kind(t: torch.Tensor) -> int:
+    if t.dtype not in (torch.bfloat16, torch.float32):
+        raise TypeError(f"attention kernels take bf16 or fp32, got {t.dtype}")
+    return 0 if t.dtype == torch.bfloat16 else 1
+
+
+def _general(q, k, v, kv_strides, scores: _Scores, out, pos, G, dk, dv, cap, ring, window, keys):
+    B, S, H, _ = q.shape
+    st = (ctypes.c_longlong * 11)(*q.stride()[:3], *kv_strides, out.stride(1) if S > 1 else out.stride(0), out.stride(2))
+    check(lib().tyr_joint_attention(ptr(q), ptr(k), ptr(v), ptr(out), ptr(pos), ctypes.byref(scores), st, B, S, H, G, dk, dv, cap, 1 if ring else 0,
+                                    int(window or 0), keys, _kind(q), ptr(err_word(q.device)), cur_stream(q.device)), "joint_attention")
+    return out
+
+
+def prompt_attention(q, k, v, *, scale: float, window: Optional[int] = None, talk: Optional[Talk] = None) -> torch.Tensor:
+    """Whole prompts (rows may end earlier: padding at the end only feeds padding).  q: [B, S, H, dk], k: [B, S, G, dk], v: [B, S, G, dv]
+    -> [B, S, H * dv].  ``talk``: mixed scores."""
+    B, S, H, dk = q.shape
+    G, dv = k.shape[2], v.shape[3]
+    if q.is_cuda:
+        out = torch.empty((B, S, H, dv), dtype=q.dtype, device=q.device)
+        scores = _Scores(scale=scale) if talk is None else talk.args(scale)
+        return _general(q, k, v, (*k.stride()[:3], *v.stride()[:3]), scores, out, None, G, dk, dv, S, False, window, S).flatten(2)
+    s = torch.einsum("bighd,bjgd->bghij", q.float().reshape(B, S, G, H // G, dk), k.float()).reshape(B, H, S, S) * scale
+    dist = torch.arange(S)[:, None] - torch.arange(S)[None, :]
+    if talk is not None:
+        s = talk.scores(s, dist)
+    seen = (dist >= 0) if window is None else (dist >= 0) & (dist < window)
+    p = torch.softmax(s.masked_fill(~seen, float("-inf")), -1).reshape(B, G, H // G, S, S)
+    return torch.einsum("bghij,bjgd->bighd", p, v.float()).reshape(B, S, H * dv).to(q.dtype)
+
+
+def step_attention(q, store, pos: torch.Tensor, dv: int, *, scale: float, window: Optional[int] = None, talk: Optional[Talk] = None,
+                   out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """One token per row against a ``KVCache`` (plain or ring) that holds it.  q: [B, 1, H, dk]; pos: int32 [B]; ``dv`` value channels (of
+    a shared store: the first of the keys) -> [B, 1, H, dv], into ``out`` (a view with contiguous channels) if given."""
+    B, _, H, dk = q.shape
+    G, cap = store.k.shape[1], store.cap
+    if out is None:
+        out = torch.empty((B, 1, H, dv), dtype=q.dtype, device=q.device)
+    if q.is_cuda:
+        st = tuple(t.stride(i) for t in (store.k, store.v) for i in (0, 2, 1))
+        scores = _Scores(scale=scale) if talk is None else talk.args(scale)
+        return _general(q, store.k, store.v, st, scores, out, pos, G, dk, dv, cap, store.ring, window, cap)
+    for b in range(B):
+        p = int(pos[b])
+        n = p + 1 if window is None else min(p + 1, window)
+        if store.ring:
+            n = min(n, cap)
+        at = torch.arange(p + 1 - n, p + 1)
+        slots = at % cap if store.ring else at
+        k, v = store.k[b][:, slots, :dk].float(), store.v[b][:, slots, :dv].float()
+        s = torch.einsum("ghd,gjd->ghj", q[b, 0].float().reshape(G, H // G, dk), k).reshape(H, 1, n) * scale
+        if talk is not None:
+            s = talk.scores(s, (p - at)[None])
+        w = torch.softmax(s[:, 0], -1).reshape(G, H // G, n)
+        out[b, 0] = torch.einsum("ghj,gjd->ghd", w, v).reshape(H, dv).to(q.dtype)
+    return out

@@ -13,14 +13,14 @@ from .._native import register_signatures
 from ._common import check, cur_stream, lib
 
 MAX_SEGMENTS = 6
-_ACT = {None: 0, "silu": 1, "relu2": 2}
+_ACT = {None: 0, "silu": 1, "relu2": 2, "xielu": 3}
 
 
 class _Seg(ctypes.Structure):
     _fields_ = [("col", ctypes.c_int), ("heads", ctypes.c_int), ("d_in", ctypes.c_int), ("d_out", ctypes.c_int), ("taps", ctypes.c_int),
                 ("act", ctypes.c_int), ("w", ctypes.c_void_p), ("bias", ctypes.c_void_p), ("window", ctypes.c_void_p), ("out", ctypes.c_void_p),
                 ("out_ld", ctypes.c_longlong), ("store", ctypes.c_void_p), ("cap", ctypes.c_int), ("store_d", ctypes.c_int),
-                ("temp_coef", ctypes.c_float), ("temp_every", ctypes.c_float)]
+                ("temp_coef", ctypes.c_float), ("temp_every", ctypes.c_float), ("act_a", ctypes.c_float), ("act_b", ctypes.c_float)]
 
 
 class _Args(ctypes.Structure):
@@ -42,7 +42,8 @@ class Segment:
     """Columns [col, col + heads * d) of the projection -> ``out`` [B, S, heads * d_out] (evenly spaced rows, contiguous channels; the
     channels of a head past d are zero).  ``w`` fp32 [heads * d, taps] and ``bias`` fp32: causal convolution whose last ``taps`` inputs
     are the ``window`` [B, heads * d, taps].  ``temp`` (coef, every): the result is multiplied by
-    1 + coef ln(floor((p + 1) / every) + 1) at position p.  ``store`` [B, heads, cap, d_store] receives whole prompts by position."""
+    1 + coef ln(floor((p + 1) / every) + 1) at position p.  ``act`` "silu", "relu2" or "xielu" (``act_args`` (a, b): a z^2 + z / 2 above
+    zero, b (e^z - 1 - z) + z / 2 below).  ``store`` [B, heads, cap, d_store] receives whole prompts by position."""
     col: int
     heads: int
     d: int
@@ -54,6 +55,13 @@ class Segment:
     act: Optional[str] = None
     temp: Optional[tuple] = None
     store: Optional[torch.Tensor] = None
+    act_args: tuple = (0.0, 0.0)
+
+
+def xielu(z: torch.Tensor, a: float, b: float) -> torch.Tensor:
+    """a z^2 + z / 2 above zero, b (e^z - 1 - z) + z / 2 below."""
+    low = z.clamp_max(0.0)
+    return torch.where(z > 0, a * z * z, b * (torch.expm1(low) - low)) + 0.5 * z
 
 
 def temperature(p: torch.Tensor, coef: float, every: float) -> torch.Tensor:
@@ -86,6 +94,8 @@ def _plain(x, segments, lens, pos, step):
             y = torch.nn.functional.silu(y)
         elif s.act == "relu2":
             y = torch.relu(y).square()
+        elif s.act == "xielu":
+            y = xielu(y, *s.act_args)
         if s.temp is not None:
             p = pos[:, None] if step else torch.arange(S)[None]
             y = y * temperature(p, *s.temp)[:, :, None]
@@ -121,6 +131,7 @@ def _run(x, segments: Sequence[Segment], lens, pos, step: bool):
             r.store, r.cap, r.store_d = s.store.data_ptr(), s.store.shape[2], s.store.shape[3]
         if s.temp is not None:
             r.temp_coef, r.temp_every = s.temp
+        r.act_a, r.act_b = s.act_args
     check(lib().tyr_mix_conv(ctypes.byref(a), 1 if step else 0, 1 if x.dtype == torch.float32 else 0, cur_stream(x.device)), "mix_conv")
 
 
@@ -132,3 +143,11 @@ def mix_prompt(x: torch.Tensor, segments: Sequence[Segment], lens: Optional[torc
 def mix_step(x: torch.Tensor, segments: Sequence[Segment], pos: torch.Tensor) -> None:
     """x: [B, 1, columns]; ``pos`` int32 [B] positions of the new tokens."""
     _run(x, segments, None, pos, True)
+
+
+def activate(x: torch.Tensor, act: str, act_args: tuple = (0.0, 0.0)) -> torch.Tensor:
+    """An activation alone, of contiguous rows [..., C]."""
+    flat = x.view(1, -1, x.shape[-1])
+    y = torch.empty_like(flat)
+    mix_prompt(flat, [Segment(0, 1, x.shape[-1], y, act=act, act_args=act_args)])
+    return y.view(x.shape)

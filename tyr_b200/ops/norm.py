@@ -14,7 +14,7 @@ from typing import Optional, Sequence
 import torch
 
 from .._native import register_signatures
-from ._common import check, cur_stream, lib, ptr
+from ._common import check, cur_stream, lib, ptr, row_stride
 
 
 @register_signatures
@@ -27,6 +27,10 @@ def _sigs(lib_):
     fn = getattr(lib_, "tyr_add_norm", None)
     if fn is not None:
         fn.argtypes = [P, L, P, P, L, P, L, I, F, I, I, P]
+        fn.restype = I
+    fn = getattr(lib_, "tyr_sandwich_norm", None)
+    if fn is not None:
+        fn.argtypes = [P, L, P, P, P, P, P, L, L, I, I, F, I, I, P]
         fn.restype = I
 
 EPS = 1e-6
@@ -190,4 +194,30 @@ def add_norm(x: Optional[torch.Tensor], gain: torch.Tensor, eps: float, resid: t
     y = torch.empty(resid.shape, dtype=out_dtype, device=resid.device)
     check(lib().tyr_add_norm(ptr(x2), 0 if x2 is None else x2.stride(0), ptr(gain), ptr(r), r.stride(0), ptr(y), r.shape[0], D, eps,
                              kinds[out_dtype if x2 is None else x2.dtype], kinds[out_dtype], cur_stream(resid.device)), "add_norm")
+    return y
+
+
+def sandwich_norm(x: torch.Tensor, post: Optional[torch.Tensor], gain: Optional[torch.Tensor], eps: float, resid: torch.Tensor, out_dtype: torch.dtype, *,
+                  bias: Optional[torch.Tensor] = None, replace: bool = False, out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """A sublayer between two norms, in one launch with the norm of the next one: ``resid += norm(x + bias) * post`` IN PLACE on an fp32
+    stream [B, S, D] (``x + bias`` itself without ``post``; ``replace``: the stream becomes it), then ``norm(resid) * gain`` (the stream
+    itself without ``gain``) in ``out_dtype`` or into ``out``, a view with evenly spaced rows."""
+    D = resid.shape[-1]
+    if not resid.is_cuda:
+        t = x.float() if bias is None else x.float() + bias
+        if post is not None:
+            t = rms_norm_ref(t, eps) * post
+        if replace:
+            resid.copy_(t)
+        else:
+            resid += t
+        y = resid if gain is None else rms_norm_ref(resid, eps) * gain
+        return y.to(out_dtype) if out is None else out.copy_(y)
+    kinds = {torch.bfloat16: 0, torch.float32: 1}
+    assert resid.dtype == torch.float32 and resid.is_contiguous() and x.shape == resid.shape
+    assert all(t is None or (t.dtype == torch.float32 and t.shape == (D,) and t.is_contiguous()) for t in (bias, post, gain))
+    y = torch.empty(resid.shape, dtype=out_dtype, device=resid.device) if out is None else out
+    assert y.dtype == out_dtype and y.shape == resid.shape
+    check(lib().tyr_sandwich_norm(ptr(x), row_stride(x), ptr(bias), ptr(post), ptr(gain), ptr(resid), ptr(y), row_stride(y), resid.numel() // D, D,
+                                  1 if replace else 0, eps, kinds[x.dtype], kinds[out_dtype], cur_stream(resid.device)), "sandwich_norm")
     return y

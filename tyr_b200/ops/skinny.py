@@ -32,6 +32,12 @@ def _sigs(lib_):
         fn.restype = I
         lib_.tyr_skinny_gemm_splits.argtypes = [I, I]
         lib_.tyr_skinny_gemm_splits.restype = I
+    F = ctypes.c_float
+    for name, args in (("tyr_skinny_gemm_act_bf16", [P, P, P, P, P, L, L, L, I, I, I, I, F, F, P]),
+                       ("tyr_skinny_heads_bf16", [P, P, P, L, L, L, L, L, L, I, I, I, I, P])):
+        fn = getattr(lib_, name, None)
+        if fn is not None:
+            fn.argtypes, fn.restype = args, I
     fn = getattr(lib_, "tyr_skinny_swiglu_bf16", None)
     if fn is not None:
         fn.argtypes = [P, P, P, P, L, L, L, I, I, I, P]
@@ -88,3 +94,35 @@ def skinny_swiglu(x2: torch.Tensor, gate_w: torch.Tensor, up_w: torch.Tensor) ->
     check(lib().tyr_skinny_swiglu_bf16(ptr(x2), ptr(gate_w), ptr(up_w), ptr(y), x2.stride(0), gate_w.stride(0), N, M, N, K, cur_stream(x2.device)),
           "skinny_swiglu")
     return y
+
+
+def skinny_xielu(x2: torch.Tensor, w: torch.Tensor, a: float, b: float) -> torch.Tensor:
+    """x2: [M <= 32, K] bf16 -> xIELU of ``x2 w^T`` (factors ``a`` above zero, ``b`` below) as [M, N] bf16, in the product's epilogue."""
+    M, K = x2.shape
+    N = w.shape[0]
+    y = torch.empty((M, N), dtype=torch.bfloat16, device=x2.device)
+    ws = _workspace(x2.device, M, N) if lib().tyr_skinny_gemm_splits(N, K) > 1 else None
+    check(lib().tyr_skinny_gemm_act_bf16(ptr(x2), ptr(w), None, ptr(y), ptr(ws), x2.stride(0), w.stride(0), N, M, N, K, 6, a, b, cur_stream(x2.device)),
+          "skinny_xielu")
+    return y
+
+
+def head_products_supported(x: torch.Tensor, w: torch.Tensor) -> bool:
+    return (x.is_cuda and x.dtype == w.dtype == torch.bfloat16 and w.shape[2] % 32 == 0 and x.stride(2) == w.stride(2) == 1
+            and all(s % 8 == 0 for s in (*x.stride()[:2], *w.stride()[:2])) and x.data_ptr() % 16 == w.data_ptr() % 16 == 0)
+
+
+def head_products(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """A matrix of its own for each head: out[m, h, :N] = x[m, h, :K] w[h]^T.  x: [M, H, >= K] and out: [M, H, >= N] (views with contiguous
+    channels), w: [H, N, K].  Channels of x past K and of out past N are left alone."""
+    M, H = x.shape[:2]
+    _, N, K = w.shape
+    if not head_products_supported(x, w):
+        out[..., :N] = torch.einsum("mhk,hnk->mhn", x[..., :K], w) if x.is_cuda else torch.einsum("mhk,hnk->mhn", x[..., :K].float(), w.float()).to(out.dtype)
+        return out
+    assert x.shape[2] >= K and out.shape[:2] == (M, H) and out.shape[2] >= N and out.stride(2) == 1 and out.dtype == x.dtype
+    for m in range(0, M, MAX_ROWS):
+        n = min(MAX_ROWS, M - m)
+        check(lib().tyr_skinny_heads_bf16(ptr(x[m:]), ptr(w), ptr(out[m:]), x.stride(0), x.stride(1), w.stride(0), w.stride(1), out.stride(0), out.stride(1),
+                                          H, n, N, K, cur_stream(x.device)), "skinny_heads")
+    return out
