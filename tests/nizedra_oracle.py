@@ -120,10 +120,11 @@ def talking_scores(q, k, mix, temp, rel, talk, i):
     return talk @ (s + rel[rows].T)
 
 
-def talking_attention(q, k, v, mix, temp, rel, talk):
+def talking_attention(q, k, v, mix, temp, rel, talk, first=0):
+    """Rows before query ``first`` stay zero."""
     out = torch.zeros(q.shape[0], q.shape[1], v.shape[2], dtype=v.dtype)
     of = torch.arange(q.shape[1]) // (q.shape[1] // k.shape[1])
-    for i in range(q.shape[0]):
+    for i in range(first, q.shape[0]):
         s = talking_scores(q, k, mix, temp, rel, talk, i)
         e = torch.exp(s - s.max(-1, keepdim=True).values)
         out[i] = torch.einsum("hj,jhd->hd", e / e.sum(-1, keepdim=True), v[:i + 1][:, of])
