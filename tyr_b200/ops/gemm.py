@@ -25,7 +25,7 @@ import torch
 from .._native import GemmArgs
 from ._common import check, cur_stream, err_word, lib
 
-_ACT = {None: 0, "none": 0, "relu2": 1, "relu": 2, "relu2_grad": 3, "swiglu": 4, "geglu": 5, "xielu": 6}
+_ACT = {None: 0, "none": 0, "relu2": 1, "relu": 2, "relu2_grad": 3, "swiglu": 4, "geglu": 5, "xielu": 6, "silu": 7}
 
 
 def _dims(t, layout, is_a):
@@ -65,6 +65,8 @@ def _reference(a, b, a_layout, b_layout, aux, alpha, beta, act, out_dtype):
     elif act == "relu2_grad":
         # aux holds y = relu(z)^2 of the forward pass: d/dz = 2*relu(z) = 2*sqrt(y)
         return (alpha * acc * 2.0 * torch.sqrt(aux.float().clamp_min(0))).to(out_dtype)
+    elif act == "silu":
+        acc = torch.nn.functional.silu(acc)
     elif act == "xielu":
         low = acc.clamp_max(0.0)
         return (torch.where(acc > 0, alpha * acc * acc, beta * (torch.expm1(low) - low)) + 0.5 * acc).to(out_dtype)
