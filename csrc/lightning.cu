@@ -9,7 +9,7 @@
 //
 // The decay comes as a double: fp32 carries it as a sum of two numbers, because a rounding of it would be applied anew at every token
 // of a long memory.  Compiled without fast math.
-#include "common.cuh"
+#include "mma_sync.cuh"
 
 namespace tyr {
 
@@ -92,20 +92,6 @@ struct __align__(16) ChunkSmem {
   float pw[LC_C + 4];                                      // powers of the decay, 0 .. LC_C
 };
 
-__device__ __forceinline__ void lc_cp16(void* dst, const void* src, bool live) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(live ? 16 : 0) : "memory");
-}
-__device__ __forceinline__ void lc_ldsm(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)) : "memory");
-}
-__device__ __forceinline__ void lc_ldsm_t(uint32_t (&r)[4], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)) : "memory");
-}
-__device__ __forceinline__ void lc_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
 // x and y as sums of three bf16 numbers each, packed in pairs
 __device__ __forceinline__ void lc_split(float x, float y, uint32_t (&r)[3]) {
 #pragma unroll
@@ -139,25 +125,25 @@ __global__ void __launch_bounds__(256, 1) lightning_chunk_kernel(LightningArgs a
       const int st = c & 1, t0 = c * LC_C, kc = a.dk / 8, vc = cols / 8;
       for (int x = tid; x < LC_C * kc; x += 256) {
         const int r = x / kc, d = (x - r * kc) * 8, tok = min(t0 + r, n - 1);
-        lc_cp16(&sm.q[st][r * LC_LDK + d], qp + tok * a.q_ss + d, t0 + r < n);
-        lc_cp16(&sm.k[st][r * LC_LDK + d], kp + tok * a.k_ss + d, t0 + r < n);
+        cp16_zfill(&sm.q[st][r * LC_LDK + d], qp + tok * a.q_ss + d, t0 + r < n);
+        cp16_zfill(&sm.k[st][r * LC_LDK + d], kp + tok * a.k_ss + d, t0 + r < n);
       }
       for (int x = tid; x < LC_C * vc; x += 256) {
         const int r = x / vc, d = (x - r * vc) * 8, tok = min(t0 + r, n - 1);
-        lc_cp16(&sm.v[st][r * LC_LDV + d], vp + tok * a.v_ss + d, t0 + r < n);
+        cp16_zfill(&sm.v[st][r * LC_LDV + d], vp + tok * a.v_ss + d, t0 + r < n);
       }
     }
-    asm volatile("cp.async.commit_group;" ::: "memory");
+    cp_commit();
   };
   fetch(0);
   float S[8][4];
 #pragma unroll
   for (int i = 0; i < 8; ++i) S[i][0] = S[i][1] = S[i][2] = S[i][3] = 0.f;
-  // addresses a lane gives ldmatrix: row lane % 16 (+ 8 columns for the upper half), and for the plain form of a B operand its rows by n
+  // a lane's row and column for ldmatrix (csrc/mma_sync.cuh)
   const int lr = lane & 15, lc = (lane >> 4) * 8, br = (lane & 7) + ((lane >> 4) << 3), bc = ((lane >> 3) & 1) * 8;
   const int m0 = (warp >> 1) * 16, n0 = (warp & 1) * 32;
   for (int c = 0; c < chunks; ++c) {
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    cp_wait<0>();
     __syncthreads();                                       // this chunk's rows and the state's mirror are there, the other stage is free
     fetch(c + 1);
     const int st = c & 1, m = min(LC_C, n - c * LC_C);
@@ -180,14 +166,14 @@ __global__ void __launch_bounds__(256, 1) lightning_chunk_kernel(LightningArgs a
 #pragma unroll 2
     for (int x = 0; x < ks; ++x) {
       uint32_t qa[4];
-      lc_ldsm(qa, q + (m0 + lr) * LC_LDK + x * 16 + lc);
+      ldsm4(qa, q + (m0 + lr) * LC_LDK + x * 16 + lc);
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         if (16 * j > m0) break;                            // later keys are not seen
         uint32_t kb[4];
-        lc_ldsm(kb, k + (16 * j + br) * LC_LDK + x * 16 + bc);
-        lc_mma(p[2 * j], qa, kb[0], kb[1]);
-        lc_mma(p[2 * j + 1], qa, kb[2], kb[3]);
+        ldsm4(kb, k + (16 * j + br) * LC_LDK + x * 16 + bc);
+        mma_bf16(p[2 * j], qa, kb[0], kb[1]);
+        mma_bf16(p[2 * j + 1], qa, kb[2], kb[3]);
       }
       if (c > 0) {
 #pragma unroll
@@ -195,9 +181,9 @@ __global__ void __launch_bounds__(256, 1) lightning_chunk_kernel(LightningArgs a
 #pragma unroll
           for (int j = 0; j < 2; ++j) {
             uint32_t sb[4];
-            lc_ldsm_t(sb, &sm.s[i][(x * 16 + lr) * LC_LDV + n0 + 16 * j + lc]);
-            lc_mma(o[2 * j], qa, sb[0], sb[1]);
-            lc_mma(o[2 * j + 1], qa, sb[2], sb[3]);
+            ldsm4_t(sb, &sm.s[i][(x * 16 + lr) * LC_LDV + n0 + 16 * j + lc]);
+            mma_bf16(o[2 * j], qa, sb[0], sb[1]);
+            mma_bf16(o[2 * j + 1], qa, sb[2], sb[3]);
           }
       }
     }
@@ -223,11 +209,11 @@ __global__ void __launch_bounds__(256, 1) lightning_chunk_kernel(LightningArgs a
 #pragma unroll
       for (int u = 0; u < 2; ++u) {
         uint32_t vb[4];
-        lc_ldsm_t(vb, v + (16 * j + lr) * LC_LDV + n0 + 16 * u + lc);
+        ldsm4_t(vb, v + (16 * j + lr) * LC_LDV + n0 + 16 * u + lc);
 #pragma unroll
         for (int i = 0; i < 3; ++i) {
-          lc_mma(o[2 * u], pa[i], vb[0], vb[1]);
-          lc_mma(o[2 * u + 1], pa[i], vb[2], vb[3]);
+          mma_bf16(o[2 * u], pa[i], vb[0], vb[1]);
+          mma_bf16(o[2 * u + 1], pa[i], vb[2], vb[3]);
         }
       }
     }
@@ -250,16 +236,16 @@ __global__ void __launch_bounds__(256, 1) lightning_chunk_kernel(LightningArgs a
 #pragma unroll 1
       for (int x = 0; x < LC_C / 16; ++x) {
         uint32_t kt[4], ka[4];
-        lc_ldsm_t(kt, k + (x * 16 + lr) * LC_LDK + warp * 16 + lc);      // 16 tokens x 16 channels, transposed: channels are the rows of A
+        ldsm4_t(kt, k + (x * 16 + lr) * LC_LDK + warp * 16 + lc);      // 16 tokens x 16 channels, transposed: channels are the rows of A
         ka[0] = kt[0]; ka[1] = kt[2]; ka[2] = kt[1]; ka[3] = kt[3];
 #pragma unroll
         for (int i = 0; i < 3; ++i)
 #pragma unroll
           for (int j = 0; j < 4; ++j) {
             uint32_t vb[4];
-            lc_ldsm_t(vb, &sm.dv[i][(x * 16 + lr) * LC_LDV + 16 * j + lc]);
-            lc_mma(S[2 * j], ka, vb[0], vb[1]);
-            lc_mma(S[2 * j + 1], ka, vb[2], vb[3]);
+            ldsm4_t(vb, &sm.dv[i][(x * 16 + lr) * LC_LDV + 16 * j + lc]);
+            mma_bf16(S[2 * j], ka, vb[0], vb[1]);
+            mma_bf16(S[2 * j + 1], ka, vb[2], vb[3]);
           }
       }
 #pragma unroll
@@ -273,7 +259,7 @@ __global__ void __launch_bounds__(256, 1) lightning_chunk_kernel(LightningArgs a
         }
     }
   }
-  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  cp_wait<0>();
   const int done = min(a.S, chunks * LC_C);                // rows a chunk wrote; the padding after them is zero
   for (long long x = tid; x < static_cast<long long>(a.S - done) * cols; x += 256) op[(done + x / cols) * a.H * a.dv + x % cols] = 0.f;
   if (warp < ks) {

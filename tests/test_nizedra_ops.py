@@ -146,8 +146,9 @@ def test_talking_heads_over_prompts(place, case):
     want = O.talking_attention(q, k, v, mix, temp, rel, talk).flatten(1)
     # two rows: the whole prompt, and one that ends early (its padding is noise)
     pad = lambda t: torch.cat([t[:T // 2], torch.randn(T - T // 2, *t.shape[1:]).bfloat16().double()])
-    batch = lambda t: torch.stack([t, pad(t)]).to(dev, dt)
-    got = ja.prompt_attention(batch(q), batch(k), batch(v), scale=mix["scale"], talk=talk_of(mix, temp, rel, talk, dev))
+    dkp, dvp = ja.store_dims(case[3], case[4], dt, dev)
+    batch = lambda t, d: torch.nn.functional.pad(torch.stack([t, pad(t)]), (0, d - t.shape[2])).to(dev, dt)
+    got = ja.prompt_attention(batch(q, dkp), batch(k, dkp), batch(v, dvp)[..., :case[4]], scale=mix["scale"], talk=talk_of(mix, temp, rel, talk, dev))
     near(got[0], want, dt)
     near(got[1, :T // 2], want[:T // 2], dt)
 

@@ -20,16 +20,22 @@ from ._common import check, cur_stream, err_word, lib, ptr
 
 class _Scores(ctypes.Structure):
     _fields_ = [("temp", ctypes.c_void_p), ("rel", ctypes.c_void_p), ("bucket", ctypes.c_void_p), ("talk", ctypes.c_void_p),
-                ("reach", ctypes.c_int), ("scale", ctypes.c_float), ("softcap", ctypes.c_float)]
+                ("reach", ctypes.c_int), ("rows", ctypes.c_int), ("talk_exact", ctypes.c_int), ("scale", ctypes.c_float), ("softcap", ctypes.c_float)]
 
 
 @register_signatures
 def _sigs(lib_):
     P, I, L = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong
-    for name, args in (("tyr_joint_attention", [P, P, P, P, P, ctypes.POINTER(_Scores), ctypes.POINTER(L)] + [I] * 11 + [P, P]),):
+    S, LL = ctypes.POINTER(_Scores), ctypes.POINTER(L)
+    for name, args in (("tyr_joint_attention", [P, P, P, P, P, S, LL] + [I] * 11 + [P, P]), ("tyr_joint_prompt_form", [I] * 6),
+                       ("tyr_joint_prompt", [P, P, P, P, S, LL] + [I] * 7 + [P]), ("tyr_joint_step_heads", [I] * 8),
+                       ("tyr_joint_step", [P, P, P, P, P, S, P, LL] + [I] * 10 + [P, P])):
         fn = getattr(lib_, name, None)
         if fn is not None:
             fn.argtypes, fn.restype = args, I
+    fn = getattr(lib_, "tyr_joint_step_workspace_bytes", None)
+    if fn is not None:
+        fn.argtypes, fn.restype = [I, I, I, I], L
 
 
 def distance_buckets(rows: int, reach: int) -> torch.Tensor:
@@ -56,6 +62,9 @@ class Talk:
     mix: torch.Tensor             # fp32 [H, H]
     softcap: float
 
+    def __post_init__(self):
+        self.exact = bool((self.mix.bfloat16().float() == self.mix).all())     # entries that TF32 holds as they are
+
     def scores(self, dots: torch.Tensor, dist: torch.Tensor) -> torch.Tensor:
         """dots: scaled products [..., H, i, j], dist: [i, j] -> mixed scores."""
         s = self.softcap * torch.tanh(dots * self.temp[:, None, None] / self.softcap)
@@ -64,14 +73,46 @@ class Talk:
 
     def args(self, scale: float) -> _Scores:
         assert all(t.dtype == torch.float32 and t.is_contiguous() for t in (self.temp, self.rel, self.mix)) and self.bucket.dtype == torch.int32
-        a = _Scores(scale=scale, softcap=self.softcap, reach=self.bucket.numel() - 1)
+        a = _Scores(scale=scale, softcap=self.softcap, reach=self.bucket.numel() - 1, rows=self.rel.shape[0], talk_exact=1 if self.exact else 0)
         a.temp, a.rel, a.bucket, a.talk = (t.data_ptr() for t in (self.temp, self.rel, self.bucket, self.mix))
         return a
 
 
 def store_dims(dk: int, dv: int, dtype, device) -> tuple:
-    """Row lengths of the K and V stores (and of the queries and new keys)."""
-    return dk, dv
+    """Row lengths of the K and V stores (and of the queries and new keys): multiples of 16 for the tensor-core forms, else the sizes
+    themselves."""
+    if torch.device(device).type != "cuda" or dtype != torch.bfloat16:
+        return dk, dv
+    return -(-dk // 16) * 16, -(-dv // 16) * 16
+
+
+_workspaces: dict = {}
+
+
+def _prompt_fused(q, k, v, talk: Talk) -> bool:
+    """The tensor-core form takes these prompts: bf16, heads of a token adjacent in rows that are multiples of 16."""
+    if q.dtype != torch.bfloat16 or not q.dtype == k.dtype == v.dtype:
+        return False
+    H, G, dk, dvp = q.shape[2], k.shape[2], q.shape[3], v.stride(2)
+    ok = lambda t, d: t.stride(3) == 1 and t.stride(2) == d and t.stride(0) % 8 == 0 and t.stride(1) % 8 == 0 and t.data_ptr() % 16 == 0
+    return (ok(q, dk) and ok(k, dk) and ok(v, dvp) and dvp >= v.shape[3] and v.stride(1) >= G * dvp
+            and lib().tyr_joint_prompt_form(H, G, dk, dvp, talk.rel.shape[0], talk.bucket.numel() - 1) != 0)
+
+
+def pick_splits(B: int, blocks: int, keys: int) -> int:
+    """Slices of the keys for one (row, block of heads): one CTA fills an SM, and a slice should outweigh its part of the merge."""
+    return max(1, min(148 // (B * blocks), -(-keys // 128), 32))
+
+
+def _step_heads(q, store, dv: int, talk: Optional[Talk]) -> int:
+    """Heads of a CTA of the tensor-core step, 0 where it does not apply."""
+    if q.dtype != torch.bfloat16 or store.k.dtype != q.dtype or q.shape[3] != store.k.shape[3] or q.stride(3) != 1:
+        return 0
+    shared = store.v is store.k
+    if shared != (talk is None) or any(s % 8 for s in (q.stride(0), q.stride(2))) or q.data_ptr() % 16:
+        return 0
+    return lib().tyr_joint_step_heads(0 if talk is None else 1, q.shape[2], store.k.shape[1], q.shape[3], dv, store.v.shape[3], 1 if shared else 0,
+                                      0 if talk is None else talk.rel.shape[0])
 
 
 def _kind(t: torch.Tensor) -> int:
@@ -96,6 +137,11 @@ def prompt_attention(q, k, v, *, scale: float, window: Optional[int] = None, tal
     if q.is_cuda:
         out = torch.empty((B, S, H, dv), dtype=q.dtype, device=q.device)
         scores = _Scores(scale=scale) if talk is None else talk.args(scale)
+        if talk is not None and window is None and _prompt_fused(q, k, v, talk):
+            st = (ctypes.c_longlong * 6)(*[t.stride(i) for t in (q, k, v) for i in range(2)])
+            check(lib().tyr_joint_prompt(ptr(q), ptr(k), ptr(v), ptr(out), ctypes.byref(scores), st, B, S, H, G, dk, dv, v.stride(2), cur_stream(q.device)),
+                  "joint_prompt")
+            return out.flatten(2)
         return _general(q, k, v, (*k.stride()[:3], *v.stride()[:3]), scores, out, None, G, dk, dv, S, False, window, S).flatten(2)
     s = torch.einsum("bighd,bjgd->bghij", q.float().reshape(B, S, G, H // G, dk), k.float()).reshape(B, H, S, S) * scale
     dist = torch.arange(S)[:, None] - torch.arange(S)[None, :]
@@ -117,6 +163,18 @@ def step_attention(q, store, pos: torch.Tensor, dv: int, *, scale: float, window
     if q.is_cuda:
         st = tuple(t.stride(i) for t in (store.k, store.v) for i in (0, 2, 1))
         scores = _Scores(scale=scale) if talk is None else talk.args(scale)
+        hb = _step_heads(q, store, dv, talk)
+        if hb:
+            splits = pick_splits(B, -(-H // hb), min(cap, window) if window else cap)
+            key = (q.device.index, B, H, dv, splits)
+            ws = _workspaces.get(key)
+            if ws is None and splits > 1:
+                ws = _workspaces[key] = torch.zeros(lib().tyr_joint_step_workspace_bytes(B, H, dv, splits) // 4, dtype=torch.int32, device=q.device)
+            so = (ctypes.c_longlong * 4)(q.stride(0), q.stride(2), out.stride(0), out.stride(2))
+            check(lib().tyr_joint_step(ptr(q), ptr(store.k), None if talk is None else ptr(store.v), ptr(out), ptr(pos), ctypes.byref(scores), ptr(ws), so, B, H, G,
+                                       dk, dv, store.v.shape[3], cap, 1 if store.ring else 0, int(window or 0), splits, ptr(err_word(q.device)),
+                                       cur_stream(q.device)), "joint_step")
+            return out
         return _general(q, store.k, store.v, st, scores, out, pos, G, dk, dv, cap, store.ring, window, cap)
     for b in range(B):
         p = int(pos[b])
