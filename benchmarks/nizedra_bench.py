@@ -145,6 +145,8 @@ def kernels(only: str = "", warmup: int = 3, steps: int = 20, device="cuda") -> 
                    f"{r['new'] / floor / (r['like'] / r['like_floor']):.2f}"
         print(txt, flush=True)
 
+    bound = 130.0                    # of unit queries and keys
+
     def talk(H):
         return ja.Talk(torch.ones(H, device=device), f32(ROWS, H) * 0.1, ja.distance_buckets(ROWS, REACH).to(device),
                        (torch.eye(H, device=device) + 0.1 * f32(H, H)).bfloat16().float(), 50.0)
@@ -154,7 +156,7 @@ def kernels(only: str = "", warmup: int = 3, steps: int = 20, device="cuda") -> 
         q, k, v, tk = mk(B, S, H, d), mk(B, S, G, d), mk(B, S, G, d), talk(H)
         q1, k1, v1 = mk(B, S, H, 128), mk(B, S, G, 128), mk(B, S, G, 128)
         pairs = B * S * (S + 1) / 2
-        case(f"talking prompt {B}x{S}, {H}/{G} heads of {d}", lambda: ja.prompt_attention(q, k, v, scale=0.09, talk=tk),
+        case(f"talking prompt {B}x{S}, {H}/{G} heads of {d}", lambda: ja.prompt_attention(q, k, v, scale=0.09, talk=tk, dot_bound=bound),
              max(tf(pairs * H * (4 * d + 2 * 2 * 2 * H)), sfu(pairs * H * 3)), lambda: flash.flash_fwd_bthd(q1, k1, v1, causal=True, window=None, scale=0.09, need_lse=False),
              max(tf(pairs * H * 4 * 128), sfu(pairs * H)))
     # mixed heads, one token per row / split-KV kernel
@@ -162,7 +164,7 @@ def kernels(only: str = "", warmup: int = 3, steps: int = 20, device="cuda") -> 
         q, kn, vn = mk(B, 1, H, 128), mk(B, 1, G, 128), mk(B, 1, G, 128)
         kc, vc, pos, tk = mk(B, G, n + 8, 128), mk(B, G, n + 8, 128), torch.full((B,), n, dtype=torch.int32, device=device), talk(H)
         st = KVCache(kc, vc)
-        case(f"talking step batch {B}, {H}/{G} heads, {n} keys", lambda: ja.step_attention(q, st, pos, 128, scale=0.09, talk=tk), gb(B * G * n * 128 * 4),
+        case(f"talking step batch {B}, {H}/{G} heads, {n} keys", lambda: ja.step_attention(q, st, pos, 128, scale=0.09, talk=tk, dot_bound=bound), gb(B * G * n * 128 * 4),
              lambda: da.decode_attention(q[:, 0], kn[:, 0], vn[:, 0], kc, vc, pos[:1], scale=0.09))
     # latent attention over prompts: windowed flash kernel with its head sizes / heads of 128, the same window
     for B, S, H, dk, dv in ((4, 2048, 32, 96, 64), (4, 2048, 32, 128, 128), (1, 8192, 32, 96, 64)):

@@ -1,0 +1,701 @@
+// Attention over all heads of a query at once (see csrc/joint_attention.cu) for sm_100a on tcgen05 / TMEM / TMA, with the keys on the
+// 128-row side of the tensor core:
+//
+//   S^T[128 keys x columns] = K Q^T        O^T[128 value channels x columns] += V^T P^T
+//
+// A column is one (head, query) pair; the columns of a key/value head are adjacent and padded to 16.  So a thread owns a key and finds
+// the scores of all heads for it in its own TMEM lane: mixing them is arithmetic on registers, and a few queries or heads leave no row
+// of the tensor core idle.
+//
+//   warps 0-3 (0-7 for prompts)   scores -> probabilities, written as bf16 to shared memory (the B operand of P V)
+//   then one warp each            MMA issuer; TMA producer of [128 keys x 64 channels] pieces in a ring of slots of one or two pieces
+//   last two warps                row sums of the probabilities (mma.sync with a column of ones), so that numerator and denominator
+//                                 hold the same rounded numbers
+//
+// Modes:
+//   * mixed heads over prompts: a CTA takes up to 32 queries of all heads; its two softmax warpgroups take half of the queries each.
+//   * mixed heads, one token per row: a slice of the keys.
+//   * latent rows, one token per row: up to 64 heads read one row per key, its first channels are the value; the rows pass through the
+//     ring twice, once for each product (the second time from L2).
+//
+// Mixed scores are bounded (the cap, or the product of unit queries and keys, times the row sums of the mix), so the softmax of the
+// first two modes takes a fixed reference; the caller checks that the range fits fp32 exponents.  With r = 1 / (1 + exp2(k2 x)) a capped
+// score is softcap (1 - 2 r), and in log2 units
+//   score_h - reference_h = init_h + near_h[distance] + sum_g w[h, g] r_g.
+// Latent scores take an online softmax whose reference moves only when a maximum grew by more than 2^8.
+#include "mma_sync.cuh"
+
+namespace tyr {
+
+constexpr int KM_KEYS = 128;                   // keys of a tile
+constexpr uint32_t KM_PIECE = KM_KEYS * 128;   // bytes of [128 keys x 64 channels]
+constexpr int KM_SLOTS = 12;                   // most ring slots
+constexpr int KM_COLS = 256;                   // most score columns
+
+enum KmMode : int { KM_PROMPT = 0, KM_STEP = 1, KM_LATENT = 2 };
+
+struct KmArgs {
+  const __nv_bfloat16* q;                      // by (batch, token, head) strides
+  __nv_bfloat16* out;
+  const int* pos;                              // step: position of each row's token
+  long long q_sb, q_ss, q_sh, out_sb, out_ss, out_sh;
+  int S, H, G, rep, dk, dv;                    // S: tokens of a prompt
+  int rn, nq, cols;                            // columns of a key/value head, queries, columns in all (G rn)
+  int kp, vp, mb;                              // pieces of a key and of a value, 128-channel blocks of a value
+  int pps, slots;                              // pieces of a ring slot, slots
+  int hb;                                      // latent: heads of a CTA
+  int cap, ring, window, splits;
+  // mixed heads: w pairs (w, w) [HT, HT], init and k2 [HT], near [H, reach + 1]
+  const float *w2, *init, *k2, *near;
+  int reach;
+  float scale_log2;                            // latent
+  float *part_acc, *part_ml;                   // [B, splits, H, dv], [B, splits, H, 2]
+  int* counters;                               // [B, blocks of heads]
+  int* err;
+};
+
+struct KmBars {
+  uint64_t full[KM_SLOTS], empty[KM_SLOTS], s_ready[2], p_ready, p_free, o_done, l_ready, wg;
+  uint32_t tmem_base;
+  int rescale_at;                              // latent: tile at which the sums and O were last scaled by `factor`
+  int last;
+};
+
+// Byte offsets from a 1024-byte aligned base.
+struct KmLayout {
+  uint32_t q, p, ring, bars, m, factor, wmax, total;
+  __host__ __device__ KmLayout(int mode, int cols, int kp, int pps, int slots) {
+    ring = 0;
+    q = slots * pps * KM_PIECE;
+    p = q + static_cast<uint32_t>(cols) * kp * 128;          // cols is a multiple of 16: both start on a swizzle atom
+    bars = p + static_cast<uint32_t>(cols) * 256;
+    m = bars + ((sizeof(KmBars) + 15) & ~15u);
+    factor = m + (mode == KM_LATENT ? cols * 4 : 0);
+    wmax = factor + (mode == KM_LATENT ? cols * 4 : 0);
+    total = wmax + (mode == KM_LATENT ? cols * 16 : 0);
+    // a value block of one piece: the MMA's upper 64 rows read whatever follows the slot (their results are not used)
+    if (pps == 1 && total < q + KM_PIECE) total = q + KM_PIECE;
+  }
+};
+
+template <int N>
+__device__ __forceinline__ void km_ld(uint32_t addr, uint32_t* r) {
+  static_assert(N == 1 || N == 2 || N == 4 || N == 32, "");
+  if constexpr (N == 1) asm volatile("tcgen05.ld.sync.aligned.32x32b.x1.b32 {%0}, [%1];" : "=r"(r[0]) : "r"(addr) : "memory");
+  if constexpr (N == 2) asm volatile("tcgen05.ld.sync.aligned.32x32b.x2.b32 {%0, %1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(addr) : "memory");
+  if constexpr (N == 4)
+    asm volatile("tcgen05.ld.sync.aligned.32x32b.x4.b32 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+__device__ __forceinline__ uint64_t km_pack(float x, float y) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(x), "f"(y));
+  return r;
+}
+__device__ __forceinline__ void km_unpack(uint64_t v, float& x, float& y) { asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(v)); }
+__device__ __forceinline__ void km_fma2(uint64_t& c, uint64_t a, uint64_t b) { asm("fma.rn.f32x2 %0, %1, %2, %0;" : "+l"(c) : "l"(a), "l"(b)); }
+__device__ __forceinline__ void km_w2(const float* p, uint64_t& a, uint64_t& b) {
+  asm("ld.global.nc.v2.u64 {%0, %1}, [%2];" : "=l"(a), "=l"(b) : "l"(p));
+}
+
+// HT: heads a thread handles (padded), QB: queries it takes at a time, WGS: softmax warpgroups.
+template <int MODE, int HT, int QB, int WGS>
+__global__ void __launch_bounds__((WGS * 4 + 4) * 32, 1)
+joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const __grid_constant__ KmArgs a) {
+  constexpr int SB = MODE == KM_PROMPT ? 1 : 2;            // score buffers
+  constexpr int SOFT = WGS * 4, THREADS = (SOFT + 4) * 32;
+  pdl_trigger();
+  extern __shared__ uint8_t km_raw[];
+  uint8_t* const smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(km_raw) + 1023) & ~static_cast<uintptr_t>(1023));
+  const KmLayout lay(MODE, a.cols, a.kp, a.pps, a.slots);
+  KmBars& s = *reinterpret_cast<KmBars*>(smem + lay.bars);
+  float* const sm_m = reinterpret_cast<float*>(smem + lay.m);
+  float* const sm_f = reinterpret_cast<float*>(smem + lay.factor);
+  float* const sm_w = reinterpret_cast<float*>(smem + lay.wmax);
+  float* const sm_l = reinterpret_cast<float*>(smem + lay.q);          // 1 / row sums, over the queries once all products are done
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  if (tid == 0) {
+    for (int i = 0; i < a.slots; ++i) {
+      mbar_init(&s.full[i], 1);
+      mbar_init(&s.empty[i], 1);
+    }
+    mbar_init(&s.s_ready[0], 1);
+    mbar_init(&s.s_ready[1], 1);
+    mbar_init(&s.p_ready, SOFT);
+    mbar_init(&s.p_free, 3);                               // P V retired, two summing warps
+    mbar_init(&s.o_done, 1);
+    mbar_init(&s.l_ready, 2);
+    mbar_init(&s.wg, 4);
+    s.rescale_at = -1;
+    s.last = 0;
+    mbar_fence_init();
+  }
+  if (warp == SOFT) {
+    tmem_alloc(&s.tmem_base, 512);
+    tmem_relinquish();
+  }
+  pdl_wait();
+  // ---- what this CTA works on
+  int b, h0 = 0, nh = a.H, i0 = 0, tiles, lo = 0, hi = 0, n_keys = 0, split = 0;
+  bool valid = true;
+  if constexpr (MODE == KM_PROMPT) {
+    b = blockIdx.y;
+    i0 = (gridDim.x - 1 - blockIdx.x) * a.nq;              // the longest rows first
+    tiles = (min(i0 + a.nq, a.S) + KM_KEYS - 1) / KM_KEYS;
+  } else {
+    split = blockIdx.x;
+    b = blockIdx.z;
+    if (MODE == KM_LATENT) {
+      h0 = blockIdx.y * a.hb;
+      nh = min(a.hb, a.H - h0);
+    }
+    const int pos = a.pos[b];
+    valid = pos >= 0 && (a.ring || pos < a.cap);
+    if (!valid && tid == 0) report_error(a.err, ERR_BOUNDS, pos);
+    // slots [lo, hi) of the store: a ring holds its last `cap` positions in an order that does not matter here
+    n_keys = pos + 1;
+    if (a.ring) n_keys = min(n_keys, a.cap);
+    const int seen = a.window > 0 ? min(n_keys, a.window) : n_keys, first = n_keys - seen;
+    int chunk = (seen + a.splits - 1) / a.splits;
+    chunk = (chunk + KM_KEYS - 1) / KM_KEYS * KM_KEYS;
+    lo = first + min(split * chunk, seen);
+    hi = min(lo + chunk, n_keys);
+    tiles = valid ? (hi - lo + KM_KEYS - 1) / KM_KEYS : 0;
+  }
+  // ---- queries -> shared memory, K-major with the 128-byte swizzle: [key/value head][piece][column][64 channels]
+  {
+    const int chunks = a.kp * 8, n = a.cols * chunks;      // 16-byte chunks of a column
+    for (int x = tid; x < n; x += THREADS) {
+      const int col = x / chunks, c = x - col * chunks, g = col / a.rn, r = col - g * a.rn;
+      uint4 v = make_uint4(0u, 0u, 0u, 0u);
+      int h = 0, i = 0;
+      bool live;
+      if constexpr (MODE == KM_PROMPT) {
+        h = g * a.rep + r / a.nq;
+        i = i0 + r % a.nq;
+        live = r / a.nq < a.rep && i < a.S;
+      } else {
+        h = MODE == KM_LATENT ? h0 + r : g * a.rep + r;
+        live = r < (MODE == KM_LATENT ? nh : a.rep);
+      }
+      if (live && valid && c * 8 < a.dk) v = *reinterpret_cast<const uint4*>(a.q + b * a.q_sb + i * a.q_ss + h * a.q_sh + c * 8);
+      *reinterpret_cast<uint4*>(smem + lay.q + (static_cast<uint32_t>(g * a.kp + (c >> 3)) * a.rn + r) * 128 + (((c & 7) ^ (r & 7)) << 4)) = v;
+    }
+    if (MODE == KM_LATENT)
+      for (int x = tid; x < a.cols; x += THREADS) { sm_m[x] = -INFINITY; sm_f[x] = 1.f; }
+  }
+  fence_proxy_async();
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = s.tmem_base, o_base = tmem + SB * a.cols;
+  const uint32_t slot_bytes = a.pps * KM_PIECE, ring = smem_u32(smem + lay.ring);
+  const int ku = (a.kp + a.pps - 1) / a.pps;               // ring slots of one key
+  const int vpb = min(2, a.vp);                            // pieces of a 128-channel value block (the last may have fewer)
+
+  if (warp == SOFT + 1) {
+    // ------------------------------------------------------------------ TMA producer
+    if (elect_one() && tiles > 0) {
+      tma_prefetch_desc(&tmK);
+      tma_prefetch_desc(&tmV);
+      uint32_t it = 0;
+      bool ok = true;
+      auto load = [&](const CUtensorMap* tm, int g, int piece, int count, int key) {
+        const int st = it % a.slots;
+        if (!mbar_wait(&s.empty[st], ((it / a.slots) & 1) ^ 1, a.err, 2500 + st)) { ok = false; return; }
+        mbar_expect_tx(&s.full[st], count * KM_PIECE);
+        for (int i = 0; i < count; ++i)
+          tma_load_4d(smem + lay.ring + st * slot_bytes + i * KM_PIECE, tm, &s.full[st], (piece + i) * 64, g, key, b);
+        ++it;
+      };
+      auto keys = [&](int j) {
+        for (int g = 0; g < a.G && ok; ++g)
+          for (int u = 0; u < ku && ok; ++u) load(&tmK, g, u * a.pps, min(a.pps, a.kp - u * a.pps), lo + j * KM_KEYS);
+      };
+      keys(0);
+      for (int j = 0; j < tiles && ok; ++j) {
+        if (j + 1 < tiles) keys(j + 1);
+        for (int g = 0; g < a.G && ok; ++g)
+          for (int m = 0; m < a.mb && ok; ++m) load(&tmV, g, m * 2, min(vpb, a.vp - m * 2), lo + j * KM_KEYS);
+      }
+      if (!ok)                                             // let the copies in flight land before the CTA unwinds
+        for (uint32_t x = (it > static_cast<uint32_t>(a.slots) ? it - a.slots : 0); x < it; ++x)
+          mbar_wait(&s.full[x % a.slots], (x / a.slots) & 1, nullptr, 0);
+    }
+  } else if (warp == SOFT) {
+    // ------------------------------------------------------------------ MMA issuer
+    if (elect_one() && tiles > 0) {
+      const uint32_t id_s = make_idesc_f16(1, 128, a.rn, 0, 0), id_o = make_idesc_f16(1, 128, a.rn, 1, 0);
+      const uint32_t q_addr = smem_u32(smem + lay.q), p_addr = smem_u32(smem + lay.p);
+      uint32_t it = 0;
+      bool ok = true;
+      auto wait_slot = [&]() {
+        ok = ok && mbar_wait(&s.full[it % a.slots], (it / a.slots) & 1, a.err, 2600 + it % a.slots);
+        tc_fence_after();
+        return ring + (it % a.slots) * slot_bytes;
+      };
+      auto scores = [&](int j) {
+        for (int g = 0; g < a.G && ok; ++g)
+          for (int u = 0; u < ku && ok; ++u) {
+            const uint32_t k_addr = wait_slot();
+            if (!ok) break;
+            const int steps = min(a.pps * 4, (a.dk - u * a.pps * 64 + 15) / 16);
+            for (int k = 0; k < steps; ++k)
+              umma_f16_ss(tmem + (SB == 2 ? (j & 1) * a.cols : 0) + g * a.rn,
+                          make_smem_desc_sw128(k_addr + (k >> 2) * KM_PIECE + (k & 3) * 32, 16, 1024),
+                          make_smem_desc_sw128(q_addr + static_cast<uint32_t>(g * a.kp + u * a.pps + (k >> 2)) * a.rn * 128 + (k & 3) * 32, 16, 1024), id_s,
+                          u > 0 || k > 0 ? 1u : 0u);
+            umma_commit(&s.empty[it % a.slots]);
+            ++it;
+          }
+        umma_commit(&s.s_ready[SB == 2 ? j & 1 : 0]);
+      };
+      scores(0);
+      for (int j = 0; j < tiles && ok; ++j) {
+        // two score buffers: the next tile's went free when the probabilities of tile j - 1 were complete
+        if (SB == 2 && j + 1 < tiles) scores(j + 1);
+        ok = ok && mbar_wait(&s.p_ready, j & 1, a.err, 2620);
+        tc_fence_after();
+        if (!ok) break;
+        if (SB == 1 && j + 1 < tiles) scores(j + 1);
+        for (int g = 0; g < a.G && ok; ++g)
+          for (int m = 0; m < a.mb && ok; ++m) {
+            const uint32_t v_addr = wait_slot();
+            if (!ok) break;
+#pragma unroll
+            for (int k = 0; k < KM_KEYS / 16; ++k)
+              umma_f16_ss(o_base + (g * a.mb + m) * a.rn, make_smem_desc_sw128(v_addr + k * 2048, KM_PIECE, 1024),
+                          make_smem_desc_sw128(p_addr + static_cast<uint32_t>(g) * a.rn * 256 + (k >> 2) * a.rn * 128 + (k & 3) * 32, 16, 1024), id_o,
+                          j > 0 || k > 0 ? 1u : 0u);
+            umma_commit(&s.empty[it % a.slots]);
+            ++it;
+          }
+        umma_commit(&s.p_free);
+      }
+      umma_commit(&s.o_done);
+    }
+  } else if (warp >= SOFT + 2) {
+    // ------------------------------------------------------------------ row sums of the probabilities
+    const int w = warp - SOFT - 2, g8 = lane >> 2;
+    float acc[KM_COLS / 32][4];
+#pragma unroll
+    for (int x = 0; x < KM_COLS / 32; ++x) acc[x][0] = acc[x][1] = acc[x][2] = acc[x][3] = 0.f;
+    bool ok = true;
+    for (int j = 0; j < tiles && ok; ++j) {
+      ok = mbar_wait(&s.p_ready, j & 1, a.err, 2630 + w);
+      ok = __all_sync(0xffffffffu, ok);
+      if (!ok) break;
+      const bool scale = MODE == KM_LATENT && *reinterpret_cast<volatile int*>(&s.rescale_at) == j;
+#pragma unroll
+      for (int x = 0; x < KM_COLS / 32; ++x) {
+        const int n0 = (2 * x + w) * 16;
+        if (n0 >= a.cols) break;
+        if (scale) {
+          const float f0 = sm_f[n0 + g8], f1 = sm_f[n0 + g8 + 8];
+          acc[x][0] *= f0; acc[x][2] *= f1;
+        }
+        const int n = n0 + (lane & 15), gg = n0 / a.rn;
+        const uint8_t* row = smem + lay.p + static_cast<uint32_t>(gg) * a.rn * 256 + (n - gg * a.rn) * 128;
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+          uint32_t f[4];
+          ldsm4(f, row + (k >> 2) * a.rn * 128 + ((((k & 3) * 2 + (lane >> 4)) ^ (n & 7)) << 4));
+          mma_bf16(acc[x], f, 0x3f803f80u, 0x3f803f80u);
+        }
+      }
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&s.p_free);
+    }
+    // the queries' space is free once every product is done
+    ok = ok && (tiles == 0 || mbar_wait(&s.o_done, 0, a.err, 2640 + w));
+    ok = __all_sync(0xffffffffu, ok);
+    if (ok) {
+#pragma unroll
+      for (int x = 0; x < KM_COLS / 32; ++x) {
+        const int n0 = (2 * x + w) * 16;
+        if (n0 < a.cols && (lane & 3) == 0) {
+          sm_l[n0 + g8] = acc[x][0];
+          sm_l[n0 + g8 + 8] = acc[x][2];
+        }
+      }
+    }
+    __syncwarp();
+    if (lane == 0) mbar_arrive(&s.l_ready);
+  } else {
+    // ------------------------------------------------------------------ scores -> probabilities
+    const int wg = warp >> 2, quarter = warp & 3, key = quarter * 32 + lane;
+    const uint32_t lane_addr = static_cast<uint32_t>(quarter * 32) << 16;
+    uint8_t* const p_row = smem + lay.p + (key >> 6) * (a.rn * 128);               // column n of head g: + g rn 256 + n 128 + swizzled p_off
+    const uint32_t p_off = (key & 63) * 2;
+    bool ok = true;
+    for (int j = 0; j < tiles && ok; ++j) {
+      ok = mbar_wait(&s.s_ready[SB == 2 ? j & 1 : 0], SB == 2 ? (j >> 1) & 1 : j & 1, a.err, 2700 + warp);
+      ok = __all_sync(0xffffffffu, ok);
+      if (!ok) break;
+      tc_fence_after();
+      const uint32_t s_addr = tmem + lane_addr + (SB == 2 ? (j & 1) * a.cols : 0);
+      const int kj = lo + j * KM_KEYS + key;                                        // this thread's key (slot of the store)
+      auto p_writable = [&]() {
+        if (j == 0) return true;
+        const bool w = mbar_wait(&s.p_free, (j - 1) & 1, a.err, 2720 + warp);
+        return static_cast<bool>(__all_sync(0xffffffffu, w));
+      };
+      if constexpr (MODE != KM_LATENT) {
+        const int nqw = MODE == KM_PROMPT ? a.nq / WGS : 1, q_first = MODE == KM_PROMPT ? wg * nqw : 0;
+        const int stride = a.nq;                                                    // columns of a head
+        const int i_first = MODE == KM_PROMPT ? i0 + q_first : n_keys - 1;          // position of the first query
+        const int tile_end = lo + j * KM_KEYS + KM_KEYS - 1;
+        const bool far = i_first - tile_end >= a.reach, edge = MODE == KM_PROMPT ? tile_end > i_first : tile_end >= hi;
+        for (int qb = 0; qb < nqw; qb += QB) {
+          const int q0 = q_first + qb;
+          uint32_t x[HT][QB];
+          {
+            int g = 0, r = 0;
+#pragma unroll
+            for (int h = 0; h < HT; ++h) {
+              km_ld<QB>(s_addr + g * a.rn + r * stride + q0, x[h]);
+              if (h + 1 < a.H && ++r == a.rep) { r = 0; ++g; }
+            }
+          }
+          tmem_wait_ld();
+          uint64_t y[HT][(QB + 1) / 2];
+#pragma unroll
+          for (int h = 0; h < HT; ++h) {
+            const float k2 = __ldg(a.k2 + h);
+            float v[QB];
+#pragma unroll
+            for (int e = 0; e < QB; ++e) v[e] = rcp(1.f + ex2(__uint_as_float(x[h][e]) * k2));
+#pragma unroll
+            for (int e = 0; e < QB; e += 2) y[h][e / 2] = km_pack(v[e], QB > 1 ? v[e + (QB > 1)] : 0.f);
+          }
+          if (qb == 0 && !(ok = p_writable())) break;
+          int g = 0, r = 0;
+#pragma unroll 1
+          for (int h = 0; h < a.H; ++h) {
+            const float init = __ldg(a.init + h);
+            uint64_t c[(QB + 1) / 2];
+#pragma unroll
+            for (int e = 0; e < QB; e += 2) c[e / 2] = km_pack(init, init);
+            const float* w = a.w2 + h * HT * 2;
+#pragma unroll
+            for (int k = 0; k < HT; k += 2) {
+              uint64_t wa, wb;
+              km_w2(w + k * 2, wa, wb);
+#pragma unroll
+              for (int e = 0; e < (QB + 1) / 2; ++e) {
+                km_fma2(c[e], y[k][e], wa);
+                km_fma2(c[e], y[k + 1][e], wb);
+              }
+            }
+            uint8_t* dst = p_row + static_cast<uint32_t>(g) * a.rn * 256;
+#pragma unroll
+            for (int e = 0; e < QB; e += 2) {
+              float v[2];
+              km_unpack(c[e / 2], v[0], v[1]);
+#pragma unroll
+              for (int z = 0; z < 2; ++z) {
+                if (e + z >= QB) break;
+                const int d = i_first + qb + e + z - kj;                            // distance of query and key
+                if (!far) v[z] += __ldg(a.near + static_cast<long long>(h) * (a.reach + 1) + min(max(d, 0), a.reach));
+                v[z] = ex2(v[z]);
+                if (edge && (MODE == KM_PROMPT ? d < 0 : kj >= hi)) v[z] = 0.f;
+                const int n = r * stride + q0 + e + z;
+                *reinterpret_cast<__nv_bfloat16*>(dst + n * 128 + (p_off ^ ((n & 7) << 4))) = __float2bfloat16(v[z]);
+              }
+            }
+            if (++r == a.rep) { r = 0; ++g; }
+          }
+        }
+        if (!ok) break;
+      } else {
+        // online softmax over the heads' columns, 32 at a time; a warp's maxima meet in shared memory
+        const bool live = kj < hi;
+        for (int c0 = 0; c0 < a.cols; c0 += 32) {
+          uint32_t x[32];
+          tmem_ld_32x32(s_addr + c0, x);                   // columns past the last may be read; they are not used
+          tmem_wait_ld();
+          float v[32];
+#pragma unroll
+          for (int e = 0; e < 32; ++e) v[e] = live ? __uint_as_float(x[e]) * a.scale_log2 : -INFINITY;
+          // lane c ends with the maximum of column c over the warp's keys
+#pragma unroll
+          for (int o = 16; o > 0; o >>= 1) {
+            const bool up = lane & o;
+#pragma unroll
+            for (int e = 0; e < o; ++e) {
+              const float send = up ? v[e] : v[e + o], keep = up ? v[e + o] : v[e];
+              v[e] = fmaxf(keep, __shfl_xor_sync(0xffffffffu, send, o));
+            }
+          }
+          if (c0 + lane < a.cols) sm_w[quarter * a.cols + c0 + lane] = v[0];
+        }
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&s.wg);
+        ok = mbar_wait(&s.wg, 0, a.err, 2740);             // phases of this barrier: two to a tile
+        ok = __all_sync(0xffffffffu, ok) && p_writable();  // also: the summing warps are done with the last factors
+        if (!ok) break;
+        // every thread of the warpgroup looks at the columns tid, tid + 128, ...; the reference and factor are written by their owner
+        bool grow = false;
+        for (int c = tid; c < a.cols; c += 128) {
+          const float mx = fmaxf(fmaxf(sm_w[c], sm_w[a.cols + c]), fmaxf(sm_w[2 * a.cols + c], sm_w[3 * a.cols + c]));
+          const float m = sm_m[c];
+          const bool up = mx > m + 8.f;                    // also the first tile: m is -inf
+          sm_f[c] = up ? ex2(m - mx) : 1.f;
+          if (up) sm_m[c] = mx;
+          grow = grow || (up && j > 0);
+        }
+        if (__any_sync(0xffffffffu, grow) && lane == 0) *reinterpret_cast<volatile int*>(&s.rescale_at) = j;
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&s.wg);
+        ok = mbar_wait(&s.wg, 1, a.err, 2741);
+        ok = __all_sync(0xffffffffu, ok);
+        if (!ok) break;
+        if (*reinterpret_cast<volatile int*>(&s.rescale_at) == j) {    // P V of the tile before has retired: O is idle
+          tc_fence_after();
+          for (int mbk = 0; mbk < a.mb; ++mbk)
+            for (int c0 = 0; c0 < a.cols; c0 += 16) {
+              uint32_t o[16];
+              tmem_ld_32x16(o_base + lane_addr + mbk * a.rn + c0, o);
+              tmem_wait_ld();
+#pragma unroll
+              for (int e = 0; e < 16; ++e) o[e] = __float_as_uint(__uint_as_float(o[e]) * sm_f[c0 + e]);
+              tmem_st_32x16(o_base + lane_addr + mbk * a.rn + c0, o);
+            }
+          tmem_wait_st();
+        }
+        for (int c0 = 0; c0 < a.cols; c0 += 16) {
+          uint32_t x[16];
+          tmem_ld_32x16(s_addr + c0, x);
+          tmem_wait_ld();
+#pragma unroll
+          for (int e = 0; e < 16; ++e) {
+            const int n = c0 + e;
+            const float p = live ? ex2(fmaf(__uint_as_float(x[e]), a.scale_log2, -sm_m[n])) : 0.f;
+            *reinterpret_cast<__nv_bfloat16*>(p_row + n * 128 + (p_off ^ ((n & 7) << 4))) = __float2bfloat16(p);
+          }
+        }
+      }
+      tc_fence_before();
+      fence_proxy_async();                                 // the probabilities are read by the tensor core
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&s.p_ready);
+    }
+    // ---------------------------------------------------------------- O^T: lane = value channel, column = (head, query)
+    if (ok && tiles > 0) ok = mbar_wait(&s.o_done, 0, a.err, 2760 + warp);
+    if (ok) ok = mbar_wait(&s.l_ready, 0, a.err, 2780 + warp);
+    ok = __all_sync(0xffffffffu, ok);
+    tc_fence_after();
+    const long long part = static_cast<long long>(b) * a.splits + split;
+    if (ok && valid) {
+      for (int m = 0; m < a.mb; ++m) {
+        const int d = m * 128 + key;
+        for (int g = 0; g < a.G; ++g)
+          for (int n0 = (WGS == 2 ? wg * 16 : 0); n0 < a.rn; n0 += 16 * WGS) {
+            uint32_t o[16];
+            if (tiles > 0) {
+              tmem_ld_32x16(o_base + lane_addr + (g * a.mb + m) * a.rn + n0, o);
+              tmem_wait_ld();
+            }
+#pragma unroll
+            for (int e = 0; e < 16; ++e) {
+              const int n = n0 + e;
+              const float l = sm_l[g * a.rn + n], v = tiles > 0 ? __uint_as_float(o[e]) : 0.f;
+              if constexpr (MODE == KM_PROMPT) {
+                const int r = n / a.nq, i = i0 + n % a.nq;
+                if (r < a.rep && i < a.S && d < a.dv) a.out[b * a.out_sb + i * a.out_ss + (g * a.rep + r) * a.out_sh + d] = __float2bfloat16(__fdividef(v, l));
+              } else {
+                const int h = MODE == KM_LATENT ? n : g * a.rep + n;
+                if (n < (MODE == KM_LATENT ? nh : a.rep)) {
+                  if (a.splits == 1) {
+                    if (d < a.dv) a.out[b * a.out_sb + (h0 + h) * a.out_sh + d] = __float2bfloat16(__fdividef(v, l));
+                  } else {
+                    if (d < a.dv) a.part_acc[(part * a.H + h0 + h) * a.dv + d] = v;
+                    if (d == 0) {
+                      a.part_ml[(part * a.H + h0 + h) * 2] = MODE == KM_LATENT ? sm_m[n] : 0.f;
+                      a.part_ml[(part * a.H + h0 + h) * 2 + 1] = tiles > 0 ? l : 0.f;
+                    }
+                  }
+                }
+              }
+            }
+          }
+      }
+    }
+  }
+  tc_fence_before();
+  if (MODE != KM_PROMPT && a.splits > 1) __threadfence();
+  __syncthreads();
+  if (warp == SOFT) {
+    tc_fence_after();
+    tmem_dealloc(tmem, 512);
+  }
+  if constexpr (MODE != KM_PROMPT) {
+    if (a.splits == 1 || !valid) return;
+    if (tid == 0) s.last = atomicAdd(a.counters + b * gridDim.y + blockIdx.y, 1) == a.splits - 1;
+    __syncthreads();
+    if (!s.last) return;
+    __threadfence();
+    float* const w = reinterpret_cast<float*>(smem + lay.q);            // [nh, splits] weights of the slices
+    for (int h = warp; h < nh; h += THREADS / 32) {
+      const float* src = a.part_ml + (static_cast<long long>(b) * a.splits * a.H + h0 + h) * 2;
+      const float mx = lane < a.splits ? __ldcg(src + static_cast<long long>(lane) * a.H * 2) : -INFINITY;
+      const float lx = lane < a.splits ? __ldcg(src + static_cast<long long>(lane) * a.H * 2 + 1) : 0.f;
+      const float M = warp_max(mx), f = ex2(mx - M), L = warp_sum(f * lx);
+      if (lane < a.splits) w[h * a.splits + lane] = f / L;
+    }
+    __syncthreads();
+    for (int x = tid; x < nh * a.dv; x += THREADS) {
+      const int h = x / a.dv, d = x - h * a.dv;
+      const float* src = a.part_acc + (static_cast<long long>(b) * a.splits * a.H + h0 + h) * a.dv + d;
+      float v = 0.f;
+#pragma unroll 8
+      for (int i = 0; i < a.splits; ++i) v += w[h * a.splits + i] * __ldcg(src + static_cast<long long>(i) * a.H * a.dv);
+      a.out[b * a.out_sb + (h0 + h) * a.out_sh + d] = __float2bfloat16(v);
+    }
+    if (tid == 0) a.counters[b * gridDim.y + blockIdx.y] = 0;
+  }
+}
+
+}  // namespace tyr
+
+using namespace tyr;
+
+namespace {
+typedef CUresult (*KmEncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
+                               const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+KmEncodeFn km_encode() {
+  static KmEncodeFn fn = nullptr;
+  if (!fn) {
+    void* ptr = nullptr;
+    cudaDriverEntryPointQueryResult q;
+    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &ptr, cudaEnableDefault, &q) == cudaSuccess && q == cudaDriverEntryPointSuccess)
+      fn = reinterpret_cast<KmEncodeFn>(ptr);
+  }
+  return fn;
+}
+// bf16 (channel, head, key, batch) by element strides; a box is 64 channels of 128 keys.
+int km_map(CUtensorMap* tm, const void* base, int D, int G, int T, int B, long long sg, long long st, long long sb) {
+  KmEncodeFn fn = km_encode();
+  if (!fn) return 1;
+  cuuint64_t dims[4] = {(cuuint64_t)D, (cuuint64_t)G, (cuuint64_t)T, (cuuint64_t)B};
+  cuuint64_t strides[3] = {(cuuint64_t)(G == 1 ? D : sg) * 2, (cuuint64_t)st * 2, (cuuint64_t)(B == 1 ? st * T : sb) * 2};
+  cuuint32_t box[4] = {64, 1, KM_KEYS, 1}, es[4] = {1, 1, 1, 1};
+  return fn(tm, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(base), dims, strides, box, es, CU_TENSOR_MAP_INTERLEAVE_NONE,
+            CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS ? 0 : 2;
+}
+
+constexpr uint32_t kKmSmem = 227 * 1024 - 1024;            // less the room for alignment
+
+// Fills in the sizes that follow from the shapes; false: the kernel does not take them.
+bool km_plan(int mode, KmArgs& a) {
+  if (a.H <= 0 || a.G <= 0 || a.H % a.G || a.dk <= 0 || a.dv <= 0 || (a.dk & 15) || a.splits < 1 || a.splits > 32) return false;
+  a.rep = a.H / a.G;
+  a.kp = (a.dk + 63) / 64;
+  a.vp = (a.dv + 63) / 64;
+  a.mb = (a.vp + 1) / 2;
+  a.pps = a.kp > 1 || a.vp > 1 ? 2 : 1;
+  const int sb = mode == KM_PROMPT ? 1 : 2;
+  auto fits = [&](int min_slots) {
+    a.cols = a.G * a.rn;
+    if (a.rn > 256 || a.cols > KM_COLS || sb * a.cols + a.cols * a.mb > 512) return false;
+    for (a.slots = KM_SLOTS; a.slots >= min_slots; --a.slots)
+      if (KmLayout(mode, a.cols, a.kp, a.pps, a.slots).total <= kKmSmem) return true;
+    return false;
+  };
+  if (mode == KM_LATENT) {
+    if (a.G != 1) return false;
+    for (a.rn = a.H >= 64 ? 64 : (a.H + 15) / 16 * 16; a.rn >= 16; a.rn -= 16) {
+      a.nq = 1;
+      a.hb = a.rn;
+      if (fits(3)) return true;
+    }
+    return false;
+  }
+  if (a.H > 32) return false;
+  if (mode == KM_STEP) {
+    a.nq = 1;
+    a.rn = (a.rep + 15) / 16 * 16;
+    return fits(2);
+  }
+  for (a.nq = 32; a.nq >= 8; a.nq /= 2) {
+    a.rn = (a.rep * a.nq + 15) / 16 * 16;
+    if (fits(2)) return true;
+  }
+  return false;
+}
+
+template <int MODE, int HT, int QB, int WGS>
+int km_launch(const CUtensorMap& tk, const CUtensorMap& tv, const KmArgs& a, dim3 grid, void* stream) {
+  auto kernel = joint_keymajor_kernel<MODE, HT, QB, WGS>;
+  static bool configured[64] = {};               // the attribute is per device
+  int dev = 0;
+  if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= 64) dev = 0;
+  if (!configured[dev]) {
+    const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kKmSmem + 1024);
+    if (e != cudaSuccess) return 1000 + (int)e;
+    configured[dev] = true;
+  }
+  const size_t smem = KmLayout(MODE, a.cols, a.kp, a.pps, a.slots).total + 1024;
+  return (int)launch_dependent(kernel, grid, dim3((WGS * 4 + 4) * 32), smem, (cudaStream_t)stream, tk, tv, a);
+}
+}  // namespace
+
+// Heads of a CTA for these sizes (0: the kernel does not take them).  mode 0 prompts, 1 steps of mixed heads, 2 steps over latent rows.
+extern "C" TYR_EXPORT int tyr_keymajor_heads(int mode, int H, int G, int dk, int dv) {
+  KmArgs a{};
+  a.H = H; a.G = G; a.dk = dk; a.dv = dv; a.splits = 1;
+  if (mode < 0 || mode > 2 || !km_plan(mode, a)) return 0;
+  return mode == KM_LATENT ? a.hb : H;
+}
+
+// Mixed heads over whole bf16 prompts.  strides: (batch, token, head) of q, k, v, out; dk multiple of 16, dv of 8, 16-byte aligned rows.
+// w2 [HT, HT] pairs, init and k2 [HT] with HT = 8, 16 or 32, the smallest that holds H; near [H, reach + 1].
+extern "C" TYR_EXPORT int tyr_keymajor_prompt(const void* q, const void* k, const void* v, void* out, const float* w2, const float* init,
+                                              const float* k2, const float* near, int reach, const long long* st, int B, int S, int H, int G,
+                                              int dk, int dv, int dvp, int* err, void* stream) {
+  KmArgs a{};
+  a.H = H; a.G = G; a.dk = dk; a.dv = dv; a.splits = 1;
+  if (B <= 0 || B > 65535 || S <= 0 || dv > dvp || (dvp & 7) || reach < 0 || !km_plan(KM_PROMPT, a)) return -1;
+  for (int i = 0; i < 9; ++i)
+    if (st[i] & 7) return -3;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v) | reinterpret_cast<uintptr_t>(w2)) & 15) return -4;
+  a.q = (const __nv_bfloat16*)q; a.out = (__nv_bfloat16*)out; a.S = S; a.err = err;
+  a.q_sb = st[0]; a.q_ss = st[1]; a.q_sh = st[2]; a.out_sb = st[9]; a.out_ss = st[10]; a.out_sh = st[11];
+  a.w2 = w2; a.init = init; a.k2 = k2; a.near = near; a.reach = reach;
+  CUtensorMap tk, tv;
+  if (int r = km_map(&tk, k, dk, G, S, B, st[5], st[4], st[3])) return 3000 + r;
+  if (int r = km_map(&tv, v, dvp, G, S, B, st[8], st[7], st[6])) return 4000 + r;
+  const dim3 grid((S + a.nq - 1) / a.nq, B);
+  return H <= 8 ? km_launch<KM_PROMPT, 8, 4, 2>(tk, tv, a, grid, stream)
+                : (H <= 16 ? km_launch<KM_PROMPT, 16, 4, 2>(tk, tv, a, grid, stream) : km_launch<KM_PROMPT, 32, 2, 2>(tk, tv, a, grid, stream));
+}
+
+// One token per row over bf16 stores that hold it.  w2 null: latent rows [B, 1, cap, dk] whose first dv channels are the values of all
+// heads (a ring must hold exactly the window), scale; else mixed heads over stores [B, G, cap, dk] and [B, G, cap, dvp].  strides:
+// (batch, head) of q, then of out.  The workspace (tyr_joint_step_workspace_bytes) must be zero-filled once.
+extern "C" TYR_EXPORT int tyr_keymajor_step(const void* q, const void* k, const void* v, void* out, const int* pos, const float* w2,
+                                            const float* init, const float* k2, const float* near, int reach, float scale, void* workspace,
+                                            const long long* st, int B, int H, int G, int dk, int dv, int dvp, int cap, int ring, int window,
+                                            int splits, int* err, void* stream) {
+  KmArgs a{};
+  const int mode = w2 == nullptr ? KM_LATENT : KM_STEP;
+  a.H = H; a.G = G; a.dk = dk; a.dv = dv; a.splits = splits;
+  if (B <= 0 || B > 65535 || cap <= 0 || window < 0 || reach < 0 || dv > dvp || (dvp & 7) || !km_plan(mode, a)) return -1;
+  if ((mode == KM_STEP && (ring || window)) || (ring && window && window < cap) || (splits > 1 && workspace == nullptr)) return -2;
+  if (((st[0] | st[1]) & 7) || ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v) | reinterpret_cast<uintptr_t>(w2)) & 15))
+    return -3;
+  a.q = (const __nv_bfloat16*)q; a.out = (__nv_bfloat16*)out; a.pos = pos; a.err = err;
+  a.q_sb = st[0]; a.q_sh = st[1]; a.out_sb = st[2]; a.out_sh = st[3];
+  a.w2 = w2; a.init = init; a.k2 = k2; a.near = near; a.reach = reach;
+  a.scale_log2 = scale * 1.4426950408889634f;
+  a.cap = cap; a.ring = ring; a.window = window;
+  a.part_acc = (float*)workspace;
+  a.part_ml = a.part_acc + static_cast<long long>(B) * H * splits * dv;
+  a.counters = (int*)(a.part_ml + static_cast<long long>(B) * H * splits * 2);
+  CUtensorMap tk, tv;
+  if (int r = km_map(&tk, k, dk, G, cap, B, static_cast<long long>(cap) * dk, dk, static_cast<long long>(G) * cap * dk)) return 3000 + r;
+  if (int r = km_map(&tv, v, dvp, G, cap, B, static_cast<long long>(cap) * dvp, dvp, static_cast<long long>(G) * cap * dvp)) return 4000 + r;
+  if (mode == KM_LATENT) return km_launch<KM_LATENT, 8, 1, 1>(tk, tv, a, dim3(splits, (H + a.hb - 1) / a.hb, B), stream);
+  const dim3 grid(splits, 1, B);
+  return H <= 8 ? km_launch<KM_STEP, 8, 1, 1>(tk, tv, a, grid, stream)
+                : (H <= 16 ? km_launch<KM_STEP, 16, 1, 1>(tk, tv, a, grid, stream) : km_launch<KM_STEP, 32, 1, 1>(tk, tv, a, grid, stream));
+}

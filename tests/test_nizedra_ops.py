@@ -148,9 +148,11 @@ def test_talking_heads_over_prompts(place, case):
     pad = lambda t: torch.cat([t[:T // 2], torch.randn(T - T // 2, *t.shape[1:]).bfloat16().double()])
     dkp, dvp = ja.store_dims(case[3], case[4], dt, dev)
     batch = lambda t, d: torch.nn.functional.pad(torch.stack([t, pad(t)]), (0, d - t.shape[2])).to(dev, dt)
-    got = ja.prompt_attention(batch(q, dkp), batch(k, dkp), batch(v, dvp)[..., :case[4]], scale=mix["scale"], talk=talk_of(mix, temp, rel, talk, dev))
-    near(got[0], want, dt)
-    near(got[1, :T // 2], want[:T // 2], dt)
+    for bound in (None, 1.02 * case[3]):                   # with and without a known bound of the products: two ways to take the softmax
+        got = ja.prompt_attention(batch(q, dkp), batch(k, dkp), batch(v, dvp)[..., :case[4]], scale=mix["scale"], talk=talk_of(mix, temp, rel, talk, dev),
+                                  dot_bound=bound)
+        near(got[0], want, dt)
+        near(got[1, :T // 2], want[:T // 2], dt)
 
 
 def stores(dev, dt, B, G, cap, dk, dv, shared=False, ring=False):
@@ -175,8 +177,9 @@ def test_talking_heads_one_token_per_row(place, case):
     for b, p in enumerate(pos):
         st.k[b, :, :p + 1], st.v[b, :, :p + 1] = fill(k, p + 1, dkp), fill(v, p + 1, dvp)
     qs = torch.nn.functional.pad(torch.stack([q[p][None] for p in pos]), (0, dkp - dk)).to(dev, dt)
-    got = ja.step_attention(qs, st, int32(pos, dev), dv, scale=mix["scale"], talk=talk_of(mix, temp, rel, talk, dev))
-    near(got[:, 0], want[pos], dt)
+    for bound in (None, 1.02 * dk):
+        got = ja.step_attention(qs, st, int32(pos, dev), dv, scale=mix["scale"], talk=talk_of(mix, temp, rel, talk, dev), dot_bound=bound)
+        near(got[:, 0], want[pos], dt)
 
 
 @pytest.mark.parametrize("place", PLACES)

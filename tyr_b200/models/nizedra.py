@@ -472,12 +472,13 @@ def latent_mixer(s: LatentSpec, m: LatentMixer, h: torch.Tensor, store: KVCache,
 def attention_mixer(s: AttentionSpec, m: AttentionMixer, h: torch.Tensor, store: KVCache, t: Tokens, eps: float) -> torch.Tensor:
     """Without the output bias, which the norm that follows adds."""
     dkp, dvp = store.k.shape[3], store.v.shape[3]
+    bound = 1.02 * s.dim                                   # queries and keys of unit root mean square, rounded
     q, k, v = qk_norm_store(lin(h, m.w_in), None, None, s.heads, s.kv_heads, s.dim, s.vdim, eps, dkp=dkp, dvp=dvp, store=store, pos=t.pos, lens=t.lens,
                             bias=m.b_in)
     if t.step:
-        o = ja.step_attention(q, store, t.pos, s.vdim, scale=s.scale, talk=m.talk).flatten(2)
+        o = ja.step_attention(q, store, t.pos, s.vdim, scale=s.scale, talk=m.talk, dot_bound=bound).flatten(2)
     else:
-        o = ja.prompt_attention(q, k, v[..., :s.vdim], scale=s.scale, talk=m.talk)
+        o = ja.prompt_attention(q, k, v[..., :s.vdim], scale=s.scale, talk=m.talk, dot_bound=bound)
     return lin(o, m.w_out)
 
 

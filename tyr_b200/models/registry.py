@@ -36,7 +36,7 @@ class Family:
 
 FAMILIES: List[Family] = [
     Family("nizedra", ("nizedra",), "nizedra", "CacheSession",
-           ("attention_fwd", "attention_general", "decode_gemm", "delta_general", "gemm_tcgen05", "joint_attention", "latent", "lightning", "mix_conv",
+           ("attention_fwd", "attention_general", "decode_gemm", "delta_general", "gemm_tcgen05", "joint_attention", "joint_tcgen05", "latent", "lightning", "mix_conv",
             "norm", "skinny_gemm"), ragged=True),
     Family("kinetar", ("kinetar",), "kinetar", "CacheSession",
            ("attention_fwd", "attention_general", "decode_attention", "decode_gemm", "delta_general", "delta_rule", "embed", "gemm_tcgen05", "mix_conv",

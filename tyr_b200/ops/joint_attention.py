@@ -29,7 +29,9 @@ def _sigs(lib_):
     S, LL = ctypes.POINTER(_Scores), ctypes.POINTER(L)
     for name, args in (("tyr_joint_attention", [P, P, P, P, P, S, LL] + [I] * 11 + [P, P]), ("tyr_joint_prompt_form", [I] * 6),
                        ("tyr_joint_prompt", [P, P, P, P, S, LL] + [I] * 7 + [P]), ("tyr_joint_step_heads", [I] * 8),
-                       ("tyr_joint_step", [P, P, P, P, P, S, P, LL] + [I] * 10 + [P, P])):
+                       ("tyr_joint_step", [P, P, P, P, P, S, P, LL] + [I] * 10 + [P, P]), ("tyr_keymajor_heads", [I] * 5),
+                       ("tyr_keymajor_prompt", [P] * 8 + [I, LL] + [I] * 7 + [P, P]),
+                       ("tyr_keymajor_step", [P] * 9 + [I, ctypes.c_float, P, LL] + [I] * 10 + [P, P])):
         fn = getattr(lib_, name, None)
         if fn is not None:
             fn.argtypes, fn.restype = args, I
@@ -63,6 +65,7 @@ class Talk:
     softcap: float
 
     def __post_init__(self):
+        self._plans: dict = {}
         self.exact = bool((self.mix.bfloat16().float() == self.mix).all())     # entries that TF32 holds as they are
 
     def scores(self, dots: torch.Tensor, dist: torch.Tensor) -> torch.Tensor:
@@ -70,6 +73,28 @@ class Talk:
         s = self.softcap * torch.tanh(dots * self.temp[:, None, None] / self.softcap)
         s = s + self.rel[self.bucket[dist.clamp(0, self.bucket.numel() - 1).long()].long()].permute(2, 0, 1)
         return torch.einsum("hg,...gij->...hij", self.mix, s)
+
+    def plan(self, scale: float, dot_bound: Optional[float]):
+        """The scores in log2 units against a fixed reference, score_h - reference_h = init_h + near_h[distance] + sum_g w[h, g] / (1 + exp2(k2_g x)):
+        (w as pairs [HT, HT, 2], init [HT], k2 [HT], near [H, reach + 1]), or None where their range could leave fp32 exponents.
+        ``dot_bound``: largest |q . k| (None: only the cap bounds a score)."""
+        key = (scale, dot_bound)
+        if key not in self._plans:
+            log2e, dev, H = 1.4426950408889634, self.mix.device, self.temp.numel()
+            T, temp, cap = self.mix.double(), self.temp.double(), self.softcap
+            near = (T @ self.rel.double()[self.bucket.long()].T) * log2e                      # [H, reach + 1], reference: the last distance
+            near = near - near[:, -1:]
+            top = torch.full_like(temp, cap) if dot_bound is None else cap * torch.tanh(dot_bound * abs(scale) * temp.abs() / cap)
+            reach = float((T.abs() @ top * log2e + near.abs().amax(1)).max())
+            if not reach <= 100.0:
+                self._plans[key] = None
+            else:
+                HT = 8 if H <= 8 else 16 if H <= 16 else 32
+                grow = lambda t, *n: torch.nn.functional.pad(t, [x for d, m in zip(reversed(t.shape), reversed(n)) for x in (0, m - d)]).float().contiguous()
+                w = grow(-2.0 * cap * log2e * T, HT, HT)
+                self._plans[key] = (w[..., None].expand(-1, -1, 2).contiguous(), grow(cap * log2e * T.sum(1), HT), grow(2.0 * log2e * scale * temp / cap, HT),
+                                    near.float().contiguous().to(dev))
+        return self._plans[key]
 
     def args(self, scale: float) -> _Scores:
         assert all(t.dtype == torch.float32 and t.is_contiguous() for t in (self.temp, self.rel, self.mix)) and self.bucket.dtype == torch.int32
@@ -129,14 +154,65 @@ def _general(q, k, v, kv_strides, scores: _Scores, out, pos, G, dk, dv, cap, rin
     return out
 
 
-def prompt_attention(q, k, v, *, scale: float, window: Optional[int] = None, talk: Optional[Talk] = None) -> torch.Tensor:
+def _rows_ok(*ts) -> bool:
+    """bf16 head rows that TMA and vector loads take: contiguous channels, strides that are multiples of 8, 16-byte aligned."""
+    return all(t.dtype == torch.bfloat16 and t.stride(3) == 1 and all(x % 8 == 0 for x in t.stride()[:3]) and t.data_ptr() % 16 == 0 for t in ts)
+
+
+def _keymajor_prompt(q, k, v, out, scale, talk: Talk, dot_bound) -> bool:
+    B, S, H, dk = q.shape
+    G, dv = k.shape[2], v.shape[3]
+    dvp = -(-dv // 8) * 8
+    if not _rows_ok(q, k, v) or v.stride(2) < dvp or not lib().tyr_keymajor_heads(0, H, G, dk, dv):
+        return False
+    plan = talk.plan(scale, dot_bound)
+    if plan is None:
+        return False
+    st = (ctypes.c_longlong * 12)(*[t.stride(i) for t in (q, k, v, out) for i in range(3)])
+    check(lib().tyr_keymajor_prompt(ptr(q), ptr(k), ptr(v), ptr(out), *(ptr(t) for t in plan), plan[3].shape[1] - 1, st, B, S, H, G, dk, dv, dvp,
+                                    ptr(err_word(q.device)), cur_stream(q.device)), "keymajor_prompt")
+    return True
+
+
+def _workspace(q, H, dv, splits):
+    key = (q.device.index, q.shape[0], H, dv, splits)
+    ws = _workspaces.get(key)
+    if ws is None and splits > 1:
+        ws = _workspaces[key] = torch.zeros(lib().tyr_joint_step_workspace_bytes(q.shape[0], H, dv, splits) // 4, dtype=torch.int32, device=q.device)
+    return ws
+
+
+def _keymajor_step(q, store, pos, out, dv, scale, window, talk: Optional[Talk], dot_bound) -> bool:
+    B, _, H, dk = q.shape
+    G, cap, dvp = store.k.shape[1], store.cap, store.v.shape[3]
+    shared = store.v is store.k
+    if not _rows_ok(q, store.k, store.v) or not (store.k.is_contiguous() and store.v.is_contiguous()) or dk != store.k.shape[3] or shared != (talk is None):
+        return False
+    if store.ring and (talk is not None or (window is not None and window < cap)) or (talk is not None and window is not None):
+        return False
+    hb = lib().tyr_keymajor_heads(2 if shared else 1, H, G, dk, dv)
+    plan = (None,) * 4 if shared else talk.plan(scale, dot_bound)
+    if not hb or plan is None:
+        return False
+    splits = pick_splits(B, -(-H // hb), min(cap, window) if window else cap)
+    st = (ctypes.c_longlong * 4)(q.stride(0), q.stride(2), out.stride(0), out.stride(2))
+    check(lib().tyr_keymajor_step(ptr(q), ptr(store.k), ptr(store.v), ptr(out), ptr(pos), *(ptr(t) for t in plan), 0 if shared else plan[3].shape[1] - 1, scale,
+                                  ptr(_workspace(q, H, dv, splits)), st, B, H, G, dk, dv, dvp, cap, 1 if store.ring else 0, int(window or 0), splits,
+                                  ptr(err_word(q.device)), cur_stream(q.device)), "keymajor_step")
+    return True
+
+
+def prompt_attention(q, k, v, *, scale: float, window: Optional[int] = None, talk: Optional[Talk] = None,
+                     dot_bound: Optional[float] = None) -> torch.Tensor:
     """Whole prompts (rows may end earlier: padding at the end only feeds padding).  q: [B, S, H, dk], k: [B, S, G, dk], v: [B, S, G, dv]
-    -> [B, S, H * dv].  ``talk``: mixed scores."""
+    -> [B, S, H * dv].  ``talk``: mixed scores; ``dot_bound``: largest |q . k| there can be, where one is known (unit queries and keys)."""
     B, S, H, dk = q.shape
     G, dv = k.shape[2], v.shape[3]
     if q.is_cuda:
         out = torch.empty((B, S, H, dv), dtype=q.dtype, device=q.device)
         scores = _Scores(scale=scale) if talk is None else talk.args(scale)
+        if talk is not None and window is None and _keymajor_prompt(q, k, v, out, scale, talk, dot_bound):
+            return out.flatten(2)
         if talk is not None and window is None and _prompt_fused(q, k, v, talk):
             st = (ctypes.c_longlong * 6)(*[t.stride(i) for t in (q, k, v) for i in range(2)])
             check(lib().tyr_joint_prompt(ptr(q), ptr(k), ptr(v), ptr(out), ctypes.byref(scores), st, B, S, H, G, dk, dv, v.stride(2), cur_stream(q.device)),
@@ -153,7 +229,7 @@ def prompt_attention(q, k, v, *, scale: float, window: Optional[int] = None, tal
 
 
 def step_attention(q, store, pos: torch.Tensor, dv: int, *, scale: float, window: Optional[int] = None, talk: Optional[Talk] = None,
-                   out: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   out: Optional[torch.Tensor] = None, dot_bound: Optional[float] = None) -> torch.Tensor:
     """One token per row against a ``KVCache`` (plain or ring) that holds it.  q: [B, 1, H, dk]; pos: int32 [B]; ``dv`` value channels (of
     a shared store: the first of the keys) -> [B, 1, H, dv], into ``out`` (a view with contiguous channels) if given."""
     B, _, H, dk = q.shape
@@ -163,13 +239,12 @@ def step_attention(q, store, pos: torch.Tensor, dv: int, *, scale: float, window
     if q.is_cuda:
         st = tuple(t.stride(i) for t in (store.k, store.v) for i in (0, 2, 1))
         scores = _Scores(scale=scale) if talk is None else talk.args(scale)
+        if _keymajor_step(q, store, pos, out, dv, scale, window, talk, dot_bound):
+            return out
         hb = _step_heads(q, store, dv, talk)
         if hb:
             splits = pick_splits(B, -(-H // hb), min(cap, window) if window else cap)
-            key = (q.device.index, B, H, dv, splits)
-            ws = _workspaces.get(key)
-            if ws is None and splits > 1:
-                ws = _workspaces[key] = torch.zeros(lib().tyr_joint_step_workspace_bytes(B, H, dv, splits) // 4, dtype=torch.int32, device=q.device)
+            ws = _workspace(q, H, dv, splits)
             so = (ctypes.c_longlong * 4)(q.stride(0), q.stride(2), out.stride(0), out.stride(2))
             check(lib().tyr_joint_step(ptr(q), ptr(store.k), None if talk is None else ptr(store.v), ptr(out), ptr(pos), ctypes.byref(scores), ptr(ws), so, B, H, G,
                                        dk, dv, store.v.shape[3], cap, 1 if store.ring else 0, int(window or 0), splits, ptr(err_word(q.device)),
