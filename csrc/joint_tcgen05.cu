@@ -23,6 +23,8 @@
 // score is softcap (1 - 2 r), and in log2 units
 //   score_h - reference_h = init_h + near_h[distance] + sum_g w[h, g] r_g.
 // Latent scores take an online softmax whose reference moves only when a maximum grew by more than 2^8.
+#include <string.h>
+
 #include "mma_sync.cuh"
 
 namespace tyr {
@@ -43,22 +45,28 @@ struct KmArgs {
   int rn, nq, cols;                            // columns of a key/value head, queries, columns in all (G rn)
   int kp, vp, mb;                              // pieces of a key and of a value, 128-channel blocks of a value
   int pps, slots;                              // pieces of a ring slot, slots
+  int lq;                                      // log2 of nq
   int hb;                                      // latent: heads of a CTA
   int cap, ring, window, splits;
-  // mixed heads: w pairs (w, w) [HT, HT], init and k2 [HT], near [H, reach + 1]
-  const float *w2, *init, *k2, *near;
+  const float* near;                           // mixed heads: [H, reach + 1]
   int reach;
+  uint16_t col[32];                            // first column of a head
+  uint32_t prow[32];                           // and the byte offset of its row of probabilities
   float scale_log2;                            // latent
-  float *part_acc, *part_ml;                   // [B, splits, H, dv], [B, splits, H, 2]
-  int* counters;                               // [B, blocks of heads]
+  float *part_acc, *part_ml;                   // [B, splits, H, dv], [B, splits, H, 2]: merged by a launch of its own
   int* err;
+};
+
+// Mixed heads: w [HT, HT], init and k2 [HT] of the scores above.  Kernel parameters, so that the arithmetic takes them as constants.
+template <int HT>
+struct KmTalk {
+  float w[HT * HT], init[HT], k2[HT];
 };
 
 struct KmBars {
   uint64_t full[KM_SLOTS], empty[KM_SLOTS], s_ready[2], p_ready, p_free, o_done, l_ready, wg;
   uint32_t tmem_base;
   int rescale_at;                              // latent: tile at which the sums and O were last scaled by `factor`
-  int last;
 };
 
 // Byte offsets from a 1024-byte aligned base.
@@ -86,21 +94,11 @@ __device__ __forceinline__ void km_ld(uint32_t addr, uint32_t* r) {
   if constexpr (N == 4)
     asm volatile("tcgen05.ld.sync.aligned.32x32b.x4.b32 {%0, %1, %2, %3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
 }
-__device__ __forceinline__ uint64_t km_pack(float x, float y) {
-  uint64_t r;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(x), "f"(y));
-  return r;
-}
-__device__ __forceinline__ void km_unpack(uint64_t v, float& x, float& y) { asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(v)); }
-__device__ __forceinline__ void km_fma2(uint64_t& c, uint64_t a, uint64_t b) { asm("fma.rn.f32x2 %0, %1, %2, %0;" : "+l"(c) : "l"(a), "l"(b)); }
-__device__ __forceinline__ void km_w2(const float* p, uint64_t& a, uint64_t& b) {
-  asm("ld.global.nc.v2.u64 {%0, %1}, [%2];" : "=l"(a), "=l"(b) : "l"(p));
-}
-
 // HT: heads a thread handles (padded), QB: queries it takes at a time, WGS: softmax warpgroups.
 template <int MODE, int HT, int QB, int WGS>
 __global__ void __launch_bounds__((WGS * 4 + 4) * 32, 1)
-joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const __grid_constant__ KmArgs a) {
+joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const __grid_constant__ KmArgs a,
+                      const __grid_constant__ KmTalk<HT> tk) {
   constexpr int SB = MODE == KM_PROMPT ? 1 : 2;            // score buffers
   constexpr int SOFT = WGS * 4, THREADS = (SOFT + 4) * 32;
   pdl_trigger();
@@ -126,7 +124,6 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
     mbar_init(&s.l_ready, 2);
     mbar_init(&s.wg, 4);
     s.rescale_at = -1;
-    s.last = 0;
     mbar_fence_init();
   }
   if (warp == SOFT) {
@@ -164,21 +161,30 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
   // ---- queries -> shared memory, K-major with the 128-byte swizzle: [key/value head][piece][column][64 channels]
   {
     const int chunks = a.kp * 8, n = a.cols * chunks;      // 16-byte chunks of a column
-    for (int x = tid; x < n; x += THREADS) {
-      const int col = x / chunks, c = x - col * chunks, g = col / a.rn, r = col - g * a.rn;
-      uint4 v = make_uint4(0u, 0u, 0u, 0u);
-      int h = 0, i = 0;
-      bool live;
-      if constexpr (MODE == KM_PROMPT) {
-        h = g * a.rep + r / a.nq;
-        i = i0 + r % a.nq;
-        live = r / a.nq < a.rep && i < a.S;
-      } else {
-        h = MODE == KM_LATENT ? h0 + r : g * a.rep + r;
-        live = r < (MODE == KM_LATENT ? nh : a.rep);
+    constexpr int U = 4;                                   // loads in flight
+    for (int x0 = tid; x0 < n; x0 += U * THREADS) {
+      uint4 v[U];
+      uint32_t at[U];
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int x = x0 + u * THREADS;
+        const int col = x / chunks, c = x - col * chunks, g = col / a.rn, r = col - g * a.rn;
+        int h, i = 0;
+        bool live = x < n && valid && c * 8 < a.dk;
+        if constexpr (MODE == KM_PROMPT) {
+          h = g * a.rep + (r >> a.lq);
+          i = i0 + (r & (a.nq - 1));
+          live = live && (r >> a.lq) < a.rep && i < a.S;
+        } else {
+          h = MODE == KM_LATENT ? h0 + r : g * a.rep + r;
+          live = live && r < (MODE == KM_LATENT ? nh : a.rep);
+        }
+        at[u] = lay.q + (static_cast<uint32_t>(g * a.kp + (c >> 3)) * a.rn + r) * 128 + (((c & 7) ^ (r & 7)) << 4);
+        v[u] = live ? *reinterpret_cast<const uint4*>(a.q + b * a.q_sb + i * a.q_ss + h * a.q_sh + c * 8) : make_uint4(0u, 0u, 0u, 0u);
       }
-      if (live && valid && c * 8 < a.dk) v = *reinterpret_cast<const uint4*>(a.q + b * a.q_sb + i * a.q_ss + h * a.q_sh + c * 8);
-      *reinterpret_cast<uint4*>(smem + lay.q + (static_cast<uint32_t>(g * a.kp + (c >> 3)) * a.rn + r) * 128 + (((c & 7) ^ (r & 7)) << 4)) = v;
+#pragma unroll
+      for (int u = 0; u < U; ++u)
+        if (x0 + u * THREADS < n) *reinterpret_cast<uint4*>(smem + at[u]) = v[u];
     }
     if (MODE == KM_LATENT)
       for (int x = tid; x < a.cols; x += THREADS) { sm_m[x] = -INFINITY; sm_f[x] = 1.f; }
@@ -279,29 +285,35 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
     float acc[KM_COLS / 32][4];
 #pragma unroll
     for (int x = 0; x < KM_COLS / 32; ++x) acc[x][0] = acc[x][1] = acc[x][2] = acc[x][3] = 0.f;
+    uint32_t row[KM_COLS / 32];                            // this lane's row of every 16-row block
+#pragma unroll
+    for (int x = 0; x < KM_COLS / 32; ++x) {
+      const int n = (2 * x + w) * 16 + (lane & 15), gg = n / a.rn;
+      row[x] = lay.p + static_cast<uint32_t>(gg) * a.rn * 256 + (n - gg * a.rn) * 128;
+    }
     bool ok = true;
     for (int j = 0; j < tiles && ok; ++j) {
       ok = mbar_wait(&s.p_ready, j & 1, a.err, 2630 + w);
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
-      const bool scale = MODE == KM_LATENT && *reinterpret_cast<volatile int*>(&s.rescale_at) == j;
+      if (MODE == KM_LATENT && *reinterpret_cast<volatile int*>(&s.rescale_at) == j) {
 #pragma unroll
-      for (int x = 0; x < KM_COLS / 32; ++x) {
-        const int n0 = (2 * x + w) * 16;
-        if (n0 >= a.cols) break;
-        if (scale) {
-          const float f0 = sm_f[n0 + g8], f1 = sm_f[n0 + g8 + 8];
-          acc[x][0] *= f0; acc[x][2] *= f1;
-        }
-        const int n = n0 + (lane & 15), gg = n0 / a.rn;
-        const uint8_t* row = smem + lay.p + static_cast<uint32_t>(gg) * a.rn * 256 + (n - gg * a.rn) * 128;
+        for (int x = 0; x < KM_COLS / 32; ++x)
+          if ((2 * x + w) * 16 < a.cols) {
+            acc[x][0] *= sm_f[(2 * x + w) * 16 + g8];
+            acc[x][2] *= sm_f[(2 * x + w) * 16 + g8 + 8];
+          }
+      }
 #pragma unroll
-        for (int k = 0; k < 8; ++k) {
+      for (int k = 0; k < 8; ++k)
+#pragma unroll
+        for (int x = 0; x < KM_COLS / 32; ++x) {
+          const int n0 = (2 * x + w) * 16;
+          if (n0 >= a.cols) break;
           uint32_t f[4];
-          ldsm4(f, row + (k >> 2) * a.rn * 128 + ((((k & 3) * 2 + (lane >> 4)) ^ (n & 7)) << 4));
+          ldsm4(f, smem + row[x] + (k >> 2) * a.rn * 128 + ((((k & 3) * 2 + (lane >> 4)) ^ (lane & 7)) << 4));
           mma_bf16(acc[x], f, 0x3f803f80u, 0x3f803f80u);
         }
-      }
       __syncwarp();
       if (lane == 0) mbar_arrive(&s.p_free);
     }
@@ -313,8 +325,9 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
       for (int x = 0; x < KM_COLS / 32; ++x) {
         const int n0 = (2 * x + w) * 16;
         if (n0 < a.cols && (lane & 3) == 0) {
-          sm_l[n0 + g8] = acc[x][0];
-          sm_l[n0 + g8 + 8] = acc[x][2];
+          const bool part = MODE != KM_PROMPT && a.splits > 1;        // parts keep the sums, results their reciprocals
+          sm_l[n0 + g8] = part ? acc[x][0] : 1.f / acc[x][0];
+          sm_l[n0 + g8 + 8] = part ? acc[x][2] : 1.f / acc[x][2];
         }
       }
     }
@@ -341,68 +354,49 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
       };
       if constexpr (MODE != KM_LATENT) {
         const int nqw = MODE == KM_PROMPT ? a.nq / WGS : 1, q_first = MODE == KM_PROMPT ? wg * nqw : 0;
-        const int stride = a.nq;                                                    // columns of a head
         const int i_first = MODE == KM_PROMPT ? i0 + q_first : n_keys - 1;          // position of the first query
         const int tile_end = lo + j * KM_KEYS + KM_KEYS - 1;
         const bool far = i_first - tile_end >= a.reach, edge = MODE == KM_PROMPT ? tile_end > i_first : tile_end >= hi;
         for (int qb = 0; qb < nqw; qb += QB) {
           const int q0 = q_first + qb;
-          uint32_t x[HT][QB];
+          float y[HT][QB];
           {
-            int g = 0, r = 0;
+            uint32_t x[HT][QB];
 #pragma unroll
-            for (int h = 0; h < HT; ++h) {
-              km_ld<QB>(s_addr + g * a.rn + r * stride + q0, x[h]);
-              if (h + 1 < a.H && ++r == a.rep) { r = 0; ++g; }
-            }
-          }
-          tmem_wait_ld();
-          uint64_t y[HT][(QB + 1) / 2];
+            for (int h = 0; h < HT; ++h) km_ld<QB>(s_addr + a.col[h] + q0, x[h]);      // heads past the last: the last again
+            tmem_wait_ld();
 #pragma unroll
-          for (int h = 0; h < HT; ++h) {
-            const float k2 = __ldg(a.k2 + h);
-            float v[QB];
+            for (int h = 0; h < HT; ++h)
 #pragma unroll
-            for (int e = 0; e < QB; ++e) v[e] = rcp(1.f + ex2(__uint_as_float(x[h][e]) * k2));
-#pragma unroll
-            for (int e = 0; e < QB; e += 2) y[h][e / 2] = km_pack(v[e], QB > 1 ? v[e + (QB > 1)] : 0.f);
+              for (int e = 0; e < QB; ++e) y[h][e] = rcp(1.f + ex2(__uint_as_float(x[h][e]) * tk.k2[h]));
           }
           if (qb == 0 && !(ok = p_writable())) break;
-          int g = 0, r = 0;
-#pragma unroll 1
-          for (int h = 0; h < a.H; ++h) {
-            const float init = __ldg(a.init + h);
-            uint64_t c[(QB + 1) / 2];
+          uint32_t off[QB];
 #pragma unroll
-            for (int e = 0; e < QB; e += 2) c[e / 2] = km_pack(init, init);
-            const float* w = a.w2 + h * HT * 2;
+          for (int e = 0; e < QB; ++e) off[e] = (q0 + e) * 128 + (p_off ^ (((q0 + e) & 7) << 4));
 #pragma unroll
-            for (int k = 0; k < HT; k += 2) {
-              uint64_t wa, wb;
-              km_w2(w + k * 2, wa, wb);
+          for (int h = 0; h < HT; ++h) {
+            if (h >= a.H) break;
+            float c[QB];
 #pragma unroll
-              for (int e = 0; e < (QB + 1) / 2; ++e) {
-                km_fma2(c[e], y[k][e], wa);
-                km_fma2(c[e], y[k + 1][e], wb);
-              }
+            for (int e = 0; e < QB; ++e) c[e] = tk.init[h];
+#pragma unroll
+            for (int k = 0; k < HT; ++k)
+#pragma unroll
+              for (int e = 0; e < QB; ++e) c[e] = fmaf(y[k][e], tk.w[h * HT + k], c[e]);
+            if (!far) {
+              const float* nr = a.near + static_cast<long long>(h) * (a.reach + 1);
+#pragma unroll
+              for (int e = 0; e < QB; ++e) c[e] += __ldg(nr + min(max(i_first + qb + e - kj, 0), a.reach));
             }
-            uint8_t* dst = p_row + static_cast<uint32_t>(g) * a.rn * 256;
+            uint8_t* const dst = p_row + a.prow[h];
 #pragma unroll
-            for (int e = 0; e < QB; e += 2) {
-              float v[2];
-              km_unpack(c[e / 2], v[0], v[1]);
-#pragma unroll
-              for (int z = 0; z < 2; ++z) {
-                if (e + z >= QB) break;
-                const int d = i_first + qb + e + z - kj;                            // distance of query and key
-                if (!far) v[z] += __ldg(a.near + static_cast<long long>(h) * (a.reach + 1) + min(max(d, 0), a.reach));
-                v[z] = ex2(v[z]);
-                if (edge && (MODE == KM_PROMPT ? d < 0 : kj >= hi)) v[z] = 0.f;
-                const int n = r * stride + q0 + e + z;
-                *reinterpret_cast<__nv_bfloat16*>(dst + n * 128 + (p_off ^ ((n & 7) << 4))) = __float2bfloat16(v[z]);
-              }
+            for (int e = 0; e < QB; ++e) {
+              float v = ex2(c[e]);
+              if (edge && (MODE == KM_PROMPT ? i_first + qb + e < kj : kj >= hi)) v = 0.f;
+              // a single query: the swizzle follows the head's row
+              *reinterpret_cast<__nv_bfloat16*>(dst + (MODE == KM_STEP ? p_off ^ ((a.prow[h] >> 3) & 0x70) : off[e])) = __float2bfloat16(v);
             }
-            if (++r == a.rep) { r = 0; ++g; }
           }
         }
         if (!ok) break;
@@ -494,26 +488,26 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
             if (tiles > 0) {
               tmem_ld_32x16(o_base + lane_addr + (g * a.mb + m) * a.rn + n0, o);
               tmem_wait_ld();
+            } else {
+#pragma unroll
+              for (int e = 0; e < 16; ++e) o[e] = 0u;
             }
+            if (d >= a.dv) continue;
+            const float* l = sm_l + g * a.rn + n0;
 #pragma unroll
             for (int e = 0; e < 16; ++e) {
               const int n = n0 + e;
-              const float l = sm_l[g * a.rn + n], v = tiles > 0 ? __uint_as_float(o[e]) : 0.f;
               if constexpr (MODE == KM_PROMPT) {
-                const int r = n / a.nq, i = i0 + n % a.nq;
-                if (r < a.rep && i < a.S && d < a.dv) a.out[b * a.out_sb + i * a.out_ss + (g * a.rep + r) * a.out_sh + d] = __float2bfloat16(__fdividef(v, l));
+                const int r = n >> a.lq, i = i0 + (n & (a.nq - 1));
+                if (r < a.rep && i < a.S) a.out[b * a.out_sb + i * a.out_ss + (g * a.rep + r) * a.out_sh + d] = __float2bfloat16(__uint_as_float(o[e]) * l[e]);
               } else {
-                const int h = MODE == KM_LATENT ? n : g * a.rep + n;
-                if (n < (MODE == KM_LATENT ? nh : a.rep)) {
-                  if (a.splits == 1) {
-                    if (d < a.dv) a.out[b * a.out_sb + (h0 + h) * a.out_sh + d] = __float2bfloat16(__fdividef(v, l));
-                  } else {
-                    if (d < a.dv) a.part_acc[(part * a.H + h0 + h) * a.dv + d] = v;
-                    if (d == 0) {
-                      a.part_ml[(part * a.H + h0 + h) * 2] = MODE == KM_LATENT ? sm_m[n] : 0.f;
-                      a.part_ml[(part * a.H + h0 + h) * 2 + 1] = tiles > 0 ? l : 0.f;
-                    }
-                  }
+                const int h = h0 + (MODE == KM_LATENT ? n : g * a.rep + n);
+                if (n >= (MODE == KM_LATENT ? nh : a.rep)) break;
+                if (a.splits == 1) a.out[b * a.out_sb + h * a.out_sh + d] = __float2bfloat16(__uint_as_float(o[e]) * l[e]);
+                else a.part_acc[(part * a.H + h) * a.dv + d] = __uint_as_float(o[e]);
+                if (a.splits > 1 && d == 0) {
+                  a.part_ml[(part * a.H + h) * 2] = MODE == KM_LATENT ? sm_m[n] : 0.f;
+                  a.part_ml[(part * a.H + h) * 2 + 1] = l[e];
                 }
               }
             }
@@ -522,36 +516,32 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
     }
   }
   tc_fence_before();
-  if (MODE != KM_PROMPT && a.splits > 1) __threadfence();
   __syncthreads();
   if (warp == SOFT) {
     tc_fence_after();
     tmem_dealloc(tmem, 512);
   }
-  if constexpr (MODE != KM_PROMPT) {
-    if (a.splits == 1 || !valid) return;
-    if (tid == 0) s.last = atomicAdd(a.counters + b * gridDim.y + blockIdx.y, 1) == a.splits - 1;
-    __syncthreads();
-    if (!s.last) return;
-    __threadfence();
-    float* const w = reinterpret_cast<float*>(smem + lay.q);            // [nh, splits] weights of the slices
-    for (int h = warp; h < nh; h += THREADS / 32) {
-      const float* src = a.part_ml + (static_cast<long long>(b) * a.splits * a.H + h0 + h) * 2;
-      const float mx = lane < a.splits ? __ldcg(src + static_cast<long long>(lane) * a.H * 2) : -INFINITY;
-      const float lx = lane < a.splits ? __ldcg(src + static_cast<long long>(lane) * a.H * 2 + 1) : 0.f;
-      const float M = warp_max(mx), f = ex2(mx - M), L = warp_sum(f * lx);
-      if (lane < a.splits) w[h * a.splits + lane] = f / L;
-    }
-    __syncthreads();
-    for (int x = tid; x < nh * a.dv; x += THREADS) {
-      const int h = x / a.dv, d = x - h * a.dv;
-      const float* src = a.part_acc + (static_cast<long long>(b) * a.splits * a.H + h0 + h) * a.dv + d;
-      float v = 0.f;
+}
+
+// Slices of a step -> result: one CTA per (row, head), a thread per channel.
+__global__ void __launch_bounds__(128) joint_merge_kernel(const float* __restrict__ acc, const float* __restrict__ ml, __nv_bfloat16* __restrict__ out, int H, int dv,
+                                                          int splits, long long out_sb, long long out_sh) {
+  __shared__ float w[32];
+  pdl_entry();
+  const int h = blockIdx.x, b = blockIdx.y, lane = threadIdx.x & 31;
+  if (threadIdx.x < 32) {
+    const float* src = ml + ((static_cast<long long>(b) * splits + lane) * H + h) * 2;
+    const float mx = lane < splits ? src[0] : -INFINITY, lx = lane < splits ? src[1] : 0.f;
+    const float M = warp_max(mx), f = ex2(mx - M), L = warp_sum(f * lx);
+    w[lane] = f / L;
+  }
+  __syncthreads();
+  for (int d = threadIdx.x; d < dv; d += 128) {
+    const float* src = acc + (static_cast<long long>(b) * splits * H + h) * dv + d;
+    float v = 0.f;
 #pragma unroll 8
-      for (int i = 0; i < a.splits; ++i) v += w[h * a.splits + i] * __ldcg(src + static_cast<long long>(i) * a.H * a.dv);
-      a.out[b * a.out_sb + (h0 + h) * a.out_sh + d] = __float2bfloat16(v);
-    }
-    if (tid == 0) a.counters[b * gridDim.y + blockIdx.y] = 0;
+    for (int i = 0; i < splits; ++i) v += w[i] * src[static_cast<long long>(i) * H * dv];
+    out[b * out_sb + h * out_sh + d] = __float2bfloat16(v);
   }
 }
 
@@ -616,15 +606,23 @@ bool km_plan(int mode, KmArgs& a) {
     a.rn = (a.rep + 15) / 16 * 16;
     return fits(2);
   }
-  for (a.nq = 32; a.nq >= 8; a.nq /= 2) {
+  for (a.nq = 32, a.lq = 5; a.nq >= 8; a.nq /= 2, --a.lq) {
     a.rn = (a.rep * a.nq + 15) / 16 * 16;
     if (fits(2)) return true;
   }
   return false;
 }
 
+// `talk`: on the host, w [HT, HT], init [HT], k2 [HT] (null for latent rows).
 template <int MODE, int HT, int QB, int WGS>
-int km_launch(const CUtensorMap& tk, const CUtensorMap& tv, const KmArgs& a, dim3 grid, void* stream) {
+int km_launch(const CUtensorMap& tk, const CUtensorMap& tv, KmArgs& a, const float* talk, dim3 grid, void* stream) {
+  KmTalk<HT> t{};
+  if (talk != nullptr) memcpy(&t, talk, sizeof(t));
+  for (int h = 0; h < HT && MODE != KM_LATENT; ++h) {
+    const int x = h < a.H ? h : a.H - 1, g = x / a.rep, r = x % a.rep;
+    a.col[h] = static_cast<uint16_t>(g * a.rn + r * a.nq);
+    a.prow[h] = static_cast<uint32_t>(g) * a.rn * 256 + r * a.nq * 128;
+  }
   auto kernel = joint_keymajor_kernel<MODE, HT, QB, WGS>;
   static bool configured[64] = {};               // the attribute is per device
   int dev = 0;
@@ -635,7 +633,7 @@ int km_launch(const CUtensorMap& tk, const CUtensorMap& tv, const KmArgs& a, dim
     configured[dev] = true;
   }
   const size_t smem = KmLayout(MODE, a.cols, a.kp, a.pps, a.slots).total + 1024;
-  return (int)launch_dependent(kernel, grid, dim3((WGS * 4 + 4) * 32), smem, (cudaStream_t)stream, tk, tv, a);
+  return (int)launch_dependent(kernel, grid, dim3((WGS * 4 + 4) * 32), smem, (cudaStream_t)stream, tk, tv, a, t);
 }
 }  // namespace
 
@@ -648,54 +646,59 @@ extern "C" TYR_EXPORT int tyr_keymajor_heads(int mode, int H, int G, int dk, int
 }
 
 // Mixed heads over whole bf16 prompts.  strides: (batch, token, head) of q, k, v, out; dk multiple of 16, dv of 8, 16-byte aligned rows.
-// w2 [HT, HT] pairs, init and k2 [HT] with HT = 8, 16 or 32, the smallest that holds H; near [H, reach + 1].
-extern "C" TYR_EXPORT int tyr_keymajor_prompt(const void* q, const void* k, const void* v, void* out, const float* w2, const float* init,
-                                              const float* k2, const float* near, int reach, const long long* st, int B, int S, int H, int G,
+// `talk` lies on the host: w [HT, HT], init [HT], k2 [HT] with HT = 8, 16 or 32, the smallest that holds H; near [H, reach + 1] on the device.
+extern "C" TYR_EXPORT int tyr_keymajor_prompt(const void* q, const void* k, const void* v, void* out, const float* talk, const float* near, int reach, const long long* st, int B, int S, int H, int G,
                                               int dk, int dv, int dvp, int* err, void* stream) {
   KmArgs a{};
   a.H = H; a.G = G; a.dk = dk; a.dv = dv; a.splits = 1;
   if (B <= 0 || B > 65535 || S <= 0 || dv > dvp || (dvp & 7) || reach < 0 || !km_plan(KM_PROMPT, a)) return -1;
   for (int i = 0; i < 9; ++i)
     if (st[i] & 7) return -3;
-  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v) | reinterpret_cast<uintptr_t>(w2)) & 15) return -4;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v)) & 15) return -4;
   a.q = (const __nv_bfloat16*)q; a.out = (__nv_bfloat16*)out; a.S = S; a.err = err;
   a.q_sb = st[0]; a.q_ss = st[1]; a.q_sh = st[2]; a.out_sb = st[9]; a.out_ss = st[10]; a.out_sh = st[11];
-  a.w2 = w2; a.init = init; a.k2 = k2; a.near = near; a.reach = reach;
+  a.near = near; a.reach = reach;
   CUtensorMap tk, tv;
   if (int r = km_map(&tk, k, dk, G, S, B, st[5], st[4], st[3])) return 3000 + r;
   if (int r = km_map(&tv, v, dvp, G, S, B, st[8], st[7], st[6])) return 4000 + r;
   const dim3 grid((S + a.nq - 1) / a.nq, B);
-  return H <= 8 ? km_launch<KM_PROMPT, 8, 4, 2>(tk, tv, a, grid, stream)
-                : (H <= 16 ? km_launch<KM_PROMPT, 16, 4, 2>(tk, tv, a, grid, stream) : km_launch<KM_PROMPT, 32, 2, 2>(tk, tv, a, grid, stream));
+  return H <= 8 ? km_launch<KM_PROMPT, 8, 4, 2>(tk, tv, a, talk, grid, stream)
+                : (H <= 16 ? km_launch<KM_PROMPT, 16, 4, 2>(tk, tv, a, talk, grid, stream) : km_launch<KM_PROMPT, 32, 2, 2>(tk, tv, a, talk, grid, stream));
 }
 
-// One token per row over bf16 stores that hold it.  w2 null: latent rows [B, 1, cap, dk] whose first dv channels are the values of all
+// One token per row over bf16 stores that hold it.  talk null: latent rows [B, 1, cap, dk] whose first dv channels are the values of all
 // heads (a ring must hold exactly the window), scale; else mixed heads over stores [B, G, cap, dk] and [B, G, cap, dvp].  strides:
-// (batch, head) of q, then of out.  The workspace (tyr_joint_step_workspace_bytes) must be zero-filled once.
-extern "C" TYR_EXPORT int tyr_keymajor_step(const void* q, const void* k, const void* v, void* out, const int* pos, const float* w2,
-                                            const float* init, const float* k2, const float* near, int reach, float scale, void* workspace,
+// (batch, head) of q, then of out.  workspace: [B, splits, H, dv + 2] floats where splits > 1.
+extern "C" TYR_EXPORT int tyr_keymajor_step(const void* q, const void* k, const void* v, void* out, const int* pos, const float* talk,
+                                            const float* near, int reach, float scale, void* workspace,
                                             const long long* st, int B, int H, int G, int dk, int dv, int dvp, int cap, int ring, int window,
                                             int splits, int* err, void* stream) {
   KmArgs a{};
-  const int mode = w2 == nullptr ? KM_LATENT : KM_STEP;
+  const int mode = talk == nullptr ? KM_LATENT : KM_STEP;
   a.H = H; a.G = G; a.dk = dk; a.dv = dv; a.splits = splits;
   if (B <= 0 || B > 65535 || cap <= 0 || window < 0 || reach < 0 || dv > dvp || (dvp & 7) || !km_plan(mode, a)) return -1;
   if ((mode == KM_STEP && (ring || window)) || (ring && window && window < cap) || (splits > 1 && workspace == nullptr)) return -2;
-  if (((st[0] | st[1]) & 7) || ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v) | reinterpret_cast<uintptr_t>(w2)) & 15))
+  if (((st[0] | st[1]) & 7) || ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v)) & 15))
     return -3;
   a.q = (const __nv_bfloat16*)q; a.out = (__nv_bfloat16*)out; a.pos = pos; a.err = err;
   a.q_sb = st[0]; a.q_sh = st[1]; a.out_sb = st[2]; a.out_sh = st[3];
-  a.w2 = w2; a.init = init; a.k2 = k2; a.near = near; a.reach = reach;
+  a.near = near; a.reach = reach;
   a.scale_log2 = scale * 1.4426950408889634f;
   a.cap = cap; a.ring = ring; a.window = window;
   a.part_acc = (float*)workspace;
   a.part_ml = a.part_acc + static_cast<long long>(B) * H * splits * dv;
-  a.counters = (int*)(a.part_ml + static_cast<long long>(B) * H * splits * 2);
   CUtensorMap tk, tv;
   if (int r = km_map(&tk, k, dk, G, cap, B, static_cast<long long>(cap) * dk, dk, static_cast<long long>(G) * cap * dk)) return 3000 + r;
   if (int r = km_map(&tv, v, dvp, G, cap, B, static_cast<long long>(cap) * dvp, dvp, static_cast<long long>(G) * cap * dvp)) return 4000 + r;
-  if (mode == KM_LATENT) return km_launch<KM_LATENT, 8, 1, 1>(tk, tv, a, dim3(splits, (H + a.hb - 1) / a.hb, B), stream);
-  const dim3 grid(splits, 1, B);
-  return H <= 8 ? km_launch<KM_STEP, 8, 1, 1>(tk, tv, a, grid, stream)
-                : (H <= 16 ? km_launch<KM_STEP, 16, 1, 1>(tk, tv, a, grid, stream) : km_launch<KM_STEP, 32, 1, 1>(tk, tv, a, grid, stream));
+  int rc;
+  if (mode == KM_LATENT) {
+    rc = km_launch<KM_LATENT, 8, 1, 1>(tk, tv, a, nullptr, dim3(splits, (H + a.hb - 1) / a.hb, B), stream);
+  } else {
+    const dim3 grid(splits, 1, B);
+    rc = H <= 8 ? km_launch<KM_STEP, 8, 1, 1>(tk, tv, a, talk, grid, stream)
+                : (H <= 16 ? km_launch<KM_STEP, 16, 1, 1>(tk, tv, a, talk, grid, stream) : km_launch<KM_STEP, 32, 1, 1>(tk, tv, a, talk, grid, stream));
+  }
+  if (rc != 0 || splits == 1) return rc;
+  return (int)launch_dependent(joint_merge_kernel, dim3(H, B), dim3(128), 0, (cudaStream_t)stream, static_cast<const float*>(a.part_acc),
+                               static_cast<const float*>(a.part_ml), a.out, H, dv, splits, a.out_sb, a.out_sh);
 }

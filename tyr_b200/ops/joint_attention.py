@@ -30,8 +30,8 @@ def _sigs(lib_):
     for name, args in (("tyr_joint_attention", [P, P, P, P, P, S, LL] + [I] * 11 + [P, P]), ("tyr_joint_prompt_form", [I] * 6),
                        ("tyr_joint_prompt", [P, P, P, P, S, LL] + [I] * 7 + [P]), ("tyr_joint_step_heads", [I] * 8),
                        ("tyr_joint_step", [P, P, P, P, P, S, P, LL] + [I] * 10 + [P, P]), ("tyr_keymajor_heads", [I] * 5),
-                       ("tyr_keymajor_prompt", [P] * 8 + [I, LL] + [I] * 7 + [P, P]),
-                       ("tyr_keymajor_step", [P] * 9 + [I, ctypes.c_float, P, LL] + [I] * 10 + [P, P])):
+                       ("tyr_keymajor_prompt", [P] * 6 + [I, LL] + [I] * 7 + [P, P]),
+                       ("tyr_keymajor_step", [P] * 7 + [I, ctypes.c_float, P, LL] + [I] * 10 + [P, P])):
         fn = getattr(lib_, name, None)
         if fn is not None:
             fn.argtypes, fn.restype = args, I
@@ -76,7 +76,7 @@ class Talk:
 
     def plan(self, scale: float, dot_bound: Optional[float]):
         """The scores in log2 units against a fixed reference, score_h - reference_h = init_h + near_h[distance] + sum_g w[h, g] / (1 + exp2(k2_g x)):
-        (w as pairs [HT, HT, 2], init [HT], k2 [HT], near [H, reach + 1]), or None where their range could leave fp32 exponents.
+        (w [HT, HT], init [HT] and k2 [HT] in one host tensor, near [H, reach + 1]), or None where their range could leave fp32 exponents.
         ``dot_bound``: largest |q . k| (None: only the cap bounds a score)."""
         key = (scale, dot_bound)
         if key not in self._plans:
@@ -90,10 +90,9 @@ class Talk:
                 self._plans[key] = None
             else:
                 HT = 8 if H <= 8 else 16 if H <= 16 else 32
-                grow = lambda t, *n: torch.nn.functional.pad(t, [x for d, m in zip(reversed(t.shape), reversed(n)) for x in (0, m - d)]).float().contiguous()
-                w = grow(-2.0 * cap * log2e * T, HT, HT)
-                self._plans[key] = (w[..., None].expand(-1, -1, 2).contiguous(), grow(cap * log2e * T.sum(1), HT), grow(2.0 * log2e * scale * temp / cap, HT),
-                                    near.float().contiguous().to(dev))
+                grow = lambda t, *n: torch.nn.functional.pad(t, [x for d, m in zip(reversed(t.shape), reversed(n)) for x in (0, m - d)]).flatten()
+                host = torch.cat([grow(-2.0 * cap * log2e * T, HT, HT), grow(cap * log2e * T.sum(1), HT), grow(2.0 * log2e * scale * temp / cap, HT)])
+                self._plans[key] = (host.float().cpu().contiguous(), near.float().contiguous().to(dev))
         return self._plans[key]
 
     def args(self, scale: float) -> _Scores:
@@ -169,7 +168,7 @@ def _keymajor_prompt(q, k, v, out, scale, talk: Talk, dot_bound) -> bool:
     if plan is None:
         return False
     st = (ctypes.c_longlong * 12)(*[t.stride(i) for t in (q, k, v, out) for i in range(3)])
-    check(lib().tyr_keymajor_prompt(ptr(q), ptr(k), ptr(v), ptr(out), *(ptr(t) for t in plan), plan[3].shape[1] - 1, st, B, S, H, G, dk, dv, dvp,
+    check(lib().tyr_keymajor_prompt(ptr(q), ptr(k), ptr(v), ptr(out), *(ptr(t) for t in plan), plan[1].shape[1] - 1, st, B, S, H, G, dk, dv, dvp,
                                     ptr(err_word(q.device)), cur_stream(q.device)), "keymajor_prompt")
     return True
 
@@ -191,12 +190,12 @@ def _keymajor_step(q, store, pos, out, dv, scale, window, talk: Optional[Talk], 
     if store.ring and (talk is not None or (window is not None and window < cap)) or (talk is not None and window is not None):
         return False
     hb = lib().tyr_keymajor_heads(2 if shared else 1, H, G, dk, dv)
-    plan = (None,) * 4 if shared else talk.plan(scale, dot_bound)
+    plan = (None,) * 2 if shared else talk.plan(scale, dot_bound)
     if not hb or plan is None:
         return False
     splits = pick_splits(B, -(-H // hb), min(cap, window) if window else cap)
     st = (ctypes.c_longlong * 4)(q.stride(0), q.stride(2), out.stride(0), out.stride(2))
-    check(lib().tyr_keymajor_step(ptr(q), ptr(store.k), ptr(store.v), ptr(out), ptr(pos), *(ptr(t) for t in plan), 0 if shared else plan[3].shape[1] - 1, scale,
+    check(lib().tyr_keymajor_step(ptr(q), ptr(store.k), ptr(store.v), ptr(out), ptr(pos), *(ptr(t) for t in plan), 0 if shared else plan[1].shape[1] - 1, scale,
                                   ptr(_workspace(q, H, dv, splits)), st, B, H, G, dk, dv, dvp, cap, 1 if store.ring else 0, int(window or 0), splits,
                                   ptr(err_word(q.device)), cur_stream(q.device)), "keymajor_step")
     return True
