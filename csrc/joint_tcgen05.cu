@@ -7,13 +7,13 @@
 // the scores of all heads for it in its own TMEM lane: mixing them is arithmetic on registers, and a few queries or heads leave no row
 // of the tensor core idle.
 //
-//   warps 0-3 (0-7 for prompts)   scores -> probabilities, written as bf16 to shared memory (the B operand of P V)
+//   warps 0-3 (0-15 for prompts)   scores -> probabilities, written as bf16 to shared memory (the B operand of P V)
 //   then one warp each            MMA issuer; TMA producer of [128 keys x 64 channels] pieces in a ring of slots of one or two pieces
 //   last two warps                row sums of the probabilities (mma.sync with a column of ones), so that numerator and denominator
 //                                 hold the same rounded numbers
 //
 // Modes:
-//   * mixed heads over prompts: a CTA takes up to 32 queries of all heads; its two softmax warpgroups take half of the queries each.
+//   * mixed heads over prompts: a CTA takes up to 32 queries of all heads; its softmax warpgroups share them.
 //   * mixed heads, one token per row: a slice of the keys.
 //   * latent rows, one token per row: up to 64 heads read one row per key, its first channels are the value; the rows pass through the
 //     ring twice, once for each product (the second time from L2).
@@ -64,7 +64,7 @@ struct KmTalk {
 };
 
 struct KmBars {
-  uint64_t full[KM_SLOTS], empty[KM_SLOTS], s_ready[2], p_ready, p_free, o_done, l_ready, wg;
+  uint64_t full[KM_SLOTS], empty[KM_SLOTS], q_ready, s_ready[2], s_free, p_ready, p_free, o_done, l_ready, wg;
   uint32_t tmem_base;
   int rescale_at;                              // latent: tile at which the sums and O were last scaled by `factor`
 };
@@ -84,6 +84,11 @@ struct KmLayout {
     // a value block of one piece: the MMA's upper 64 rows read whatever follows the slot (their results are not used)
     if (pps == 1 && total < q + KM_PIECE) total = q + KM_PIECE;
   }
+};
+
+template <bool V>
+struct KmFlag {
+  static constexpr bool value = V;
 };
 
 template <int N>
@@ -118,6 +123,8 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
     }
     mbar_init(&s.s_ready[0], 1);
     mbar_init(&s.s_ready[1], 1);
+    mbar_init(&s.q_ready, SOFT + 2);
+    mbar_init(&s.s_free, SOFT);
     mbar_init(&s.p_ready, SOFT);
     mbar_init(&s.p_free, 3);                               // P V retired, two summing warps
     mbar_init(&s.o_done, 1);
@@ -158,16 +165,29 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
     hi = min(lo + chunk, n_keys);
     tiles = valid ? (hi - lo + KM_KEYS - 1) / KM_KEYS : 0;
   }
-  // ---- queries -> shared memory, K-major with the 128-byte swizzle: [key/value head][piece][column][64 channels]
-  {
+  if (MODE == KM_LATENT)
+    for (int x = tid; x < a.cols; x += THREADS) { sm_m[x] = -INFINITY; sm_f[x] = 1.f; }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = s.tmem_base, o_base = tmem + SB * a.cols;
+  const uint32_t slot_bytes = a.pps * KM_PIECE, ring = smem_u32(smem + lay.ring);
+  const int ku = (a.kp + a.pps - 1) / a.pps;               // ring slots of one key
+  const int vpb = min(2, a.vp);                            // pieces of a 128-channel value block (the last may have fewer)
+
+  // ---- queries -> shared memory, K-major with the 128-byte swizzle: [key/value head][piece][column][64 channels]; by the softmax and
+  // summing warps, while the first keys are on their way
+  if (warp < SOFT || warp >= SOFT + 2) {
+    constexpr int STAGERS = (SOFT + 2) * 32;
+    const int me = warp < SOFT ? tid : tid - 64;
     const int chunks = a.kp * 8, n = a.cols * chunks;      // 16-byte chunks of a column
     constexpr int U = 4;                                   // loads in flight
-    for (int x0 = tid; x0 < n; x0 += U * THREADS) {
+    for (int x0 = me; x0 < n; x0 += U * STAGERS) {
       uint4 v[U];
       uint32_t at[U];
 #pragma unroll
       for (int u = 0; u < U; ++u) {
-        const int x = x0 + u * THREADS;
+        const int x = x0 + u * STAGERS;
         const int col = x / chunks, c = x - col * chunks, g = col / a.rn, r = col - g * a.rn;
         int h, i = 0;
         bool live = x < n && valid && c * 8 < a.dk;
@@ -184,19 +204,12 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
       }
 #pragma unroll
       for (int u = 0; u < U; ++u)
-        if (x0 + u * THREADS < n) *reinterpret_cast<uint4*>(smem + at[u]) = v[u];
+        if (x0 + u * STAGERS < n) *reinterpret_cast<uint4*>(smem + at[u]) = v[u];
     }
-    if (MODE == KM_LATENT)
-      for (int x = tid; x < a.cols; x += THREADS) { sm_m[x] = -INFINITY; sm_f[x] = 1.f; }
+    fence_proxy_async();
+    __syncwarp();
+    if (lane == 0) mbar_arrive(&s.q_ready);
   }
-  fence_proxy_async();
-  tc_fence_before();
-  __syncthreads();
-  tc_fence_after();
-  const uint32_t tmem = s.tmem_base, o_base = tmem + SB * a.cols;
-  const uint32_t slot_bytes = a.pps * KM_PIECE, ring = smem_u32(smem + lay.ring);
-  const int ku = (a.kp + a.pps - 1) / a.pps;               // ring slots of one key
-  const int vpb = min(2, a.vp);                            // pieces of a 128-channel value block (the last may have fewer)
 
   if (warp == SOFT + 1) {
     // ------------------------------------------------------------------ TMA producer
@@ -231,49 +244,61 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
     // ------------------------------------------------------------------ MMA issuer
     if (elect_one() && tiles > 0) {
       const uint32_t id_s = make_idesc_f16(1, 128, a.rn, 0, 0), id_o = make_idesc_f16(1, 128, a.rn, 1, 0);
-      const uint32_t q_addr = smem_u32(smem + lay.q), p_addr = smem_u32(smem + lay.p);
-      uint32_t it = 0;
-      bool ok = true;
+      // descriptors of the operands' first rows; the issuing thread only adds to their low words
+      const uint64_t dq = make_smem_desc_sw128(smem_u32(smem + lay.q), 16, 1024), dp = make_smem_desc_sw128(smem_u32(smem + lay.p), 16, 1024);
+      const uint64_t dk = make_smem_desc_sw128(ring, 16, 1024), dv = make_smem_desc_sw128(ring, KM_PIECE, 1024);
+      const uint32_t piece_q = a.rn * 128;                 // bytes of 64 channels (or keys) of a key/value head's columns
+      uint32_t st = 0, phase = 0;
+      bool ok = mbar_wait(&s.q_ready, 0, a.err, 2590);
       auto wait_slot = [&]() {
-        ok = ok && mbar_wait(&s.full[it % a.slots], (it / a.slots) & 1, a.err, 2600 + it % a.slots);
+        ok = ok && mbar_wait(&s.full[st], phase, a.err, 2600 + st);
         tc_fence_after();
-        return ring + (it % a.slots) * slot_bytes;
+        return st * slot_bytes;
+      };
+      auto free_slot = [&]() {
+        umma_commit(&s.empty[st]);
+        if (++st == static_cast<uint32_t>(a.slots)) { st = 0; phase ^= 1; }
       };
       auto scores = [&](int j) {
+        const uint32_t s_col = tmem + (SB == 2 ? (j & 1) * a.cols : 0);
         for (int g = 0; g < a.G && ok; ++g)
           for (int u = 0; u < ku && ok; ++u) {
-            const uint32_t k_addr = wait_slot();
+            const uint64_t ka = smem_desc_advance(dk, wait_slot());
             if (!ok) break;
             const int steps = min(a.pps * 4, (a.dk - u * a.pps * 64 + 15) / 16);
-            for (int k = 0; k < steps; ++k)
-              umma_f16_ss(tmem + (SB == 2 ? (j & 1) * a.cols : 0) + g * a.rn,
-                          make_smem_desc_sw128(k_addr + (k >> 2) * KM_PIECE + (k & 3) * 32, 16, 1024),
-                          make_smem_desc_sw128(q_addr + static_cast<uint32_t>(g * a.kp + u * a.pps + (k >> 2)) * a.rn * 128 + (k & 3) * 32, 16, 1024), id_s,
-                          u > 0 || k > 0 ? 1u : 0u);
-            umma_commit(&s.empty[it % a.slots]);
-            ++it;
+            const uint64_t qa = smem_desc_advance(dq, (g * a.kp + u * a.pps) * piece_q);
+            const uint32_t d = s_col + g * a.rn;
+#pragma unroll
+            for (int k = 0; k < 8; ++k)
+              if (k < steps)
+                umma_f16_ss(d, smem_desc_advance(ka, (k >> 2) * KM_PIECE + (k & 3) * 32), smem_desc_advance(qa, (k >> 2) * piece_q + (k & 3) * 32), id_s,
+                            u > 0 || k > 0 ? 1u : 0u);
+            free_slot();
           }
         umma_commit(&s.s_ready[SB == 2 ? j & 1 : 0]);
       };
-      scores(0);
+      if (ok) scores(0);
       for (int j = 0; j < tiles && ok; ++j) {
-        // two score buffers: the next tile's went free when the probabilities of tile j - 1 were complete
-        if (SB == 2 && j + 1 < tiles) scores(j + 1);
+        // the next tile's scores: two buffers, of which the other went free when the probabilities of tile j - 1 were complete, or one,
+        // free as soon as every thread has taken its scores
+        if (j + 1 < tiles) {
+          if (SB == 1) {
+            ok = mbar_wait(&s.s_free, j & 1, a.err, 2610);
+            tc_fence_after();
+          }
+          if (ok) scores(j + 1);
+        }
         ok = ok && mbar_wait(&s.p_ready, j & 1, a.err, 2620);
         tc_fence_after();
-        if (!ok) break;
-        if (SB == 1 && j + 1 < tiles) scores(j + 1);
         for (int g = 0; g < a.G && ok; ++g)
           for (int m = 0; m < a.mb && ok; ++m) {
-            const uint32_t v_addr = wait_slot();
+            const uint64_t va = smem_desc_advance(dv, wait_slot()), pa = smem_desc_advance(dp, g * a.rn * 256);
             if (!ok) break;
+            const uint32_t d = o_base + (g * a.mb + m) * a.rn;
 #pragma unroll
             for (int k = 0; k < KM_KEYS / 16; ++k)
-              umma_f16_ss(o_base + (g * a.mb + m) * a.rn, make_smem_desc_sw128(v_addr + k * 2048, KM_PIECE, 1024),
-                          make_smem_desc_sw128(p_addr + static_cast<uint32_t>(g) * a.rn * 256 + (k >> 2) * a.rn * 128 + (k & 3) * 32, 16, 1024), id_o,
-                          j > 0 || k > 0 ? 1u : 0u);
-            umma_commit(&s.empty[it % a.slots]);
-            ++it;
+              umma_f16_ss(d, smem_desc_advance(va, k * 2048), smem_desc_advance(pa, (k >> 2) * piece_q + (k & 3) * 32), id_o, j > 0 || k > 0 ? 1u : 0u);
+            free_slot();
           }
         umma_commit(&s.p_free);
       }
@@ -356,7 +381,7 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
         const int nqw = MODE == KM_PROMPT ? a.nq / WGS : 1, q_first = MODE == KM_PROMPT ? wg * nqw : 0;
         const int i_first = MODE == KM_PROMPT ? i0 + q_first : n_keys - 1;          // position of the first query
         const int tile_end = lo + j * KM_KEYS + KM_KEYS - 1;
-        const bool far = i_first - tile_end >= a.reach, edge = MODE == KM_PROMPT ? tile_end > i_first : tile_end >= hi;
+        const bool edge = i_first - tile_end < a.reach || (MODE == KM_STEP && tile_end >= hi);
         for (int qb = 0; qb < nqw; qb += QB) {
           const int q0 = q_first + qb;
           float y[HT][QB];
@@ -370,34 +395,45 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
 #pragma unroll
               for (int e = 0; e < QB; ++e) y[h][e] = rcp(1.f + ex2(__uint_as_float(x[h][e]) * tk.k2[h]));
           }
+          if (SB == 1 && qb + QB >= nqw) {                 // the last scores of the tile are in registers
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&s.s_free);
+          }
           if (qb == 0 && !(ok = p_writable())) break;
           uint32_t off[QB];
 #pragma unroll
           for (int e = 0; e < QB; ++e) off[e] = (q0 + e) * 128 + (p_off ^ (((q0 + e) & 7) << 4));
+          // EDGE: some of the tile's pairs are masked or nearer than the last distance
+          auto mix = [&](auto edge_t) {
+            constexpr bool EDGE = decltype(edge_t)::value;
 #pragma unroll
-          for (int h = 0; h < HT; ++h) {
-            if (h >= a.H) break;
-            float c[QB];
+            for (int h = 0; h < HT; ++h) {
+              if (h >= a.H) break;
+              float c[QB];
 #pragma unroll
-            for (int e = 0; e < QB; ++e) c[e] = tk.init[h];
+              for (int e = 0; e < QB; ++e) c[e] = tk.init[h];
 #pragma unroll
-            for (int k = 0; k < HT; ++k)
+              for (int k = 0; k < HT; ++k)
 #pragma unroll
-              for (int e = 0; e < QB; ++e) c[e] = fmaf(y[k][e], tk.w[h * HT + k], c[e]);
-            if (!far) {
-              const float* nr = a.near + static_cast<long long>(h) * (a.reach + 1);
+                for (int e = 0; e < QB; ++e) c[e] = fmaf(y[k][e], tk.w[h * HT + k], c[e]);
+              if constexpr (EDGE) {
+                const float* nr = a.near + static_cast<long long>(h) * (a.reach + 1);
 #pragma unroll
-              for (int e = 0; e < QB; ++e) c[e] += __ldg(nr + min(max(i_first + qb + e - kj, 0), a.reach));
-            }
-            uint8_t* const dst = p_row + a.prow[h];
-#pragma unroll
-            for (int e = 0; e < QB; ++e) {
-              float v = ex2(c[e]);
-              if (edge && (MODE == KM_PROMPT ? i_first + qb + e < kj : kj >= hi)) v = 0.f;
+                for (int e = 0; e < QB; ++e) {
+                  const int d = i_first + qb + e - kj;
+                  c[e] += __ldg(nr + min(max(d, 0), a.reach));
+                  if (MODE == KM_PROMPT ? d < 0 : kj >= hi) c[e] = -INFINITY;
+                }
+              }
+              uint8_t* const dst = p_row + a.prow[h];
               // a single query: the swizzle follows the head's row
-              *reinterpret_cast<__nv_bfloat16*>(dst + (MODE == KM_STEP ? p_off ^ ((a.prow[h] >> 3) & 0x70) : off[e])) = __float2bfloat16(v);
+#pragma unroll
+              for (int e = 0; e < QB; ++e)
+                *reinterpret_cast<__nv_bfloat16*>(dst + (MODE == KM_STEP ? p_off ^ ((a.prow[h] >> 3) & 0x70) : off[e])) = __float2bfloat16(ex2(c[e]));
             }
-          }
+          };
+          if (edge) mix(KmFlag<true>{}); else mix(KmFlag<false>{});
         }
         if (!ok) break;
       } else {
@@ -479,11 +515,13 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
     ok = __all_sync(0xffffffffu, ok);
     tc_fence_after();
     const long long part = static_cast<long long>(b) * a.splits + split;
+    __nv_bfloat16* const sm_o = reinterpret_cast<__nv_bfloat16*>(smem + lay.p);
+    const uint32_t o_row = a.H * a.dv;
     if (ok && valid) {
       for (int m = 0; m < a.mb; ++m) {
         const int d = m * 128 + key;
         for (int g = 0; g < a.G; ++g)
-          for (int n0 = (WGS == 2 ? wg * 16 : 0); n0 < a.rn; n0 += 16 * WGS) {
+          for (int n0 = wg * 16; n0 < a.rn; n0 += 16 * WGS) {
             uint32_t o[16];
             if (tiles > 0) {
               tmem_ld_32x16(o_base + lane_addr + (g * a.mb + m) * a.rn + n0, o);
@@ -497,9 +535,9 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
 #pragma unroll
             for (int e = 0; e < 16; ++e) {
               const int n = n0 + e;
-              if constexpr (MODE == KM_PROMPT) {
-                const int r = n >> a.lq, i = i0 + (n & (a.nq - 1));
-                if (r < a.rep && i < a.S) a.out[b * a.out_sb + i * a.out_ss + (g * a.rep + r) * a.out_sh + d] = __float2bfloat16(__uint_as_float(o[e]) * l[e]);
+              if constexpr (MODE == KM_PROMPT) {           // over the probabilities: [query][head][channel]
+                const int r = n >> a.lq;
+                if (r < a.rep) sm_o[static_cast<uint32_t>(n & (a.nq - 1)) * o_row + (g * a.rep + r) * a.dv + d] = __float2bfloat16(__uint_as_float(o[e]) * l[e]);
               } else {
                 const int h = h0 + (MODE == KM_LATENT ? n : g * a.rep + n);
                 if (n >= (MODE == KM_LATENT ? nh : a.rep)) break;
@@ -520,6 +558,14 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
   if (warp == SOFT) {
     tc_fence_after();
     tmem_dealloc(tmem, 512);
+  }
+  if constexpr (MODE == KM_PROMPT) {                       // rows of 8 channels
+    const int chunks = a.H * a.dv / 8, per = a.dv / 8;
+    for (int x = tid; x < a.nq * chunks; x += THREADS) {
+      const int i = x / chunks, c = x - i * chunks, h = c / per, d = (c - h * per) * 8;
+      if (i0 + i < a.S)
+        *reinterpret_cast<uint4*>(a.out + b * a.out_sb + (i0 + i) * a.out_ss + h * a.out_sh + d) = *reinterpret_cast<const uint4*>(smem + lay.p + static_cast<uint32_t>(x) * 16);
+    }
   }
 }
 
@@ -606,6 +652,7 @@ bool km_plan(int mode, KmArgs& a) {
     a.rn = (a.rep + 15) / 16 * 16;
     return fits(2);
   }
+  if ((a.dv & 7) || a.mb > 1) return false;                // results leave through the probabilities' space, in rows of 8 channels
   for (a.nq = 32, a.lq = 5; a.nq >= 8; a.nq /= 2, --a.lq) {
     a.rn = (a.rep * a.nq + 15) / 16 * 16;
     if (fits(2)) return true;
@@ -652,9 +699,9 @@ extern "C" TYR_EXPORT int tyr_keymajor_prompt(const void* q, const void* k, cons
   KmArgs a{};
   a.H = H; a.G = G; a.dk = dk; a.dv = dv; a.splits = 1;
   if (B <= 0 || B > 65535 || S <= 0 || dv > dvp || (dvp & 7) || reach < 0 || !km_plan(KM_PROMPT, a)) return -1;
-  for (int i = 0; i < 9; ++i)
+  for (int i = 0; i < 12; ++i)
     if (st[i] & 7) return -3;
-  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v)) & 15) return -4;
+  if ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v) | reinterpret_cast<uintptr_t>(out)) & 15) return -4;
   a.q = (const __nv_bfloat16*)q; a.out = (__nv_bfloat16*)out; a.S = S; a.err = err;
   a.q_sb = st[0]; a.q_ss = st[1]; a.q_sh = st[2]; a.out_sb = st[9]; a.out_ss = st[10]; a.out_sh = st[11];
   a.near = near; a.reach = reach;
@@ -662,8 +709,8 @@ extern "C" TYR_EXPORT int tyr_keymajor_prompt(const void* q, const void* k, cons
   if (int r = km_map(&tk, k, dk, G, S, B, st[5], st[4], st[3])) return 3000 + r;
   if (int r = km_map(&tv, v, dvp, G, S, B, st[8], st[7], st[6])) return 4000 + r;
   const dim3 grid((S + a.nq - 1) / a.nq, B);
-  return H <= 8 ? km_launch<KM_PROMPT, 8, 4, 2>(tk, tv, a, talk, grid, stream)
-                : (H <= 16 ? km_launch<KM_PROMPT, 16, 4, 2>(tk, tv, a, talk, grid, stream) : km_launch<KM_PROMPT, 32, 2, 2>(tk, tv, a, talk, grid, stream));
+  return H <= 8 ? km_launch<KM_PROMPT, 8, 2, 4>(tk, tv, a, talk, grid, stream)
+                : (H <= 16 ? km_launch<KM_PROMPT, 16, 2, 4>(tk, tv, a, talk, grid, stream) : km_launch<KM_PROMPT, 32, 2, 4>(tk, tv, a, talk, grid, stream));
 }
 
 // One token per row over bf16 stores that hold it.  talk null: latent rows [B, 1, cap, dk] whose first dv channels are the values of all
