@@ -83,6 +83,60 @@ __global__ void __launch_bounds__(256) qk_norm_store_kernel(QkNormArgs a) {
   }
 }
 
+// bf16 heads of up to 128 channels in 16-byte vectors: one CTA per token, half a warp per head.
+__global__ void __launch_bounds__(256) qk_norm_store_vec_kernel(QkNormArgs a) {
+  pdl_entry();
+  const int sub = threadIdx.x >> 4, l8 = (threadIdx.x & 15) * 8;
+  const long long row = blockIdx.x;
+  const int b = static_cast<int>(row / a.S), s = static_cast<int>(row % a.S);
+  const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(a.y) + row * a.ld;
+  long long slot = -1;
+  if (a.k_store != nullptr) {
+    const int n = a.lens ? a.lens[b] : a.S, p0 = a.pos ? a.pos[b] : 0, p = p0 + s;
+    if (s < n && p >= 0 && (a.ring ? p0 + n - p <= a.cap : p < a.cap)) slot = a.ring ? p % a.cap : p;
+  }
+  for (int hd0 = 0; hd0 < a.H + 2 * a.G; hd0 += 16) {
+    const int hd = hd0 + sub;
+    const bool on = hd < a.H + 2 * a.G, is_q = hd < a.H, is_v = hd >= a.H + a.G;
+    const int g = is_q ? hd : (is_v ? hd - a.H - a.G : hd - a.H);
+    const int d_in = is_v ? a.dv : a.dk, d_out = is_v ? a.dvp : a.dkp;
+    const int col = (is_v ? (a.H + a.G) * a.dk + g * a.dv : hd * a.dk) + l8;
+    float f[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) f[e] = 0.f;
+    if (on && l8 < d_in) {
+      const uint4 u = *reinterpret_cast<const uint4*>(src + col);
+      const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const float2 t = unpack_bf16x2(w[e]);
+        f[2 * e] = t.x; f[2 * e + 1] = t.y;
+      }
+      if (a.bias) {
+        const float4 b0 = *reinterpret_cast<const float4*>(a.bias + col), b1 = *reinterpret_cast<const float4*>(a.bias + col + 4);
+        f[0] += b0.x; f[1] += b0.y; f[2] += b0.z; f[3] += b0.w; f[4] += b1.x; f[5] += b1.y; f[6] += b1.z; f[7] += b1.w;
+      }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss += f[e] * f[e];
+#pragma unroll
+    for (int o = 8; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (!on || l8 >= d_out) continue;
+    if (!is_v) {
+      const float rstd = 1.f / sqrtf(ss / d_in + a.eps);
+      const float* w = is_q ? a.q_w : a.k_w;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[e] *= w && l8 < d_in ? rstd * w[l8 + e] : rstd;
+    }
+    const uint4 r = make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7]));
+    void* dst = is_q ? a.q_out : (is_v ? a.v_out : a.k_out);
+    if (dst) *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(dst) + (row * (is_q ? a.H : a.G) + g) * d_out + l8) = r;
+    if (!is_q && slot >= 0)
+      *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(is_v ? a.v_store : a.k_store) + ((static_cast<long long>(b) * a.G + g) * a.cap + slot) * d_out + l8) = r;
+  }
+}
+
 struct GeneralAttnArgs {
   const void *q, *k, *v;       // q: [B, S, H, .]; k / v: [B, ., G, .] by (batch, position or slot, head) element strides
   void* out;                   // [B * S, .] rows of out_ld elements, channel h * dv + d
@@ -175,6 +229,11 @@ extern "C" TYR_EXPORT int tyr_qk_norm_store(const void* y, long long ld, const f
   if (B <= 0 || S <= 0 || H <= 0 || G < 0 || dk <= 0 || dkp < dk || dvp < dv || (G > 0 && dv <= 0)) return -1;
   if ((k_store != nullptr) != (v_store != nullptr) || (k_store != nullptr && cap <= 0)) return -2;
   QkNormArgs a{y, ld, q_w, k_w, bias, q_out, k_out, v_out, k_store, v_store, pos, lens, B, S, H, G, dk, dv, dkp, dvp, cap, ring, eps};
+  const uintptr_t al = reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(q_out) | reinterpret_cast<uintptr_t>(k_out) |
+                       reinterpret_cast<uintptr_t>(v_out) | reinterpret_cast<uintptr_t>(k_store) | reinterpret_cast<uintptr_t>(v_store) |
+                       reinterpret_cast<uintptr_t>(bias);
+  if (dtype == 0 && ((ld | dk | dv | dkp | dvp) & 7) == 0 && dkp <= 128 && dvp <= 128 && (al & 15) == 0)
+    return (int)launch_dependent(qk_norm_store_vec_kernel, dim3(static_cast<unsigned>(static_cast<long long>(B) * S)), dim3(256), 0, (cudaStream_t)stream, a);
   const long long want = (static_cast<long long>(B) * S * (H + 2 * G) + 7) / 8;
   const dim3 grid(static_cast<unsigned>(want < 148LL * 32 ? want : 148LL * 32));
   return (int)(dtype == 1 ? launch_dependent(qk_norm_store_kernel<float>, grid, dim3(256), 0, (cudaStream_t)stream, a)

@@ -64,7 +64,7 @@ struct KmTalk {
 };
 
 struct KmBars {
-  uint64_t full[KM_SLOTS], empty[KM_SLOTS], q_ready, s_ready[2], s_free, p_ready, p_free, o_done, l_ready, wg;
+  uint64_t full[KM_SLOTS], empty[KM_SLOTS], q_ready, s_ready[2], s_free, p_ready, p_free, o_done, l_ready, wg[2];
   uint32_t tmem_base;
   int rescale_at;                              // latent: tile at which the sums and O were last scaled by `factor`
 };
@@ -129,7 +129,8 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
     mbar_init(&s.p_free, 3);                               // P V retired, two summing warps
     mbar_init(&s.o_done, 1);
     mbar_init(&s.l_ready, 2);
-    mbar_init(&s.wg, 4);
+    mbar_init(&s.wg[0], 4);
+    mbar_init(&s.wg[1], 4);
     s.rescale_at = -1;
     mbar_fence_init();
   }
@@ -437,9 +438,10 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
         }
         if (!ok) break;
       } else {
-        // online softmax over the heads' columns, 32 at a time; a warp's maxima meet in shared memory
+        // online softmax over this warpgroup's share of the columns, 32 at a time; a warp's maxima meet in shared memory
         const bool live = kj < hi;
-        for (int c0 = 0; c0 < a.cols; c0 += 32) {
+        const int half = WGS == 2 ? (a.cols / 16 + 1) / 2 * 16 : a.cols, c_lo = wg * half, c_hi = min(a.cols, c_lo + half);
+        for (int c0 = c_lo; c0 < c_hi; c0 += 32) {
           uint32_t x[32];
           tmem_ld_32x32(s_addr + c0, x);                   // columns past the last may be read; they are not used
           tmem_wait_ld();
@@ -456,33 +458,34 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
               v[e] = fmaxf(keep, __shfl_xor_sync(0xffffffffu, send, o));
             }
           }
-          if (c0 + lane < a.cols) sm_w[quarter * a.cols + c0 + lane] = v[0];
+          if (c0 + lane < c_hi) sm_w[quarter * a.cols + c0 + lane] = v[0];
         }
         __syncwarp();
-        if (lane == 0) mbar_arrive(&s.wg);
-        ok = mbar_wait(&s.wg, 0, a.err, 2740);             // phases of this barrier: two to a tile
+        if (lane == 0) mbar_arrive(&s.wg[wg]);
+        ok = mbar_wait(&s.wg[wg], 0, a.err, 2740);         // phases of this barrier: two to a tile
         ok = __all_sync(0xffffffffu, ok) && p_writable();  // also: the summing warps are done with the last factors
         if (!ok) break;
-        // every thread of the warpgroup looks at the columns tid, tid + 128, ...; the reference and factor are written by their owner
+        // a thread owns a column: its reference, and the factor that a move of it asks for
         bool grow = false;
-        for (int c = tid; c < a.cols; c += 128) {
+        if (c_lo + key < c_hi) {
+          const int c = c_lo + key;
           const float mx = fmaxf(fmaxf(sm_w[c], sm_w[a.cols + c]), fmaxf(sm_w[2 * a.cols + c], sm_w[3 * a.cols + c]));
           const float m = sm_m[c];
           const bool up = mx > m + 8.f;                    // also the first tile: m is -inf
           sm_f[c] = up ? ex2(m - mx) : 1.f;
           if (up) sm_m[c] = mx;
-          grow = grow || (up && j > 0);
+          grow = up && j > 0;
         }
         if (__any_sync(0xffffffffu, grow) && lane == 0) *reinterpret_cast<volatile int*>(&s.rescale_at) = j;
         __syncwarp();
-        if (lane == 0) mbar_arrive(&s.wg);
-        ok = mbar_wait(&s.wg, 1, a.err, 2741);
+        if (lane == 0) mbar_arrive(&s.wg[wg]);
+        ok = mbar_wait(&s.wg[wg], 1, a.err, 2741);
         ok = __all_sync(0xffffffffu, ok);
         if (!ok) break;
         if (*reinterpret_cast<volatile int*>(&s.rescale_at) == j) {    // P V of the tile before has retired: O is idle
           tc_fence_after();
           for (int mbk = 0; mbk < a.mb; ++mbk)
-            for (int c0 = 0; c0 < a.cols; c0 += 16) {
+            for (int c0 = c_lo; c0 < c_hi; c0 += 16) {
               uint32_t o[16];
               tmem_ld_32x16(o_base + lane_addr + mbk * a.rn + c0, o);
               tmem_wait_ld();
@@ -492,7 +495,7 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
             }
           tmem_wait_st();
         }
-        for (int c0 = 0; c0 < a.cols; c0 += 16) {
+        for (int c0 = c_lo; c0 < c_hi; c0 += 16) {
           uint32_t x[16];
           tmem_ld_32x16(s_addr + c0, x);
           tmem_wait_ld();
@@ -653,7 +656,8 @@ bool km_plan(int mode, KmArgs& a) {
     return fits(2);
   }
   if ((a.dv & 7) || a.mb > 1) return false;                // results leave through the probabilities' space, in rows of 8 channels
-  for (a.nq = 32, a.lq = 5; a.nq >= 8; a.nq /= 2, --a.lq) {
+  const int least = a.H <= 8 ? 16 : 8;                     // a warpgroup takes a quarter of the queries, 4 or 2 at a time
+  for (a.nq = 32, a.lq = 5; a.nq >= least; a.nq /= 2, --a.lq) {
     a.rn = (a.rep * a.nq + 15) / 16 * 16;
     if (fits(2)) return true;
   }
@@ -709,7 +713,7 @@ extern "C" TYR_EXPORT int tyr_keymajor_prompt(const void* q, const void* k, cons
   if (int r = km_map(&tk, k, dk, G, S, B, st[5], st[4], st[3])) return 3000 + r;
   if (int r = km_map(&tv, v, dvp, G, S, B, st[8], st[7], st[6])) return 4000 + r;
   const dim3 grid((S + a.nq - 1) / a.nq, B);
-  return H <= 8 ? km_launch<KM_PROMPT, 8, 2, 4>(tk, tv, a, talk, grid, stream)
+  return H <= 8 ? km_launch<KM_PROMPT, 8, 4, 4>(tk, tv, a, talk, grid, stream)
                 : (H <= 16 ? km_launch<KM_PROMPT, 16, 2, 4>(tk, tv, a, talk, grid, stream) : km_launch<KM_PROMPT, 32, 2, 4>(tk, tv, a, talk, grid, stream));
 }
 
@@ -739,7 +743,8 @@ extern "C" TYR_EXPORT int tyr_keymajor_step(const void* q, const void* k, const 
   if (int r = km_map(&tv, v, dvp, G, cap, B, static_cast<long long>(cap) * dvp, dvp, static_cast<long long>(G) * cap * dvp)) return 4000 + r;
   int rc;
   if (mode == KM_LATENT) {
-    rc = km_launch<KM_LATENT, 8, 1, 1>(tk, tv, a, nullptr, dim3(splits, (H + a.hb - 1) / a.hb, B), stream);
+    const dim3 grid(splits, (H + a.hb - 1) / a.hb, B);
+    rc = a.rn >= 32 ? km_launch<KM_LATENT, 8, 1, 2>(tk, tv, a, nullptr, grid, stream) : km_launch<KM_LATENT, 8, 1, 1>(tk, tv, a, nullptr, grid, stream);
   } else {
     const dim3 grid(splits, 1, B);
     rc = H <= 8 ? km_launch<KM_STEP, 8, 1, 1>(tk, tv, a, talk, grid, stream)

@@ -122,34 +122,37 @@ struct RotateArgs {
   int B, S, H, rot, dims, width;      // channels [rot, width) of y are set to zero
 };
 
-// A thread per (token, head, channel pair); the pairs of all heads of a token are adjacent.
+constexpr int ROT_HEADS = 8;
+
+// A thread per (token, channel pair, eight heads), which share the angle.
 template <typename T>
 __global__ void __launch_bounds__(256) rotate_heads_kernel(RotateArgs a) {
   pdl_entry();
-  const int pairs = (a.width + 1) / 2;
-  const long long total = static_cast<long long>(a.B) * a.S * a.H * pairs;
+  const int pairs = (a.width + 1) / 2, groups = (a.H + ROT_HEADS - 1) / ROT_HEADS;
+  const long long total = static_cast<long long>(a.B) * a.S * groups * pairs;
   for (long long i = blockIdx.x * 256LL + threadIdx.x; i < total; i += gridDim.x * 256LL) {
-    const int d = 2 * static_cast<int>(i % pairs), h = static_cast<int>(i / pairs % a.H);
-    const long long row = i / pairs / a.H;
+    const int d = 2 * static_cast<int>(i % pairs), h0 = static_cast<int>(i / pairs % groups) * ROT_HEADS;
+    const long long row = i / pairs / groups;
     const int b = static_cast<int>(row / a.S), s = static_cast<int>(row % a.S);
-    const T* x = static_cast<const T*>(a.x) + b * a.x_sb + s * a.x_ss + h * a.x_sh;
-    T* y = static_cast<T*>(a.y) + b * a.y_sb + s * a.y_ss + h * a.y_sh;
-    const int p = (a.pos ? a.pos[b] : 0) + s;
-    float v[2];
+    const T* x = static_cast<const T*>(a.x) + b * a.x_sb + s * a.x_ss + h0 * a.x_sh + d;
+    T* y = static_cast<T*>(a.y) + b * a.y_sb + s * a.y_ss + h0 * a.y_sh + d;
+    float sn = 0.f, cs = 1.f;
     if (d + 1 < a.dims) {
-      const double t = p * a.turns[d >> 1];
-      float sn, cs;
+      const double t = ((a.pos ? a.pos[b] : 0) + s) * a.turns[d >> 1];
       sincospif(2.f * static_cast<float>(t - rint(t)), &sn, &cs);
-      const float u = la_load(x + d), w = la_load(x + d + 1);
-      v[0] = u * cs - w * sn;
-      v[1] = w * cs + u * sn;
-    } else {
+    }
+    float u[ROT_HEADS], w[ROT_HEADS];
 #pragma unroll
-      for (int e = 0; e < 2; ++e) v[e] = d + e < a.rot ? la_load(x + d + e) : 0.f;
+    for (int h = 0; h < ROT_HEADS; ++h) {
+      u[h] = h0 + h < a.H && d < a.rot ? la_load(x + h * a.x_sh) : 0.f;
+      w[h] = h0 + h < a.H && d + 1 < a.rot ? la_load(x + h * a.x_sh + 1) : 0.f;
     }
 #pragma unroll
-    for (int e = 0; e < 2; ++e)
-      if (d + e < a.width) la_store(y + d + e, v[e]);
+    for (int h = 0; h < ROT_HEADS; ++h) {
+      if (h0 + h >= a.H) break;
+      la_store(y + h * a.y_sh, u[h] * cs - w[h] * sn);
+      if (d + 1 < a.width) la_store(y + h * a.y_sh + 1, w[h] * cs + u[h] * sn);
+    }
   }
 }
 
@@ -175,7 +178,7 @@ extern "C" TYR_EXPORT int tyr_rotate_heads(const void* x, void* y, const double*
                                            int rot, int dims, int width, int dtype, void* stream) {
   if (B <= 0 || S <= 0 || H <= 0 || rot < 0 || dims < 0 || dims > rot || (dims & 1) || width < rot || width <= 0) return -1;
   RotateArgs a{x, y, turns, pos, strides[0], strides[1], strides[2], strides[3], strides[4], strides[5], B, S, H, rot, dims, width};
-  const long long want = (static_cast<long long>(B) * S * H * ((width + 1) / 2) + 255) / 256;
+  const long long want = (static_cast<long long>(B) * S * ((H + ROT_HEADS - 1) / ROT_HEADS) * ((width + 1) / 2) + 255) / 256;
   const dim3 grid(static_cast<unsigned>(want < 148LL * 32 ? want : 148LL * 32));
   return (int)(dtype == 1 ? launch_dependent(rotate_heads_kernel<float>, grid, dim3(256), 0, (cudaStream_t)stream, a)
                           : launch_dependent(rotate_heads_kernel<__nv_bfloat16>, grid, dim3(256), 0, (cudaStream_t)stream, a));

@@ -24,7 +24,7 @@ struct SkinnyArgs {
   float* ws;                   // [M, N] fp32, zero on entry and exit; used when the reduction is split over gridDim.y CTAs
   long long ldx, ldw, ldy;
   int M, N, K;
-  long long hx, hw, hy;        // per-head form: elements from head to head (gridDim.z heads)
+  long long hx, hw, hy;        // per-head form: elements from head to head
   int act;                     // 6: xIELU with factors act_a, act_b, as in csrc/gemm_tcgen05.cu; 0: none
   float act_a, act_b;
 };
@@ -47,9 +47,6 @@ __global__ void __launch_bounds__(kSkWarps * 32) skinny_gemm_kernel(SkinnyArgs a
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int g = lane >> 2, t = lane & 3;
   const int row0 = blockIdx.x * 16;
-  a.w += blockIdx.z * a.hw;
-  a.x += blockIdx.z * a.hx;
-  a.y += blockIdx.z * a.hy;
   // The weights are constants: while the kernel that produces `x` still runs (this one may already be resident, see
   // launch_dependent), pull the head of every weight row of this CTA into the L2.  The whole grid asks for at most
   // kSkPrefetchBytes, so what it brings in is still there when the loop below reads it.
@@ -59,7 +56,7 @@ __global__ void __launch_bounds__(kSkWarps * 32) skinny_gemm_kernel(SkinnyArgs a
     const int chunks = a.K >> 5;
     const int c0 = static_cast<int>(static_cast<long long>(chunks) * blockIdx.y / gridDim.y);
     const int c1 = static_cast<int>(static_cast<long long>(chunks) * (blockIdx.y + 1) / gridDim.y);
-    long long per_row = kSkPrefetchBytes / (static_cast<long long>(gridDim.x) * gridDim.y * gridDim.z * (GATED ? 32 : 16));
+    long long per_row = kSkPrefetchBytes / (static_cast<long long>(gridDim.x) * gridDim.y * (GATED ? 32 : 16));
     per_row = min(per_row & ~127LL, static_cast<long long>(c1 - c0) * 64);
     if (r < a.N && per_row >= 128)
       bulk_prefetch_l2((tid < 16 ? a.w : a.w2) + static_cast<long long>(r) * a.ldw + 32LL * c0, static_cast<uint32_t>(per_row));
@@ -144,6 +141,65 @@ __global__ void __launch_bounds__(kSkWarps * 32) skinny_gemm_kernel(SkinnyArgs a
       }
     }
   }
+}
+
+// A small matrix of its own for each head: gridDim.y heads, a warp owns 16 rows of the head's matrix and its whole contraction.
+template <int TILES>
+__global__ void __launch_bounds__(kSkWarps * 32) skinny_heads_kernel(SkinnyArgs a) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+  const int row0 = (blockIdx.x * kSkWarps + warp) * 16;
+  pdl_trigger();
+  if (row0 >= a.N) return;
+  const __nv_bfloat16* w = a.w + blockIdx.y * a.hw;
+  const __nv_bfloat16* w_lo = w + min(row0 + g, a.N - 1) * a.ldw + 8 * t;        // clamped rows are not written
+  const __nv_bfloat16* w_hi = w + min(row0 + g + 8, a.N - 1) * a.ldw + 8 * t;
+  constexpr int U = 4;                             // the weights need nothing from the kernel in front of this one
+  const int chunks = a.K >> 5;
+  uint4 lo[U], hi[U];
+#pragma unroll
+  for (int u = 0; u < U; ++u)
+    if (u < chunks) {
+      lo[u] = __ldg(reinterpret_cast<const uint4*>(w_lo + 32 * u));
+      hi[u] = __ldg(reinterpret_cast<const uint4*>(w_hi + 32 * u));
+    }
+  pdl_wait();
+  const __nv_bfloat16* xr[TILES];
+  bool live[TILES];
+  float acc[TILES][4];
+#pragma unroll
+  for (int i = 0; i < TILES; ++i) {
+    const int tok = 8 * i + g;
+    live[i] = tok < a.M;
+    xr[i] = a.x + blockIdx.y * a.hx + (live[i] ? tok : 0) * a.ldx + 8 * t;
+    acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+  }
+  for (int c0 = 0; c0 < chunks; c0 += U) {
+    uint4 xv[U][TILES];
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+#pragma unroll
+      for (int i = 0; i < TILES; ++i) xv[u][i] = c0 + u < chunks && live[i] ? *reinterpret_cast<const uint4*>(xr[i] + 32 * (c0 + u)) : make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      if (c0 + u >= chunks) break;
+#pragma unroll
+      for (int i = 0; i < TILES; ++i) {
+        mma_16816(acc[i], lo[u].x, hi[u].x, lo[u].y, hi[u].y, xv[u][i].x, xv[u][i].y);
+        mma_16816(acc[i], lo[u].z, hi[u].z, lo[u].w, hi[u].w, xv[u][i].z, xv[u][i].w);
+      }
+      if (c0 + u + U < chunks) {
+        lo[u] = __ldg(reinterpret_cast<const uint4*>(w_lo + 32 * (c0 + u + U)));
+        hi[u] = __ldg(reinterpret_cast<const uint4*>(w_hi + 32 * (c0 + u + U)));
+      }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < TILES; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int tok = 8 * i + 2 * t + (e & 1), row = row0 + g + (e >> 1) * 8;
+      if (tok < a.M && row < a.N) a.y[blockIdx.y * a.hy + tok * a.ldy + row] = __float2bfloat16(acc[i][e]);
+    }
 }
 
 // Second pass of a split reduction: round the fp32 sums (+ bias) and leave the workspace zeroed for the next call.
@@ -246,12 +302,10 @@ extern "C" TYR_EXPORT int tyr_skinny_heads_bf16(const void* x, const void* w, vo
   if ((ldx | ldw | hx | hw) & 7) return -2;
   if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) return -3;
   SkinnyArgs a{(const __nv_bfloat16*)x, (const __nv_bfloat16*)w, nullptr, nullptr, (__nv_bfloat16*)y, nullptr, ldx, ldw, ldy, M, N, K, hx, hw, hy, 0, 0.f, 0.f};
-  const dim3 grid((N + 15) / 16, 1, heads), block(kSkWarps * 32);
-  skinny_prefer_l1();
+  const dim3 grid((N + 16 * kSkWarps - 1) / (16 * kSkWarps), heads), block(kSkWarps * 32);
   const cudaStream_t st = (cudaStream_t)stream;
-  return (int)(M <= 8 ? launch_dependent(skinny_gemm_kernel<1, false>, grid, block, 0, st, a)
-                      : M <= 16 ? launch_dependent(skinny_gemm_kernel<2, false>, grid, block, 0, st, a)
-                                : launch_dependent(skinny_gemm_kernel<4, false>, grid, block, 0, st, a));
+  return (int)(M <= 8 ? launch_dependent(skinny_heads_kernel<1>, grid, block, 0, st, a)
+                      : M <= 16 ? launch_dependent(skinny_heads_kernel<2>, grid, block, 0, st, a) : launch_dependent(skinny_heads_kernel<4>, grid, block, 0, st, a));
 }
 
 // y[M, N] = silu(x wg^T) * (x wu^T): the gate and up projections of a SwiGLU MLP for decode-sized M in one pass over both
