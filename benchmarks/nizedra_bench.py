@@ -209,9 +209,9 @@ def kernels(only: str = "", warmup: int = 3, steps: int = 20, device="cuda") -> 
         pos = torch.full((B,), 5000, dtype=torch.int32, device=device) if S == 1 else None
         case(f"latent norms, rotation and store {B}x{S}", lambda: lt.latent_norm_store(y, qw, kw, turns, 64, 1e-6, q_width=768, width=576, store=st, pos=pos),
              gb(B * S * (1344 * 4 + min(1.0, 1024 / S) * 576 * 2)), lambda: rms_norm_weighted(y, None, 1e-6), gb(B * S * 1344 * 4))
-        q, x = mk(B, S, 32, 128), mk(B, S, 24 * 128)
+        q, x, bias = mk(B, S, 32, 128), mk(B, S, 24 * 128), f32(24 * 128)
         case(f"rotation of query heads {B}x{S}, 32 heads, 32 of 128 channels", lambda: lt.rotate_heads(q[..., 96:], turns[:16], pos), gb(B * S * 32 * 32 * 4))
-        case(f"unit queries and keys and store {B}x{S}, 16/4 heads", lambda: qk_norm_store(x, None, None, 16, 4, 128, 128, 1e-6, dkp=128, dvp=128, bias=f32(24 * 128)),
+        case(f"unit queries and keys and store {B}x{S}, 16/4 heads", lambda: qk_norm_store(x, None, None, 16, 4, 128, 128, 1e-6, dkp=128, dvp=128, bias=bias),
              gb(B * S * 24 * 128 * 4), lambda: rms_norm_weighted(x, None, 1e-6), gb(B * S * 24 * 128 * 4))
     for M, H, N, K in ((1, 32, 512, 64), (32, 32, 512, 64), (32, 32, 64, 512), (32, 128, 512, 128)):
         x, w, y, w2 = mk(M, H, K), mk(H, N, K), mk(M, H, N), mk(H * N * K // 2048, 2048)

@@ -537,7 +537,9 @@ __device__ __forceinline__ float pn_block_sum(float v, float* red, int tid, int 
   return tot;
 }
 
-template <typename TX, typename TY, bool VEC>
+// NV: vectors of 8 channels a thread holds (0: any size, element by element).  The weights are constants: they are on their way while the
+// kernel in front of this one still runs.
+template <typename TX, typename TY, int NV>
 __global__ void __launch_bounds__(256) sandwich_norm_kernel(SandwichNormArgs a) {
   __shared__ float red[2][8];
   const long long row = blockIdx.x;
@@ -545,14 +547,26 @@ __global__ void __launch_bounds__(256) sandwich_norm_kernel(SandwichNormArgs a) 
   const TX* x = static_cast<const TX*>(a.x) + row * a.x_stride;
   float* resid = a.resid + row * a.D;
   TY* y = static_cast<TY*>(a.y) + row * a.y_stride;
-  pdl_entry();
-  float f[kPnVecs][8], ss = 0.f;
-  if constexpr (VEC) {
+  pdl_trigger();
+  if constexpr (NV > 0) {
+    constexpr bool EARLY = NV <= 2;                // registers for both gains
+    float f[NV][8], r[NV][8], wp[EARLY ? NV : 1][8], wg[EARLY ? NV : 1][8], ss = 0.f;
+    if constexpr (EARLY) {
 #pragma unroll
-    for (int j = 0; j < kPnVecs; ++j) {
+      for (int j = 0; j < NV; ++j) {
+        const int v = (tid + j * blockDim.x) * 8;
+        if (v >= a.D) continue;
+        if (a.post) pn_load8(a.post + v, wp[j]);
+        if (a.gain) pn_load8(a.gain + v, wg[j]);
+      }
+    }
+    pdl_wait();
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
       const int v = (tid + j * blockDim.x) * 8;
       if (v >= a.D) continue;
       pn_load8(x + v, f[j]);
+      if (!a.replace) pn_load8(resid + v, r[j]);
       if (a.bias) {
         float b[8];
         pn_load8(a.bias + v, b);
@@ -562,36 +576,48 @@ __global__ void __launch_bounds__(256) sandwich_norm_kernel(SandwichNormArgs a) 
 #pragma unroll
       for (int e = 0; e < 8; ++e) ss += f[j][e] * f[j][e];
     }
-  } else {
-    for (int d = tid; d < a.D; d += blockDim.x) {
-      const float t = pn_get(x + d) + (a.bias ? a.bias[d] : 0.f);
-      ss += t * t;
-    }
-  }
-  const float inner = a.post ? rsqrtf(pn_block_sum(ss, red[0], tid, nw) / a.D + a.eps) : 1.f;
-  ss = 0.f;
-  if constexpr (VEC) {
+    const float inner = a.post ? rsqrtf(pn_block_sum(ss, red[0], tid, nw) / a.D + a.eps) : 1.f;
+    ss = 0.f;
 #pragma unroll
-    for (int j = 0; j < kPnVecs; ++j) {
+    for (int j = 0; j < NV; ++j) {
       const int v = (tid + j * blockDim.x) * 8;
       if (v >= a.D) continue;
       if (a.post) {
         float w[8];
-        pn_load8(a.post + v, w);
+        if constexpr (!EARLY) pn_load8(a.post + v, w);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) f[j][e] *= inner * w[e];
+        for (int e = 0; e < 8; ++e) f[j][e] *= inner * (EARLY ? wp[EARLY ? j : 0][e] : w[e]);
       }
       if (!a.replace) {
-        float r[8];
-        pn_load8(resid + v, r);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) f[j][e] += r[e];
+        for (int e = 0; e < 8; ++e) f[j][e] += r[j][e];
       }
       pn_store8(resid + v, f[j]);
 #pragma unroll
       for (int e = 0; e < 8; ++e) ss += f[j][e] * f[j][e];
     }
+    const float outer = a.gain ? rsqrtf(pn_block_sum(ss, red[1], tid, nw) / a.D + a.eps) : 1.f;
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+      const int v = (tid + j * blockDim.x) * 8;
+      if (v >= a.D) continue;
+      if (a.gain) {
+        float w[8];
+        if constexpr (!EARLY) pn_load8(a.gain + v, w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[j][e] *= outer * (EARLY ? wg[EARLY ? j : 0][e] : w[e]);
+      }
+      pn_store8(y + v, f[j]);
+    }
   } else {
+    pdl_wait();
+    float ss = 0.f;
+    for (int d = tid; d < a.D; d += blockDim.x) {
+      const float t = pn_get(x + d) + (a.bias ? a.bias[d] : 0.f);
+      ss += t * t;
+    }
+    const float inner = a.post ? rsqrtf(pn_block_sum(ss, red[0], tid, nw) / a.D + a.eps) : 1.f;
+    ss = 0.f;
     for (int d = tid; d < a.D; d += blockDim.x) {
       float t = pn_get(x + d) + (a.bias ? a.bias[d] : 0.f);
       if (a.post) t *= inner * a.post[d];
@@ -599,22 +625,7 @@ __global__ void __launch_bounds__(256) sandwich_norm_kernel(SandwichNormArgs a) 
       resid[d] = t;
       ss += t * t;
     }
-  }
-  const float outer = a.gain ? rsqrtf(pn_block_sum(ss, red[1], tid, nw) / a.D + a.eps) : 1.f;
-  if constexpr (VEC) {
-#pragma unroll
-    for (int j = 0; j < kPnVecs; ++j) {
-      const int v = (tid + j * blockDim.x) * 8;
-      if (v >= a.D) continue;
-      if (a.gain) {
-        float w[8];
-        pn_load8(a.gain + v, w);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) f[j][e] *= outer * w[e];
-      }
-      pn_store8(y + v, f[j]);
-    }
-  } else {
+    const float outer = a.gain ? rsqrtf(pn_block_sum(ss, red[1], tid, nw) / a.D + a.eps) : 1.f;
     for (int d = tid; d < a.D; d += blockDim.x) pn_put(y + d, a.gain ? resid[d] * outer * a.gain[d] : resid[d]);
   }
 }
@@ -742,8 +753,11 @@ extern "C" TYR_EXPORT int tyr_sandwich_norm(const void* x, long long x_stride, c
   while (threads > 32 && threads * 4 >= D) threads >>= 1;       // narrow rows: no idle warps
   const dim3 grid(static_cast<unsigned>(rows)), block(threads);
   cudaStream_t st = (cudaStream_t)stream;
-#define TYR_SN(TX, TY) (vec ? launch_dependent(sandwich_norm_kernel<TX, TY, true>, grid, block, 0, st, a) \
-                            : launch_dependent(sandwich_norm_kernel<TX, TY, false>, grid, block, 0, st, a))
+  const int nv = !vec ? 0 : D <= threads * 8 ? 1 : D <= threads * 16 ? 2 : 4;
+#define TYR_SN(TX, TY)                                                                          \
+  (nv == 0 ? launch_dependent(sandwich_norm_kernel<TX, TY, 0>, grid, block, 0, st, a)           \
+           : nv == 1 ? launch_dependent(sandwich_norm_kernel<TX, TY, 1>, grid, block, 0, st, a) \
+                     : nv == 2 ? launch_dependent(sandwich_norm_kernel<TX, TY, 2>, grid, block, 0, st, a) : launch_dependent(sandwich_norm_kernel<TX, TY, 4>, grid, block, 0, st, a))
   if (x_dtype == 0) return (int)(y_dtype == 0 ? TYR_SN(__nv_bfloat16, __nv_bfloat16) : TYR_SN(__nv_bfloat16, float));
   return (int)(y_dtype == 0 ? TYR_SN(float, __nv_bfloat16) : TYR_SN(float, float));
 #undef TYR_SN

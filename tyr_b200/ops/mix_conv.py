@@ -147,7 +147,8 @@ def mix_step(x: torch.Tensor, segments: Sequence[Segment], pos: torch.Tensor) ->
 
 def activate(x: torch.Tensor, act: str, act_args: tuple = (0.0, 0.0)) -> torch.Tensor:
     """An activation alone, of contiguous rows [..., C]."""
-    flat = x.view(1, -1, x.shape[-1])
+    rows = x.numel() // x.shape[-1]
+    flat = x.view(rows, 1, -1) if rows < 4096 else x.view(1, rows, -1)        # few rows: a thread each instead of a thread per 64
     y = torch.empty_like(flat)
     mix_prompt(flat, [Segment(0, 1, x.shape[-1], y, act=act, act_args=act_args)])
     return y.view(x.shape)
