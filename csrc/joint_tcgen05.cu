@@ -343,8 +343,8 @@ joint_keymajor_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
       __syncwarp();
       if (lane == 0) mbar_arrive(&s.p_free);
     }
-    // the queries' space is free once every product is done
-    ok = ok && (tiles == 0 || mbar_wait(&s.o_done, 0, a.err, 2640 + w));
+    // the queries' space is free once every product is done (an empty slice: once everybody has written to it)
+    ok = ok && mbar_wait(tiles == 0 ? &s.q_ready : &s.o_done, 0, a.err, 2640 + w);
     ok = __all_sync(0xffffffffu, ok);
     if (ok) {
 #pragma unroll

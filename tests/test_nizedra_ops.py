@@ -134,7 +134,8 @@ def talk_of(mix, temp, rel, talk, dev):
 
 TALK = [(40, 6, 2, 24, 40, 2.0, 16, 20), (70, 1, 1, 8, 8, 1.0, 2, 2), (33, 5, 5, 130, 20, 30.0, 9, 31), (150, 4, 2, 64, 64, 3.0, 8, 100),
         (150, 8, 2, 128, 128, 5.0, 32, 128), (100, 16, 4, 64, 128, 20.0, 16, 60), (90, 12, 4, 32, 64, 4.0, 10, 300), (60, 32, 8, 128, 64, 4.0, 12, 40),
-        (50, 20, 1, 64, 64, 4.0, 12, 40), (37, 40, 8, 16, 24, 4.0, 12, 40), (130, 7, 7, 48, 80, 6.0, 16, 90), (45, 32, 2, 128, 128, 6.0, 16, 90)]
+        (50, 20, 1, 64, 64, 4.0, 12, 40), (37, 40, 8, 16, 24, 4.0, 12, 40), (130, 7, 7, 48, 80, 6.0, 16, 90), (45, 32, 2, 128, 128, 6.0, 16, 90),
+        (400, 4, 1, 64, 64, 3.0, 16, 1000), (300, 2, 1, 32, 16, 3.0, 4, 64)]
 
 
 @pytest.mark.parametrize("place", PLACES)
@@ -172,7 +173,7 @@ def test_talking_heads_one_token_per_row(place, case):
     want = O.talking_attention(q, k, v, mix, temp, rel, talk)
     dkp, dvp = ja.store_dims(dk, dv, dt, dev)
     st = stores(dev, dt, 4, G, T + 3, dkp, dvp)
-    pos = [T - 1, 0, T // 2, 1]
+    pos = [T - 1, 0, T // 2, 1]                            # in a long store, the early rows leave slices of the keys empty
     fill = lambda t, n, d: torch.nn.functional.pad(t[:n].transpose(0, 1), (0, d - t.shape[2])).to(dev, dt)
     for b, p in enumerate(pos):
         st.k[b, :, :p + 1], st.v[b, :, :p + 1] = fill(k, p + 1, dkp), fill(v, p + 1, dvp)
