@@ -294,7 +294,7 @@ def test_rotation_of_query_heads(place):
 
 
 @pytest.mark.parametrize("place", PLACES)
-@pytest.mark.parametrize("T,H,dk,dv,win", [(40, 3, 24, 16, 7), (300, 2, 96, 64, 136), (300, 2, 96, 64, 128), (260, 4, 64, 128, 1), (140, 2, 128, 40, None),
+@pytest.mark.parametrize("T,H,dk,dv,win", [(40, 3, 24, 16, 7), (300, 2, 96, 64, 140), (300, 2, 96, 64, 128), (260, 4, 64, 128, 1), (140, 2, 128, 40, None),
                                            (150, 1, 200, 136, 30), (50, 2, 300, 20, 12), (500, 2, 48, 48, 131)])
 def test_windowed_attention_over_prompts(place, T, H, dk, dv, win):
     dev, dt = place
@@ -333,7 +333,7 @@ def test_key_just_inside_and_just_outside_the_window(place, win):
 
 
 @pytest.mark.parametrize("place", PLACES)
-@pytest.mark.parametrize("H,rank,rot,win,ring", [(3, 24, 8, 9, True), (4, 128, 32, 40, True), (1, 8, 0, None, False), (20, 64, 32, 33, False), (5, 520, 24, 64, True),
+@pytest.mark.parametrize("H,rank,rot,win,ring", [(3, 24, 8, 9, True), (4, 112, 32, 40, True), (1, 8, 0, None, False), (20, 64, 32, 33, False), (5, 520, 24, 64, True),
                                                  (33, 96, 32, 50, True), (16, 512, 64, 100, True), (40, 1100, 20, 17, True)])
 def test_attention_over_latent_rows(place, H, rank, rot, win, ring):
     """Every head reads the row of a position as its key and the row's first channels as its value; rows at unequal positions."""
