@@ -4,7 +4,8 @@
 //   score_h   = sum_g talk[h, g] s_g                          (each step optional), j <= i, 0 <= i - j < window,
 //
 // softmax over the visible keys of every head.  Keys and values are separate rows, or the values are the first channels of the keys
-// (one latent row for all heads).
+// (one latent row for all heads).  csrc/joint_tcgen05.cu has the form for scores of bounded range; these take every score, and the sizes
+// that one does not hold.
 //
 //   * prompt:  mixed heads over bf16 prompts.  One CTA owns 16 (or 8) queries with all their heads and walks the keys in tiles: Q K^T of all
 //              heads, cap and bias on the way to shared memory; the mix as a product of `talk` with the scores of every (query, key) pair
