@@ -35,6 +35,10 @@
 // Sink and gate (BIAS 3): the same head sizes without a penalty, with an optional window; the softmax denominator also holds exp(sink_h), and the output is
 // multiplied by out_scale * sigmoid(gate), both in the epilogue.
 //
+// Kept first keys and turned values (BIAS 4): the sink form in which the first `keep` keys stay visible beyond the window (their blocks come
+// first, then the window's), the gate may be one number per head, and the output's channel pairs (m, m + dv / 2) are turned back by
+// the query's angles (values that were rotated by their positions).
+//
 // The reference calls at::scaled_dot_product_attention, or a query-chunked masked-math fallback
 // for windows (cc/include/tyr_attention.h:58-130).
 #include "common.cuh"
@@ -65,6 +69,11 @@ struct AttnParams {
   const __nv_bfloat16* gate;
   long long g_row_stride, g_batch_stride, g_head_stride;
   float out_scale;
+  // form with kept keys only
+  int keep;           // keys 0 .. keep - 1 are visible past the window
+  int gate_head;      // the gate is one number per (row, head)
+  const float2* back; // [Tq, back_half] (cos, sin) of the query's turns (nullable)
+  int back_half;
 };
 
 constexpr int ATT_TBL_PAD = 256;       // table entries below distance 0 and past the window that boundary blocks can touch
@@ -128,6 +137,12 @@ __device__ __forceinline__ void tmem_ld_32x32_nowait(uint32_t taddr, uint32_t* r
       : "r"(taddr)
       : "memory");
 }
+__device__ __forceinline__ void tmem_ld_32x8_nowait(uint32_t taddr, uint32_t (&r)[8]) {
+  asm volatile("tcgen05.ld.sync.aligned.32x32b.x8.b32 {%0, %1, %2, %3, %4, %5, %6, %7}, [%8];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7])
+               : "r"(taddr)
+               : "memory");
+}
 __device__ __forceinline__ void tmem_st_32x32(uint32_t taddr, const uint32_t* r) {
   asm volatile(
       "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
@@ -159,6 +174,7 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
                       const __grid_constant__ CUtensorMap tmK,
                       const __grid_constant__ CUtensorMap tmV, AttnParams p) {
   constexpr bool kPenalty = BIAS == 1 || BIAS == 2;
+  constexpr bool kKept = BIAS == 4, kGated = BIAS == 3 || kKept;
   pdl_trigger();
   extern __shared__ uint8_t smem_raw[];
   AttnSmem& s = *reinterpret_cast<AttnSmem*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
@@ -180,6 +196,11 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
   if (!tile1_live) { lo[1] = 0; hi[1] = 0; }
   int jlo = lo[0], jhi = hi[0];
   if (tile1_live) { jlo = min(lo[0], lo[1]); jhi = max(hi[0], hi[1]); }
+  // Key blocks in the order they are walked: those of the kept keys, then those from a tile's first window key on.
+  const int kept = kKept && p.window > 0 ? (p.keep + ATT_BN - 1) / ATT_BN : 0;
+  const int jfirst = kept > 0 ? 0 : jlo;
+  auto after = [&](int j, int low) { return kKept && j + 1 >= kept && j + 1 < low ? low : j + 1; };
+  auto active = [&](int t, int j) { return j < hi[t] && (j >= lo[t] || (kKept && j < kept)); };
 
   if (threadIdx.x == 0) {
     mbar_init(&s.q_full, 1);
@@ -237,7 +258,7 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
           tma_load_4d(s.q[t] + c * kChunk, &tmQ, &s.q_full, c * 64, head, row0 + t * ATT_BM, batch);
       uint32_t it = 0;
       bool ok = true;
-      for (int j = jlo; j < jhi && ok; ++j, ++it) {
+      for (int j = jfirst; j < jhi && ok; j = after(j, jlo), ++it) {
         const int st = it % ATT_STAGES;
         const uint32_t ph = (it / ATT_STAGES) & 1;
         // K and V have separate rings: a K stage is released a whole iteration before the V stage of the same block, so
@@ -288,31 +309,32 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
       uint32_t p_cnt[2] = {0, 0};
       uint32_t it = 0;
       // prologue: S for the first block of each live tile
-      if (ok && jhi > jlo) {
+      if (ok && jhi > jfirst) {
         ok = mbar_wait(&s.k_full[0], 0, p.err, 610);
         tc_fence_after();
         for (int t = 0; t < 2 && ok; ++t)
-          if (jlo >= lo[t] && jlo < hi[t]) issue_s(t, 0);
+          if (active(t, jfirst)) issue_s(t, 0);
         umma_commit(&s.k_empty[0]);                              // K of the first block: its S products are queued
       }
-      for (int j = jlo; j < jhi && ok; ++j, ++it) {
+      for (int j = jfirst; j < jhi && ok; j = after(j, jlo), ++it) {
+        const int jn = after(j, jlo);
         const int st = it % ATT_STAGES;
         const uint32_t ph = (it / ATT_STAGES) & 1;
         const int st_n = (it + 1) % ATT_STAGES;
         const uint32_t ph_n = ((it + 1) / ATT_STAGES) & 1;
         bool next_k_ready = false;
         for (int t = 0; t < 2 && ok; ++t) {
-          const bool cur = (j >= lo[t] && j < hi[t]);
+          const bool cur = active(t, j);
           if (cur) {
             if (!mbar_wait(&s.v_full[st], ph, p.err, 620 + st)) { ok = false; break; }
             if (!mbar_wait(&s.p_ready[t], p_cnt[t] & 1, p.err, 630 + t)) { ok = false; break; }
             ++p_cnt[t];
             tc_fence_after();
-            issue_pv(t, st, j == lo[t]);
+            issue_pv(t, st, j == (kept > 0 ? 0 : lo[t]));
             if (j + 1 == hi[t]) umma_commit(&s.o_done[t]);
           }
           // next block's S for this tile (its S/P columns are free once PV above is queued)
-          const bool nxt = (j + 1 >= lo[t] && j + 1 < hi[t]);
+          const bool nxt = active(t, jn);
           if (nxt) {
             if (!next_k_ready) {
               if (!mbar_wait(&s.k_full[st_n], ph_n, p.err, 640 + st_n)) { ok = false; break; }
@@ -324,7 +346,7 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
         }
         if (ok) {
           umma_commit(&s.v_empty[st]);                           // V_j: both PV products are queued
-          if (j + 1 < jhi) umma_commit(&s.k_empty[st_n]);        // K_{j+1}: both S products are queued
+          if (jn < jhi) umma_commit(&s.k_empty[st_n]);        // K_{j+1}: both S products are queued
         }
       }
     }
@@ -350,7 +372,8 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
     bool ok = true;
     uint32_t cnt = 0;
     if (tile_live) {
-      for (int j = lo[t]; j < hi[t] && ok; ++j, ++cnt) {
+      const int j0 = kept > 0 ? 0 : lo[t];
+      for (int j = j0; j < hi[t] && ok; j = after(j, lo[t]), ++cnt) {
         if (!mbar_wait(&s.s_ready[t], cnt & 1, p.err, 700 + t)) { ok = false; break; }
         tc_fence_after();
         const int col0 = j * ATT_BN + h * 64;
@@ -364,7 +387,7 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
             const int col = base + c;
             bool keep = col < p.Tk;
             if (p.causal) keep = keep && (col <= qi);
-            if (p.window > 0) keep = keep && (col > qi - p.window);
+            if (p.window > 0) keep = keep && (col > qi - p.window || (kKept && col < p.keep));
             if (!keep) v[c] = __float_as_uint(-INFINITY);
           }
         };
@@ -416,7 +439,7 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
         }
         // lazy rescale: move the reference maximum only when it grew by more than 8 (log2 units); both halves of a row
         // take the same decision because they see the same maximum
-        const bool first = (j == lo[t]);
+        const bool first = (j == j0);
         float m_new = fmaxf(m_used, mx);
         const bool want = first || (m_new > m_used + 8.f);
         if (__any_sync(0xffffffffu, want && !first)) {
@@ -485,16 +508,46 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
         float inv = l_sum > 0.f ? 1.f / l_sum : 0.f;
         const bool row_ok = row < p.Tq;
         const __nv_bfloat16* gate = nullptr;
-        if constexpr (BIAS == 3) {
+        if constexpr (kGated) {
           if (p.sink) {                          // both terms relative to the larger of the row's reference and the sink
             const float sk = p.sink[head] * 1.4426950408889634f, m = fmaxf(m_used, sk), f = exp2f(m_used - m);
             inv = f / (l_sum * f + exp2f(sk - m));
           }
           inv *= p.out_scale;
-          if (p.gate) gate = p.gate + batch * p.g_batch_stride + static_cast<long long>(row) * p.g_row_stride + head * p.g_head_stride + h * 64;
+          if (p.gate && !(kKept && p.gate_head))
+            gate = p.gate + batch * p.g_batch_stride + static_cast<long long>(row) * p.g_row_stride + head * p.g_head_stride + h * 64;
+          if (kKept && p.gate && p.gate_head && row_ok)
+            inv = __fdividef(inv, 1.f + __expf(-__bfloat162float(p.gate[batch * p.g_batch_stride + static_cast<long long>(row) * p.g_row_stride + head * p.g_head_stride])));
         }
         __nv_bfloat16* out = p.O + batch * p.o_batch_stride + static_cast<long long>(row) * p.o_row_stride +
                              head * p.o_head_stride + h * 64;
+        if (kKept && p.back != nullptr) {
+          // eight channel pairs at a time, the two halves of the row taking turns
+          const float2* turn = p.back + static_cast<long long>(row) * p.back_half;
+          const uint32_t o_row = tmem_base + 256 + t * 128 + lane_addr;
+          __nv_bfloat16* out0 = out - h * 64;
+#pragma unroll 1
+          for (int c = h * 8; c < p.back_half; c += 16) {
+            uint32_t u[8], w[8];
+            tmem_ld_32x8_nowait(o_row + c, u);
+            tmem_ld_32x8_nowait(o_row + p.back_half + c, w);
+            tmem_wait_ld();
+            if (row_ok) {
+              float a[8], b[8];
+#pragma unroll
+              for (int e = 0; e < 8; e += 2) {
+                const float4 cs = *reinterpret_cast<const float4*>(turn + c + e);
+                const float u0 = __uint_as_float(u[e]) * inv, w0 = __uint_as_float(w[e]) * inv;
+                const float u1 = __uint_as_float(u[e + 1]) * inv, w1 = __uint_as_float(w[e + 1]) * inv;
+                a[e] = u0 * cs.x + w0 * cs.y; b[e] = w0 * cs.x - u0 * cs.y;
+                a[e + 1] = u1 * cs.z + w1 * cs.w; b[e + 1] = w1 * cs.z - u1 * cs.w;
+              }
+              *reinterpret_cast<uint4*>(out0 + c) = make_uint4(pack_bf16x2(a[0], a[1]), pack_bf16x2(a[2], a[3]), pack_bf16x2(a[4], a[5]), pack_bf16x2(a[6], a[7]));
+              *reinterpret_cast<uint4*>(out0 + p.back_half + c) =
+                  make_uint4(pack_bf16x2(b[0], b[1]), pack_bf16x2(b[2], b[3]), pack_bf16x2(b[4], b[5]), pack_bf16x2(b[6], b[7]));
+            }
+          }
+        } else {
 #pragma unroll
         for (int c = 0; c < 2; ++c) {
           uint32_t o[32];
@@ -504,7 +557,7 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
 #pragma unroll
             for (int q = 0; q < 4; ++q) {
               if (BIAS != 0 && h * 64 + c * 32 + q * 8 >= p.dv) break;
-              if (BIAS == 3 && gate) {
+              if (kGated && gate) {
                 const uint4 gu = *reinterpret_cast<const uint4*>(gate + c * 32 + q * 8);
                 const uint32_t gw[4] = {gu.x, gu.y, gu.z, gu.w};
 #pragma unroll
@@ -522,6 +575,7 @@ flash_fwd_d128_kernel(const __grid_constant__ CUtensorMap tmQ,
               *reinterpret_cast<uint4*>(out + c * 32 + q * 8) = u;
             }
           }
+        }
         }
         if (p.lse && row_ok && h == 0)
           p.lse[(static_cast<long long>(batch) * p.Hq + head) * p.Tq + row] =
@@ -582,6 +636,9 @@ struct FlashExtra {           // sink and gate form
   const void* gate;
   const long long* gate_strides;
   float out_scale;
+  int kept = 0;               // the form with kept keys
+  int keep = 0, gate_head = 0, back_half = 0;
+  const float2* back = nullptr;
 };
 
 static int flash_fwd_launch(const void* q, const void* k, const void* v, void* o, float* lse, int B, int Hq, int Hkv, int Tq, int Tk,
@@ -599,11 +656,12 @@ static int flash_fwd_launch(const void* q, const void* k, const void* v, void* o
   constexpr size_t kBase = sizeof(AttnSmem) + 1024, kMax = 227 * 1024;
   const size_t table = (static_cast<size_t>(window) + 2 * ATT_TBL_PAD) * sizeof(float);
   // the table covers a causal window whose distances start at 0 in the query's own block (no key offset)
-  const int bias = extra != nullptr ? 3 : r1 == nullptr ? 0 : (causal && window > 0 && q_offset == 0 && kBase + table <= kMax ? 1 : 2);
+  const int bias = extra != nullptr ? (extra->kept ? 4 : 3) : r1 == nullptr ? 0 : (causal && window > 0 && q_offset == 0 && kBase + table <= kMax ? 1 : 2);
   const size_t smem = bias == 1 ? kBase + table : kBase;
   auto kernel = bias == 0 ? flash_fwd_d128_kernel<0>
-                          : (bias == 1 ? flash_fwd_d128_kernel<1> : (bias == 2 ? flash_fwd_d128_kernel<2> : flash_fwd_d128_kernel<3>));
-  static bool configured_dev[64][4] = {};       // the attribute is per device
+                          : (bias == 1 ? flash_fwd_d128_kernel<1>
+                                       : (bias == 2 ? flash_fwd_d128_kernel<2> : (bias == 3 ? flash_fwd_d128_kernel<3> : flash_fwd_d128_kernel<4>)));
+  static bool configured_dev[64][5] = {};       // the attribute is per device
   int cfg_dev = 0;
   if (cudaGetDevice(&cfg_dev) != cudaSuccess || cfg_dev < 0 || cfg_dev >= 64) cfg_dev = 0;
   bool& configured = configured_dev[cfg_dev][bias];
@@ -618,6 +676,7 @@ static int flash_fwd_launch(const void* q, const void* k, const void* v, void* o
     p.gate = static_cast<const __nv_bfloat16*>(extra->gate);
     p.g_batch_stride = extra->gate_strides[0]; p.g_row_stride = extra->gate_strides[1]; p.g_head_stride = extra->gate_strides[2];
     p.out_scale = extra->out_scale;
+    p.keep = extra->keep; p.gate_head = extra->gate_head; p.back = extra->back; p.back_half = extra->back_half;
   }
   p.B = B; p.Hq = Hq; p.Hkv = Hkv; p.Tq = Tq; p.Tk = Tk;
   p.q_offset = q_offset; p.causal = causal; p.window = window;
@@ -661,5 +720,20 @@ extern "C" TYR_EXPORT int tyr_flash_fwd_sink(const void* q, const void* k, const
   if (dk <= 0 || dv <= 0 || dk > ATT_D || dv > ATT_D || (dk & 7) || (dv & 7) || window < 0 || scale <= 0.f) return -1;
   if (gate != nullptr && (((strides[12] | strides[13] | strides[14]) & 7) || (reinterpret_cast<uintptr_t>(gate) & 15))) return -3;
   const FlashExtra ex{sink, gate, strides + 12, out_scale};
+  return flash_fwd_launch(q, k, v, o, nullptr, B, Hq, Hkv, T, T, dk, dv, strides, 1, window, 0, scale, nullptr, nullptr, err, stream, &ex);
+}
+
+// The sink form whose window (0: none) leaves the first `keep` keys visible.  gate_head: the gate is one number per (row, head), any strides.
+// back (nullable): [T, dv / 2] pairs (cos, sin) by which the output's channel pairs (m, m + dv / 2) are turned back; dv a multiple of 16 then.
+extern "C" TYR_EXPORT int tyr_flash_fwd_kept(const void* q, const void* k, const void* v, void* o, const float* sink, const void* gate, int gate_head,
+                                             const void* back, int B, int Hq, int Hkv, int T, int dk, int dv, const long long* strides, int window,
+                                             int keep, float scale, float out_scale, int* err, void* stream) {
+  if (dk <= 0 || dv <= 0 || dk > ATT_D || dv > ATT_D || (dk & 7) || (dv & 7) || window < 0 || keep < 0 || scale <= 0.f) return -1;
+  if (back != nullptr && ((dv & 15) || (reinterpret_cast<uintptr_t>(back) & 15) || (gate != nullptr && !gate_head))) return -5;
+  if (gate != nullptr && !gate_head && (((strides[12] | strides[13] | strides[14]) & 7) || (reinterpret_cast<uintptr_t>(gate) & 15))) return -3;
+  FlashExtra ex{sink, gate, strides + 12, out_scale};
+  ex.kept = 1;
+  ex.keep = keep; ex.gate_head = gate_head; ex.back_half = dv / 2;
+  ex.back = static_cast<const float2*>(back);
   return flash_fwd_launch(q, k, v, o, nullptr, B, Hq, Hkv, T, T, dk, dv, strides, 1, window, 0, scale, nullptr, nullptr, err, stream, &ex);
 }

@@ -2,7 +2,8 @@
 //
 //   score(i, j) = scale q_i . k_j - r1_h ln(1 + r2_h (i - j)),   0 <= i - j < window,
 //
-// a sink (the softmax denominator also holds exp(sink_h)) and an output gate (element by element, out_scale sigmoid(gate)).
+// a sink (the softmax denominator also holds exp(sink_h)), an output gate (element by element or one number per head, out_scale sigmoid(gate)),
+// first positions that stay visible past the window, and an output whose channel pairs (m, m + dv / 2) are turned back by the query's angles.
 //
 //   * qk_norm_store: per-head RMSNorm of q and k (no rotation; weights and projection biases optional), v copied, rows of the padded batch written to the K/V store at
 //                    their own positions (plain or ring).
@@ -148,6 +149,9 @@ struct GeneralAttnArgs {
   int B, S, H, G, dk, dv, cap, ring, window, keys;
   float scale, out_scale;
   int* err;
+  int keep;                    // positions 0 .. keep - 1 are visible past the window; a ring store holds them in its first slots
+  int gate_head;               // the gate is one number per (row, head): channel h
+  const float2* back;          // [positions, dv / 2] (cos, sin) (nullable)
 };
 constexpr int GA_WARPS = 4;
 constexpr int GA_DMAX = 256;
@@ -176,16 +180,22 @@ __global__ void __launch_bounds__(GA_WARPS * 32) general_attention_kernel(Genera
   for (int d = lane; d < a.dk; d += 32) sq[warp][d] = ag_load(qp + d);
   __syncwarp();
   const float r1 = a.r1 ? a.r1[h] : 0.f, r2 = a.r1 ? a.r2[h] : 0.f;
+  const int ring_len = a.cap - a.keep;
   int lo = a.window > 0 ? max(0, p - a.window + 1) : 0;
-  if (a.ring) lo = max(lo, p - a.cap + 1);
+  if (a.ring) lo = max(lo, p - ring_len + 1);
+  const int k0 = min(a.keep, lo), gap = lo - k0, n = p + 1 - gap;      // key i of n: position i, past the k0 kept ones i + gap
+  auto slot_of = [&](int i) {
+    const int j = i < k0 ? i : i + gap;
+    return static_cast<long long>(a.ring && j >= a.keep ? a.keep + (j - a.keep) % ring_len : j);
+  };
   float m = a.sink ? a.sink[h] : -INFINITY, l = a.sink ? 1.f : 0.f, acc[GA_DMAX / 32];
 #pragma unroll
   for (int j = 0; j < GA_DMAX / 32; ++j) acc[j] = 0.f;
-  for (int base = lo; base <= p; base += 32) {
-    const int j = base + lane;
+  for (int base = 0; base < n; base += 32) {
+    const int i = base + lane, j = i < k0 ? i : i + gap;
     float sc = -INFINITY;
-    if (j <= p) {
-      const T* kr = kb + static_cast<long long>(a.ring ? j % a.cap : j) * a.k_ss;
+    if (i < n) {
+      const T* kr = kb + slot_of(i) * a.k_ss;
       float dot = 0.f;
       for (int d = 0; d < a.dk; ++d) dot += sq[warp][d] * ag_load(kr + d);
       sc = dot * a.scale - r1 * log1pf(r2 * static_cast<float>(p - j));
@@ -198,10 +208,10 @@ __global__ void __launch_bounds__(GA_WARPS * 32) general_attention_kernel(Genera
     __syncwarp();
 #pragma unroll
     for (int c = 0; c < GA_DMAX / 32; ++c) acc[c] *= f;
-    const int nk = min(32, p - base + 1);
+    const int nk = min(32, n - base);
     for (int t = 0; t < nk; ++t) {
       const float wt = sp[warp][t];
-      const T* vr = vb + static_cast<long long>(a.ring ? (base + t) % a.cap : base + t) * a.v_ss;
+      const T* vr = vb + slot_of(base + t) * a.v_ss;
 #pragma unroll
       for (int c = 0; c < GA_DMAX / 32; ++c)
         if (lane + 32 * c < a.dv) acc[c] += wt * ag_load(vr + lane + 32 * c);
@@ -209,11 +219,25 @@ __global__ void __launch_bounds__(GA_WARPS * 32) general_attention_kernel(Genera
     __syncwarp();
   }
   T* op = static_cast<T*>(a.out) + row * a.out_ld + static_cast<long long>(h) * a.dv;
-  const T* gp = a.gate ? static_cast<const T*>(a.gate) + row * a.gate_ld + static_cast<long long>(h) * a.dv : nullptr;
+  const T* gp = a.gate ? static_cast<const T*>(a.gate) + row * a.gate_ld + static_cast<long long>(h) * (a.gate_head ? 1 : a.dv) : nullptr;
+  if (a.back != nullptr) {                         // the queries are done with: a channel's partner is in another lane
+#pragma unroll
+    for (int c = 0; c < GA_DMAX / 32; ++c)
+      if (lane + 32 * c < a.dv) sq[warp][lane + 32 * c] = acc[c];
+    __syncwarp();
+    const int half = a.dv / 2;
+    const float2* cs = a.back + static_cast<long long>(p) * half;
+#pragma unroll
+    for (int c = 0; c < GA_DMAX / 32; ++c) {
+      const int d = lane + 32 * c;
+      if (d < half) acc[c] = sq[warp][d] * cs[d].x + sq[warp][d + half] * cs[d].y;
+      else if (d < a.dv) acc[c] = sq[warp][d] * cs[d - half].x - sq[warp][d - half] * cs[d - half].y;
+    }
+  }
 #pragma unroll
   for (int c = 0; c < GA_DMAX / 32; ++c)
     if (lane + 32 * c < a.dv) {
-      const float g = gp ? a.out_scale / (1.f + expf(-ag_load(gp + lane + 32 * c))) : a.out_scale;
+      const float g = gp ? a.out_scale / (1.f + expf(-ag_load(gp + (a.gate_head ? 0 : lane + 32 * c)))) : a.out_scale;
       ag_store(op + lane + 32 * c, acc[c] / l * g);
     }
 }
@@ -275,5 +299,20 @@ extern "C" TYR_EXPORT int tyr_general_attention_sink(const void* q, const void* 
   a.B = B; a.S = S; a.H = H; a.G = G; a.dk = dk; a.dv = dv; a.cap = keys; a.keys = keys;
   a.gate_ld = strides[9]; a.out_ld = strides[10];
   a.scale = scale; a.out_scale = out_scale; a.err = err;
+  return general_attention_launch(a, strides, dtype, stream);
+}
+
+// A window (0: none) that leaves the first `keep` positions visible, in rows of a prompt, a plain store or one of `keep` slots followed by a
+// ring; one gate per head (nullable: rows of strides[9] elements); `back` (nullable): [positions, dv / 2] pairs (cos, sin).  strides: as for
+// the sink form.
+extern "C" TYR_EXPORT int tyr_general_attention_kept(const void* q, const void* k, const void* v, void* out, const int* pos, const void* head_gate,
+                                                     const void* back, const long long* strides, int B, int S, int H, int G, int dk, int dv, int cap,
+                                                     int ring, int window, int keep, int keys, float scale, int dtype, int* err, void* stream) {
+  if (keep < 0 || (ring && keep >= cap) || (back != nullptr && (dv & 1))) return -3;
+  GeneralAttnArgs a{};
+  a.q = q; a.k = k; a.v = v; a.out = out; a.pos = pos; a.gate = head_gate; a.gate_head = 1; a.back = static_cast<const float2*>(back);
+  a.B = B; a.S = S; a.H = H; a.G = G; a.dk = dk; a.dv = dv; a.cap = cap; a.ring = ring; a.window = window; a.keep = keep; a.keys = keys;
+  a.gate_ld = strides[9]; a.out_ld = strides[10];
+  a.scale = scale; a.out_scale = 1.f; a.err = err;
   return general_attention_launch(a, strides, dtype, stream);
 }

@@ -13,6 +13,8 @@
 // modulo its capacity), so a window may be smaller than the ring and a penalty r1_h ln(1 + r2_h distance) can be taken off the
 // scores (template parameter BIAS).  Key size DK and value size DV may differ.  The softmax denominator may also hold exp(sink_h),
 // added once when a row's result is written, and the values may be the keys (one store: its rows are read from memory once).
+// The first `keep` positions may stay visible past the window; a ring store then holds them in its first slots and the ring after them.
+// Values that were rotated by their positions: the output's channel pairs (m, m + dv / 2) are turned back by the query's angles.
 //
 // The reference takes the library SDPA over a sliced cache for this step (cc/include/tyr_attention.h:58-130,
 // Tyr/Inference/KVCache.lean:41-215).
@@ -43,7 +45,7 @@ struct DecodeAttnArgs {
   int B, Hq, Hkv, cap, ring, window, splits, append;
   float scale_log2;
   int* err;
-  // optional output gate, applied when the result is written: mode 1 = one value per (batch, head), out *= softplus(g)
+  // optional output gate, applied when the result is written (mode 3: one value per (batch, head), out *= sigmoid(g)): mode 1 = one value per (batch, head), out *= softplus(g)
   // (Laguna); mode 2 = one value per element, out *= sigmoid(g) (Qwen3.5).  Element (b, h, d) is at gate + b * gate_bs +
   // h * gate_hs (+ d in mode 2).
   const __nv_bfloat16* gate;
@@ -53,6 +55,9 @@ struct DecodeAttnArgs {
   long long out_bs;              // batch stride of out
   int dv;                        // channels of a head that are written (heads of out are packed)
   float out_scale;
+  int keep;                      // positions 0 .. keep - 1 are visible past the window
+  const float2* back;            // [positions, back_half] (cos, sin) of a position's turns (nullable)
+  int back_half;
 };
 
 __device__ __forceinline__ float decode_gate(const DecodeAttnArgs& a, int b, int h, int d) {
@@ -60,8 +65,8 @@ __device__ __forceinline__ float decode_gate(const DecodeAttnArgs& a, int b, int
     const float g = __bfloat162float(a.gate[b * a.gate_bs + h * a.gate_hs]);
     return g > 20.f ? g : log1pf(__expf(g));
   }
-  if (a.gate_mode == 2) {
-    const float g = __bfloat162float(a.gate[b * a.gate_bs + h * a.gate_hs + d]);
+  if (a.gate_mode >= 2) {
+    const float g = __bfloat162float(a.gate[b * a.gate_bs + h * a.gate_hs + (a.gate_mode == 2 ? d : 0)]);
     return 1.f / (1.f + __expf(-g));
   }
   return 1.f;
@@ -102,6 +107,13 @@ __device__ __forceinline__ uint32_t prmt(uint32_t a, uint32_t b, uint32_t sel) {
   return r;
 }
 
+// Channels d and d + back_half of a head, turned back by the angles of position `pos`.
+__device__ __forceinline__ void decode_write_turned(const DecodeAttnArgs& a, int b, int h, int d, int pos, float M, float L, float u, float w) {
+  const float2 cs = a.back[static_cast<long long>(pos) * a.back_half + d];
+  decode_write(a, b, h, d, M, L, u * cs.x + w * cs.y);
+  decode_write(a, b, h, d + a.back_half, M, L, w * cs.x - u * cs.y);
+}
+
 // The end of both kernels: combine the four warps' states {s_m, s_l, acc} (acc_warp: floats between two warps' accumulators), write the
 // result of a single slice, or leave the partial and let the last CTA of this (batch, K/V head) merge all slices.
 template <int DV, int GM>
@@ -116,17 +128,22 @@ __device__ __forceinline__ void decode_combine(const DecodeAttnArgs& a, int b, i
     float M = -INFINITY;
 #pragma unroll
     for (int w = 0; w < kDecWarps; ++w) M = fmaxf(M, s_m[w][g]);
-    float L = 0.f, A = 0.f;
+    float L = 0.f, A = 0.f, A2 = 0.f;
+    const bool turned = a.splits == 1 && a.back != nullptr;
+    if (turned && d >= a.back_half) continue;
     if (M > -INFINITY) {
 #pragma unroll
       for (int w = 0; w < kDecWarps; ++w) {
         const float f = exp2f(s_m[w][g] - M);
         L += s_l[w][g] * f;
         A += acc[w * (acc_warp / DV) + g][d] * f;
+        if (turned) A2 += acc[w * (acc_warp / DV) + g][d + a.back_half] * f;
       }
     }
     const long long row = static_cast<long long>(b) * a.Hq + hq0 + g;
-    if (a.splits == 1) {
+    if (turned) {
+      decode_write_turned(a, b, hq0 + g, d, a.pos[b * a.pos_stride], M, L, A, A2);
+    } else if (a.splits == 1) {
       decode_write(a, b, hq0 + g, d, M, L, A);
     } else {
       a.part_acc[(row * a.splits + split) * DV + d] = A;
@@ -149,16 +166,19 @@ __device__ __forceinline__ void decode_combine(const DecodeAttnArgs& a, int b, i
     const int g = i / DV, d = i - g * DV;
     const long long row = static_cast<long long>(b) * a.Hq + hq0 + g;
     float M = -INFINITY;
+    if (a.back != nullptr && d >= a.back_half) continue;
     for (int sp = 0; sp < a.splits; ++sp) M = fmaxf(M, __ldcg(&a.part_ml[(row * a.splits + sp) * 2]));
-    float L = 0.f, A = 0.f;
+    float L = 0.f, A = 0.f, A2 = 0.f;
     if (M > -INFINITY) {
       for (int sp = 0; sp < a.splits; ++sp) {
         const float f = exp2f(__ldcg(&a.part_ml[(row * a.splits + sp) * 2]) - M);
         L += __ldcg(&a.part_ml[(row * a.splits + sp) * 2 + 1]) * f;
         A += __ldcg(&a.part_acc[(row * a.splits + sp) * DV + d]) * f;
+        if (a.back != nullptr) A2 += __ldcg(&a.part_acc[(row * a.splits + sp) * DV + d + a.back_half]) * f;
       }
     }
-    decode_write(a, b, hq0 + g, d, M, L, A);
+    if (a.back != nullptr) decode_write_turned(a, b, hq0 + g, d, a.pos[b * a.pos_stride], M, L, A, A2);
+    else decode_write(a, b, hq0 + g, d, M, L, A);
   }
   if (tid == 0) a.counters[b * a.Hkv + hkv] = 0;
 }
@@ -190,16 +210,18 @@ __global__ void __launch_bounds__(kDecWarps * 32) decode_attention_kernel(Decode
     if (tid == 0) report_error(a.err, ERR_BOUNDS, pos);
     return;
   }
-  // key index i of 0 .. n_keys - 1 is at distance n_keys - 1 - i from the new token and in slot slot0 + i (modulo cap)
-  int n_keys = pos + 1;
-  if (a.window > 0 && n_keys > a.window) n_keys = a.window;
-  if (a.ring && n_keys > a.cap) n_keys = a.cap;
-  const int start = pos + 1 - n_keys;
-  const int slot0 = a.ring ? start % a.cap : start;
-  const int slot_new = a.ring ? pos % a.cap : pos;
+  // Key index i of 0 .. n_keys - 1: the first k0 are the kept positions that the window has left behind, in slots of their own; the rest
+  // is at distance n_keys - 1 - i from the new token and in slot slot0 + i - k0 (a ring: modulo its length).
+  const int ring_len = a.cap - a.keep;
+  int start = a.window > 0 && pos + 1 > a.window ? pos + 1 - a.window : 0;
+  if (a.ring && pos + 1 - ring_len > start) start = pos + 1 - ring_len;
+  const int k0 = min(a.keep, start);
+  const int n_keys = k0 + pos + 1 - start;
+  const int slot0 = (a.ring && start >= a.keep ? a.keep + (start - a.keep) % ring_len : start) - k0;
+  const int slot_new = a.ring && pos >= a.keep ? a.keep + (pos - a.keep) % ring_len : pos;
   auto slot_of = [&](int i) {
-    int sl = slot0 + i;
-    return sl >= a.cap ? sl - a.cap : sl;
+    const int sl = slot0 + i;
+    return i < k0 ? i : (sl >= a.cap ? sl - ring_len : sl);
   };
   int chunk = (n_keys + a.splits - 1) / a.splits;
   chunk = (chunk + 63) & ~63;
@@ -210,8 +232,9 @@ __global__ void __launch_bounds__(kDecWarps * 32) decode_attention_kernel(Decode
   const long long kv_row = (static_cast<long long>(b) * a.Hkv + hkv) * a.cap;
   __nv_bfloat16* kc = a.k_cache + kv_row * DK;
   __nv_bfloat16* vc = a.v_cache + kv_row * DV;
-  const __nv_bfloat16* kn = a.k_new + b * a.kn_bs + static_cast<long long>(hkv) * DK;
-  const __nv_bfloat16* vn = a.v_new + b * a.vn_bs + static_cast<long long>(hkv) * DV;
+  const bool fresh = a.k_new != nullptr;         // otherwise the store already holds the new token
+  const __nv_bfloat16* kn = fresh ? a.k_new + b * a.kn_bs + static_cast<long long>(hkv) * DK : nullptr;
+  const __nv_bfloat16* vn = fresh ? a.v_new + b * a.vn_bs + static_cast<long long>(hkv) * DV : nullptr;
 
   if (a.append && split == 0) {                  // fused append; nobody reads this slot from the store in this launch
     for (int i = tid; i < DK / 8; i += kDecWarps * 32)
@@ -256,7 +279,7 @@ __global__ void __launch_bounds__(kDecWarps * 32) decode_attention_kernel(Decode
     for (int tile = 0; tile < 2; ++tile) {
       int row = base + 8 * tile + g;
       row = row < hi ? row : hi - 1;             // clamped rows are masked below
-      const __nv_bfloat16* krow = (row == n_keys - 1) ? kn : kc + static_cast<long long>(slot_of(row)) * DK;
+      const __nv_bfloat16* krow = (fresh && row == n_keys - 1) ? kn : kc + static_cast<long long>(slot_of(row)) * DK;
       uint4 kf[NJ];
 #pragma unroll
       for (int j = 0; j < NJ; ++j) kf[j] = *reinterpret_cast<const uint4*>(krow + 32 * j + 8 * t);
@@ -288,7 +311,7 @@ __global__ void __launch_bounds__(kDecWarps * 32) decode_attention_kernel(Decode
     for (int i = 0; i < 4; ++i) {
       int row = base + 2 * t + (i & 1) + 8 * (i >> 1);
       row = row < hi ? row : hi - 1;
-      vrow[i] = (row == n_keys - 1) ? vn : vc + static_cast<long long>(slot_of(row)) * DV;
+      vrow[i] = (fresh && row == n_keys - 1) ? vn : vc + static_cast<long long>(slot_of(row)) * DV;
     }
     uint4 vf[NC][4];
 #pragma unroll
@@ -500,9 +523,9 @@ static int decode_attention_launch(const void* q, const void* k_new, const void*
                                    int Hq, int Hkv, int DK, int DV, int cap, int ring, int window, int splits, int append, float scale,
                                    const void* gate, long long gate_bs, long long gate_hs, int gate_mode, const float* r1,
                                    const float* r2, void* err, void* stream, const float* sink = nullptr, int dv_out = 0,
-                                   long long out_bs = 0, float out_scale = 1.f) {
+                                   long long out_bs = 0, float out_scale = 1.f, int keep = 0, const void* back = nullptr) {
   using namespace tyr;
-  if (gate_mode < 0 || gate_mode > 2 || (gate_mode != 0 && gate == nullptr)) return -5;
+  if (gate_mode < 0 || gate_mode > 3 || (gate_mode != 0 && gate == nullptr)) return -5;
   if (B <= 0 || Hq <= 0 || Hkv <= 0 || Hq % Hkv != 0 || Hq / Hkv > 16 || cap <= 0 || splits < 1 || splits > 64) return -1;
   const bool wide = Hq / Hkv > 8;
   if ((q_bs | kn_bs | vn_bs) & 7) return -3;                       // 16-byte rows
@@ -523,10 +546,15 @@ static int decode_attention_launch(const void* q, const void* k_new, const void*
   a.dv = dv_out > 0 ? dv_out : DV;
   a.out_bs = out_bs > 0 ? out_bs : static_cast<long long>(Hq) * DV;
   a.out_scale = out_scale;
+  if (keep < 0 || keep >= cap || (keep > 0 && r1 != nullptr) || (append && k_new == nullptr) || (k_new == nullptr) != (v_new == nullptr)) return -7;
+  a.keep = keep;
+  a.back = (const float2*)back;
+  a.back_half = a.dv / 2;
+  if (back != nullptr && (a.dv & 1)) return -8;
   const dim3 grid(splits, Hkv, B);
   const cudaStream_t st = (cudaStream_t)stream;
   const dim3 block(kDecWarps * 32);
-  if (k_cache == v_cache && k_new == v_new && DK == DV && (DK == 64 || DK == 128) && !wide && r1 == nullptr && !ring && window == 0) {
+  if (k_cache == v_cache && k_new == v_new && DK == DV && (DK == 64 || DK == 128) && !wide && r1 == nullptr && !ring && window == 0 && k_new != nullptr) {
     const size_t smem = static_cast<size_t>(kDecWarps) * kRing * 16 * DK * 2;
     auto kernel = DK == 64 ? decode_attention_shared_kernel<64> : decode_attention_shared_kernel<128>;
     static bool configured[64][2] = {};          // the attribute is per device
@@ -547,6 +575,8 @@ static int decode_attention_launch(const void* q, const void* k_new, const void*
   TYR_DEC(64, 64, false, false) TYR_DEC(64, 64, true, false)
   TYR_DEC(128, 128, false, false) TYR_DEC(128, 128, true, false)
   TYR_DEC(256, 256, false, false)                                  // 16 heads x 256 channels of accumulators do not fit a warp
+  TYR_DEC(64, 128, false, false) TYR_DEC(64, 128, true, false)
+  TYR_DEC(128, 64, false, false) TYR_DEC(128, 64, true, false)
   TYR_DEC(64, 64, false, true) TYR_DEC(64, 64, true, true)
   TYR_DEC(128, 128, false, true) TYR_DEC(128, 128, true, true)
   TYR_DEC(64, 128, false, true) TYR_DEC(64, 128, true, true)
@@ -597,4 +627,18 @@ extern "C" TYR_EXPORT int tyr_decode_attention_sink(const void* q, const void* k
   return decode_attention_launch(q, k_new, v_new, k_cache, v_cache, pos, pos_stride, out, workspace, q_bs, kn_bs, vn_bs, B, Hq, Hkv, D, D, cap, 0, 0,
                                  splits, append, scale, gate, gate_bs, dv, gate == nullptr ? 0 : 2, nullptr, nullptr, err, stream, sink, dv,
                                  out_bs, out_scale);
+}
+
+// Window (0: none) that leaves the first `keep` positions visible, in a plain store or one of `keep` slots followed by a ring; output gate
+// sigmoid(head_gate[b * gate_bs + h]) (nullable); `back` (nullable): [positions, dv / 2] pairs (cos, sin) by which the output's channel pairs
+// (m, m + dv / 2) are turned back.  k_new / v_new null: the store holds the new token already.  DK, DV in {64, 128}.
+extern "C" TYR_EXPORT int tyr_decode_attention_kept(const void* q, const void* k_new, const void* v_new, void* k_cache, void* v_cache, const void* pos,
+                                                    int pos_stride, void* out, void* workspace, long long q_bs, long long kn_bs, long long vn_bs,
+                                                    int B, int Hq, int Hkv, int DK, int DV, int dv, int cap, int ring, int window, int keep, int splits,
+                                                    int append, float scale, const void* head_gate, long long gate_bs, const void* back,
+                                                    long long out_bs, void* err, void* stream) {
+  if (dv <= 0 || dv > DV) return -2;
+  return decode_attention_launch(q, k_new, v_new, k_cache, v_cache, pos, pos_stride, out, workspace, q_bs, kn_bs, vn_bs, B, Hq, Hkv, DK, DV, cap, ring,
+                                 window, splits, append, scale, head_gate, gate_bs, 1, head_gate == nullptr ? 0 : 3, nullptr, nullptr, err, stream,
+                                 nullptr, dv, out_bs, 1.f, keep, back);
 }

@@ -70,7 +70,7 @@ embed_grad_sorted_kernel(const __nv_bfloat16* __restrict__ dy, const long long* 
 
 // Input rows of a decoder with sinusoidal positions: x[r, d] = table[ids[r], d] * scale + sin / cos(p * freq[d / 2]), fp32, channel 2i the
 // sine and 2i + 1 the cosine.  `turns` holds the frequencies over 2 pi in double, so that the angle is reduced to a fraction of a turn
-// before it is rounded and far positions keep their accuracy.  p = pos[r] (a decode step), else r % S.
+// before it is rounded and far positions keep their accuracy.  p = pos[r] (a decode step), else r % S.  Without `turns` nothing is added.
 // A thread owns EP_PAIRS channel pairs of one position and walks the rows of the batch that share it (all of a prompt's; one of a step's).
 constexpr int EP_PAIRS = 4;
 __device__ __forceinline__ void ep_load(const __nv_bfloat16* p, float (&f)[8]) {
@@ -100,6 +100,10 @@ __global__ void __launch_bounds__(256) embed_positions_kernel(const long long* _
     float add[2 * EP_PAIRS];
 #pragma unroll
     for (int j = 0; j < EP_PAIRS; ++j) {
+      if (turns == nullptr) {
+        add[2 * j] = add[2 * j + 1] = 0.f;
+        continue;
+      }
       const double t = k0 + j < half ? p * turns[k0 + j] : 0.0;
       sincospif(2.f * static_cast<float>(t - rint(t)), &add[2 * j], &add[2 * j + 1]);
     }
@@ -143,7 +147,7 @@ extern "C" TYR_EXPORT int tyr_embed_grad_sorted(const void* dy, const long long*
   return static_cast<int>(cudaGetLastError());
 }
 
-// ids int64 [B, S]; table [vocab, D] (dtype 0 = bf16, 1 = fp32); turns double [(D + 1) / 2]; pos int32 [B] (S == 1) or null; x fp32 [B, S, D].
+// ids int64 [B, S]; table [vocab, D] (dtype 0 = bf16, 1 = fp32); turns double [(D + 1) / 2] or null; pos int32 [B] (S == 1) or null; x fp32 [B, S, D].
 // An id outside the table is recorded in `err` and its row left alone.
 extern "C" TYR_EXPORT int tyr_embed_positions(const void* ids, const void* table, const double* turns, const int* pos, float* x, int B,
                                               int S, int D, int vocab, float scale, int dtype, int* err, void* stream) {

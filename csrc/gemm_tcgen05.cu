@@ -22,6 +22,7 @@
 // What the reference does for the same products: cuBLAS through torch::linear / mm / bmm
 // (cc/src/tyr.cpp:1003-1036, 1267-1300) followed by separate elementwise kernels.
 #include "common.cuh"
+#include "gates.cuh"
 #include <cstdio>
 #include <cstdlib>
 #include <mutex>
@@ -38,7 +39,8 @@ struct GemmParams {
   const __nv_bfloat16* aux;
   long long ldc, ldaux, sC, sAux;
   float alpha, beta;
-  int act;        // 0 none, 1 relu(x)^2, 2 relu, 3 acc * 2*sqrt(aux), 4 SwiGLU of column halves, 5 GELU(tanh)-gate of column halves
+  int act;        // 0 none, 1 relu(x)^2, 2 relu, 3 acc * 2*sqrt(aux), 4 SwiGLU of column halves, 5 GELU(tanh)-gate of column halves,
+                  // 6 xIELU, 7 SiLU, 8 clamped SwiGLU of column halves (limit alpha, slope beta), 9 tanh-GELU times aux
   int out_mode;   // 0 bf16 store, 1 fp32 store, 2 fp32 atomic add (stream-K)
   // out_mode 2 only.  > 0: the first (tiles / grid) * grid tiles are reduced whole, one per CTA and round, and every
   // remaining tile is cut into sk_slabs equal k ranges that are dealt round-robin, slab by slab.  All CTAs then sweep the
@@ -111,6 +113,7 @@ __device__ __forceinline__ float apply_act(float v, int act) {
 //   ACT 0: v = alpha * acc (+ beta * aux)      1: alpha * relu(acc)^2 (+ ...)      2: alpha * relu(acc) (+ ...)
 //   ACT 3: v = alpha * acc * 2 * sqrt(aux)     (gradient of y = relu(z)^2 given aux = y)
 //   ACT 7: alpha * silu(acc) (+ ...)
+//   ACT 9: gelu(acc) * aux
 //   ACT 6: xIELU of acc: alpha z^2 + z / 2 above zero, beta (e^z - 1 - z) + z / 2 below (no aux)
 template <int ACT>
 __device__ __forceinline__ void epi_chunk(const uint32_t (&r)[32], const float (&ax)[32], bool use_aux, float alpha,
@@ -118,6 +121,9 @@ __device__ __forceinline__ void epi_chunk(const uint32_t (&r)[32], const float (
   if constexpr (ACT == 3) {
 #pragma unroll
     for (int j = 0; j < 32; ++j) v[j] = alpha * __uint_as_float(r[j]) * 2.f * sqrtf(fmaxf(ax[j], 0.f));
+  } else if constexpr (ACT == 9) {
+#pragma unroll
+    for (int j = 0; j < 32; ++j) v[j] = gelu_tanh(__uint_as_float(r[j])) * ax[j];
   } else if constexpr (ACT == 6) {
 #pragma unroll
     for (int j = 0; j < 32; ++j) {
@@ -515,7 +521,7 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA,
     // bf16 outputs leave through shared memory and TMA stores (full 128-byte rows; also the efficient
     // packet size for stores that cross NVLink in tp_mode 1); grouped / SwiGLU outputs need row masks
     // and keep the direct stores.
-    const bool tma_out = p.out_mode == 0 && p.group_offsets == nullptr && p.act != 4 && p.act != 5;
+    const bool tma_out = p.out_mode == 0 && p.group_offsets == nullptr && p.act != 4 && p.act != 5 && p.act != 8;
     uint32_t n_stores = 0;
     while (ok && next_segment(cursor, tile, kb0, kb1)) {
       int bi, m0, n0;
@@ -547,9 +553,9 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA,
         c_base = p.peer_c[owner];
         c_off = (static_cast<long long>(p.tp_rank) * p.rows_per_rank + (row - owner * p.rows_per_rank)) * p.ldc;
       }
-      if (p.act == 4 || p.act == 5) {
+      if (p.act == 4 || p.act == 5 || p.act == 8) {
         // gated MLP over column halves of the tile: out[:, n0/2 + j] = act(acc[:, j]) * acc[:, BN/2 + j], act = SiLU (4) or
-        // tanh-GELU (5)
+        // tanh-GELU (5), or the clamped form (8)
         // with eight epilogue warps (CTA pairs) each set of four takes half of the output columns
         const int gc0 = (EPI_WARPS == 8) ? (epi >> 2) * (BN / 128) : 0;
         const int gc1 = (EPI_WARPS == 8) ? gc0 + BN / 128 : BN / 64;
@@ -571,6 +577,10 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA,
           if (!row_ok || col >= p.N / 2) continue;
           __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(p.C) + c_off + col;
           float v[32];
+          if (p.act == 8) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) v[j] = clamped_swiglu(__uint_as_float(rg[j]), __uint_as_float(ru[j]), p.alpha, p.beta);
+          } else
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
             const float g = p.alpha * __uint_as_float(rg[j]);
@@ -623,7 +633,7 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA,
         }
         float v[32];
         const bool full = (col + 32 <= p.N);
-        const bool use_aux = p.aux != nullptr && (p.beta != 0.f || p.act == 3) && row_ok;
+        const bool use_aux = p.aux != nullptr && (p.beta != 0.f || p.act == 3 || p.act == 9) && row_ok;
         float ax[32];
         if (use_aux) {
           const __nv_bfloat16* axp = p.aux + x_off + col;
@@ -648,6 +658,7 @@ gemm_bf16_tcgen05_kernel(const __grid_constant__ CUtensorMap tmA,
         else if (p.act == 1) epi_chunk<1>(r, ax, use_aux, p.alpha, p.beta, v);
         else if (p.act == 2) epi_chunk<2>(r, ax, use_aux, p.alpha, p.beta, v);
         else if (p.act == 7) epi_chunk<7>(r, ax, use_aux, p.alpha, p.beta, v);
+        else if (p.act == 9) epi_chunk<9>(r, ax, use_aux, p.alpha, p.beta, v);
         else if (p.act == 6) epi_chunk<6>(r, ax, use_aux, p.alpha, p.beta, v);
         else epi_chunk<3>(r, ax, use_aux, p.alpha, p.beta, v);
         if (tma_out) {
@@ -1020,7 +1031,7 @@ static int gemm_impl(const TyrGemmArgs& a, const TyrTpArgs* tpa) {
     r = make_tmap_bf16_3d(&tmB, a.B, a.N, a.K, a.batch, a.ldb, a.sB, BK);
   if (r) return 4000 + r;
   CUtensorMap tmC{};
-  if (a.out_mode == 0 && a.group_offsets == nullptr && a.act != 4 && a.act != 5) {
+  if (a.out_mode == 0 && a.group_offsets == nullptr && a.act != 4 && a.act != 5 && a.act != 8) {
     if (tpa != nullptr && tpa->mode == 1) {
       for (int i = 0; i < tpa->world; ++i) {
         r = make_tmap_bf16_3d(&tmP.m[i], tpa->peers[i], a.N, static_cast<uint64_t>(tpa->world) * tpa->rows_per_rank, 1,

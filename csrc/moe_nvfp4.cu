@@ -105,7 +105,7 @@ nvfp4_dequant_kernel(const uint8_t* __restrict__ packed, const uint8_t* __restri
 // routing: one warp per token, E <= 512
 // ---------------------------------------------------------------------------------------------
 struct RouteArgs {
-  const float* logits;   // [T, E]
+  const float* logits;   // [T, ld], the first E columns
   const float* bias;     // [E] selection bias (nullable)
   int* ids;              // [T, k]
   float* weights;        // [T, k]
@@ -115,6 +115,7 @@ struct RouteArgs {
   int renorm;
   float softcap, scale;
   int groups, keep;      // groups > 1: E / groups neighbouring experts form a group; only the `keep` groups with the best expert compete
+  int ld;                // columns of a row of logits: E, or more where other projections of the token follow the router's
 };
 
 // One warp routes one token from its row of logits.  The row may have been written by other CTAs of the same launch, so it is
@@ -225,7 +226,7 @@ __global__ void __launch_bounds__(256) moe_route_kernel(RouteArgs a) {
   const int lane = threadIdx.x & 31;
   const int tok = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (tok >= a.T) return;
-  route_token(a, a.logits + static_cast<long long>(tok) * a.E, tok, lane);
+  route_token(a, a.logits + static_cast<long long>(tok) * a.ld, tok, lane);
 }
 
 // Decode-sized batches: router logits and routing in one launch.  CTA (token group, expert group) takes kRouteTok tokens and
@@ -257,7 +258,7 @@ __global__ void __launch_bounds__(256) moe_route_fused_kernel(RouteArgs a, const
   float acc[kRouteTok];
 #pragma unroll
   for (int t = 0; t < kRouteTok; ++t) acc[t] = 0.f;
-  if (e < a.E) {
+  if (e < a.ld) {
     const float4* w4 = reinterpret_cast<const float4*>(wr + static_cast<long long>(e) * h);
     const int q4 = h >> 2;                            // float4 groups per row; this warp takes [half * q4 / 2, ...)
     const int lo = half * (q4 >> 1), hi = half ? q4 : (q4 >> 1);
@@ -281,10 +282,10 @@ __global__ void __launch_bounds__(256) moe_route_fused_kernel(RouteArgs a, const
     for (int t = 0; t < kRouteTok; ++t) s_part[el][t] = acc[t];
   }
   __syncthreads();
-  if (half == 0 && lane == 0 && e < a.E) {
+  if (half == 0 && lane == 0 && e < a.ld) {
 #pragma unroll
     for (int t = 0; t < kRouteTok; ++t)
-      if (t < nt) logits[static_cast<long long>(tok0 + t) * a.E + e] = acc[t] + s_part[el][t];
+      if (t < nt) logits[static_cast<long long>(tok0 + t) * a.ld + e] = acc[t] + s_part[el][t];
   }
   __threadfence();
   __syncthreads();
@@ -292,7 +293,7 @@ __global__ void __launch_bounds__(256) moe_route_fused_kernel(RouteArgs a, const
   __syncthreads();
   if (!s_last) return;
   __threadfence();
-  if (warp < nt) route_token(a, logits + static_cast<long long>(tok0 + warp) * a.E, tok0 + warp, lane);
+  if (warp < nt) route_token(a, logits + static_cast<long long>(tok0 + warp) * a.ld, tok0 + warp, lane);
 }
 
 // offsets[E+1] from counts[E]; cursors[E] zeroed; tiles[E+1] (nullable) = prefix sum of
@@ -367,6 +368,94 @@ moe_gather_rows_kernel(const __nv_bfloat16* src, const int* pair_order, __nv_bfl
     if (!TYR_INDEX_OK(pair_order[pos], pairs, 12)) continue;
     reinterpret_cast<uint4*>(dst + static_cast<long long>(pos) * h)[c] =
         reinterpret_cast<const uint4*>(src + static_cast<long long>(tok) * h)[c];
+  }
+}
+
+// The same with the rows multiplied by their pairs' weights: experts that take the weighted token.
+__global__ void __launch_bounds__(256)
+moe_gather_scaled_kernel(const __nv_bfloat16* src, const int* pair_order, const float* weights, __nv_bfloat16* dst, int pairs, int k, int h) {
+  pdl_entry();
+  const int vec = h >> 3;
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < static_cast<long long>(pairs) * vec;
+       i += static_cast<long long>(gridDim.x) * blockDim.x) {
+    const int pos = static_cast<int>(i / vec), c = static_cast<int>(i % vec), pair = pair_order[pos];
+    if (!TYR_INDEX_OK(pair, pairs, 13)) continue;
+    const float w = weights[pair];
+    const uint4 u = reinterpret_cast<const uint4*>(src + static_cast<long long>(pair / k) * h)[c];
+    const float2 a0 = unpack_bf16x2(u.x), a1 = unpack_bf16x2(u.y), a2 = unpack_bf16x2(u.z), a3 = unpack_bf16x2(u.w);
+    reinterpret_cast<uint4*>(dst + static_cast<long long>(pos) * h)[c] =
+        make_uint4(pack_bf16x2(w * a0.x, w * a0.y), pack_bf16x2(w * a1.x, w * a1.y), pack_bf16x2(w * a2.x, w * a2.y), pack_bf16x2(w * a3.x, w * a3.y));
+  }
+}
+
+// The sum over a token's k pairs (unweighted) and sigmoid(gate[tok]) times the shared expert's row, added to the fp32 stream in place;
+// the stream also goes out as T.  Without pair_pos the rows of y are in pair order.  A thread takes V neighbouring channels.
+struct CombineResidualArgs {
+  const void* y;               // [rows, h]
+  const int* pair_pos;         // [T * k] (nullable)
+  const void* shared;          // [T, h] (nullable)
+  const float* gate;           // gate[tok * gate_ld] (nullable: 1)
+  long long gate_ld;
+  float* resid;                // [T, h]
+  void* out;                   // [T, h] (nullable)
+  int T, k, h;
+};
+template <typename T, int V>
+__device__ __forceinline__ void cr_load(const T* p, float (&f)[V]) {
+  if constexpr (V == 8 && sizeof(T) == 2) {
+    const uint4 u = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float2 t = unpack_bf16x2(w[e]);
+      f[2 * e] = t.x; f[2 * e + 1] = t.y;
+    }
+  } else if constexpr (V == 8) {
+    const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+  } else {
+    f[0] = static_cast<float>(*p);
+  }
+}
+template <typename T, int V>
+__global__ void __launch_bounds__(256) moe_combine_residual_kernel(CombineResidualArgs a) {
+  pdl_entry();
+  const int parts = a.h / V;
+  for (long long i = blockIdx.x * 256LL + threadIdx.x; i < static_cast<long long>(a.T) * parts; i += gridDim.x * 256LL) {
+    const int tok = static_cast<int>(i / parts);
+    const long long c = static_cast<long long>(i % parts) * V, at = static_cast<long long>(tok) * a.h + c;
+    float r[V], f[V], acc[V];
+    cr_load<float, V>(a.resid + at, r);
+#pragma unroll
+    for (int e = 0; e < V; ++e) acc[e] = 0.f;
+    for (int s = 0; s < a.k; ++s) {
+      const int pair = tok * a.k + s, pp = a.pair_pos ? a.pair_pos[pair] : pair;
+      cr_load<T, V>(static_cast<const T*>(a.y) + static_cast<long long>(pp) * a.h + c, f);
+#pragma unroll
+      for (int e = 0; e < V; ++e) acc[e] += f[e];
+    }
+    if (a.shared) {
+      const float g = a.gate ? 1.f / (1.f + expf(-a.gate[tok * a.gate_ld])) : 1.f;
+      cr_load<T, V>(static_cast<const T*>(a.shared) + at, f);
+#pragma unroll
+      for (int e = 0; e < V; ++e) acc[e] += g * f[e];
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) r[e] += acc[e];
+    if constexpr (V == 8) {
+      reinterpret_cast<float4*>(a.resid + at)[0] = make_float4(r[0], r[1], r[2], r[3]);
+      reinterpret_cast<float4*>(a.resid + at)[1] = make_float4(r[4], r[5], r[6], r[7]);
+    } else {
+      a.resid[at] = r[0];
+    }
+    if (a.out) {
+      T* o = static_cast<T*>(a.out) + at;
+      if constexpr (V == 8 && sizeof(T) == 2)
+        *reinterpret_cast<uint4*>(o) = make_uint4(pack_bf16x2(r[0], r[1]), pack_bf16x2(r[2], r[3]), pack_bf16x2(r[4], r[5]), pack_bf16x2(r[6], r[7]));
+      else
+#pragma unroll
+        for (int e = 0; e < V; ++e) o[e] = static_cast<T>(r[e]);
+    }
   }
 }
 
@@ -666,20 +755,22 @@ extern "C" TYR_EXPORT int tyr_nvfp4_dequant(const void* packed, const void* scal
 
 extern "C" TYR_EXPORT int tyr_moe_route(const float* logits, const float* bias, int* ids, float* weights, int* counts,
                                         int T, int E, int k, int softmax, int renorm, float softcap, float scale,
-                                        int groups, int keep, void* stream) {
+                                        int groups, int keep, int ld, void* stream) {
+  if (ld < E) return -5;
   if (T <= 0 || E <= 0 || E > 512 || k <= 0 || k > 32 || k > E) return -1;
   if (groups > 1 && (groups > 32 || E % groups || keep <= 0 || keep > groups || k > keep * (E / groups))) return -4;
-  RouteArgs a{logits, bias, ids, weights, counts, T, E, k, softmax, renorm, softcap, scale, groups, keep};
+  RouteArgs a{logits, bias, ids, weights, counts, T, E, k, softmax, renorm, softcap, scale, groups, keep, ld};
   moe_route_kernel<<<(T + 7) / 8, 256, 0, (cudaStream_t)stream>>>(a);
   return (int)cudaGetLastError();
 }
 
-// Router GEMV + routing in one launch: x bf16 [T, h] (h a multiple of 8), router weight fp32 [E, h], `logits` a scratch of
-// T * E floats, `tickets` ceil(T / 4) zeroed ints.
+// Router GEMV + routing in one launch: x bf16 [T, h] (h a multiple of 8), router weight fp32 [ld, h] whose first E rows route (the
+// logits of the others are written too), `logits` [T, ld] floats, `tickets` ceil(T / 4) zeroed ints.
 extern "C" TYR_EXPORT int tyr_moe_route_fused(const void* x, const float* router_w, const float* bias, float* logits,
                                               int* tickets, int* ids, float* weights, int* counts, int T, int E, int k,
                                               int h, int softmax, int renorm, float softcap, float scale, int groups, int keep,
-                                              void* stream) {
+                                              int ld, void* stream) {
+  if (ld < E) return -5;
   if (T <= 0 || E <= 0 || E > 512 || k <= 0 || k > 32 || k > E || h <= 0 || (h & 7)) return -1;
   if (groups > 1 && (groups > 32 || E % groups || keep <= 0 || keep > groups || k > keep * (E / groups))) return -4;
   if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(router_w)) & 15) return -2;
@@ -690,8 +781,8 @@ extern "C" TYR_EXPORT int tyr_moe_route_fused(const void* x, const float* router
     cudaFuncSetAttribute(moe_route_fused_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     configured = smem;
   }
-  RouteArgs a{nullptr, bias, ids, weights, counts, T, E, k, softmax, renorm, softcap, scale, groups, keep};
-  dim3 grid((T + kRouteTok - 1) / kRouteTok, (E + kRouteExp - 1) / kRouteExp);
+  RouteArgs a{nullptr, bias, ids, weights, counts, T, E, k, softmax, renorm, softcap, scale, groups, keep, ld};
+  dim3 grid((T + kRouteTok - 1) / kRouteTok, (ld + kRouteExp - 1) / kRouteExp);
   return (int)launch_dependent(moe_route_fused_kernel, grid, dim3(256), smem, (cudaStream_t)stream, a, (const __nv_bfloat16*)x,
                                router_w, logits, tickets, h);
 }
@@ -727,6 +818,29 @@ extern "C" TYR_EXPORT int tyr_moe_combine(const void* y, const int* pair_pos, co
   if (T <= 0 || (h & 7)) return -1;
   return (int)launch_dependent(moe_combine_kernel, dim3(blocks_for(1LL * T * (h / 8))), dim3(256), 0, (cudaStream_t)stream,
                                (const __nv_bfloat16*)y, pair_pos, weights, (const __nv_bfloat16*)add, (__nv_bfloat16*)out, T, k, h);
+}
+
+extern "C" TYR_EXPORT int tyr_moe_gather_scaled(const void* src, const int* pair_order, const float* weights, void* dst, int pairs, int k, int h,
+                                                void* stream) {
+  if (pairs <= 0 || k <= 0 || (h & 7)) return -1;
+  return (int)launch_dependent(moe_gather_scaled_kernel, dim3(blocks_for(1LL * pairs * (h / 8))), dim3(256), 0, (cudaStream_t)stream,
+                               (const __nv_bfloat16*)src, pair_order, weights, (__nv_bfloat16*)dst, pairs, k, h);
+}
+
+// dtype of y, shared and out: 0 = bf16, 1 = fp32.
+extern "C" TYR_EXPORT int tyr_moe_combine_residual(const void* y, const int* pair_pos, const void* shared, const float* gate, long long gate_ld,
+                                                   float* resid, void* out, int T, int k, int h, int dtype, void* stream) {
+  if (T <= 0 || k < 0 || h <= 0) return -1;
+  CombineResidualArgs a{y, pair_pos, shared, gate, gate_ld, resid, out, T, k, h};
+  const uintptr_t al = reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(shared) | reinterpret_cast<uintptr_t>(resid) | reinterpret_cast<uintptr_t>(out);
+  const bool vec = (h & 7) == 0 && (al & 15) == 0;
+  const dim3 grid(blocks_for(1LL * T * (vec ? h / 8 : h))), block(256);
+  cudaStream_t st = (cudaStream_t)stream;
+  if (dtype == 1)
+    return (int)(vec ? launch_dependent(moe_combine_residual_kernel<float, 8>, grid, block, 0, st, a)
+                     : launch_dependent(moe_combine_residual_kernel<float, 1>, grid, block, 0, st, a));
+  return (int)(vec ? launch_dependent(moe_combine_residual_kernel<__nv_bfloat16, 8>, grid, block, 0, st, a)
+                   : launch_dependent(moe_combine_residual_kernel<__nv_bfloat16, 1>, grid, block, 0, st, a));
 }
 
 static int pick_split(int ctas, int steps, int sm_count) {

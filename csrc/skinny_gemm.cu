@@ -10,6 +10,7 @@
 #include <stdint.h>
 
 #include "common.cuh"
+#include "gates.cuh"
 
 namespace tyr {
 
@@ -25,11 +26,14 @@ struct SkinnyArgs {
   long long ldx, ldw, ldy;
   int M, N, K;
   long long hx, hw, hy;        // per-head form: elements from head to head
-  int act;                     // 6: xIELU with factors act_a, act_b, as in csrc/gemm_tcgen05.cu; 0: none
+  int act;                     // 6: xIELU with factors act_a, act_b, 9: tanh-GELU times aux, as in csrc/gemm_tcgen05.cu; 0: none
   float act_a, act_b;
+  const __nv_bfloat16* aux;    // [M, N], row stride ldaux
+  long long ldaux;
 };
 
-__device__ __forceinline__ float sk_act(float z, const SkinnyArgs& a) {
+__device__ __forceinline__ float sk_act(float z, const SkinnyArgs& a, int tok, int row) {
+  if (a.act == 9) return gelu_tanh(z) * __bfloat162float(a.aux[tok * a.ldaux + row]);
   return a.act == 6 ? fmaf(0.5f, z, z > 0.f ? a.act_a * z * z : a.act_b * (__expf(z) - 1.f - z)) : z;
 }
 
@@ -135,7 +139,7 @@ __global__ void __launch_bounds__(kSkWarps * 32) skinny_gemm_kernel(SkinnyArgs a
         a.y[tok * a.ldy + row] = __float2bfloat16(s / (1.f + __expf(-s)) * u);
       } else if (gridDim.y == 1) {
         if (a.bias) s += __bfloat162float(a.bias[row]);
-        a.y[tok * a.ldy + row] = __float2bfloat16(sk_act(s, a));
+        a.y[tok * a.ldy + row] = __float2bfloat16(sk_act(s, a, tok, row));
       } else {
         atomicAdd(a.ws + static_cast<long long>(tok) * a.N + row, s);
       }
@@ -211,7 +215,7 @@ __global__ void __launch_bounds__(256) skinny_finish_kernel(SkinnyArgs a) {
     float s = a.ws[i];
     a.ws[i] = 0.f;
     if (a.bias) s += __bfloat162float(a.bias[row]);
-    a.y[tok * a.ldy + row] = __float2bfloat16(sk_act(s, a));
+    a.y[tok * a.ldy + row] = __float2bfloat16(sk_act(s, a, tok, row));
   }
 }
 
@@ -260,14 +264,14 @@ extern "C" TYR_EXPORT int tyr_skinny_gemm_splits(int N, int K) {
 }
 
 static int skinny_launch(const void* x, const void* w, const void* bias, void* y, void* ws, long long ldx, long long ldw, long long ldy, int M,
-                         int N, int K, int act, float act_a, float act_b, void* stream) {
+                         int N, int K, int act, float act_a, float act_b, void* stream, const void* aux = nullptr, long long ldaux = 0) {
   using namespace tyr;
-  if (act != 0 && act != 6) return -4;
+  if ((act != 0 && act != 6 && act != 9) || (act == 9) != (aux != nullptr)) return -4;
   if (M < 1 || M > 32 || N < 1 || K < 32 || (K & 31)) return -1;
   if ((ldx | ldw) & 7) return -2;                                    // 16-byte loads
   if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) return -3;
   SkinnyArgs a{(const __nv_bfloat16*)x, (const __nv_bfloat16*)w, nullptr, (const __nv_bfloat16*)bias, (__nv_bfloat16*)y, (float*)ws, ldx, ldw, ldy, M, N, K,
-               0, 0, 0, act, act_a, act_b};
+               0, 0, 0, act, act_a, act_b, (const __nv_bfloat16*)aux, ldaux};
   const int splits = ws != nullptr ? tyr_skinny_gemm_splits(N, K) : 1;
   const dim3 grid((N + 15) / 16, splits);
   skinny_prefer_l1();
@@ -291,6 +295,12 @@ extern "C" TYR_EXPORT int tyr_skinny_gemm_bf16(const void* x, const void* w, con
 extern "C" TYR_EXPORT int tyr_skinny_gemm_act_bf16(const void* x, const void* w, const void* bias, void* y, void* ws, long long ldx, long long ldw,
                                                    long long ldy, int M, int N, int K, int act, float act_a, float act_b, void* stream) {
   return skinny_launch(x, w, bias, y, ws, ldx, ldw, ldy, M, N, K, act, act_a, act_b, stream);
+}
+
+// y[M, N] = gelu(x W^T) * aux (tanh form); aux [M, N] with row stride ldaux.
+extern "C" TYR_EXPORT int tyr_skinny_gelu_mul_bf16(const void* x, const void* w, const void* aux, void* y, void* ws, long long ldx, long long ldw,
+                                                   long long ldaux, long long ldy, int M, int N, int K, void* stream) {
+  return skinny_launch(x, w, nullptr, y, ws, ldx, ldw, ldy, M, N, K, 9, 0.f, 0.f, stream, aux, ldaux);
 }
 
 // A product of its own for each head: y[m, h, :N] = x[m, h, :K] @ W[h]^T for `heads` heads, rows (ldx, ldy) and heads (hx, hw, hy) apart

@@ -36,7 +36,8 @@ NVCC_FLAGS = [
 ]
 # Units whose results are carried through thousands of steps or stand for the fp32 mode: correctly rounded division, square root
 # and library exponentials.  Every other unit is compiled with fast math.
-PRECISE_UNITS = ("delta_general", "attention_general", "joint_attention", "latent", "lightning", "mix_conv", "selective_scan")
+PRECISE_UNITS = ("delta_general", "attention_general", "depth_average", "gates", "joint_attention", "latent", "lightning", "mix_conv", "rotary_store",
+                 "selective_scan")
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-pthread"]
 
 

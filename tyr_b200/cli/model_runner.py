@@ -3,7 +3,7 @@ executables: Qwen3, Qwen2.5-Omni thinker, Qwen3.5 / 3.6, Gemma 4, Zatorax, Kinet
 
     python -m tyr_b200.cli.model_runner --family gemma4 --source google/gemma-4-e2b --prompt "Hi" --max-new-tokens 64 --stream
     python -m tyr_b200.cli.model_runner --family qwen3 --source Qwen/Qwen3-4B --prompt-file prompts.txt --batch-size 4
-    python -m tyr_b200.cli.model_runner --source <zatorax, kinetar or nizedra dir> --prompt "5 17 3" --max-new-tokens 16        # family from config.json
+    python -m tyr_b200.cli.model_runner --source <zatorax, kinetar, nizedra or vonulix dir> --prompt "5 17 3" --max-new-tokens 16        # family from config.json
     python -m tyr_b200.cli.model_runner --family whisper --source openai/whisper-small --audio speech.wav
 
 Common flags: ``--family`` (default ``auto``: by config.json, ``models/registry.py``), ``--source`` (directory or hub repo id), ``--prompt`` / ``--prompt-file``, ``--batch-size``, ``--max-new-tokens``,
@@ -23,7 +23,7 @@ from ..models import registry
 from ..models.generation import SamplingStrategy
 from ..tokenizer import hf as tok_hf
 
-TEXT_FAMILIES = ("qwen3", "qwen25omni", "qwen35", "gemma4", "zatorax", "kinetar", "nizedra")
+TEXT_FAMILIES = ("qwen3", "qwen25omni", "qwen35", "gemma4", "zatorax", "kinetar", "nizedra", "vonulix")
 SPEECH_FAMILIES = ("whisper", "qwen3asr")
 
 

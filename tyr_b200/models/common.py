@@ -104,6 +104,17 @@ def norm_w(x, w, eps, one_plus_w: bool = False, residual=None, return_residual: 
     return rms_norm_weighted(x, w, eps, one_plus_w=one_plus_w, residual=residual, return_residual=return_residual)
 
 
+def config_fields(design: str, j: dict, what: str, required: Sequence[str], optional: Sequence[str] = ()) -> dict:
+    """The entries of a config object that are not null; names what is missing and what is unknown."""
+    j = {k: v for k, v in j.items() if v is not None}
+    missing = [k for k in required if k not in j]
+    unknown = [k for k in j if k not in required and k not in optional]
+    if missing or unknown:
+        raise ValueError(f"Invalid {design} config: {what} " + "; ".join(
+            [f"lacks {', '.join(missing)}"] * bool(missing) + [f"has unknown {', '.join(unknown)}"] * bool(unknown)))
+    return j
+
+
 # ---- rotary ---------------------------------------------------------------------------------------
 def plain_inv_freq(half: int, base: float) -> List[float]:
     dim = 2.0 * half
@@ -159,25 +170,40 @@ def head_norm(x: torch.Tensor, w: torch.Tensor, eps: float, one_plus_w: bool = F
 @dataclass
 class KVCache:
     """K/V stores ``[B, Hkv, cap, D]``.  ``ring`` stores keep the last ``cap`` positions at slot
-    ``position % cap``; RoPE is already applied so slot order is irrelevant to a single query."""
+    ``position % cap``; RoPE is already applied so slot order is irrelevant to a single query.  With ``keep`` the first ``keep``
+    positions stay in the first slots for good, and the ring is made of the slots after them."""
     k: torch.Tensor
     v: torch.Tensor
     ring: bool = False
     length: int = 0           # absolute positions written so far
+    keep: int = 0
 
     @staticmethod
     def allocate(batch: int, kv_heads: int, cap: int, head_dim: int, device, dtype, ring: bool = False, v_dim: Optional[int] = None,
-                 shared: bool = False) -> "KVCache":
-        """``shared``: the values are the keys, and one store serves both."""
+                 shared: bool = False, keep: int = 0) -> "KVCache":
+        """``shared``: the values are the keys, and one store serves both.  ``cap`` counts the ``keep`` slots of a ring store too."""
         if cap <= 0:
             raise ValueError("cache capacity must be positive")
+        if keep < 0 or (ring and keep >= cap):
+            raise ValueError("a ring store needs slots beyond the kept ones")
         zeros = lambda d: torch.zeros((batch, kv_heads, cap, d), device=device, dtype=dtype)
         k = zeros(head_dim)
-        return KVCache(k, k if shared else zeros(head_dim if v_dim is None else v_dim), ring)
+        return KVCache(k, k if shared else zeros(head_dim if v_dim is None else v_dim), ring, keep=keep)
 
     @property
     def cap(self) -> int:
         return self.k.shape[2]
+
+    def slots(self, positions: torch.Tensor) -> torch.Tensor:
+        """Where these positions lie."""
+        if not self.ring:
+            return positions
+        return torch.where(positions < self.keep, positions, self.keep + (positions - self.keep) % (self.cap - self.keep))
+
+    def held(self, first: int, last: int) -> torch.Tensor:
+        """The positions of first .. last that are still there once ``last`` is written."""
+        p = torch.arange(first, last + 1)
+        return p[(p < self.keep) | (p > last - (self.cap - self.keep))] if self.ring else p
 
     def write(self, k_new: torch.Tensor, v_new: torch.Tensor) -> None:
         """Append ``[B, Hkv, S, D]`` at absolute position ``self.length``."""
@@ -187,6 +213,10 @@ class KVCache:
                 raise ValueError(f"KV cache overflow: {pos}+{S} > {cap}")
             self.k[:, :, pos:pos + S].copy_(k_new)
             self.v[:, :, pos:pos + S].copy_(v_new)
+        elif self.keep:
+            at = self.held(pos, pos + S - 1)
+            self.k[:, :, self.slots(at)] = k_new[:, :, at - pos]
+            self.v[:, :, self.slots(at)] = v_new[:, :, at - pos]
         else:
             keep = min(S, cap)
             src0 = S - keep
@@ -204,7 +234,7 @@ class KVCache:
         return self.k[:, :, :n], self.v[:, :, :n]
 
     def clone(self) -> "KVCache":
-        return KVCache(self.k.clone(), self.v.clone(), self.ring, self.length)
+        return KVCache(self.k.clone(), self.v.clone(), self.ring, self.length, self.keep)
 
     def retain(self, rows: torch.Tensor) -> None:
         """Keep only these rows of the batch, in this order; the others' memory is given back."""

@@ -35,6 +35,9 @@ class Family:
 
 
 FAMILIES: List[Family] = [
+    Family("vonulix", ("vonulix",), "vonulix", "CacheSession",
+           ("attention_fwd", "attention_general", "decode_attention", "decode_gemm", "depth_average", "embed", "gates", "gemm_tcgen05", "moe_nvfp4", "moe_stream",
+            "norm", "rotary_store", "skinny_gemm"), ragged=True),
     Family("nizedra", ("nizedra",), "nizedra", "CacheSession",
            ("attention_fwd", "attention_general", "decode_gemm", "delta_general", "gemm_tcgen05", "joint_attention", "joint_tcgen05", "latent", "lightning", "mix_conv",
             "norm", "skinny_gemm"), ragged=True),

@@ -52,19 +52,25 @@ def position_turns(width: int, base: float = 10000.0, device="cpu") -> torch.Ten
     return (base ** (-2.0 * i / width) / (2.0 * math.pi)).to(device)
 
 
-def embed_positions(ids: torch.Tensor, table: torch.Tensor, turns: torch.Tensor, scale: float, pos: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """fp32 [B, S, D]: ``table[ids] * scale`` plus the sinusoidal vector of each position (channel 2i the sine, 2i + 1 the cosine).
+def embed_positions(ids: torch.Tensor, table: torch.Tensor, turns: Optional[torch.Tensor], scale: float, pos: Optional[torch.Tensor] = None,
+                    out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """fp32 [B, S, D]: ``table[ids] * scale`` plus the sinusoidal vector of each position (channel 2i the sine, 2i + 1 the cosine; nothing
+    without ``turns``), into ``out`` when given.
     ``pos``: int32 [B] positions of single tokens (S == 1); without it positions count from 0 in every row."""
     B, S = ids.shape
     V, D = table.shape
     if not ids.is_cuda:
+        x = torch.nn.functional.embedding(ids, table).float() * scale
+        if turns is None:
+            return x if out is None else out.copy_(x)
         p = (torch.arange(S)[None] if pos is None else pos[:, None]).double()
         angle = 2.0 * math.pi * torch.frac(p[..., None] * turns)
         vec = torch.stack([torch.sin(angle), torch.cos(angle)], -1).flatten(-2)[..., :D].float()
-        return torch.nn.functional.embedding(ids, table).float() * scale + vec
-    assert ids.dtype == torch.int64 and table.is_contiguous() and turns.dtype == torch.float64 and turns.numel() == (D + 1) // 2
+        return x + vec if out is None else out.copy_(x + vec)
+    assert ids.dtype == torch.int64 and table.is_contiguous() and (turns is None or (turns.dtype == torch.float64 and turns.numel() == (D + 1) // 2))
     assert pos is None or (S == 1 and pos.dtype == torch.int32 and pos.numel() == B)
-    x = torch.empty((B, S, D), dtype=torch.float32, device=ids.device)
+    x = torch.empty((B, S, D), dtype=torch.float32, device=ids.device) if out is None else out
+    assert x.dtype == torch.float32 and x.shape == (B, S, D) and x.is_contiguous()
     kind = {torch.bfloat16: 0, torch.float32: 1}[table.dtype]
     check(lib().tyr_embed_positions(ptr(ids.contiguous()), ptr(table), ptr(turns), ptr(pos), ptr(x), B, S, D, V, scale, kind, ptr(err_word(ids.device)),
                                     cur_stream(ids.device)), "embed_positions")

@@ -39,6 +39,10 @@ def _sigs(lib_):
     if fn is not None:
         fn.argtypes = [P, P, P, P, P, P, I, I, I, I, I, I, ctypes.POINTER(L), I, F, F, P, P]
         fn.restype = ctypes.c_int
+    fn = getattr(lib_, "tyr_flash_fwd_kept", None)
+    if fn is not None:
+        fn.argtypes = [P, P, P, P, P, P, I, P, I, I, I, I, I, I, ctypes.POINTER(L), I, I, F, F, P, P]
+        fn.restype = ctypes.c_int
     fn = getattr(lib_, "tyr_flash_bwd_workspace_bytes", None)
     if fn is not None:
         fn.argtypes = [I, I, I]
@@ -198,3 +202,20 @@ def flash_fwd_sink(q, k, v, *, scale: float, sink=None, gate=None, out_scale: fl
     check(lib().tyr_flash_fwd_sink(ptr(q), ptr(k), ptr(v), ptr(out), ptr(sink), ptr(gate), B, Hq, Hkv, T, dk, dv, strides, int(window or 0), scale, out_scale,
                                    ptr(err_word(q.device)), cur_stream(q.device)), "flash_fwd_sink")
     return out
+
+
+def flash_fwd_kept(q, k, v, *, scale: float, window: Optional[int], keep: int, head_gate: Optional[torch.Tensor] = None,
+                   back: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Causal attention of whole prompts in which the first ``keep`` keys stay visible beyond ``window`` keys (None: no window); every head's
+    output times the sigmoid of its number in ``head_gate`` [B, T, Hq]; ``back`` [>= T, dv / 2, 2] (cos, sin): the output's channel
+    pairs (m, m + dv / 2) turned back (dv a multiple of 16).  q: [B, T, Hq, dk], k: [B, T, Hkv, dk], v: [B, T, Hkv, dv] -> [B, T, Hq * dv]."""
+    import ctypes
+    B, T, Hq, dk = q.shape
+    Hkv, dv = k.shape[2], v.shape[3]
+    out = torch.empty((B, T, Hq, dv), dtype=q.dtype, device=q.device)
+    assert back is None or (back.dtype == torch.float32 and back.is_contiguous() and back.shape[0] >= T and back.shape[1:] == (dv // 2, 2))
+    assert head_gate is None or (head_gate.dtype == torch.bfloat16 and head_gate.shape == (B, T, Hq))
+    strides = (ctypes.c_longlong * 15)(*[x for t in (q, k, v, out) for x in _bthd_strides(t)], *((0, 0, 0) if head_gate is None else head_gate.stride()))
+    check(lib().tyr_flash_fwd_kept(ptr(q), ptr(k), ptr(v), ptr(out), None, ptr(head_gate), 1, ptr(back), B, Hq, Hkv, T, dk, dv, strides, int(window or 0),
+                                   keep, scale, 1.0, ptr(err_word(q.device)), cur_stream(q.device)), "flash_fwd_kept")
+    return out.flatten(2)

@@ -9,7 +9,8 @@ Operand layouts (no transposes are ever materialised):
 * ``b_layout='MN'`` : ``b`` has shape ``[..., K, N]``
 
 ``out = alpha * act(A @ B) + beta * aux`` (``act='relu2_grad'``: ``alpha * (A @ B) * 2*sqrt(aux)``; ``act='xielu'``: xIELU of A @ B with
-factors ``alpha`` above zero and ``beta`` below, no ``aux``); ``out_dtype`` bf16 or fp32; ``accumulate=True`` adds
+factors ``alpha`` above zero and ``beta`` below, no ``aux``; ``act='gelu_mul'``: tanh-GELU of A @ B times ``aux``; the gated
+``act='clamped_swiglu'`` has limit ``alpha`` and slope ``beta``); ``out_dtype`` bf16 or fp32; ``accumulate=True`` adds
 into an existing fp32 ``out`` with an even stream-K split (used for weight gradients).
 
 The reference reaches cuBLAS for these products (cc/src/tyr.cpp:1003-1036, 1267-1300) and runs
@@ -25,7 +26,8 @@ import torch
 from .._native import GemmArgs
 from ._common import check, cur_stream, err_word, lib
 
-_ACT = {None: 0, "none": 0, "relu2": 1, "relu": 2, "relu2_grad": 3, "swiglu": 4, "geglu": 5, "xielu": 6, "silu": 7}
+_ACT = {None: 0, "none": 0, "relu2": 1, "relu": 2, "relu2_grad": 3, "swiglu": 4, "geglu": 5, "xielu": 6, "silu": 7, "clamped_swiglu": 8, "gelu_mul": 9}
+_GATED = ("swiglu", "geglu", "clamped_swiglu")
 
 
 def _dims(t, layout, is_a):
@@ -47,14 +49,21 @@ def _dims(t, layout, is_a):
     return r1, r0, ld, batch, bs
 
 
+def clamped_swiglu(gate: torch.Tensor, up: torch.Tensor, limit: float, slope: float) -> torch.Tensor:
+    g, u = gate.float().clamp(max=limit), up.float().clamp(-limit, limit)
+    return g * torch.sigmoid(slope * g) * (u + 1.0)
+
+
 def _reference(a, b, a_layout, b_layout, aux, alpha, beta, act, out_dtype):
     A = a.float() if a_layout == "K" else a.float().transpose(-1, -2)
     B = b.float().transpose(-1, -2) if b_layout == "K" else b.float()
     acc = A @ B
-    if act in ("swiglu", "geglu"):
+    if act in _GATED:
         # column blocks of 256: 128 gate columns followed by the matching 128 up columns
         N = acc.shape[-1]
         blk = acc.reshape(*acc.shape[:-1], N // 256, 2, 128)
+        if act == "clamped_swiglu":
+            return clamped_swiglu(blk[..., 0, :], blk[..., 1, :], alpha, beta).reshape(*acc.shape[:-1], N // 2).to(out_dtype)
         gate, up = alpha * blk[..., 0, :], beta * blk[..., 1, :]
         fn = torch.nn.functional.silu if act == "swiglu" else (lambda t: torch.nn.functional.gelu(t, approximate="tanh"))
         return (fn(gate) * up).reshape(*acc.shape[:-1], N // 2).to(out_dtype)
@@ -67,6 +76,8 @@ def _reference(a, b, a_layout, b_layout, aux, alpha, beta, act, out_dtype):
         return (alpha * acc * 2.0 * torch.sqrt(aux.float().clamp_min(0))).to(out_dtype)
     elif act == "silu":
         acc = torch.nn.functional.silu(acc)
+    elif act == "gelu_mul":
+        return (torch.nn.functional.gelu(acc, approximate="tanh") * aux.float()).to(out_dtype)
     elif act == "xielu":
         low = acc.clamp_max(0.0)
         return (torch.where(acc > 0, alpha * acc * acc, beta * (torch.expm1(low) - low)) + 0.5 * acc).to(out_dtype)
@@ -88,7 +99,9 @@ def gemm(a: torch.Tensor, b: torch.Tensor, *, a_layout: str = "K", b_layout: str
     batch = max(batch_a, batch_b)
     if batch_a not in (1, batch) or batch_b not in (1, batch):
         raise ValueError("gemm batch mismatch")
-    gated = act in ("swiglu", "geglu")
+    gated = act in _GATED
+    if act == "gelu_mul" and aux is None:
+        raise ValueError("gelu_mul takes its factor as aux")
     if gated:
         # b holds, per block of 256 rows, 128 gate rows then the matching 128 up rows (`interleave_gate_up`); the result
         # is silu(alpha * gate) * (beta * up) (tanh-GELU for "geglu"), N / 2 columns wide
@@ -226,7 +239,7 @@ def grouped_gemm(a: torch.Tensor, b: torch.Tensor, group_offsets: torch.Tensor,
     total, K = a.shape
     G, N, K2 = b.shape
     assert K == K2 and group_offsets.numel() == G + 1
-    swiglu = act in ("swiglu", "geglu")          # gated pairs: SiLU or tanh-GELU on the gate half
+    swiglu = act in _GATED                       # gated pairs: SiLU, tanh-GELU or the clamped form (limit alpha, slope beta) on the gate half
     n_out = N // 2 if swiglu else N
     if not a.is_cuda:
         offs = group_offsets.tolist()
@@ -238,6 +251,9 @@ def grouped_gemm(a: torch.Tensor, b: torch.Tensor, group_offsets: torch.Tensor,
             acc = a[lo:hi].float() @ b[g].float().T
             if swiglu:
                 blk = acc.reshape(hi - lo, N // 256, 2, 128)
+                if act == "clamped_swiglu":
+                    res[lo:hi] = clamped_swiglu(blk[:, :, 0], blk[:, :, 1], alpha, beta).reshape(hi - lo, n_out).to(a.dtype)
+                    continue
                 gate, up = alpha * blk[:, :, 0], beta * blk[:, :, 1]
                 fn = torch.nn.functional.silu if act == "swiglu" else (lambda t: torch.nn.functional.gelu(t, approximate="tanh"))
                 acc = (fn(gate) * up).reshape(hi - lo, n_out)
@@ -259,7 +275,7 @@ def grouped_gemm(a: torch.Tensor, b: torch.Tensor, group_offsets: torch.Tensor,
     args.lda, args.ldb, args.ldc = a.stride(0), b.stride(1), out.stride(0)
     args.sA, args.sB = total, b.stride(0)
     args.out_mode = 0
-    args.act = (4 if act == "swiglu" else 5) if swiglu else _ACT[act]
+    args.act = _ACT[act]
     args.alpha = alpha
     args.beta = beta if swiglu else 0.0
     args.bn = 256

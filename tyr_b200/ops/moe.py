@@ -31,10 +31,12 @@ def _sigs(lib_):
     P, I, L, F = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong, ctypes.c_float
     table = {
         "tyr_nvfp4_quantize": [P, P, P, P, L, L, P], "tyr_nvfp4_dequant": [P, P, P, P, L, L, P],
-        "tyr_moe_route": [P, P, P, P, P, I, I, I, I, I, F, F, I, I, P],
-        "tyr_moe_route_fused": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, F, I, I, P],
+        "tyr_moe_route": [P, P, P, P, P, I, I, I, I, I, F, F, I, I, I, P],
+        "tyr_moe_route_fused": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, F, I, I, I, P],
         "tyr_moe_layout": [P, P, P, P, P, P, P, P, I, I, P], "tyr_moe_count": [P, P, I, I, P],
         "tyr_moe_gather_rows": [P, P, P, I, I, I, P], "tyr_moe_combine": [P, P, P, P, P, I, I, I, P],
+        "tyr_moe_gather_scaled": [P, P, P, P, I, I, I, P], "tyr_moe_combine_residual": [P, P, P, P, L, P, P, I, I, I, I, P],
+        "tyr_moe_stream_up": [P] * 6 + [L, L, L] + [I] * 6 + [F, F, F, P], "tyr_moe_stream_down": [P] * 5 + [L, L, L, L] + [I] * 6 + [P],
         "tyr_moe_fp4_gemv": [P] * 17 + [I, I, I, I, I, P], "tyr_moe_finalize": [P, P, P, L, P],
     }
     for name, args in table.items():
@@ -112,13 +114,14 @@ def nvfp4_dequant(packed: torch.Tensor, scales: torch.Tensor, global_scale: torc
 
 # ---- routing -------------------------------------------------------------------------------------------
 def route(logits: torch.Tensor, k: int, *, softmax: bool = False, bias: Optional[torch.Tensor] = None,
-          renorm: bool = True, softcap: float = 0.0, scale: float = 1.0, want_counts: bool = True, groups: int = 1, keep: int = 1):
-    """logits fp32 [T, E] -> (ids int32 [T, k], weights fp32 [T, k], counts int32 [E]).
+          renorm: bool = True, softcap: float = 0.0, scale: float = 1.0, want_counts: bool = True, groups: int = 1, keep: int = 1,
+          experts: Optional[int] = None):
+    """logits fp32 [T, E] (or more columns, of which the first ``experts`` count) -> (ids int32 [T, k], weights fp32 [T, k], counts int32 [E]).
     Sigmoid (Laguna, Tyr/Model/Laguna/MoE.lean:71-90) or softmax (Qwen3.5) scores; the selection
     bias only influences WHICH experts are picked; ties go to the lower expert index.  With ``groups`` > 1 the experts form
     that many equal groups of neighbours, a group counts by its best selection score (bias included), and only experts of the
     ``keep`` best groups compete."""
-    T, E = logits.shape
+    T, E = logits.shape[0], experts or logits.shape[1]
     if logits.is_cuda:
         lg = logits.float().contiguous()
         ids = torch.empty((T, k), dtype=torch.int32, device=logits.device)
@@ -126,9 +129,9 @@ def route(logits: torch.Tensor, k: int, *, softmax: bool = False, bias: Optional
         counts = torch.zeros(E, dtype=torch.int32, device=logits.device)
         b = bias.float().contiguous() if bias is not None else None
         check(lib().tyr_moe_route(ptr(lg), ptr(b), ptr(ids), ptr(w), ptr(counts), T, E, k, 1 if softmax else 0,
-                                  1 if renorm else 0, softcap, scale, groups, keep, cur_stream(logits.device)), "moe_route")
+                                  1 if renorm else 0, softcap, scale, groups, keep, lg.shape[1], cur_stream(logits.device)), "moe_route")
         return ids, w, counts
-    l = logits.float()
+    l = logits[:, :E].float()
     if softcap > 0:
         l = softcap * torch.tanh(l / softcap)
     scores = torch.softmax(l, -1) if softmax else torch.sigmoid(l)
@@ -170,19 +173,22 @@ def route_fused_supported(x: torch.Tensor, router_w: torch.Tensor) -> bool:
 
 
 def route_fused(x: torch.Tensor, router_w: torch.Tensor, k: int, *, softmax: bool = False, bias: Optional[torch.Tensor] = None,
-                renorm: bool = True, softcap: float = 0.0, scale: float = 1.0, groups: int = 1, keep: int = 1):
+                renorm: bool = True, softcap: float = 0.0, scale: float = 1.0, groups: int = 1, keep: int = 1, experts: Optional[int] = None,
+                want_logits: bool = False):
     """x bf16 [T, h], router_w fp32 [E, h] -> (ids, weights, counts) as :func:`route` of ``x.float() @ router_w.T`` (fp32
-    accumulation inside the kernel; the logits are never written out)."""
-    T, E = x.shape[0], router_w.shape[0]
+    accumulation inside the kernel).  ``router_w`` may have more rows than the ``experts`` that are chosen from; ``want_logits``: all
+    rows' logits [T, rows] are a fourth result."""
+    T, rows = x.shape[0], router_w.shape[0]
+    E = experts or rows
     ids = torch.empty((T, k), dtype=torch.int32, device=x.device)
     w = torch.empty((T, k), dtype=torch.float32, device=x.device)
     zeros = torch.zeros(E + (T + 3) // 4, dtype=torch.int32, device=x.device)       # expert counts, then one ticket per group of 4 tokens
     counts, tickets = zeros[:E], zeros[E:]
-    logits = torch.empty((T, E), dtype=torch.float32, device=x.device)
+    logits = torch.empty((T, rows), dtype=torch.float32, device=x.device)
     b = bias.float().contiguous() if bias is not None else None
     check(lib().tyr_moe_route_fused(ptr(x), ptr(router_w), ptr(b), ptr(logits), ptr(tickets), ptr(ids), ptr(w), ptr(counts), T, E, k, x.shape[1], 1 if softmax else 0,
-                                    1 if renorm else 0, softcap, scale, groups, keep, cur_stream(x.device)), "moe_route_fused")
-    return ids, w, counts
+                                    1 if renorm else 0, softcap, scale, groups, keep, rows, cur_stream(x.device)), "moe_route_fused")
+    return (ids, w, counts, logits) if want_logits else (ids, w, counts)
 
 
 def layout(ids: torch.Tensor, counts: torch.Tensor, want_tiles: bool = False, want_active: bool = False):
@@ -409,6 +415,11 @@ class ExpertBank:
         self._tiled: Optional[Tuple[torch.Tensor, torch.Tensor]] = None
 
     @property
+    def padded(self) -> int:
+        """Hidden channels of an expert in the grouped GEMM's layout."""
+        return -(-self.moe_int // 128) * 128
+
+    @property
     def gate_up(self) -> torch.Tensor:
         return self._plain[0] if self._plain is not None else _deinterleave(self._tiled[0], self.moe_int)
 
@@ -466,4 +477,90 @@ def _moe_grouped(x, ids, weights, gu, dn, counts, add, act):
     out = torch.empty_like(x)
     check(lib().tyr_moe_combine(ptr(y), ptr(pos), ptr(weights.float().contiguous()), ptr(add.contiguous() if add is not None else None),
                                 ptr(out), T, k, h, st), "moe_combine")
+    return out
+
+
+# ---- experts of the weighted input ---------------------------------------------------------------------------------------
+@dataclass(frozen=True)
+class ClampedExpert:
+    """Form of an expert: g = min(gate x, limit), u = clamp(up x, +-limit); down (g sigmoid(slope g) (u + 1))."""
+    limit: float
+    slope: float
+
+
+STREAM_MAX_TOKENS, STREAM_MAX_PAIRS = 64, 2048
+
+
+def _stream_rows(bank: ExpertBank) -> int:
+    """Hidden channels the weight-streaming kernel works on: the bank's, up to a multiple of 32 (its padding is zero)."""
+    return -(-bank.moe_int // 32) * 32
+
+
+def stream_supported(x: torch.Tensor, pairs: int) -> bool:
+    """A few tokens: the weight-streaming products of csrc/moe_stream.cu."""
+    return (x.is_cuda and x.dtype == torch.bfloat16 and x.shape[0] <= STREAM_MAX_TOKENS and pairs <= STREAM_MAX_PAIRS and x.shape[1] % 32 == 0
+            and x.stride(1) == 1 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 and hasattr(lib(), "tyr_moe_stream_up"))
+
+
+def _clamped_mlp(x: torch.Tensor, bank: ExpertBank, form: ClampedExpert, scale: Optional[torch.Tensor] = None, e: int = 0) -> torch.Tensor:
+    """One expert on rows [T, h] with the library's products (``scale``: a factor per row on the input)."""
+    from .gates import clamped_swiglu
+    if scale is not None:
+        x = (x.float() * scale[:, None]).to(x.dtype)
+    lin, tiled = torch.nn.functional.linear, bank._plain is None
+    gu, dn = bank._tiled if tiled else bank._plain
+    return lin(clamped_swiglu(lin(x, gu[e]), dn.shape[2], form.limit, form.slope, block=128 if tiled else 0), dn[e])
+
+
+def weighted_input_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, bank: ExpertBank, form: ClampedExpert, resid: torch.Tensor, *,
+                           shared: Optional[ExpertBank] = None, shared_form: Optional[ClampedExpert] = None, shared_gate: Optional[torch.Tensor] = None,
+                           counts: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``resid += sum_s expert_{ids[t, s]}(weights[t, s] x[t]) + sigmoid(shared_gate[t]) shared(x[t])`` IN PLACE on an fp32 stream [T, h], and
+    the sum in x's dtype.  x: [T, h]; ``shared``: a bank of one expert; ``shared_gate``: fp32 [T] (a column of a wider matrix)."""
+    T, h = x.shape
+    k, E = ids.shape[1], bank.num_experts
+    st = cur_stream(x.device) if x.is_cuda else None
+    y, pos, extra = None, None, None
+    if stream_supported(x, T * k) and (shared is None or shared_form.slope == form.slope):
+        gu, dn = bank.tiled()
+        sgu, sdn = shared.tiled() if shared is not None else (None, None)
+        n1, n1s = _stream_rows(bank), _stream_rows(shared) if shared is not None else 0
+        hid = torch.empty((T * k + T, max(n1, n1s)), dtype=x.dtype, device=x.device)
+        y = torch.empty((T * k + T, h), dtype=x.dtype, device=x.device)
+        check(lib().tyr_moe_stream_up(ptr(x), ptr(gu), ptr(sgu), ptr(ids), ptr(weights), ptr(hid), x.stride(0), gu.stride(0), hid.stride(0), T, k, E, n1, n1s,
+                                      h, form.limit, shared_form.limit if shared is not None else 0.0, form.slope, st), "moe_stream_up")
+        check(lib().tyr_moe_stream_down(ptr(hid), ptr(dn), ptr(sdn), ptr(ids), ptr(y), hid.stride(0), dn.stride(1), 0 if sdn is None else sdn.stride(1),
+                                        dn.stride(0), T, k, E, h, n1, n1s, st), "moe_stream_down")
+        extra = y[T * k:] if shared is not None else None
+    else:
+        if grouped_supported(x, bank.padded):
+            gu, dn = bank.tiled()
+            if counts is None:
+                counts = count_experts(ids, E)
+            offsets, order, pos, tiles = layout(ids, counts, want_tiles=True)
+            xs = torch.empty((T * k, h), dtype=x.dtype, device=x.device)
+            check(lib().tyr_moe_gather_scaled(ptr(x.contiguous()), ptr(order), ptr(weights), ptr(xs), T * k, k, h, st), "moe_gather_scaled")
+            y = grouped_gemm(grouped_gemm(xs, gu, offsets, tiles, act="clamped_swiglu", alpha=form.limit, beta=form.slope), dn, offsets, tiles)
+        else:
+            acc = torch.zeros((T, h), dtype=torch.float32, device=x.device)
+            for e in torch.unique(ids).tolist():
+                tok, slot = torch.nonzero(ids == e, as_tuple=True)
+                acc.index_add_(0, tok, _clamped_mlp(x[tok], bank, form, weights[tok, slot], e).float())
+            y, k = acc.to(x.dtype), 1
+        if shared is not None:
+            if T >= 128 and grouped_supported(x, shared.padded):
+                from .gemm import gemm
+                sgu, sdn = shared.tiled()
+                extra = gemm(gemm(x, sgu[0], act="clamped_swiglu", alpha=shared_form.limit, beta=shared_form.slope), sdn[0])
+            else:
+                extra = _clamped_mlp(x, shared, shared_form)
+    if not x.is_cuda:
+        resid += y
+        if extra is not None:
+            resid += extra if shared_gate is None else torch.sigmoid(shared_gate.float())[:, None] * extra
+        return resid.to(x.dtype)
+    out = torch.empty_like(x)
+    assert resid.dtype == torch.float32 and resid.is_contiguous() and (shared_gate is None or shared_gate.dtype == torch.float32)
+    check(lib().tyr_moe_combine_residual(ptr(y), ptr(pos), ptr(extra), ptr(shared_gate), 0 if shared_gate is None else shared_gate.stride(0), ptr(resid), ptr(out),
+                                         T, k, h, 0 if x.dtype == torch.bfloat16 else 1, st), "moe_combine_residual")
     return out

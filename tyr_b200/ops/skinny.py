@@ -34,7 +34,8 @@ def _sigs(lib_):
         lib_.tyr_skinny_gemm_splits.restype = I
     F = ctypes.c_float
     for name, args in (("tyr_skinny_gemm_act_bf16", [P, P, P, P, P, L, L, L, I, I, I, I, F, F, P]),
-                       ("tyr_skinny_heads_bf16", [P, P, P, L, L, L, L, L, L, I, I, I, I, P])):
+                       ("tyr_skinny_heads_bf16", [P, P, P, L, L, L, L, L, L, I, I, I, I, P]),
+                       ("tyr_skinny_gelu_mul_bf16", [P, P, P, P, P, L, L, L, L, I, I, I, P])):
         fn = getattr(lib_, name, None)
         if fn is not None:
             fn.argtypes, fn.restype = args, I
@@ -104,6 +105,18 @@ def skinny_xielu(x2: torch.Tensor, w: torch.Tensor, a: float, b: float) -> torch
     ws = _workspace(x2.device, M, N) if lib().tyr_skinny_gemm_splits(N, K) > 1 else None
     check(lib().tyr_skinny_gemm_act_bf16(ptr(x2), ptr(w), None, ptr(y), ptr(ws), x2.stride(0), w.stride(0), N, M, N, K, 6, a, b, cur_stream(x2.device)),
           "skinny_xielu")
+    return y
+
+
+def skinny_gelu_mul(x2: torch.Tensor, w: torch.Tensor, e: torch.Tensor) -> torch.Tensor:
+    """x2: [M <= 32, K] bf16 -> tanh-GELU of ``x2 w^T`` times ``e`` [M, N] (rows may be strided) as [M, N] bf16, in the product's epilogue."""
+    M, K = x2.shape
+    N = w.shape[0]
+    assert e.shape == (M, N) and e.dtype == torch.bfloat16 and e.stride(1) == 1
+    y = torch.empty((M, N), dtype=torch.bfloat16, device=x2.device)
+    ws = _workspace(x2.device, M, N) if lib().tyr_skinny_gemm_splits(N, K) > 1 else None
+    check(lib().tyr_skinny_gelu_mul_bf16(ptr(x2), ptr(w), ptr(e), ptr(y), ptr(ws), x2.stride(0), w.stride(0), e.stride(0), N, M, N, K, cur_stream(x2.device)),
+          "skinny_gelu_mul")
     return y
 
 
