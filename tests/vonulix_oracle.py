@@ -41,13 +41,13 @@ def visible(i, size: Optional[int], keep):
     return [j for j in range(i + 1) if size is None or i - j < size or j < keep]
 
 
-def attend(q, k, v, scale, size, keep):
-    """q: [T, H, d], k: [T, G, d], v: [T, G, dv] -> [T, H, dv]."""
-    T, H, _ = q.shape
+def attend(q, k, v, scale, size, keep, first=0):
+    """q: [n, H, d] at positions ``first`` .., k: [T, G, d], v: [T, G, dv] at 0 .. -> [n, H, dv]."""
+    n, H, _ = q.shape
     rep = H // k.shape[1]
-    out = torch.zeros(T, H, v.shape[2], dtype=v.dtype)
-    for i in range(T):
-        js = torch.tensor(visible(i, size, keep))
+    out = torch.zeros(n, H, v.shape[2], dtype=v.dtype)
+    for i in range(n):
+        js = torch.tensor(visible(first + i, size, keep))
         for h in range(H):
             s = (k[js, h // rep] @ q[i, h]) * scale
             e = torch.exp(s - s.max())
