@@ -46,9 +46,9 @@ def parse_args():
     ap.add_argument("--device-batch", type=int, default=32)
     ap.add_argument("--seq-len", type=int, default=2048)
     ap.add_argument("--vocab", type=int, default=65536)
-    ap.add_argument("--workload", default="nanochat", choices=["nanochat", "zatorax", "kinetar", "nizedra"],
-                    help="zatorax / kinetar / nizedra: prefill / decode throughput beside Qwen3.5 MoE / Qwen3.5 / Qwen3.5 at equal size on one GPU "
-                         "(benchmarks/{zatorax,kinetar,nizedra}_bench.py)")
+    ap.add_argument("--workload", default="nanochat", choices=["nanochat", "zatorax", "kinetar", "nizedra", "vonulix"],
+                    help="zatorax / kinetar / nizedra / vonulix: prefill / decode throughput beside Qwen3.5 MoE / Qwen3.5 / Qwen3.5 / Zatorax at equal size on one GPU "
+                         "(benchmarks/{zatorax,kinetar,nizedra,vonulix}_bench.py)")
     ap.add_argument("--no-e2e", action="store_true")
     ap.add_argument("--no-laguna", action="store_true", help="skip the Laguna MoE decode half of the metric")
     ap.add_argument("--laguna-steps", type=int, default=48)

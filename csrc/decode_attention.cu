@@ -546,7 +546,7 @@ static int decode_attention_launch(const void* q, const void* k_new, const void*
   a.dv = dv_out > 0 ? dv_out : DV;
   a.out_bs = out_bs > 0 ? out_bs : static_cast<long long>(Hq) * DV;
   a.out_scale = out_scale;
-  if (keep < 0 || keep >= cap || (keep > 0 && r1 != nullptr) || (append && k_new == nullptr) || (k_new == nullptr) != (v_new == nullptr)) return -7;
+  if (keep < 0 || (ring && keep >= cap) || (keep > 0 && r1 != nullptr) || (append && k_new == nullptr) || (k_new == nullptr) != (v_new == nullptr)) return -7;
   a.keep = keep;
   a.back = (const float2*)back;
   a.back_half = a.dv / 2;
