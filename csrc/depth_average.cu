@@ -51,9 +51,10 @@ __device__ __forceinline__ void dp_fma(float4& a, float w, const float4& v) {
 }
 __device__ __forceinline__ float dp_square(const float4& v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
 
-// NV vectors of four channels per thread, `blockDim.x` vectors apart.
-template <typename TY, typename TH, int NV>
-__global__ void __launch_bounds__(512) depth_average_kernel(DepthArgs a) {
+// NV vectors of four channels per thread, `blockDim.x` vectors apart.  FEW rows: no second CTA on an SM hides the loads, so more of them
+// are on their way at a time.
+template <typename TY, typename TH, int NV, bool FEW>
+__global__ void __launch_bounds__(512, FEW ? 1 : NV == 1 ? 3 : NV == 2 ? 2 : 1) depth_average_kernel(DepthArgs a) {
   __shared__ float part[2][32];
   const int vecs = a.D / 4;
   float4 post[NV], gain[NV];
@@ -83,7 +84,8 @@ __global__ void __launch_bounds__(512) depth_average_kernel(DepthArgs a) {
       }
       ss += dp_square(y[i]);
     }
-#pragma unroll 4
+    constexpr int kUnroll = FEW ? 8 : 4;
+#pragma unroll kUnroll
     for (int j = 0; j < a.n; ++j) {
       const float w = __ldg(a.weights + j);
       const float* src = a.history + j * a.between + base;
@@ -157,10 +159,14 @@ static int depth_launch(const DepthArgs& a, bool vec, cudaStream_t st) {
   if (!vec || vecs > 4096) return (int)launch_dependent(depth_average_any_kernel<TY, TH>, dim3(rows), dim3(256), 0, st, a);
   const int nv = vecs <= 512 ? 1 : (vecs <= 1024 ? 2 : (vecs <= 2048 ? 4 : 8));
   const dim3 block(static_cast<unsigned>(((vecs + nv - 1) / nv + 31) / 32 * 32));
-  return (int)(nv == 1 ? launch_dependent(depth_average_kernel<TY, TH, 1>, dim3(rows), block, 0, st, a)
-               : nv == 2 ? launch_dependent(depth_average_kernel<TY, TH, 2>, dim3(rows), block, 0, st, a)
-               : nv == 4 ? launch_dependent(depth_average_kernel<TY, TH, 4>, dim3(rows), block, 0, st, a)
-                         : launch_dependent(depth_average_kernel<TY, TH, 8>, dim3(rows), block, 0, st, a));
+  const dim3 grid(rows);
+  if (a.rows <= 148 && nv <= 2)
+    return (int)(nv == 1 ? launch_dependent(depth_average_kernel<TY, TH, 1, true>, grid, block, 0, st, a)
+                         : launch_dependent(depth_average_kernel<TY, TH, 2, true>, grid, block, 0, st, a));
+  return (int)(nv == 1 ? launch_dependent(depth_average_kernel<TY, TH, 1, false>, grid, block, 0, st, a)
+               : nv == 2 ? launch_dependent(depth_average_kernel<TY, TH, 2, false>, grid, block, 0, st, a)
+               : nv == 4 ? launch_dependent(depth_average_kernel<TY, TH, 4, false>, grid, block, 0, st, a)
+                         : launch_dependent(depth_average_kernel<TY, TH, 8, false>, grid, block, 0, st, a));
 }
 
 // dtypes: 0 = bf16, 1 = fp32 of y and of h.

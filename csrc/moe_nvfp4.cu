@@ -428,6 +428,7 @@ __global__ void __launch_bounds__(256) moe_combine_residual_kernel(CombineResidu
     cr_load<float, V>(a.resid + at, r);
 #pragma unroll
     for (int e = 0; e < V; ++e) acc[e] = 0.f;
+#pragma unroll 4
     for (int s = 0; s < a.k; ++s) {
       const int pair = tok * a.k + s, pp = a.pair_pos ? a.pair_pos[pair] : pair;
       cr_load<T, V>(static_cast<const T*>(a.y) + static_cast<long long>(pp) * a.h + c, f);

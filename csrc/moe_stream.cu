@@ -7,7 +7,8 @@
 // The products are bound by reading each active expert's weights once.  As in csrc/skinny_gemm.cu a CTA owns 16 weight rows, its 8 warps
 // split the contraction and stream 16 bytes per lane and row into mma.sync A fragments, with 8 pairs of one expert on the narrow side.
 // A CTA finds the pairs of its expert in the token-major list of ids itself: with fewer pairs than experts, CTA row p stands for the
-// expert of pair p and leaves when an earlier pair has the same one; otherwise CTA rows are experts.  The first CTA row is the shared expert.
+// expert of pair p and leaves when an earlier pair has the same one; otherwise CTA rows are experts, whose weights are on their way
+// into L2 before the kernel in front of this one has ended.  The first CTA row is the shared expert.
 //
 // Gate and up rows come in the grouped GEMM's layout: per 256 rows, 128 gate rows, then the matching 128 up rows.
 #include "common.cuh"
@@ -112,17 +113,19 @@ __global__ void __launch_bounds__(MS_WARPS * 32, UP ? 2 : 3) moe_stream_kernel(M
   auto part = reinterpret_cast<float(*)[MS_WARPS][4][16][9]>(ms_smem);
   int* list = reinterpret_cast<int*>(ms_smem + sizeof(float) * (UP ? 2 : 1) * MS_WARPS * 4 * 16 * 9);
   __shared__ int s_count;
-  const int tid = threadIdx.x, lane = tid & 31, row0 = blockIdx.x * 16, pairs = a.T * a.k;
+  const int tid = threadIdx.x, row0 = blockIdx.x * 16, pairs = a.T * a.k;
   const bool shared = a.ws != nullptr && blockIdx.y == 0;
   const int N = shared ? a.Ns : a.N, K = shared ? a.Ks : a.K;
   const long long ldw = shared ? a.ldws : a.ldw;
   pdl_trigger();
   if (row0 >= N) return;
   const int wrow = UP ? (row0 >> 7) * 256 + (row0 & 127) : row0;
+  auto prefetch = [&](const __nv_bfloat16* w) {    // constants: on their way into L2 while the kernel in front of this one runs
+    if (tid < (UP ? 32 : 16)) bulk_prefetch_l2(w + (tid < 16 ? tid : 112 + tid) * ldw, static_cast<uint32_t>(min(K, 4096)) * 2u);
+  };
   if (shared) {
     const __nv_bfloat16* w = a.ws + wrow * ldw;
-    if (tid < (UP ? 32 : 16))                      // constants: on their way into L2 while the kernel in front of this one runs
-      bulk_prefetch_l2(w + (tid < 16 ? tid : 112 + tid) * ldw, static_cast<uint32_t>(min(K, 4096)) * 2u);
+    prefetch(w);
     pdl_wait();
     for (int t0 = 0; t0 < a.T; t0 += 32) {
       __syncthreads();
@@ -134,27 +137,17 @@ __global__ void __launch_bounds__(MS_WARPS * 32, UP ? 2 : 3) moe_stream_kernel(M
     }
     return;
   }
-  pdl_wait();
   const int unit = blockIdx.y - (a.ws != nullptr ? 1 : 0);
-  int e = unit, from = 0;
-  if (a.by_pair) {
-    e = a.ids[unit];
-    int earlier = 0;
+  if (!a.by_pair) prefetch(a.w + unit * a.w_expert + wrow * ldw);
+  pdl_wait();
+  const int e = a.by_pair ? a.ids[unit] : unit;
+  int earlier = e < 0 || e >= a.E;
+  if (tid == 0) s_count = 0;
+  if (a.by_pair)
     for (int p = tid; p < unit; p += MS_WARPS * 32) earlier |= a.ids[p] == e;
-    if (__syncthreads_or(earlier)) return;         // an earlier CTA row has this expert
-    from = unit;
-  }
-  if (e < 0 || e >= a.E) return;
-  if (tid < 32) {                                  // the pairs of the expert, in order
-    int n = 0;
-    for (int p0 = from; p0 < pairs; p0 += 32) {
-      const bool mine = p0 + lane < pairs && a.ids[p0 + lane] == e;
-      const unsigned ballot = __ballot_sync(0xffffffffu, mine);
-      if (mine) list[n + __popc(ballot & ((1u << lane) - 1u))] = p0 + lane;
-      n += __popc(ballot);
-    }
-    if (lane == 0) s_count = n;
-  }
+  if (__syncthreads_or(earlier)) return;           // an earlier CTA row has this expert
+  for (int p = tid; p < pairs; p += MS_WARPS * 32)
+    if (a.ids[p] == e) list[atomicAdd(&s_count, 1)] = p;          // in any order: the pairs do not meet
   __syncthreads();
   const int count = s_count;
   const __nv_bfloat16* w = a.w + e * a.w_expert + wrow * ldw;
@@ -178,9 +171,9 @@ static int moe_stream_launch(MoeStreamArgs a, cudaStream_t st) {
   if ((a.ldx | a.ldw | a.ldws | a.w_expert) & 7) return -3;
   if ((reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.w) | reinterpret_cast<uintptr_t>(a.ws)) & 15) return -4;
   a.by_pair = pairs <= a.E ? 1 : 0;
-  const int n = a.ws != nullptr && a.Ns > a.N ? a.Ns : a.N;
-  const dim3 grid(n / 16, (a.by_pair ? pairs : a.E) + (a.ws != nullptr ? 1 : 0));
-  if (grid.y > 65535) return -5;
+  const int n = a.ws != nullptr && a.Ns > a.N ? a.Ns : a.N, rows = (a.by_pair ? pairs : a.E) + (a.ws != nullptr ? 1 : 0);
+  if (rows > 65535) return -5;
+  const dim3 grid(n / 16, rows);
   const size_t smem = sizeof(float) * (UP ? 2 : 1) * MS_WARPS * 4 * 16 * 9 + sizeof(int) * ((pairs + 3) & ~3);
   static bool configured[64] = {};                 // the attribute is per device
   int dev = 0;

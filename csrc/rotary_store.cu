@@ -118,7 +118,7 @@ struct Turns8 {
 };
 
 // bf16 heads of up to 128 channels in 16-byte vectors: one CTA per token, half a warp per head.
-__global__ void __launch_bounds__(256) rotary_store_vec_kernel(RotaryStoreArgs a) {
+__global__ void __launch_bounds__(256, 5) rotary_store_vec_kernel(RotaryStoreArgs a) {
   pdl_entry();
   const int sub = threadIdx.x >> 4, l8 = (threadIdx.x & 15) * 8, subs = blockDim.x >> 4;
   const long long row = blockIdx.x;
@@ -134,6 +134,7 @@ __global__ void __launch_bounds__(256) rotary_store_vec_kernel(RotaryStoreArgs a
   auto pack = [](const float (&f)[8]) { return make_uint4(pack_bf16x2(f[0], f[1]), pack_bf16x2(f[2], f[3]), pack_bf16x2(f[4], f[5]), pack_bf16x2(f[6], f[7])); };
   Turns8 turn;
   turn.load(a.key_turns, p, a.key_half, l8);
+#pragma unroll 2
   for (int hd = sub; hd < a.H + a.G; hd += subs) {
     const __nv_bfloat16* src = y + hd * a.dk + l8;
     uint4 r = zero;
