@@ -151,7 +151,8 @@ struct GeneralAttnArgs {
   int* err;
   int keep;                    // positions 0 .. keep - 1 are visible past the window; a ring store holds them in its first slots
   int gate_head;               // the gate is one number per (row, head): channel h
-  const float2* back;          // [positions, dv / 2] (cos, sin) (nullable)
+  const float2* back;          // [back_rows, dv / 2] (cos, sin) (nullable)
+  int back_rows;
 };
 constexpr int GA_WARPS = 4;
 constexpr int GA_DMAX = 256;
@@ -170,7 +171,7 @@ __global__ void __launch_bounds__(GA_WARPS * 32) general_attention_kernel(Genera
   const int b = static_cast<int>(row / a.S), s = static_cast<int>(row % a.S);
   const int g = h / (a.H / a.G);
   const int p = (a.pos ? a.pos[b] : 0) + s;
-  if (p < 0 || (!a.ring && p >= a.keys)) {         // a query without its own key in the store: report, leave the output
+  if (p < 0 || (!a.ring && p >= a.keys) || (a.back != nullptr && p >= a.back_rows)) {         // a query without its own key in the store or turns: report, leave the output
     if (lane == 0) report_error(a.err, ERR_BOUNDS, p);
     return;
   }
@@ -303,14 +304,14 @@ extern "C" TYR_EXPORT int tyr_general_attention_sink(const void* q, const void* 
 }
 
 // A window (0: none) that leaves the first `keep` positions visible, in rows of a prompt, a plain store or one of `keep` slots followed by a
-// ring; one gate per head (nullable: rows of strides[9] elements); `back` (nullable): [positions, dv / 2] pairs (cos, sin).  strides: as for
+// ring; one gate per head (nullable: rows of strides[9] elements); `back` (nullable): [back_rows, dv / 2] pairs (cos, sin).  strides: as for
 // the sink form.
 extern "C" TYR_EXPORT int tyr_general_attention_kept(const void* q, const void* k, const void* v, void* out, const int* pos, const void* head_gate,
-                                                     const void* back, const long long* strides, int B, int S, int H, int G, int dk, int dv, int cap,
+                                                     const void* back, int back_rows, const long long* strides, int B, int S, int H, int G, int dk, int dv, int cap,
                                                      int ring, int window, int keep, int keys, float scale, int dtype, int* err, void* stream) {
   if (keep < 0 || (ring && keep >= cap) || (back != nullptr && (dv & 1))) return -3;
   GeneralAttnArgs a{};
-  a.q = q; a.k = k; a.v = v; a.out = out; a.pos = pos; a.gate = head_gate; a.gate_head = 1; a.back = static_cast<const float2*>(back);
+  a.q = q; a.k = k; a.v = v; a.out = out; a.pos = pos; a.gate = head_gate; a.gate_head = 1; a.back = static_cast<const float2*>(back); a.back_rows = back_rows;
   a.B = B; a.S = S; a.H = H; a.G = G; a.dk = dk; a.dv = dv; a.cap = cap; a.ring = ring; a.window = window; a.keep = keep; a.keys = keys;
   a.gate_ld = strides[9]; a.out_ld = strides[10];
   a.scale = scale; a.out_scale = 1.f; a.err = err;

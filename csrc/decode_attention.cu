@@ -57,7 +57,7 @@ struct DecodeAttnArgs {
   float out_scale;
   int keep;                      // positions 0 .. keep - 1 are visible past the window
   const float2* back;            // [positions, back_half] (cos, sin) of a position's turns (nullable)
-  int back_half;
+  int back_half, back_rows;
 };
 
 __device__ __forceinline__ float decode_gate(const DecodeAttnArgs& a, int b, int h, int d) {
@@ -206,7 +206,7 @@ __global__ void __launch_bounds__(kDecWarps * 32) decode_attention_kernel(Decode
   const int g = lane >> 2, t = lane & 3;
   const int G = a.Hq / a.Hkv;
   const int pos = a.pos[b * a.pos_stride];
-  if (pos < 0 || (!a.ring && pos >= a.cap)) {    // position outside the store: report, leave the output untouched
+  if (pos < 0 || (!a.ring && pos >= a.cap) || (a.back != nullptr && pos >= a.back_rows)) {    // position outside the store or the turns: report, leave the output untouched
     if (tid == 0) report_error(a.err, ERR_BOUNDS, pos);
     return;
   }
@@ -523,7 +523,7 @@ static int decode_attention_launch(const void* q, const void* k_new, const void*
                                    int Hq, int Hkv, int DK, int DV, int cap, int ring, int window, int splits, int append, float scale,
                                    const void* gate, long long gate_bs, long long gate_hs, int gate_mode, const float* r1,
                                    const float* r2, void* err, void* stream, const float* sink = nullptr, int dv_out = 0,
-                                   long long out_bs = 0, float out_scale = 1.f, int keep = 0, const void* back = nullptr) {
+                                   long long out_bs = 0, float out_scale = 1.f, int keep = 0, const void* back = nullptr, int back_rows = 0) {
   using namespace tyr;
   if (gate_mode < 0 || gate_mode > 3 || (gate_mode != 0 && gate == nullptr)) return -5;
   if (B <= 0 || Hq <= 0 || Hkv <= 0 || Hq % Hkv != 0 || Hq / Hkv > 16 || cap <= 0 || splits < 1 || splits > 64) return -1;
@@ -550,6 +550,7 @@ static int decode_attention_launch(const void* q, const void* k_new, const void*
   a.keep = keep;
   a.back = (const float2*)back;
   a.back_half = a.dv / 2;
+  a.back_rows = back_rows;
   if (back != nullptr && (a.dv & 1)) return -8;
   const dim3 grid(splits, Hkv, B);
   const cudaStream_t st = (cudaStream_t)stream;
@@ -630,15 +631,15 @@ extern "C" TYR_EXPORT int tyr_decode_attention_sink(const void* q, const void* k
 }
 
 // Window (0: none) that leaves the first `keep` positions visible, in a plain store or one of `keep` slots followed by a ring; output gate
-// sigmoid(head_gate[b * gate_bs + h]) (nullable); `back` (nullable): [positions, dv / 2] pairs (cos, sin) by which the output's channel pairs
+// sigmoid(head_gate[b * gate_bs + h]) (nullable); `back` (nullable): [back_rows, dv / 2] pairs (cos, sin) by which the output's channel pairs
 // (m, m + dv / 2) are turned back.  k_new / v_new null: the store holds the new token already.  DK, DV in {64, 128}.
 extern "C" TYR_EXPORT int tyr_decode_attention_kept(const void* q, const void* k_new, const void* v_new, void* k_cache, void* v_cache, const void* pos,
                                                     int pos_stride, void* out, void* workspace, long long q_bs, long long kn_bs, long long vn_bs,
                                                     int B, int Hq, int Hkv, int DK, int DV, int dv, int cap, int ring, int window, int keep, int splits,
                                                     int append, float scale, const void* head_gate, long long gate_bs, const void* back,
-                                                    long long out_bs, void* err, void* stream) {
+                                                    int back_rows, long long out_bs, void* err, void* stream) {
   if (dv <= 0 || dv > DV) return -2;
   return decode_attention_launch(q, k_new, v_new, k_cache, v_cache, pos, pos_stride, out, workspace, q_bs, kn_bs, vn_bs, B, Hq, Hkv, DK, DV, cap, ring,
                                  window, splits, append, scale, head_gate, gate_bs, 1, head_gate == nullptr ? 0 : 3, nullptr, nullptr, err, stream,
-                                 nullptr, dv, out_bs, 1.f, keep, back);
+                                 nullptr, dv, out_bs, 1.f, keep, back, back_rows);
 }

@@ -214,6 +214,11 @@ def test_a_position_outside_store_and_tables_is_recorded():
     ka.step_attention(q, store, pos, 64, 64, scale=1.0, back=table)
     with pytest.raises(RuntimeError, match="code=3"):
         raise_on_device_error("cuda")
+    for dt in (torch.bfloat16, torch.float32):                      # a ring takes any position, the table does not
+        ring = KVCache.allocate(1, 1, 6, 64, "cuda", dt, ring=True)
+        ka.step_attention(q.to(dt), ring, pos, 64, 64, scale=1.0, window=6, back=table)
+        with pytest.raises(RuntimeError, match="code=3"):
+            raise_on_device_error("cuda")
 
 
 # ---- experts ------------------------------------------------------------------------------------------------------

@@ -29,8 +29,8 @@ _KIND = {torch.bfloat16: 0, torch.float32: 1}
 def _sigs(lib_):
     P, I, L, F = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong, ctypes.c_float
     for name, args in (("tyr_rotary_store", [P, L] + [P] * 9 + [ctypes.POINTER(I), F, I, P, P]),
-                       ("tyr_general_attention_kept", [P] * 7 + [ctypes.POINTER(L)] + [I] * 11 + [F, I, P, P]),
-                       ("tyr_decode_attention_kept", [P] * 6 + [I, P, P, L, L, L] + [I] * 12 + [F, P, L, P, L, P, P])):
+                       ("tyr_general_attention_kept", [P] * 7 + [I, ctypes.POINTER(L)] + [I] * 11 + [F, I, P, P]),
+                       ("tyr_decode_attention_kept", [P] * 6 + [I, P, P, L, L, L] + [I] * 12 + [F, P, L, P, I, L, P, P])):
         fn = getattr(lib_, name, None)
         if fn is not None:
             fn.argtypes, fn.restype = args, I
@@ -113,7 +113,8 @@ def _general(q, k, v, kv_strides, head_gate, back, pos, G, dk, dv, cap, ring, wi
         raise ValueError(f"attention heads hold at most {MAX_HEAD} channels, got {dk} and {dv}")
     out = torch.empty((B, S, H * dv), dtype=q.dtype, device=q.device)
     st = (ctypes.c_longlong * 11)(*q.stride()[:3], *kv_strides, 0 if head_gate is None else row_stride(head_gate), row_stride(out))
-    check(lib().tyr_general_attention_kept(ptr(q), ptr(k), ptr(v), ptr(out), ptr(pos), ptr(head_gate), ptr(back), st, B, S, H, G, dk, dv, cap, 1 if ring else 0,
+    check(lib().tyr_general_attention_kept(ptr(q), ptr(k), ptr(v), ptr(out), ptr(pos), ptr(head_gate), ptr(back), 0 if back is None else back.shape[0], st, B, S, H, G, dk, dv,
+                                           cap, 1 if ring else 0,
                                            int(window or 0), keep, keys, scale, _KIND[q.dtype], ptr(err_word(q.device)), cur_stream(q.device)),
           "general_attention_kept")
     return out
@@ -168,7 +169,7 @@ def step_attention(q, store, pos: torch.Tensor, dk: int, dv: int, *, scale: floa
         out = torch.empty((B, 1, H * dv), dtype=q.dtype, device=q.device)
         check(lib().tyr_decode_attention_kept(ptr(q), None, None, ptr(store.k), ptr(store.v), ptr(pos), 1, ptr(out), ptr(ws), q.stride(0), 0, 0, B, H, G, dkp, dvp,
                                               dv, cap, 1 if store.ring else 0, int(window or 0), keep, splits, 0, scale, ptr(head_gate),
-                                              0 if head_gate is None else head_gate.stride(0), ptr(back), out.stride(0), ptr(err_word(q.device)),
+                                              0 if head_gate is None else head_gate.stride(0), ptr(back), 0 if back is None else back.shape[0], out.stride(0), ptr(err_word(q.device)),
                                               cur_stream(q.device)), "decode_attention_kept")
         return out
     if q.is_cuda:
